@@ -45,7 +45,8 @@ enum {
 enum { RB_U8 = 0, RB_U32 = 1, RB_I64 = 2, RB_F16 = 3, RB_BF16 = 4, RB_F32 = 5, RB_F64 = 6 };
 
 /* ---- activations, rai-nn/src/activations.rs:5-30 and rai-core/src/hlops/activations.rs:5-32 ---- */
-enum { RB_ACT_NONE = 0, RB_ACT_SILU = 1, RB_ACT_GELU_TANH = 2, RB_ACT_GELU_ERF = 3, RB_ACT_RELU = 4 };
+enum { RB_ACT_NONE = 0, RB_ACT_SILU = 1, RB_ACT_GELU_TANH = 2, RB_ACT_GELU_ERF = 3, RB_ACT_RELU = 4,
+       RB_ACT_XIELU = 5 /* two learned numbers, see rb_linear_act; no counterpart in the reference */ };
 
 /* ---- norm kinds ---- */
 enum {
@@ -55,7 +56,11 @@ enum {
 };
 
 /* ---- decoder families, rai-models/src/llm/{qwen2,phi2,phi3,gemma}.rs ---- */
-enum { RB_ARCH_QWEN2 = 0, RB_ARCH_PHI2 = 1, RB_ARCH_PHI3 = 2, RB_ARCH_GEMMA = 3 };
+enum { RB_ARCH_QWEN2 = 0, RB_ARCH_PHI2 = 1, RB_ARCH_PHI3 = 2, RB_ARCH_GEMMA = 3,
+       RB_ARCH_MALASUN = 4 /* described layer by layer (rb_model_create_layers); no counterpart in the reference */ };
+
+/* ---- sequence mixers of a layer-by-layer design (rb_layer_config) ---- */
+enum { RB_MIXER_ATTENTION = 0, RB_MIXER_HGRN2 = 1 };
 
 /* ---- elementwise / reduce op tags of the primitive set (rai-core/src/dispatch.rs:41-157) ---- */
 enum {
@@ -227,6 +232,66 @@ int32_t rb_rope_attention_decode(rb_ctx* ctx, const void* qkv_dev, const float* 
                                  rb_kv_cache* cache, int32_t layer, float scale, void* q_scratch_dev, void* out_dev,
                                  int32_t dtype);
 
+/* ======================================================================================
+ * Mechanisms of designs beyond the reference's four families (no counterpart in the reference).  Rows of
+ * activations have a pitch `ld` in elements, a multiple of 8; what lies between the row's width and its pitch is
+ * written as zero.  "Model dtype" is `dtype`, RB_BF16 or RB_F32.
+ * ====================================================================================== */
+
+/* rb_linear with an activation that has parameters of its own: RB_ACT_XIELU takes two numbers (model dtype).  With
+ * a = softplus(act_params[0]) and b = 1/2 + softplus(act_params[1]) it is x/2 + a x^2 for positive x and
+ * x/2 + b (expm1(x) - x) otherwise. */
+int32_t rb_linear_act(rb_ctx* ctx, const void* x_dev, const void* w_dev, const void* bias_dev, void* out_dev, int64_t m,
+                      int64_t n, int64_t k, int32_t act, const void* act_params_dev, int32_t dtype);
+/* Embedding into a float32 residual stream: h[i, :] = table[ids[i], :] and, unless x_dev is NULL, the same rows in the
+ * model dtype (the operand of the next product). */
+int32_t rb_embed_stream(rb_ctx* ctx, const void* table_dev, int32_t dtype, int64_t vocab, int64_t width, int64_t ld,
+                        const uint32_t* ids_dev, int64_t n_ids, float* h_dev, void* x_dev);
+/* Norm on a sublayer's output, added to a float32 residual stream: with y = y_dev + sum_s acc[s] (either may be NULL),
+ *   h += gain * rms(y),  x = h in the model dtype (x_dev may be NULL), where rms(y) is y scaled by 1 / sqrt(eps + mean of
+ * its squares) and gain a single number. */
+int32_t rb_add_scaled_norm(rb_ctx* ctx, const void* y_dev, const float* acc_dev, int32_t n_acc, const void* gain_dev, float eps,
+                           int64_t rows, int64_t width, int64_t ld, float* h_dev, void* x_dev, int32_t dtype);
+/* out[i, :] = gain * rms(h[r_i, :]), with r_i = rows_dev[i], or (i + 1) * row_step - 1 when
+ * rows_dev is NULL: the norm before the vocabulary product, of the rows whose logits are wanted. */
+int32_t rb_scalar_norm_rows(rb_ctx* ctx, const float* h_dev, const int32_t* rows_dev, int64_t row_step, const void* gain_dev,
+                            float eps, int64_t n_rows, int64_t width, int64_t ld, void* out_dev, int32_t dtype);
+/* Short causal convolution over time on each channel of q, k and v, RMS norm of the whole of q and the whole of k, head
+ * split and cache append, for one fused projection.  Its columns are [q | k | v | gate], each part padded to a
+ * multiple of 8; kv_heads == 0 means [q | gate] (a layer that reads another layer's keys and values).
+ *   u = src + sum_s acc[s] + bias                    (src or acc may be NULL; with acc, s_new must be 1)
+ *   y[t] = sum over b = 0..taps-1 of conv[taps - 1 - b] u[t - b]      conv is [taps][columns of q, k, v]; u[<0] = 0
+ *   q, k: weight * rms(y), one rms over all the part's columns       (weight NULL: no norm)
+ * q goes to q_out [rows, q_heads, cache head_dim] and k, v to the cache at the tokens' positions, each head padded
+ * with zeros to the cache's head_dim.  The last taps - 1 values of u per sequence live in `ring`
+ * [cache max_batch][taps - 1][columns of q, k, v] (float32, at index position % (taps - 1), by state slot); new_lens_dev
+ * ([batch], NULL = s_new each) says how many of the s_new rows are tokens.  gate_out (may be NULL): the gate columns of u. */
+int32_t rb_conv_norm_append(rb_ctx* ctx, const void* src_dev, const float* acc_dev, int32_t n_acc, const void* bias_dev,
+                            const void* conv_dev, int32_t taps, const void* q_weight_dev, const void* k_weight_dev, float eps,
+                            int32_t batch, int32_t s_new, int32_t q_heads, int32_t kv_heads, int32_t key_dim, int32_t value_dim,
+                            int64_t src_ld, rb_kv_cache* cache, int32_t layer, float* ring_dev, const int32_t* new_lens_dev,
+                            void* q_out_dev, void* gate_out_dev, int32_t dtype);
+/* rb_attention with a rolling window, a distance bias and an output gate.  The row at position i sees the `window` keys
+ * i - window + 1 .. i (0 = every earlier key), in prompts and single-token steps alike; the score is q.k * scale, less
+ * 2^(-8 (h + 1) / q_heads) * (i - j) for head h when `alibi` is set; out[row, h * value_dim + e] (pitch out_ld) is
+ * multiplied by sigmoid(gate[row, h * value_dim + e]) when gate is given (model dtype, pitch gate_ld). */
+int32_t rb_attention_window(rb_ctx* ctx, const void* q_dev, rb_kv_cache* cache, int32_t layer, int32_t batch, int32_t s_new,
+                            int32_t q_heads, int32_t value_dim, float scale, int32_t window, int32_t alibi, const void* gate_dev,
+                            int64_t gate_ld, void* out_dev, int64_t out_ld, int32_t dtype);
+/* The HGRN2 recurrence: a head's state is a key_dim x value_dim matrix, and what a row forgets makes room for what it
+ * takes in.  One fused projection u = src + sum_s acc[s] (with acc, s_new must be 1) has columns [q | f | v], each padded
+ * to a multiple of 8.  Per token and head, for state row r with keep = lower + (1 - lower) sigmoid(u_f + f_bias):
+ *   state[r][:] = keep[r] state[r][:] + (1 - keep[r]) u_v[:];      out = norm_weight * rms(sum over r of silu(u_q[r]) state[r][:]).
+ * Everything after the projection is float32.  `state` is [cache max_batch][heads][key_dim][value_dim] float32, by
+ * state slot; a sequence whose first token is among these rows starts from zero.  Lengths and slots come from `cache`
+ * (see rb_conv_norm_append for new_lens_dev).  chunk > 0 cuts a prompt into pieces of that many tokens that run in
+ * parallel (two passes over the tokens and a scan over the pieces; the same recurrence, so the same rounding up to
+ * the scan); 0 lets the library choose. */
+int32_t rb_hgrn2(rb_ctx* ctx, const void* src_dev, const float* acc_dev, int32_t n_acc, int64_t src_ld, const void* f_bias_dev,
+                 const void* lower_dev, const void* norm_weight_dev, float eps, int32_t heads, int32_t key_dim, int32_t value_dim,
+                 int32_t batch, int32_t s_new, rb_kv_cache* cache, const int32_t* new_lens_dev, float* state_dev, int32_t chunk,
+                 void* out_dev, int64_t out_ld, int32_t dtype);
+
 /* sample_argmax, examples/qwen2/src/main.rs:32-40: per row, the index of the maximum under f32
  * total order, the LAST index among equal maxima.  Bit-exact by construction. */
 int32_t rb_argmax_rows(rb_ctx* ctx, const void* logits_dev, int32_t dtype, int64_t rows, int64_t cols,
@@ -346,6 +411,31 @@ typedef struct rb_model_config {
 } rb_model_config;
 
 int32_t rb_model_create(rb_ctx* ctx, const rb_model_config* cfg, rb_model** out);
+
+/* One layer of a design that is described layer by layer: its sequence mixer and its feed-forward. */
+typedef struct rb_layer_config {
+  int32_t mixer;                   /* RB_MIXER_* */
+  int32_t heads;
+  int32_t kv_heads;                /* attention: heads / kv_heads query heads share a key/value head */
+  int32_t key_dim;                 /* per-head query / key size */
+  int32_t value_dim;               /* per-head value size */
+  int32_t conv_taps;               /* attention: taps of the short convolution on q, k and v */
+  int32_t window;                  /* attention: how many keys, its own included, a token sees; 0 = all of them */
+  int32_t kv_from;                 /* attention: the earlier layer whose keys and values this one reads; -1 = its own */
+  int32_t mlp_size;                /* dense feed-forward, RB_ACT_XIELU; 0 = the layer has none */
+  int32_t reserved0;               /* set to 0 */
+  double scale;                    /* attention: factor on q.k */
+} rb_layer_config;
+
+/* A model of RB_ARCH_MALASUN: `layers` has cfg->num_hidden_layers entries.  Of cfg, the fields arch, dtype, vocab_size,
+ * hidden_size, num_hidden_layers, norm_eps and the capacities are read.  The residual stream and the logits are float32
+ * whatever the model dtype; every other rb_model_* entry point works as for the other families.  Single GPU. */
+int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out);
+/* RB_F32 or RB_BF16: the type in which rb_model_forward* return logits (the model dtype for the reference's families). */
+int32_t rb_model_logits_dtype(rb_model* m);
+/* Test hook: from now on every forward call copies the residual stream after each layer to dst_dev
+ * [layers][batch * seq][hidden_size] (float32); NULL stops it.  RB_ARCH_MALASUN only; not with the captured decode step. */
+int32_t rb_model_set_layer_trace(rb_model* m, float* dst_dev);
 int32_t rb_model_destroy(rb_model* m);
 /* Tensor::update_by_name, rai-core/src/nn.rs:192-205: copies (and casts to the model dtype) one named
  * parameter; names follow the derive rule of rai-core/src/nn.rs:256-269, e.g.
@@ -400,6 +490,15 @@ int32_t rb_model_forward(rb_model* m, const uint32_t* tokens_dev, int32_t batch,
  * examples run one sequence; a server batching prompts of different lengths needs this. */
 int32_t rb_model_forward_ragged(rb_model* m, const uint32_t* tokens_dev, int32_t batch, int32_t seq, int32_t pos,
                                 const int32_t* lens_host, void* logits_dev);
+/* The general step of a server: sequence b feeds lens_host[b] (0..seq) of the seq tokens in its row (NULL = seq each), and
+ * logits are returned for the positions rows_host[i] = b * seq + s of this call, [n_rows, vocab] (n_rows may be 0).
+ * pos >= 0 must be every sequence's cached length; pos = -1 continues each at its own, so that single tokens and whole
+ * prompts, or later portions of prompts, can share a call. */
+int32_t rb_model_forward_rows(rb_model* m, const uint32_t* tokens_dev, int32_t batch, int32_t seq, int32_t pos,
+                              const int32_t* lens_host, const int32_t* rows_host, int32_t n_rows, void* logits_dev);
+/* Sequences keep_host[0..n) (distinct) become sequences 0..n-1; every other sequence is released: its cache pages and
+ * state slots are free for new sequences.  No cached data moves, only the tables that name it. */
+int32_t rb_model_keep_sequences(rb_model* m, const int32_t* keep_host, int32_t n);
 /* rb_model_generate_step for the prompts of a right-padded batch, from an empty cache: host tokens
  * [batch, seq] and lens_host in, one sampled token per sequence out.  Synchronous.  Continue with
  * rb_model_generate_step / rb_model_decode_loop passing pos = -1 ("each sequence at its own length"). */
@@ -440,7 +539,7 @@ int64_t rb_launch_count(rb_ctx* ctx);
  * and fills out4 = {launches, total milliseconds, algorithmic bytes, floating-point operations} for
  * one kernel class (RB_PROF_*). */
 enum { RB_PROF_GEMM = 0, RB_PROF_ATTENTION = 1, RB_PROF_NORM = 2, RB_PROF_ROPE_KV = 3, RB_PROF_EMBED = 4,
-       RB_PROF_ARGMAX = 5, RB_PROF_OTHER = 6, RB_PROF_CLASSES = 7 };
+       RB_PROF_ARGMAX = 5, RB_PROF_OTHER = 6, RB_PROF_RECURRENCE = 7, RB_PROF_CLASSES = 8 };
 int32_t rb_profile_start(rb_ctx* ctx);
 int32_t rb_profile_read(rb_ctx* ctx, int32_t kernel_class, double* out4);
 /* Bytes of device memory the model holds for parameters (after sharding). */

@@ -65,6 +65,23 @@ pub struct rb_model {
 pub struct rb_safetensors {
     _p: [u8; 0],
 }
+/// `struct rb_layer_config` of include/rai_b200.h, field for field.
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct rb_layer_config {
+    pub mixer: i32,
+    pub heads: i32,
+    pub kv_heads: i32,
+    pub key_dim: i32,
+    pub value_dim: i32,
+    pub conv_taps: i32,
+    pub window: i32,
+    pub kv_from: i32,
+    pub mlp_size: i32,
+    pub reserved0: i32,
+    pub scale: f64,
+}
+
 /// `struct rb_model_config` of include/rai_b200.h, field for field.
 #[repr(C)]
 #[derive(Clone, Copy, Debug, Default)]
@@ -128,6 +145,13 @@ extern "C" {
     pub fn rb_attention(ctx: *mut rb_ctx, q_dev: *const c_void, cache: *mut rb_kv_cache, layer: i32, batch: i32, s_new: i32, q_heads: i32, scale: f32, out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_attention_decode_static(ctx: *mut rb_ctx, q_dev: *const c_void, cache: *mut rb_kv_cache, layer: i32, batch: i32, q_heads: i32, scale: f32, out_dev: *mut c_void) -> i32;
     pub fn rb_rope_attention_decode(ctx: *mut rb_ctx, qkv_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, cos_dev: *const f32, sin_dev: *const f32, rot: i32, batch: i32, q_heads: i32, cache: *mut rb_kv_cache, layer: i32, scale: f32, q_scratch_dev: *mut c_void, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_linear_act(ctx: *mut rb_ctx, x_dev: *const c_void, w_dev: *const c_void, bias_dev: *const c_void, out_dev: *mut c_void, m: i64, n: i64, k: i64, act: i32, act_params_dev: *const c_void, dtype: i32) -> i32;
+    pub fn rb_embed_stream(ctx: *mut rb_ctx, table_dev: *const c_void, dtype: i32, vocab: i64, width: i64, ld: i64, ids_dev: *const u32, n_ids: i64, h_dev: *mut f32, x_dev: *mut c_void) -> i32;
+    pub fn rb_add_scaled_norm(ctx: *mut rb_ctx, y_dev: *const c_void, acc_dev: *const f32, n_acc: i32, gain_dev: *const c_void, eps: f32, rows: i64, width: i64, ld: i64, h_dev: *mut f32, x_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_scalar_norm_rows(ctx: *mut rb_ctx, h_dev: *const f32, rows_dev: *const i32, row_step: i64, gain_dev: *const c_void, eps: f32, n_rows: i64, width: i64, ld: i64, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_conv_norm_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, conv_dev: *const c_void, taps: i32, q_weight_dev: *const c_void, k_weight_dev: *const c_void, eps: f32, batch: i32, s_new: i32, q_heads: i32, kv_heads: i32, key_dim: i32, value_dim: i32, src_ld: i64, cache: *mut rb_kv_cache, layer: i32, ring_dev: *mut f32, new_lens_dev: *const i32, q_out_dev: *mut c_void, gate_out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_attention_window(ctx: *mut rb_ctx, q_dev: *const c_void, cache: *mut rb_kv_cache, layer: i32, batch: i32, s_new: i32, q_heads: i32, value_dim: i32, scale: f32, window: i32, alibi: i32, gate_dev: *const c_void, gate_ld: i64, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
+    pub fn rb_hgrn2(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, f_bias_dev: *const c_void, lower_dev: *const c_void, norm_weight_dev: *const c_void, eps: f32, heads: i32, key_dim: i32, value_dim: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, new_lens_dev: *const i32, state_dev: *mut f32, chunk: i32, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
     pub fn rb_argmax_rows(ctx: *mut rb_ctx, logits_dev: *const c_void, dtype: i32, rows: i64, cols: i64, out_dev: *mut u32) -> i32;
     pub fn rb_sample_greedy(ctx: *mut rb_ctx, logits_dev: *const c_void, dtype: i32, rows: i64, cols: i64, penalty: f32, context_dev: *const i32, context_stride: i32, context_count_dev: *const i32, eos_token: i32, finished_dev: *mut u8, out_dev: *mut u32) -> i32;
     pub fn rb_unary(ctx: *mut rb_ctx, op: i32, x_dev: *const c_void, out_dev: *mut c_void, n: i64, scalar: f32, dtype: i32) -> i32;
@@ -151,6 +175,9 @@ extern "C" {
     pub fn rb_pool2d(ctx: *mut rb_ctx, is_max: i32, x_dev: *const c_void, x_shape4: *const i32, kernel2: *const i32, stride2: *const i32, padding2: *const i32, dilation2: *const i32, out_dev: *mut c_void, out_shape4: *mut i32, dtype: i32) -> i32;
     pub fn rb_upsample_nearest2d(ctx: *mut rb_ctx, x_dev: *const c_void, x_shape4: *const i32, out_h: i32, out_w: i32, out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_model_create(ctx: *mut rb_ctx, cfg: *const rb_model_config, out: *mut *mut rb_model) -> i32;
+    pub fn rb_model_create_layers(ctx: *mut rb_ctx, cfg: *const rb_model_config, layers: *const rb_layer_config, out: *mut *mut rb_model) -> i32;
+    pub fn rb_model_logits_dtype(m: *mut rb_model) -> i32;
+    pub fn rb_model_set_layer_trace(m: *mut rb_model, dst_dev: *mut f32) -> i32;
     pub fn rb_model_destroy(m: *mut rb_model) -> i32;
     pub fn rb_model_load_param(m: *mut rb_model, name: *const c_char, data: *const c_void, on_device: i32, src_dtype: i32, rank: i32, shape: *const i64) -> i32;
     pub fn rb_model_read_param(m: *mut rb_model, name: *const c_char, dst_host: *mut c_void, dst_bytes: usize) -> i32;
@@ -166,6 +193,8 @@ extern "C" {
     pub fn rb_tp_unique_id(out128: *mut c_void) -> i32;
     pub fn rb_model_forward(m: *mut rb_model, tokens_dev: *const u32, batch: i32, seq: i32, pos: i32, logits_dev: *mut c_void) -> i32;
     pub fn rb_model_forward_ragged(m: *mut rb_model, tokens_dev: *const u32, batch: i32, seq: i32, pos: i32, lens_host: *const i32, logits_dev: *mut c_void) -> i32;
+    pub fn rb_model_forward_rows(m: *mut rb_model, tokens_dev: *const u32, batch: i32, seq: i32, pos: i32, lens_host: *const i32, rows_host: *const i32, n_rows: i32, logits_dev: *mut c_void) -> i32;
+    pub fn rb_model_keep_sequences(m: *mut rb_model, keep_host: *const i32, n: i32) -> i32;
     pub fn rb_model_generate_ragged(m: *mut rb_model, tokens_host: *const u32, batch: i32, seq: i32, lens_host: *const i32, next_host: *mut u32) -> i32;
     pub fn rb_model_generate_step(m: *mut rb_model, tokens_host: *const u32, batch: i32, seq: i32, pos: i32, next_host: *mut u32) -> i32;
     pub fn rb_model_decode_loop(m: *mut rb_model, tokens_dev: *const u32, batch: i32, pos: i32, steps: i32, out_dev: *mut u32) -> i32;

@@ -20,9 +20,10 @@ LIB_PATH = PKG / ("librai_b200_dbg.so" if __import__("os").environ.get("RAI_B200
 # status codes / tags of the header, mirrored for Python callers
 RB_OK = 0
 U8, U32, I64, F16, BF16, F32, F64 = range(7)
-ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF, ACT_RELU = range(5)
+ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF, ACT_RELU, ACT_XIELU = range(6)
 NORM_RMS, NORM_RMS_ONE_PLUS, NORM_LAYER = range(3)
-ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA = range(4)
+ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA, ARCH_MALASUN = range(5)
+MIXER_ATTENTION, MIXER_HGRN2 = range(2)
 (UN_NEG, UN_EXP, UN_SQRT, UN_RSQRT, UN_SQUARE, UN_TANH, UN_ERF, UN_SIN, UN_COS, UN_POWF, UN_SILU, UN_GELU_TANH,
  UN_GELU_ERF, UN_RELU, UN_LOG, UN_ABS, UN_RECIP, UN_ADD_SCALAR, UN_MUL_SCALAR, UN_SIGN, UN_LOG2, UN_LOG10) = range(22)
 CMP_EQ, CMP_NE, CMP_GT, CMP_GE, CMP_LT, CMP_LE = range(6)
@@ -46,6 +47,13 @@ class ModelConfig(ctypes.Structure):
         "num_attention_heads", "num_key_value_heads", "max_position_embeddings", "rotary_dim", "hidden_act",
         "tie_word_embeddings", "max_batch", "max_seq", "max_tokens", "tp_rank", "tp_size", "sliding_window", "reserved0")] + [
         ("rope_theta", ctypes.c_double), ("norm_eps", ctypes.c_double)]
+
+
+class LayerConfig(ctypes.Structure):
+    """struct rb_layer_config of include/rai_b200.h."""
+    _fields_ = [(n, ctypes.c_int32) for n in (
+        "mixer", "heads", "kv_heads", "key_dim", "value_dim", "conv_taps", "window", "kv_from", "mlp_size",
+        "reserved0")] + [("scale", ctypes.c_double)]
 
 
 _SCALARS = {"int32_t": ctypes.c_int32, "int64_t": ctypes.c_int64, "size_t": ctypes.c_size_t, "float": ctypes.c_float,

@@ -1,6 +1,7 @@
 """Decoder configurations.
 
-Field names follow the reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24,
+Malasun, a design described layer by layer (no counterpart in the reference), has a configuration of its own shape: see
+`malasun_config`.  For the others, field names follow the reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24,
 phi3.rs:9-24, gemma.rs:12-27) as they appear in a Hugging Face config.json, plus `arch`.
 `BASELINE` holds the five benchmark configurations; `TINY` holds small models of the same four
 architectures for parity tests.
@@ -8,11 +9,16 @@ architectures for parity tests.
 from __future__ import annotations
 
 import copy
+import ctypes
+import json
+import os
 from typing import Dict
 
 from . import _lib
 
-ARCH_IDS = {"qwen2": _lib.ARCH_QWEN2, "phi2": _lib.ARCH_PHI2, "phi3": _lib.ARCH_PHI3, "gemma": _lib.ARCH_GEMMA}
+ARCH_IDS = {"qwen2": _lib.ARCH_QWEN2, "phi2": _lib.ARCH_PHI2, "phi3": _lib.ARCH_PHI3, "gemma": _lib.ARCH_GEMMA,
+            "malasun": _lib.ARCH_MALASUN}
+MIXER_IDS = {"attention": _lib.MIXER_ATTENTION, "hgrn2": _lib.MIXER_HGRN2}
 # serde names of rai-nn/src/activations.rs:5-17
 ACT_IDS = {"silu": _lib.ACT_SILU, "gelu_new": _lib.ACT_GELU_TANH, "newgelu": _lib.ACT_GELU_TANH,
            "gelu": _lib.ACT_GELU_ERF, "relu": _lib.ACT_RELU}
@@ -76,8 +82,80 @@ TINY: Dict[str, dict] = {
 }
 
 
+def malasun_layer(kind: str, heads: int, dim: int, vdim: int, mlp: int = 0, kv_heads: int = 0, conv: int = 1, window: int = 0,
+                  scale: float = 0.0, kv_from=None) -> dict:
+    """One entry of a Malasun configuration's `layers`; mlp = 0 leaves the feed-forward out."""
+    mixer = dict(type=kind, heads=heads, dim=dim, vdim=vdim)
+    if kind == "attention":
+        mixer.update(kv_heads=kv_heads or heads, conv=conv, window=window, scale=scale or dim ** -0.5, kv_from=kv_from)
+    return dict(mixer=mixer, mlp=dict(kind="dense", ff=mlp) if mlp else None)
+
+
+def _malasun(vocab: int, width: int, layers, eps: float = 1e-6) -> dict:
+    return dict(arch="malasun", vocab_size=vocab, hidden_size=width, norm_eps=eps, layers=layers)
+
+
+def _malasun_bench(vocab: int, width: int, heads: int, kv_heads: int, ff: int, pairs: int, window: int) -> dict:
+    """Alternating hgrn2 and attention layers of 128-wide heads, each with a feed-forward."""
+    layers = []
+    for _ in range(pairs):
+        layers.append(malasun_layer("hgrn2", heads, 128, 128, ff))
+        layers.append(malasun_layer("attention", heads, 128, 128, ff, kv_heads, 4, window))
+    return _malasun(vocab, width, layers)
+
+
+MALASUN: Dict[str, dict] = {
+    # sizes that resemble a real model's layers, for throughput measurements (random weights)
+    "malasun-1k": _malasun_bench(32000, 1024, 8, 2, 4096, 2, 1024),
+    "malasun-2k": _malasun_bench(32000, 2048, 16, 4, 8192, 2, 1024),
+    "malasun-4k": _malasun_bench(32000, 4096, 32, 8, 16384, 2, 1024),
+    # small models for tests
+    "tiny-malasun": _malasun(320, 160, [
+        malasun_layer("attention", 4, 40, 32, 200, 2, 4, 21), malasun_layer("hgrn2", 3, 32, 48, 0),
+        malasun_layer("hgrn2", 2, 72, 24, 88), malasun_layer("attention", 4, 40, 32, 0, 2, 2, 75, kv_from=0),
+        malasun_layer("attention", 6, 64, 64, 120, 6, 1, 33, 0.17)]),
+}
+
+
+def malasun_config(raw: dict) -> dict:
+    """A Malasun config.json -> the configuration the library takes."""
+    layers = []
+    for i, entry in enumerate(raw["layers"]):
+        kind, mix, mlp = entry["type"], entry["mixer"], entry.get("mlp")
+        if kind not in MIXER_IDS:
+            raise _lib.RaiB200Error(-7, f"layer {i}: mixer {kind!r} is not implemented")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise _lib.RaiB200Error(-7, f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented")
+        ff = int(mlp["ff"]) if mlp is not None else 0
+        if kind == "attention":
+            src = mix.get("kv_from")
+            layers.append(malasun_layer(kind, int(mix["heads"]), int(mix["dim"]), int(mix["vdim"]), ff, int(mix["kv_heads"]),
+                                        int(mix["conv"]), int(mix["mask"]["size"]), float(mix["scale"]),
+                                        None if src is None else int(src)))
+        else:
+            layers.append(malasun_layer(kind, int(mix["heads"]), int(mix["dim"]), int(mix["vdim"]), ff))
+    return _malasun(int(raw["vocab"]), int(raw["width"]), layers, float(raw["norm"]["eps"]))
+
+
+_MODEL_TYPES = {"qwen2": "qwen2", "phi": "phi2", "phi2": "phi2", "phi3": "phi3", "gemma": "gemma"}
+
+
+def from_json(path: str) -> dict:
+    """The configuration in a checkpoint folder's (or file's) config.json, whichever architecture it names."""
+    if os.path.isdir(path):
+        path = os.path.join(path, "config.json")
+    with open(path) as f:
+        raw = json.load(f)
+    if raw.get("architecture") == "Malasun":
+        return malasun_config(raw)
+    name = raw.get("arch") or _MODEL_TYPES.get(raw.get("model_type"))
+    if name not in ARCH_IDS or name == "malasun":
+        raise _lib.RaiB200Error(-7, f"{path}: architecture {raw.get('architecture') or raw.get('model_type')!r} is not implemented")
+    return dict(raw, arch=name)
+
+
 def get(name: str) -> dict:
-    src = BASELINE.get(name) or TINY.get(name)
+    src = BASELINE.get(name) or TINY.get(name) or MALASUN.get(name)
     if src is None:
         raise KeyError(f"unknown configuration {name!r}")
     return copy.deepcopy(src)
@@ -100,6 +178,29 @@ def tied(cfg: dict) -> bool:
     return cfg["arch"] == "gemma" or bool(cfg.get("tie_word_embeddings", False))
 
 
+def layer_structs(cfg: dict):
+    """The rb_layer_config array of a layer-by-layer configuration."""
+    arr = (_lib.LayerConfig * len(cfg["layers"]))()
+    for s, layer in zip(arr, cfg["layers"]):
+        mix, mlp = layer["mixer"], layer["mlp"]
+        s.mixer = MIXER_IDS[mix["type"]]
+        s.heads, s.key_dim, s.value_dim = mix["heads"], mix["dim"], mix["vdim"]
+        s.kv_from = -1
+        s.mlp_size = mlp["ff"] if mlp else 0
+        if mix["type"] == "attention":
+            s.kv_heads, s.conv_taps, s.window, s.scale = mix["kv_heads"], mix["conv"], mix["window"], mix["scale"]
+            s.kv_from = -1 if mix["kv_from"] is None else mix["kv_from"]
+    return arr
+
+
+def create_model(ctx, cfg: dict, struct, out) -> None:
+    """rb_model_create or rb_model_create_layers, by architecture."""
+    if cfg["arch"] == "malasun":
+        _lib.call("rb_model_create_layers", ctx, ctypes.byref(struct), ctypes.byref(layer_structs(cfg)), ctypes.byref(out))
+    else:
+        _lib.call("rb_model_create", ctx, ctypes.byref(struct), ctypes.byref(out))
+
+
 def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: int, tp_rank: int = 0,
               tp_size: int = 1) -> "_lib.ModelConfig":
     if cfg["arch"] == "phi2" and cfg.get("qk_layernorm"):
@@ -107,6 +208,12 @@ def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: i
     s = _lib.ModelConfig()
     s.arch = ARCH_IDS[cfg["arch"]]
     s.dtype = dtype
+    s.max_batch, s.max_seq, s.max_tokens = int(max_batch), int(max_seq), int(max_tokens)
+    s.tp_rank, s.tp_size = int(tp_rank), int(tp_size)
+    if cfg["arch"] == "malasun":
+        s.vocab_size, s.hidden_size, s.num_hidden_layers = cfg["vocab_size"], cfg["hidden_size"], len(cfg["layers"])
+        s.norm_eps = cfg["norm_eps"]
+        return s
     for k in ("vocab_size", "hidden_size", "intermediate_size", "num_hidden_layers", "num_attention_heads",
               "max_position_embeddings"):
         setattr(s, k, int(cfg[k]))
@@ -114,8 +221,6 @@ def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: i
     s.rotary_dim = rotary_dim(cfg)
     s.hidden_act = ACT_IDS[cfg["hidden_act"]]
     s.tie_word_embeddings = int(tied(cfg))
-    s.max_batch, s.max_seq, s.max_tokens = int(max_batch), int(max_seq), int(max_tokens)
-    s.tp_rank, s.tp_size = int(tp_rank), int(tp_size)
     # only qwen2's mask has the sliding-window term (qwen2.rs:316-327); the other families' masks are plain causal
     s.sliding_window = int(cfg.get("sliding_window") or 0) if cfg["arch"] == "qwen2" else 0
     s.reserved0 = 0

@@ -102,6 +102,7 @@ extern "C" int32_t rb_destroy(rb_ctx* ctx) {
   if (ctx->argmax_best) cudaFree(ctx->argmax_best);
   if (ctx->argmax_count) cudaFree(ctx->argmax_count);
   if (ctx->attn_scratch) cudaFree(ctx->attn_scratch);
+  if (ctx->chunk_scratch) cudaFree(ctx->chunk_scratch);
   for (void* r : ctx->retired) cudaFree(r);
   if (ctx->gemm_scratch) cudaFree(ctx->gemm_scratch);
   if (ctx->gemm_tile_count) cudaFree(ctx->gemm_tile_count);
@@ -247,39 +248,75 @@ extern "C" int32_t rb_download(rb_ctx* ctx, void* dst, const void* src, size_t b
 }
 
 // ------------------------------------------------------------------------------------------ KV cache
+int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_heads, int head_dim, int max_batch, int max_seq,
+                        int dtype, rb_kv_cache** out) {
+  rb_kv_cache* c = new rb_kv_cache(shared);
+  c->ctx = ctx;
+  c->layers = layers; c->kv_heads = kv_heads; c->head_dim = head_dim;
+  c->max_batch = shared ? shared->max_batch : max_batch;
+  c->dtype = dtype;
+  c->pages_per_seq = ((shared ? shared->max_seq : max_seq) + kPageTokens - 1) / kPageTokens;
+  c->max_seq = c->pages_per_seq * kPageTokens;
+  c->num_pages = c->pages_per_seq * c->max_batch;
+  const size_t bytes = (size_t)layers * c->layer_stride_elems() * dtype_size(dtype);
+  int st = rb_malloc(ctx, bytes, &c->k);
+  if (st == RB_OK) st = rb_malloc(ctx, bytes, &c->v);
+  if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->num_pages * sizeof(int32_t), (void**)&c->block_table);
+  if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->seq_lens);
+  if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->slots);
+  if (st == RB_OK) st = rb_malloc(ctx, (size_t)c->max_batch * kv_heads * sizeof(uint32_t), (void**)&c->split_count);
+  if (st != RB_OK) { rb_kv_cache_destroy(c); return st; }
+  // Zero the pages: the tail of a sequence's last page is read (and masked) by the attention
+  // kernels, so it must hold finite values.
+  if (bytes) RB_CUDA(cudaMemsetAsync(c->k, 0, bytes, ctx->stream));
+  if (bytes) RB_CUDA(cudaMemsetAsync(c->v, 0, bytes, ctx->stream));
+  if (shared) {
+    c->block_table = shared->block_table;
+    c->seq_lens = shared->seq_lens;
+    c->slots = shared->slots;
+  } else {
+    c->host_table.resize(c->num_pages);
+    for (int i = 0; i < c->num_pages; ++i) c->host_table[i] = i;  // sequence b owns pages [b*pages_per_seq, ...)
+    c->host_slots.resize(c->max_batch);
+    for (int i = 0; i < c->max_batch; ++i) c->host_slots[i] = i;
+    RB_CUDA(cudaMemcpyAsync(c->block_table, c->host_table.data(), c->host_table.size() * sizeof(int32_t), cudaMemcpyHostToDevice,
+                            ctx->stream));
+    RB_CUDA(cudaMemcpyAsync(c->slots, c->host_slots.data(), c->host_slots.size() * sizeof(int32_t), cudaMemcpyHostToDevice,
+                            ctx->stream));
+    RB_CUDA(cudaMemsetAsync(c->seq_lens, 0, (size_t)c->max_batch * sizeof(int32_t), ctx->stream));
+    c->own_lens.assign(c->max_batch, 0);
+  }
+  RB_CUDA(cudaMemsetAsync(c->split_count, 0, (size_t)c->max_batch * kv_heads * sizeof(uint32_t), ctx->stream));
+  RB_CUDA(cudaStreamSynchronize(ctx->stream));
+  ctx->caches.push_back(c);
+  *out = c;
+  return RB_OK;
+}
+
 extern "C" int32_t rb_kv_cache_create(rb_ctx* ctx, int32_t layers, int32_t kv_heads, int32_t head_dim,
                                       int32_t max_batch, int32_t max_seq, int32_t dtype, rb_kv_cache** out) {
   RB_REQUIRE(ctx && out, "rb_kv_cache_create: null argument");
   RB_REQUIRE(layers > 0 && kv_heads > 0 && head_dim > 0 && max_batch > 0 && max_seq > 0, "rb_kv_cache_create: bad sizes");
   RB_REQUIRE(dtype == RB_BF16 || dtype == RB_F32, "rb_kv_cache_create: dtype %d unsupported", dtype);
   RB_REQUIRE(head_dim % 8 == 0 && head_dim <= 256, "rb_kv_cache_create: head_dim %d unsupported", head_dim);
-  rb_kv_cache* c = new rb_kv_cache();
-  c->ctx = ctx;
-  c->layers = layers; c->kv_heads = kv_heads; c->head_dim = head_dim;
-  c->max_batch = max_batch; c->dtype = dtype;
-  c->pages_per_seq = (max_seq + kPageTokens - 1) / kPageTokens;
-  c->max_seq = c->pages_per_seq * kPageTokens;
-  c->num_pages = c->pages_per_seq * max_batch;
-  const size_t bytes = (size_t)layers * c->layer_stride_elems() * dtype_size(dtype);
-  int st = rb_malloc(ctx, bytes, &c->k);
-  if (st == RB_OK) st = rb_malloc(ctx, bytes, &c->v);
-  if (st == RB_OK) st = rb_malloc(ctx, (size_t)c->num_pages * sizeof(int32_t), (void**)&c->block_table);
-  if (st == RB_OK) st = rb_malloc(ctx, (size_t)max_batch * sizeof(int32_t), (void**)&c->seq_lens);
-  if (st == RB_OK) st = rb_malloc(ctx, (size_t)max_batch * kv_heads * sizeof(uint32_t), (void**)&c->split_count);
-  if (st != RB_OK) { rb_kv_cache_destroy(c); return st; }
-  // Zero the pages: the tail of a sequence's last page is read (and masked) by the attention
-  // kernels, so it must hold finite values.
-  RB_CUDA(cudaMemsetAsync(c->k, 0, bytes, ctx->stream));
-  RB_CUDA(cudaMemsetAsync(c->v, 0, bytes, ctx->stream));
-  std::vector<int32_t> bt(c->num_pages);
-  for (int i = 0; i < c->num_pages; ++i) bt[i] = i;  // sequence b owns pages [b*pages_per_seq, ...)
-  RB_CUDA(cudaMemcpyAsync(c->block_table, bt.data(), bt.size() * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
-  RB_CUDA(cudaMemsetAsync(c->seq_lens, 0, (size_t)max_batch * sizeof(int32_t), ctx->stream));
-  RB_CUDA(cudaMemsetAsync(c->split_count, 0, (size_t)max_batch * kv_heads * sizeof(uint32_t), ctx->stream));
-  RB_CUDA(cudaStreamSynchronize(ctx->stream));
-  c->host_lens.assign(max_batch, 0);
-  ctx->caches.push_back(c);
-  *out = c;
+  return kv_cache_create(ctx, nullptr, layers, kv_heads, head_dim, max_batch, max_seq, dtype, out);
+}
+
+int rb::kv_cache_permute(rb_kv_cache* c, const std::vector<int32_t>& order) {
+  const size_t pp = (size_t)c->pages_per_seq;
+  std::vector<int32_t> table(c->host_table.size()), slots(c->host_slots.size()), lens(c->host_lens.size());
+  for (size_t i = 0; i < order.size(); ++i) {
+    const size_t from = (size_t)order[i];
+    for (size_t j = 0; j < pp; ++j) table[i * pp + j] = c->host_table[from * pp + j];
+    slots[i] = c->host_slots[from];
+    lens[i] = c->host_lens[from];
+  }
+  c->host_table = table; c->host_slots = slots; c->host_lens = lens;
+  cudaStream_t s = c->ctx->stream;
+  RB_CUDA(cudaMemcpyAsync(c->block_table, c->host_table.data(), table.size() * sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  RB_CUDA(cudaMemcpyAsync(c->slots, c->host_slots.data(), slots.size() * sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  RB_CUDA(cudaMemcpyAsync(c->seq_lens, c->host_lens.data(), lens.size() * sizeof(int32_t), cudaMemcpyHostToDevice, s));
+  RB_CUDA(cudaStreamSynchronize(s));
   return RB_OK;
 }
 
@@ -290,8 +327,11 @@ extern "C" int32_t rb_kv_cache_destroy(rb_kv_cache* c) {
     if (*it == c) { c->ctx->caches.erase(it); break; }
   if (c->k) cudaFree(c->k);
   if (c->v) cudaFree(c->v);
-  if (c->block_table) cudaFree(c->block_table);
-  if (c->seq_lens) cudaFree(c->seq_lens);
+  if (!c->tables) {
+    if (c->block_table) cudaFree(c->block_table);
+    if (c->seq_lens) cudaFree(c->seq_lens);
+    if (c->slots) cudaFree(c->slots);
+  }
   if (c->split_count) cudaFree(c->split_count);
   delete c;
   return RB_OK;
@@ -332,7 +372,7 @@ extern "C" int32_t rb_kv_cache_read(rb_kv_cache* c, int32_t layer, int32_t seq, 
   RB_CUDA(cudaStreamSynchronize(c->ctx->stream));
   for (int i = 0; i < n; ++i) {
     const int t = t0 + i;
-    const int page = seq * c->pages_per_seq + t / kPageTokens;  // identity block table
+    const int page = (c->tables ? c->tables : c)->host_table[(size_t)seq * c->pages_per_seq + t / kPageTokens];
     const size_t off = ((size_t)layer * c->layer_stride_elems() +
                         (((size_t)page * c->kv_heads + kv_head) * kPageTokens + t % kPageTokens) * c->head_dim) * es;
     RB_CUDA(cudaMemcpy((char*)k_host + i * row, (char*)c->k + off, row, cudaMemcpyDeviceToHost));
@@ -353,6 +393,21 @@ extern "C" int32_t rb_linear(rb_ctx* ctx, const void* x, const void* w, const vo
   const double es = (double)dtype_size(dtype);
   ProfScope prof(ctx, RB_PROF_GEMM, es * ((double)n * k + (double)m * k + (double)m * n * (residual ? 2 : 1) + (bias ? n : 0)),
                  2.0 * m * n * k);
+  if (dtype == RB_BF16 && !ctx->debug_simple_gemm) return gemm_tc_bf16(ctx, a);
+  return gemm_simple(ctx, a, dtype);
+}
+
+extern "C" int32_t rb_linear_act(rb_ctx* ctx, const void* x, const void* w, const void* bias, void* out, int64_t m, int64_t n,
+                                 int64_t k, int32_t act, const void* act_params, int32_t dtype) {
+  RB_REQUIRE(ctx && x && w && out, "rb_linear_act: null argument");
+  RB_REQUIRE(m >= 0 && n > 0 && k > 0, "rb_linear_act: bad sizes");
+  RB_REQUIRE(act != RB_ACT_XIELU || act_params, "rb_linear_act: the activation needs its parameters");
+  GemmArgs a;
+  a.x = x; a.w = w; a.bias = bias; a.out = out;
+  a.m = m; a.n = n; a.k = k; a.act = act; a.act_params = act_params;
+  a.reduce = ctx->gemm_reduce;
+  const double es = (double)dtype_size(dtype);
+  ProfScope prof(ctx, RB_PROF_GEMM, es * ((double)n * k + (double)m * k + (double)m * n), 2.0 * m * n * k);
   if (dtype == RB_BF16 && !ctx->debug_simple_gemm) return gemm_tc_bf16(ctx, a);
   return gemm_simple(ctx, a, dtype);
 }
@@ -442,4 +497,38 @@ extern "C" int32_t rb_attention(rb_ctx* ctx, const void* q, rb_kv_cache* c, int3
                  es * (2.0 * kv_tokens * c->kv_heads * d + 2.0 * batch * s_new * q_heads * d), 4.0 * pairs * q_heads * d);
   if (dtype == RB_BF16 && !ctx->debug_simple_attn) return attention_mma_bf16(ctx, q, c, layer, batch, s_new, q_heads, scale, out);
   return attention_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype);
+}
+
+extern "C" int32_t rb_attention_window(rb_ctx* ctx, const void* q, rb_kv_cache* c, int32_t layer, int32_t batch, int32_t s_new,
+                                       int32_t q_heads, int32_t value_dim, float scale, int32_t window, int32_t alibi,
+                                       const void* gate, int64_t gate_ld, void* out, int64_t out_ld, int32_t dtype) {
+  RB_REQUIRE(ctx && q && c && out, "rb_attention_window: null argument");
+  RB_REQUIRE(dtype == c->dtype, "rb_attention_window: cache dtype differs");
+  RB_REQUIRE(layer >= 0 && layer < c->layers, "rb_attention_window: layer %d out of range", layer);
+  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0, "rb_attention_window: bad batch/seq");
+  RB_REQUIRE(q_heads > 0 && q_heads % c->kv_heads == 0, "rb_attention_window: %d query heads over %d KV heads", q_heads, c->kv_heads);
+  RB_REQUIRE(value_dim > 0 && value_dim <= c->head_dim, "rb_attention_window: value size %d of a %d-wide cache", value_dim, c->head_dim);
+  RB_REQUIRE(window >= 0 && window <= (1 << 30), "rb_attention_window: bad window %d", window);
+  RB_REQUIRE(scale > 0.f, "rb_attention_window: the scale must be positive");
+  RB_REQUIRE(out_ld >= (int64_t)q_heads * value_dim && (out_ld % 8) == 0 && (!gate || (gate_ld % 8) == 0),
+             "rb_attention_window: row pitches must be multiples of 8 and hold every head");
+  double kv_tokens = 0.0, pairs = 0.0;  // keys read; visible (query, key) pairs
+  for (int b = 0; b < batch; ++b) {
+    RB_REQUIRE(c->host_lens[b] >= s_new, "rb_attention_window: sequence %d holds %d tokens, fewer than the %d new ones", b,
+               c->host_lens[b], s_new);
+    const double len = c->host_lens[b], base = len - s_new, w = window > 0 ? window : 1e18;
+    kv_tokens += window > 0 ? (len < w + s_new - 1 ? len : w + s_new - 1) : len;
+    // sum over the new rows i of min(i + 1, w)
+    const double full = base + 1 >= w ? s_new : (len <= w ? 0.0 : len - w);
+    const double grow = s_new - full;
+    pairs += (full > 0 ? full * w : 0.0) + grow * (base + 1) + 0.5 * grow * (grow - 1.0);
+  }
+  AttnExtra x;
+  x.window = window; x.alibi = alibi != 0; x.gate = gate; x.gate_ld = gate_ld; x.value_dim = value_dim; x.out_ld = out_ld;
+  const double es = (double)dtype_size(dtype), d = c->head_dim;
+  ProfScope prof(ctx, RB_PROF_ATTENTION,
+                 es * (2.0 * kv_tokens * c->kv_heads * d + (gate ? 3.0 : 2.0) * batch * s_new * q_heads * d), 4.0 * pairs * q_heads * d);
+  if (!ctx->debug_simple_attn && attention_mma_takes(c, q_heads))
+    return attention_mma_bf16(ctx, q, c, layer, batch, s_new, q_heads, scale, out, &x);
+  return attention_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, &x);
 }

@@ -109,6 +109,10 @@ struct AParams {
   float* part_ml;  // [batch*q_heads][n_splits][2]
   uint32_t* split_count;  // [batch][kv_heads] arrivals; non-null: the last split block of a (sequence, KV head) merges
   uint32_t* status;
+  // Beyond the plain causal form (the EXT instantiations; see AttnExtra)
+  int x_window, x_alibi, x_value_dim;  // x_window: 2^30 = none
+  const bf16* x_gate;
+  int64_t x_gate_ld, x_out_ld;
   // Fused single-token step (decode, tiled-copy path): the new token's q, k and v are taken straight from
   // the q/k/v projection's output (bf16 rows and/or float32 split-K partials, plus bias), rotated, and the
   // k/v rows appended to the cache by this kernel, which then needs no separate RoPE/append launch and
@@ -126,7 +130,15 @@ struct AParams {
   bf16* f_v;
 };
 
-template <int D, bool DECODE, bool TMA>
+// EXT output: element dd of head `head` in row `row` of the packed output, gated
+__device__ __forceinline__ void store_ext(const AParams& p, size_t row, int head, int dd, float v) {
+  if (dd >= p.x_value_dim) return;
+  const int col = head * p.x_value_dim + dd;
+  if (p.x_gate) v *= sigmoid_f(__bfloat162float(p.x_gate[row * p.x_gate_ld + col]));
+  p.out[row * p.x_out_ld + col] = __float2bfloat16_rn(v);
+}
+
+template <int D, bool DECODE, bool TMA, bool EXT>
 __global__ void __launch_bounds__(128, (D <= 128) ? 2 : 1)
 attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v) {
   using C = ACfg<D, DECODE, TMA>;
@@ -170,15 +182,17 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
   // key tiles this CTA walks
   int tile_lo, tile_hi;
   if (DECODE) {
+    const int first = EXT ? max(0, len - p.x_window) / kTile : 0;  // tiles wholly outside the rolling window are not walked
     const int total = (len + kTile - 1) / kTile;
-    const int per = (total + p.n_splits - 1) / p.n_splits;
-    tile_lo = split * per;
+    const int per = (total - first + p.n_splits - 1) / p.n_splits;
+    tile_lo = first + split * per;
     tile_hi = min(total, tile_lo + per);
   } else {
     // The reference's window term acts among the tokens of ONE call only (qwen2.rs:316-334: the mask block of the
     // cached prefix is all zeros, and a single-token call builds no mask at all, qwen2.rs:340-342), so whole tiles
     // can be skipped only when nothing is cached.
-    tile_lo = base == 0 ? max(0, q0 - p.window) / kTile : 0;
+    if (EXT) tile_lo = max(0, base + q0 - p.x_window + 1) / kTile;
+    else tile_lo = base == 0 ? max(0, q0 - p.window) / kTile : 0;
     tile_hi = (min(base + q0 + 64, len) + kTile - 1) / kTile;
   }
   if (fuse && (len < 1 || len > p.f_max_seq)) {  // the same guard the separate RoPE/append kernel has
@@ -339,6 +353,11 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
   if (DECODE) { lim[0] = lim[1] = len - 1; }
   else { lim[0] = base + q0 + qrow0 + g; lim[1] = lim[0] + 8; }
 
+  float slope2[2] = {0.f, 0.f};  // distance bias per row half, in log2 units
+  if (EXT && p.x_alibi) {
+    slope2[0] = alibi_slope(DECODE ? head + g : head, p.q_heads) * kLog2e;
+    slope2[1] = DECODE ? alibi_slope(head + g + 8, p.q_heads) * kLog2e : slope2[0];
+  }
   bool q_loaded = false;
   bool aborted = false;
   for (int tile = tile_lo; tile < tile_hi; ++tile) {
@@ -406,8 +425,16 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
           const int key_abs = tile_start + kw0 + nt * 8 + 2 * t + (e & 1);
           const int hf = e >> 1;
           // causal limit (lim is the row's own position) and, among the new tokens only, the sliding window
-          const bool seen = key_abs <= lim[hf] && (DECODE || key_abs < base || key_abs + p.window >= lim[hf]);
-          const float v = seen ? s[nt][e] * p.scale_log2 : -INFINITY;
+          bool seen;
+          float score = s[nt][e] * p.scale_log2;
+          if (EXT) {  // rolling window, in prompts and single-token steps alike; then the distance bias
+            const int dist = lim[hf] - key_abs;
+            seen = dist >= 0 && dist < p.x_window;
+            score = fmaf(-slope2[hf], (float)dist, score);
+          } else {
+            seen = key_abs <= lim[hf] && (DECODE || key_abs < base || key_abs + p.window >= lim[hf]);
+          }
+          const float v = seen ? score : -INFINITY;
           s[nt][e] = v;
           mx[hf] = fmaxf(mx[hf], v);
         }
@@ -477,6 +504,14 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
       const int row = q0 + qrow0 + g + hf * 8;
       if (row >= p.s_new) continue;
       const float inv = 1.0f / l_run[hf];
+      if (EXT) {
+#pragma unroll
+        for (int i = 0; i < D / 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+            store_ext(p, (size_t)b * p.s_new + row, head, i * 8 + 2 * t + e, o[i][hf * 2 + e] * inv);
+        continue;
+      }
       bf16* dst = p.out + (((size_t)b * p.s_new + row) * p.q_heads + head) * D;
 #pragma unroll
       for (int i = 0; i < D / 8; ++i)
@@ -516,7 +551,8 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     }
     const size_t bh = (size_t)b * p.q_heads + head + row;
     if (p.n_splits == 1) {
-      p.out[bh * D + dd] = __float2bfloat16_rn(O / L);
+      if (EXT) store_ext(p, b, head + row, dd, O / L);
+      else p.out[bh * D + dd] = __float2bfloat16_rn(O / L);
     } else {
       p.part_o[(bh * p.n_splits + split) * D + dd] = O;
       if (dd == 0) { p.part_ml[(bh * p.n_splits + split) * 2] = M; p.part_ml[(bh * p.n_splits + split) * 2 + 1] = L; }
@@ -573,7 +609,8 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
       for (int k = 0; k < 8; ++k)
         if (s0 + k < ns) O += t[k] * w_s[row * 32 + s0 + k];
     }
-    p.out[bh * D + dd] = __float2bfloat16_rn(O / w_s[1024 + row]);
+    if (EXT) store_ext(p, b, head + row, dd, O / w_s[1024 + row]);
+    else p.out[bh * D + dd] = __float2bfloat16_rn(O / w_s[1024 + row]);
   }
 }
 
@@ -597,11 +634,11 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
 }
 
 // Launches attention_kernel<D, DECODE> with tiled-copy loading when the head size allows it.
-template <int D, bool DECODE>
+template <int D, bool DECODE, bool EXT = false>
 int launch_attn_kernel(rb_ctx* ctx, rb_kv_cache* c, const AParams& p, dim3 grid) {
   constexpr bool kTma = (D % 64) == 0;
   using C = ACfg<D, DECODE, kTma>;
-  auto kern = attention_kernel<D, DECODE, kTma>;
+  auto kern = attention_kernel<D, DECODE, kTma, EXT>;
   static bool set[64] = {};  // the attribute belongs to the (kernel, device) pair
   const int dv = ctx->device & 63;
   if (!set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes)); set[dv] = true; }
@@ -617,12 +654,12 @@ int launch_attn_kernel(rb_ctx* ctx, rb_kv_cache* c, const AParams& p, dim3 grid)
   return RB_OK;
 }
 
-template <int D>
+template <int D, bool EXT = false>
 int launch_attention(rb_ctx* ctx, rb_kv_cache* c, AParams& p, int batch, int max_len) {
   if (p.s_new > 1) {
     dim3 grid((unsigned)((p.s_new + 63) / 64), (unsigned)p.q_heads, (unsigned)batch);
     p.n_splits = 1;
-    return launch_attn_kernel<D, false>(ctx, c, p, grid);
+    return launch_attn_kernel<D, false, EXT>(ctx, c, p, grid);
   }
   // Split the keys of a sequence over several blocks only when (sequence, KV head) pairs alone leave
   // the GPU under-filled: one long block per pair keeps its copy pipeline full and needs no merge.
@@ -635,8 +672,8 @@ int launch_attention(rb_ctx* ctx, rb_kv_cache* c, AParams& p, int batch, int max
   }
   dim3 grid((unsigned)splits, (unsigned)p.kv_heads, (unsigned)batch);
   static const bool separate_merge = getenv("RAI_B200_ATTN_MERGE_KERNEL") != nullptr;  // debugging aid
-  p.split_count = (splits > 1 && !separate_merge) ? c->split_count : nullptr;
-  RB_TRY((launch_attn_kernel<D, true>(ctx, c, p, grid)));
+  p.split_count = (splits > 1 && (EXT || !separate_merge)) ? c->split_count : nullptr;
+  RB_TRY((launch_attn_kernel<D, true, EXT>(ctx, c, p, grid)));
   if (splits > 1 && !p.split_count) {
     RB_CUDA(launch_kernel(attention_merge_kernel, dim3((unsigned)(batch * p.q_heads)), dim3(128), 0, ctx->stream, ctx->pdl,
                           (const float*)p.part_o, (const float*)p.part_ml, splits, D, p.out));
@@ -709,8 +746,14 @@ int attention_decode_splits(rb_ctx* ctx, int batch, int kv_heads, int max_len, i
   return best;
 }
 
+bool attention_mma_takes(const rb_kv_cache* c, int q_heads) {
+  const int d = c->head_dim;
+  return c->dtype == RB_BF16 && (d == 64 || d == 80 || d == 96 || d == 128 || d == 256) && q_heads % c->kv_heads == 0 &&
+         q_heads / c->kv_heads <= 16;
+}
+
 int attention_mma_bf16(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
-                       float scale, void* out) {
+                       float scale, void* out, const AttnExtra* ext) {
   AParams p{};
   const size_t loff = (size_t)layer * c->layer_stride_elems();
   p.q = (const bf16*)q;
@@ -732,9 +775,26 @@ int attention_mma_bf16(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, in
              "attention: %d query heads per KV head unsupported (1..16)", p.group);
   // prefill with at least one 128-row query tile and head size 64 or 128: the tcgen05 kernel
   if (ctx->attn_tc && attention_prefill_tc_supported(c, s_new, q_heads, q, out))
-    return attention_prefill_tc(ctx, q, c, layer, batch, s_new, q_heads, scale, out);
+    return attention_prefill_tc(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
   int max_len = 0;
   for (int b = 0; b < batch; ++b) max_len = std::max(max_len, c->host_lens[b]);
+  if (ext) {
+    p.x_window = ext->window > 0 ? ext->window : (1 << 30);
+    p.x_alibi = ext->alibi;
+    p.x_value_dim = ext->value_dim;
+    p.x_gate = (const bf16*)ext->gate;
+    p.x_gate_ld = ext->gate_ld;
+    p.x_out_ld = ext->out_ld;
+    max_len = attention_walk_len(max_len, ext->window);
+    switch (c->head_dim) {
+      case 64: return launch_attention<64, true>(ctx, c, p, batch, max_len);
+      case 80: return launch_attention<80, true>(ctx, c, p, batch, max_len);
+      case 96: return launch_attention<96, true>(ctx, c, p, batch, max_len);
+      case 128: return launch_attention<128, true>(ctx, c, p, batch, max_len);
+      case 256: return launch_attention<256, true>(ctx, c, p, batch, max_len);
+    }
+    return fail(RB_ERR_UNIMPLEMENTED, "attention: head_dim %d has no tensor-core kernel (64, 80, 96, 128, 256)", c->head_dim);
+  }
   switch (c->head_dim) {
     case 64: return launch_attention<64>(ctx, c, p, batch, max_len);
     case 80: return launch_attention<80>(ctx, c, p, batch, max_len);

@@ -69,6 +69,10 @@ struct TParams {
   bf16* out;
   uint32_t* status;
   long long wait_cycles;
+  // the EXT instantiation (see AttnExtra): rolling window (2^30 = none), distance bias, gated and packed output
+  int x_window, x_alibi, x_value_dim;
+  const bf16* x_gate;
+  int64_t x_gate_ld, x_out_ld;
 #ifdef RB_DEBUG_AIDS
   unsigned long long* trace;  // developer build: cycles per phase of one softmax thread (see launch_tc)
 #endif
@@ -88,7 +92,7 @@ struct Ctrl {  // lives in dynamic shared memory behind the tiles
 };
 static_assert(sizeof(Ctrl) <= 256, "control block exceeds its reservation");
 
-template <int D>
+template <int D, bool EXT>
 __global__ void __launch_bounds__(kThreads, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                             const __grid_constant__ CUtensorMap tm_v, const TParams p) {
@@ -136,7 +140,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   const int base = len - p.s_new;  // absolute position of query row 0
   // Key tiles this CTA walks.  The window term acts among the tokens of one call only (qwen2.rs:316-334), so whole
   // tiles can be skipped only when nothing is cached.
-  const int tile_lo = base == 0 ? max(0, q0 - p.window) / kBN : 0;
+  const int tile_lo = EXT ? max(0, base + q0 - p.x_window + 1) / kBN : base == 0 ? max(0, q0 - p.window) / kBN : 0;
   const int tile_hi = (min(base + q0 + kBM, len) + kBN - 1) / kBN;
   const int n = tile_hi - tile_lo;
   // The tiles must sit on a 1024-byte boundary (swizzle atoms); nothing else lives in shared memory before them.
@@ -222,7 +226,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     const int row = quarter * 32 + lane;      // query row inside the tile
     const int row_abs = base + q0 + row;      // its absolute position = its causal limit
     const uint32_t t_row = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    const bool windowed = p.window < (1 << 30);
+    const bool windowed = EXT ? p.x_window < (1 << 30) : p.window < (1 << 30);
+    const float slope2 = EXT && p.x_alibi ? alibi_slope(head, p.q_heads) * kLog2e : 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
 #ifdef RB_DEBUG_AIDS
@@ -254,12 +259,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // mask (only tiles that the causal diagonal or the window actually cuts), then the row max over the raw scores;
       // the scale is positive, so it commutes with the max and rides in the exponent's multiply-add below
       const bool causal_edge = key0 + kBN - 1 > base + q0;
-      const bool window_edge = windowed && key0 + kBN > base && base + q0 + kBM - 1 - p.window > key0;
+      const bool window_edge = EXT ? windowed && base + q0 + kBM - 1 - key0 >= p.x_window
+                                   : windowed && key0 + kBN > base && base + q0 + kBM - 1 - p.window > key0;
+      if (EXT) {  // log2-scaled score less the distance bias; what follows then needs no scale of its own
+        const float b0 = slope2 * (float)(key0 - row_abs);
+#pragma unroll
+        for (int i = 0; i < kBN; ++i) s[i] = fmaf(s[i], p.scale_log2, fmaf(slope2, (float)i, b0));
+      }
       if (causal_edge || window_edge) {
 #pragma unroll
         for (int i = 0; i < kBN; ++i) {
           const int key = key0 + i;
-          const bool seen = key <= row_abs && (key < base || key + p.window >= row_abs);
+          const bool seen = EXT ? key <= row_abs && row_abs - key < p.x_window
+                                : key <= row_abs && (key < base || key + p.window >= row_abs);
           s[i] = seen ? s[i] : -INFINITY;
         }
       }
@@ -269,7 +281,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         mx4[0] = fmaxf(mx4[0], s[i]); mx4[1] = fmaxf(mx4[1], s[i + 1]);
         mx4[2] = fmaxf(mx4[2], s[i + 2]); mx4[3] = fmaxf(mx4[3], s[i + 3]);
       }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+      const float unit = EXT ? 1.0f : p.scale_log2;
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * unit;
       // The reference point of the exponentials follows the running max lazily: it moves only when the max has grown
       // by more than 2^kSlack since it was last set.  softmax is invariant to the reference point (numerator and
       // denominator carry the same factor), the terms stay below 2^kSlack, well inside float32 and bf16 range, and the
@@ -283,8 +296,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       uint32_t packed[kBN / 2];
 #pragma unroll
       for (int i = 0; i < kBN; i += 4) {
-        const float p0 = ex2_fast(fmaf(s[i], p.scale_log2, -m_use)), p1 = ex2_fast(fmaf(s[i + 1], p.scale_log2, -m_use));
-        const float p2 = ex2_fast(fmaf(s[i + 2], p.scale_log2, -m_use)), p3 = ex2_fast(fmaf(s[i + 3], p.scale_log2, -m_use));
+        const float p0 = ex2_fast(fmaf(s[i], unit, -m_use)), p1 = ex2_fast(fmaf(s[i + 1], unit, -m_use));
+        const float p2 = ex2_fast(fmaf(s[i + 2], unit, -m_use)), p3 = ex2_fast(fmaf(s[i + 3], unit, -m_use));
         sum4[0] += p0; sum4[1] += p1; sum4[2] += p2; sum4[3] += p3;
         __nv_bfloat162 h0 = __floats2bfloat162_rn(p0, p1), h1 = __floats2bfloat162_rn(p2, p3);
         packed[i >> 1] = *reinterpret_cast<uint32_t*>(&h0);
@@ -341,7 +354,36 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         uint32_t r[32];
         ptx::tmem_ld_32x32(t_row + C::kOCol + (uint32_t)c0, r);
         ptx::tmem_wait_ld();
-        if (store) {
+        if (EXT && store) {
+          const size_t m = (size_t)b * p.s_new + q0 + row;
+          const int vd = p.x_value_dim, col0 = head * vd;
+          bf16* xo = p.out + m * p.x_out_ld + col0;
+          const bf16* xg = p.x_gate ? p.x_gate + m * p.x_gate_ld + col0 : nullptr;
+          if ((vd & 7) == 0) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 8) {
+              if (c0 + i >= vd) break;
+              float v[8];
+#pragma unroll
+              for (int k = 0; k < 8; ++k) v[k] = __uint_as_float(r[i + k]) * inv;
+              if (xg) {
+                float gt[8];
+                load8(xg + c0 + i, gt);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) v[k] = __fdividef(v[k], 1.0f + __expf(-gt[k]));
+              }
+              *reinterpret_cast<uint4*>(xo + c0 + i) = pack8_bf16(v);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (c0 + i < vd) {
+                float v = __uint_as_float(r[i]) * inv;
+                if (xg) v = __fdividef(v, 1.0f + __expf(-__bfloat162float(xg[c0 + i])));
+                xo[c0 + i] = __float2bfloat16_rn(v);
+              }
+          }
+        } else if (store) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             float v[8];
@@ -376,8 +418,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   }
 }
 
-template <int D>
-int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out) {
+template <int D, bool EXT>
+int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+              const AttnExtra* ext) {
   using C = TCfg<D>;
   const size_t loff = (size_t)layer * c->layer_stride_elems();
   const bf16* kbase = (const bf16*)c->k + loff;
@@ -389,7 +432,7 @@ int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, 
   const int64_t rows = (int64_t)c->num_pages * c->kv_heads * kBN;
   RB_TRY(tmap_2d_bf16(ctx, kbase, rows, D, D, kBN, &tk));
   RB_TRY(tmap_2d_bf16(ctx, vbase, rows, D, D, kBN, &tv));
-  auto kern = attention_prefill_tc_kernel<D>;
+  auto kern = attention_prefill_tc_kernel<D, EXT>;
   static bool set[64] = {};  // the attribute belongs to the (kernel, device) pair
   const int dv = ctx->device & 63;
   if (!set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes)); set[dv] = true; }
@@ -406,6 +449,14 @@ int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, 
   p.out = (bf16*)out;
   p.status = ctx->status_dev;
   p.wait_cycles = ctx->local_wait_cycles();
+  if (EXT) {
+    p.x_window = ext->window > 0 ? ext->window : (1 << 30);
+    p.x_alibi = ext->alibi;
+    p.x_value_dim = ext->value_dim;
+    p.x_gate = (const bf16*)ext->gate;
+    p.x_gate_ld = ext->gate_ld;
+    p.x_out_ld = ext->out_ld;
+  }
   dim3 grid((unsigned)((s_new + kBM - 1) / kBM), (unsigned)q_heads, (unsigned)batch);
 #ifdef RB_DEBUG_AIDS
   static const bool trace = getenv("RAI_B200_ATTN_TRACE") != nullptr;
@@ -443,9 +494,11 @@ bool attention_prefill_tc_supported(const rb_kv_cache* c, int s_new, int q_heads
 }
 
 int attention_prefill_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
-                         void* out) {
-  if (c->head_dim == 64) return launch_tc<64>(ctx, q, c, layer, batch, s_new, q_heads, scale, out);
-  if (c->head_dim == 128) return launch_tc<128>(ctx, q, c, layer, batch, s_new, q_heads, scale, out);
+                         void* out, const AttnExtra* ext) {
+  if (ext && c->head_dim == 64) return launch_tc<64, true>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
+  if (ext && c->head_dim == 128) return launch_tc<128, true>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
+  if (c->head_dim == 64) return launch_tc<64, false>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, nullptr);
+  if (c->head_dim == 128) return launch_tc<128, false>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, nullptr);
   return fail(RB_ERR_UNIMPLEMENTED, "tensor-core prefill attention: head_dim %d unsupported (64, 128)", c->head_dim);
 }
 

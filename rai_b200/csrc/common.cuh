@@ -183,10 +183,27 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
+// log(1 + e^z) without overflow
+__device__ __forceinline__ float softplus_f(float z) { return log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f); }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// RB_ACT_XIELU: z/2 plus a curve, a z^2 for positive z and b (expm1(z) - z) otherwise; these are a and b from the two
+// learned numbers
+template <typename T>
+__device__ __forceinline__ float2 xielu_consts(const T* pq) {
+  return make_float2(softplus_f(Cvt<T>::to_f(pq[0])), 0.5f + softplus_f(Cvt<T>::to_f(pq[1])));
+}
+__device__ __forceinline__ float xielu_f(float z, float2 c) {
+  return z > 0.f ? fmaf(c.x * z, z, 0.5f * z) : fmaf(c.y, expm1f(z) - z, 0.5f * z);
+}
+
 // Activation tags shared by the GEMM epilogues and the elementwise kernels
 // (rai-core/src/hlops/activations.rs:20-32).
-__device__ __forceinline__ float act_apply(int act, float x) {
+// `c` holds the constants of an activation that has any (RB_ACT_XIELU).
+__device__ __forceinline__ float act_apply(int act, float x, float2 c = make_float2(0.f, 0.f)) {
   switch (act) {
+    case RB_ACT_XIELU: return xielu_f(x, c);
     case RB_ACT_SILU: return x / (__expf(-x) + 1.0f);
     case RB_ACT_GELU_TANH: {
       const float c = 0.7978845608028654f;

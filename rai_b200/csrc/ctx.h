@@ -35,6 +35,8 @@ struct rb_ctx {
   // argmax across blocks: running best (key << 32 | index) and arrival count per row; self-resetting
   unsigned long long* argmax_best = nullptr;
   unsigned int* argmax_count = nullptr;
+  float* chunk_scratch = nullptr;   // states between the pieces of a recurrence that is run piecewise; grow-only
+  size_t chunk_scratch_bytes = 0;
   // split-KV partials of the decode attention: grown on demand, owned by the context (one stream at a time)
   bool pool_ready = false;  // the device's default memory pool has been told to keep freed blocks
   float* attn_scratch = nullptr;
@@ -52,7 +54,15 @@ struct rb_ctx {
 };
 
 // Pages of 64 tokens.  K and V each: [layer][page][kv_head][64][head_dim] in the cache dtype.
+//
+// A design whose layers differ in head counts or sizes has one cache per geometry over ONE set of sequences: the
+// first owns the tables (block table, lengths, state slots), the others are views that share them (`tables`).  A
+// cache with layers == 0 is only the tables.
 struct rb_kv_cache {
+  explicit rb_kv_cache(rb_kv_cache* shared = nullptr)
+      : tables(shared), host_lens(shared ? shared->host_lens : own_lens) {}
+  rb_kv_cache* tables = nullptr;   // the cache whose tables this one uses; null = its own
+  std::vector<int32_t> own_lens;
   rb_ctx* ctx = nullptr;
   int layers = 0, kv_heads = 0, head_dim = 0, max_batch = 0, max_seq = 0, dtype = RB_BF16;
   int pages_per_seq = 0, num_pages = 0;
@@ -61,8 +71,10 @@ struct rb_kv_cache {
   void* v = nullptr;
   int32_t* block_table = nullptr;  // device [max_batch][pages_per_seq]
   int32_t* seq_lens = nullptr;     // device [max_batch]
+  int32_t* slots = nullptr;        // device [max_batch]: where sequence b keeps its recurrent and convolution state
+  std::vector<int32_t> host_table, host_slots;  // host copies of block_table and slots
   uint32_t* split_count = nullptr;  // device [max_batch][kv_heads]: arrivals of a split decode attention; self-resetting
-  std::vector<int32_t> host_lens;
+  std::vector<int32_t>& host_lens;
   size_t layer_stride_elems() const { return (size_t)num_pages * kv_heads * 64 * head_dim; }
 };
 
@@ -97,6 +109,11 @@ struct TpPeers {
 };
 
 namespace rb {
+// api.cu: layers >= 0; `shared` makes a view over another cache's sequences (max_batch and max_seq are then its)
+int kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_heads, int head_dim, int max_batch, int max_seq, int dtype,
+                    rb_kv_cache** out);
+// sequences order[0 .. max_batch) (a permutation) become 0, 1, ...: pages, slots and lengths move with them
+int kv_cache_permute(rb_kv_cache* c, const std::vector<int32_t>& order);
 constexpr int kPageTokens = 64;
 constexpr int kArgmaxRows = 4096;  // rows one argmax launch can reduce across blocks
 
@@ -131,6 +148,7 @@ struct GemmArgs {
   void* out = nullptr;          // [M, N] (model dtype) or float partials [n_split][M][N]
   int64_t m = 0, n = 0, k = 0;
   int act = RB_ACT_NONE;
+  const void* act_params = nullptr;  // RB_ACT_XIELU: its two numbers, model dtype
   int n_split = 1;              // > 1: write float partials, no epilogue
   bool partials = false;
   bool reduce = false;            // M <= 64: if K is split, sum the splits inside the kernel and apply the epilogue
@@ -140,8 +158,21 @@ int gemm_tc_pick_splits(rb_ctx* ctx, int64_t m, int64_t n, int64_t k);
 int gemm_reserve_scratch(rb_ctx* ctx, size_t bytes);
 int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype);
 
+// What an attention layer may have beyond the plain causal form.
+struct AttnExtra {
+  int window = 0;              // rolling window: how many keys, its own included, a row sees; 0 = all
+  bool alibi = false;          // distance bias: 2^(-8 (h + 1) / q_heads) * (i - j) off the score of head h
+  const void* gate = nullptr;  // out *= sigmoid(gate), model dtype, row pitch gate_ld
+  int64_t gate_ld = 0;
+  int value_dim = 0;           // columns of a head that are stored (the cache may hold padded heads)
+  int64_t out_ld = 0;          // row pitch of the output
+};
+// slope of the distance bias, 2^(-8 (h + 1) / heads)
+__device__ __forceinline__ float alibi_slope(int head, int heads) { return exp2f(-8.0f * (float)(head + 1) / (float)heads); }
+
 int attention_mma_bf16(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
-                       float scale, void* out);
+                       float scale, void* out, const AttnExtra* ext = nullptr);
+bool attention_mma_takes(const rb_kv_cache* c, int q_heads);
 // decoder_kernels.cu: the tensor-parallel sum of a row-parallel product (split-K slabs + bias, or a finished bf16
 // tensor `part`) over the exchange buffers, the residual add and the following norm, in one kernel.
 // sum_out = h + sum over ranks; out = norm(sum_out) (out may be NULL).  `parity` alternates 0,1,0,1.. launch by launch.
@@ -150,7 +181,7 @@ int exchange_norm(rb_ctx* ctx, const TpPeers& tp, int parity, int kind, const vo
                   int64_t hidden, void* out, void* sum_out);
 // decoder_kernels.cu: out[r, j] = act(sum_s part[s][r][j] + bias[j]) (* sum_s part[s][r][j + n_out] when gated)
 int act_from_partials(rb_ctx* ctx, const float* part, int n_split, int64_t rows, int64_t n_all, int64_t n_out, bool gated,
-                      const void* bias, int act, void* out);
+                      const void* bias, int act, void* out, const void* act_params = nullptr);
 // Single-token step with the RoPE / KV-append work folded into the decode attention kernel (bf16 caches,
 // head sizes that are multiples of 64).  `attention_can_fuse_rope` says whether the shapes and pointers allow it.
 bool attention_can_fuse_rope(const rb_kv_cache* c, int q_heads, int rot, const void* qkv, const float* acc, int n_acc,
@@ -159,11 +190,13 @@ int attention_decode_fused_rope(rb_ctx* ctx, const void* qkv, const float* acc, 
                                 const float* cos_t, const float* sin_t, int rot, rb_kv_cache* c, int layer, int batch,
                                 int q_heads, float scale, void* out);
 int attention_decode_splits(rb_ctx* ctx, int batch, int kv_heads, int max_len, int head_dim);
+// keys a single-token step may have to walk under a rolling window, for the split decision above
+inline int attention_walk_len(int max_len, int window) { return (window > 0 && window < max_len - 64) ? window + 64 : max_len; }
 int attention_reserve_scratch(rb_ctx* ctx, size_t bytes);
 // attention_tc.cu: causal prefill attention on tcgen05 (head sizes 64 and 128, query length >= 128)
 bool attention_prefill_tc_supported(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const void* out);
 int attention_prefill_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
-                         void* out);
+                         void* out, const AttnExtra* ext = nullptr);
 int attention_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
-                     float scale, void* out, int dtype);
+                     float scale, void* out, int dtype, const AttnExtra* ext = nullptr);
 }  // namespace rb

@@ -541,8 +541,10 @@ __global__ void __launch_bounds__(512) exchange_norm_kernel(int kind, const T* _
 // product (qwen2.rs:101-103).  8 outputs per thread.
 __global__ void act_from_partials_kernel(const float* __restrict__ part, int n_split, size_t slab, int n_all, int n_out,
                                          int gated, const __nv_bfloat16* __restrict__ bias, int act,
-                                         __nv_bfloat16* __restrict__ out, int64_t total_chunks) {
+                                         const __nv_bfloat16* __restrict__ act_params, __nv_bfloat16* __restrict__ out,
+                                         int64_t total_chunks) {
   pdl_launch_dependents();
+  const float2 ac = act == RB_ACT_XIELU ? xielu_consts(act_params) : make_float2(0.f, 0.f);
   pdl_wait();
   const int chunks_per_row = n_out >> 3;
   for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total_chunks; i += (int64_t)gridDim.x * blockDim.x) {
@@ -565,7 +567,7 @@ __global__ void act_from_partials_kernel(const float* __restrict__ part, int n_s
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       // gate and up are tensors of the model dtype before the product in the reference; round like the fused kernel does not
-      const float a = act_apply(act, g[k]);
+      const float a = act_apply(act, g[k], ac);
       g[k] = gated ? a * u[k] : a;
     }
     store8(out + (size_t)r * n_out + j, g);
@@ -970,14 +972,14 @@ int exchange_norm(rb_ctx* ctx, const TpPeers& tp, int parity, int kind, const vo
 }
 
 int act_from_partials(rb_ctx* ctx, const float* part, int n_split, int64_t rows, int64_t n_all, int64_t n_out, bool gated,
-                      const void* bias, int act, void* out) {
+                      const void* bias, int act, void* out, const void* act_params) {
   RB_REQUIRE(part && out && rows > 0 && n_out > 0 && (n_out % 8) == 0 && (n_all % 4) == 0, "act_from_partials: bad shape");
   ProfScope prof(ctx, RB_PROF_OTHER, (double)rows * (4.0 * n_split * n_all + 2.0 * n_out), 0.0);
   const int64_t chunks = rows * (n_out / 8);
   const int blocks = (int)std::min<int64_t>((chunks + 127) / 128, 8 * ctx->sm_count);
   RB_CUDA(launch_kernel(act_from_partials_kernel, dim3((unsigned)blocks), dim3(128), 0, ctx->stream, ctx->pdl, part, n_split,
                         (size_t)rows * n_all, (int)n_all, (int)n_out, gated ? 1 : 0, (const __nv_bfloat16*)bias, act,
-                        (__nv_bfloat16*)out, chunks));
+                        (const __nv_bfloat16*)act_params, (__nv_bfloat16*)out, chunks));
   ctx->launches++;
   return RB_OK;
 }

@@ -83,6 +83,7 @@ struct Params {
   bf16* out;
   float* part;
   int act;
+  const bf16* act_params;  // RB_ACT_XIELU
   int stages;           // ring depth of this launch, 2..Cfg::kStages
   int reduce;           // split-K reduced inside the kernel: the splits of a tile wait for one another (see the epilogue)
   uint32_t* tile_count; // reduce: arrivals per tile, and readers done per tile; both self-resetting
@@ -152,7 +153,7 @@ __device__ __forceinline__ float tanh_fast(float x) {
 // Activation over a register array with the selector hoisted out of the element loop
 // (rai-core/src/hlops/activations.rs:20-32); fast-math forms, results are rounded to bf16 anyway.
 template <int N>
-__device__ __forceinline__ void act_inplace(int act, float (&v)[N]) {
+__device__ __forceinline__ void act_inplace(int act, float (&v)[N], float2 ac) {
   if (act == RB_ACT_SILU) {
 #pragma unroll
     for (int i = 0; i < N; ++i) v[i] = __fdividef(v[i], 1.0f + __expf(-v[i]));
@@ -168,6 +169,13 @@ __device__ __forceinline__ void act_inplace(int act, float (&v)[N]) {
   } else if (act == RB_ACT_RELU) {
 #pragma unroll
     for (int i = 0; i < N; ++i) v[i] = fmaxf(v[i], 0.f);
+  } else if (act == RB_ACT_XIELU) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float z = v[i];
+      const float curve = z > 0.f ? ac.x * z * z : ac.y * (__expf(fminf(z, 0.f)) - 1.0f - z);
+      v[i] = fmaf(0.5f, z, curve);
+    }
   }
 }
 
@@ -315,6 +323,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
     pdl_wait();  // bias/residual reads and every store below must follow the predecessor's completion
     const int quarter = warp & 3;              // the 32 TMEM lanes this warp may read
     const int lane_row = quarter * 32 + lane;  // row of the P operand inside the tile
+    const float2 ac = p.act == RB_ACT_XIELU ? xielu_consts(p.act_params) : make_float2(0.f, 0.f);
     int as = 0;
     uint32_t aphase = 0;
     bool ok = true;
@@ -384,14 +393,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
             }
           } else {
             if (GATED) {
-              act_inplace(p.act, g);
+              act_inplace(p.act, g, ac);
 #pragma unroll
               for (int j = 0; j < CH; ++j) v[j] *= g[j];
             } else {
               const float bias = (p.bias && gn < p.n) ? __bfloat162float(p.bias[gn]) : 0.f;
 #pragma unroll
               for (int j = 0; j < CH; ++j) v[j] += bias;
-              act_inplace(p.act, v);
+              act_inplace(p.act, v, ac);
             }
             // The accumulator holds the tile transposed (lane = output column).  Turn it through
             // shared memory so that the global stores are 16-byte pieces of output rows.
@@ -430,7 +439,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
         } else {
           const int gm = pt * kBM + lane_row;
           const int gn0 = qt * BN + c0;
-          if (GATED) act_inplace(p.act, g);
+          if (GATED) act_inplace(p.act, g, ac);
           if (gm < p.m) {
             const bool vec_ok = (p.n % 8) == 0;
 #pragma unroll
@@ -454,7 +463,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
                     for (int j = 0; j < 8 && gn + j < p.n; ++j) y[j] += __bfloat162float(p.bias[gn + j]);
                   }
                 }
-                act_inplace(p.act, y);
+                act_inplace(p.act, y, ac);
                 if (p.residual) {
                   if (vec_ok) {
                     float r8[8];
@@ -543,13 +552,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
                 }
             }
             if (GATED) {
-              act_inplace(p.act, a);
+              act_inplace(p.act, a, ac);
 #pragma unroll
               for (int i = 0; i < 4; ++i) a[i] *= u[i];
             } else {
 #pragma unroll
               for (int i = 0; i < 4; ++i) a[i] += bias;
-              act_inplace(p.act, a);
+              act_inplace(p.act, a, ac);
             }
 #pragma unroll
             for (int i = 0; i < 4; ++i)
@@ -759,6 +768,8 @@ int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a) {
   p.out = a.partials ? nullptr : (bf16*)a.out;
   p.part = a.partials ? (float*)a.out : nullptr;
   p.act = a.act;
+  p.act_params = (const bf16*)a.act_params;
+  RB_REQUIRE(a.act != RB_ACT_XIELU || (a.act_params && !gated), "GEMM: RB_ACT_XIELU needs its parameters and an ungated product");
   p.status = ctx->status_dev;
   const bool swap = a.m <= 256 && !(gated && a.m > 128);
   if (a.partials) {

@@ -1,0 +1,330 @@
+// Decoders described layer by layer: every layer has its own sequence mixer (windowed attention or the HGRN2 recurrence),
+// its own sizes and an optional feed-forward, with the norm on each sublayer's output and a float32 residual stream:
+//
+//   attention   x -> [q|k|v|gate] GEMM -> convolution + q/k norm + cache append -> attention (window, distance bias, gate)
+//               -> output GEMM -> x += norm(.)
+//   hgrn2       x -> [q|f|v] GEMM -> recurrence (+ per-head norm) -> output GEMM -> x += norm(.)
+//   feed-forward  x -> up GEMM (+ xIELU) -> down GEMM -> x += norm(.)
+//
+// Single-token GEMMs leave float32 split-K slabs that the next kernel sums, as in the other families.  The driver around
+// this walk (lengths, the captured decode step, sampling, loading) is model.cu's.
+#include <algorithm>
+#include <map>
+
+#include "model.h"
+
+using namespace rb;
+
+namespace {
+
+int pad8(int64_t v) { return (int)((v + 7) / 8 * 8); }
+
+// head size of the cache: the next one the tensor-core attention kernels have (bf16), or a multiple of 8 (float32)
+int cache_dim(int dtype, int key_dim, int value_dim) {
+  const int d = std::max(key_dim, value_dim);
+  if (dtype == RB_BF16)
+    for (int have : {64, 80, 96, 128, 256})
+      if (d <= have) return have;
+  return pad8(d);
+}
+
+// float32 split-K slabs in m->scratch of x . W^T; returns how many, or 0 when the product has to be a tensor
+int slab_count(rb_model* m, int64_t rows, int64_t n, int64_t k) {
+  if (m->cfg.dtype != RB_BF16 || rows > 256) return 0;
+  const int fit = (int)std::min<size_t>(16, m->scratch_floats / ((size_t)rows * n));
+  return std::min(rb_linear_pick_splits(m->ctx, rows, n, k), fit);
+}
+
+// stream += norm(x . W^T), and its copy in the model dtype
+int sublayer_out(rb_model* m, const void* x, const void* w, int k, const void* gain, int64_t rows) {
+  rb_ctx* ctx = m->ctx;
+  void* copy = m->cfg.dtype == RB_F32 ? nullptr : m->h;  // float32: the stream itself is the next operand
+  const int s = slab_count(m, rows, m->ld, k);
+  if (s > 0) {
+    RB_TRY(rb_linear_partials(ctx, x, w, m->scratch, rows, m->ld, k, s));
+    return rb_add_scaled_norm(ctx, nullptr, m->scratch, s, gain, (float)m->cfg.norm_eps, rows, m->cfg.hidden_size, m->ld, m->stream,
+                              copy, m->cfg.dtype);
+  }
+  RB_TRY(rb_linear(ctx, x, w, nullptr, nullptr, m->sub_out, rows, m->ld, k, RB_ACT_NONE, m->cfg.dtype));
+  return rb_add_scaled_norm(ctx, m->sub_out, nullptr, 0, gain, (float)m->cfg.norm_eps, rows, m->cfg.hidden_size, m->ld, m->stream, copy,
+                            m->cfg.dtype);
+}
+
+int mixer(rb_model* m, const MixLayer& w, int batch, int seq, const int32_t* new_lens) {
+  rb_ctx* ctx = m->ctx;
+  const int dt = m->cfg.dtype;
+  const int64_t rows = (int64_t)batch * seq;
+  const float eps = (float)m->cfg.norm_eps;
+  const rb_layer_config& c = w.c;
+  // input projection: slabs for the consumer to sum at single-token steps, a tensor otherwise
+  const int s = seq == 1 ? slab_count(m, rows, w.n_in, m->ld) : 0;
+  const void* src = nullptr;
+  const float* acc = nullptr;
+  if (s > 0) {
+    RB_TRY(rb_linear_partials(ctx, m->h, w.in_w, m->scratch, rows, w.n_in, m->ld, s));
+    acc = m->scratch;
+  } else {
+    RB_TRY(rb_linear(ctx, m->h, w.in_w, w.in_b, nullptr, m->mix_in, rows, w.n_in, m->ld, RB_ACT_NONE, dt));
+    src = m->mix_in;
+  }
+  if (c.mixer == RB_MIXER_HGRN2)
+    return rb_hgrn2(ctx, src, acc, s, w.n_in, w.f_bias, w.lower, w.out_norm, eps, c.heads, c.key_dim, c.value_dim, batch, seq, m->cache,
+                    new_lens, w.state, 0, m->attn, w.mix_k, dt);
+  const int kv_heads = c.kv_from < 0 ? c.kv_heads : 0;
+  RB_TRY(rb_conv_norm_append(ctx, src, acc, s, w.in_b, w.conv, c.conv_taps, w.q_norm, w.k_norm, eps, batch, seq, c.heads, kv_heads,
+                             c.key_dim, c.value_dim, w.n_in, w.kv, w.kv_layer, w.state, new_lens, m->q, s > 0 ? m->gate : nullptr, dt));
+  const void* gate = s > 0 ? m->gate : (const char*)m->mix_in + (size_t)w.gate_col * m->es;
+  const int64_t gate_ld = s > 0 ? w.n_in - w.gate_col : w.n_in;
+  return rb_attention_window(ctx, m->q, w.kv, w.kv_layer, batch, seq, c.heads, c.value_dim, (float)c.scale, c.window, 1, gate, gate_ld,
+                             m->attn, w.mix_k, dt);
+}
+
+// m->act = xIELU(x . Wup^T): in the GEMM's epilogue, or, when that would leave most SMs idle, from split-K slabs
+int mlp_up(rb_model* m, const MixLayer& w, int64_t rows) {
+  rb_ctx* ctx = m->ctx;
+  const int64_t tiles = (w.mlp_k + 127) / 128;
+  if (!ctx->debug_simple && tiles * 4 < (int64_t)ctx->sm_count * 3) {
+    const int s = slab_count(m, rows, w.mlp_k, m->ld);
+    if (s > 1) {
+      RB_TRY(rb_linear_partials(ctx, m->h, w.up, m->scratch, rows, w.mlp_k, m->ld, s));
+      return act_from_partials(ctx, m->scratch, s, rows, w.mlp_k, w.mlp_k, false, nullptr, RB_ACT_XIELU, m->act, w.act);
+    }
+  }
+  return rb_linear_act(ctx, m->h, w.up, nullptr, m->act, rows, w.mlp_k, m->ld, RB_ACT_XIELU, w.act, m->cfg.dtype);
+}
+
+}  // namespace
+
+int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq, const int32_t* new_lens) {
+  const rb_model_config& c = m->cfg;
+  rb_ctx* ctx = m->ctx;
+  const int64_t rows = (int64_t)batch * seq;
+  RB_TRY(rb_embed_stream(ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->stream,
+                         c.dtype == RB_F32 ? nullptr : m->h));
+  for (size_t l = 0; l < m->mix.size(); ++l) {
+    const MixLayer& w = m->mix[l];
+    RB_TRY(mixer(m, w, batch, seq, new_lens));
+    RB_TRY(sublayer_out(m, m->attn, w.o_w, w.mix_k, w.norm1, rows));
+    if (w.c.mlp_size > 0) {
+      RB_TRY(mlp_up(m, w, rows));
+      RB_TRY(sublayer_out(m, m->act, w.down, w.mlp_k, w.norm2, rows));
+    }
+    if (m->layer_trace)
+      RB_CUDA(cudaMemcpy2DAsync(m->layer_trace + (size_t)l * rows * c.hidden_size, (size_t)c.hidden_size * 4, m->stream, (size_t)m->ld * 4,
+                                (size_t)c.hidden_size * 4, (size_t)rows, cudaMemcpyDeviceToDevice, ctx->stream));
+  }
+  return RB_OK;
+}
+
+int rb::layered_logits(rb_model* m, const int32_t* rows, int seq, int n, float* out) {
+  const rb_model_config& c = m->cfg;
+  RB_TRY(rb_scalar_norm_rows(m->ctx, m->stream, rows, seq, m->norm_w, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
+  if (c.dtype == RB_F32)
+    return rb_linear(m->ctx, m->xn, m->lm_head, nullptr, nullptr, out, n, c.vocab_size, m->ld, RB_ACT_NONE, RB_F32);
+  for (int r = 0; r < n; r += 256)  // one float32 slab is a float32 product
+    RB_TRY(rb_linear_partials(m->ctx, (const char*)m->xn + (size_t)r * m->ld * m->es, m->lm_head, out + (size_t)r * c.vocab_size,
+                              std::min(256, n - r), c.vocab_size, m->ld, 1));
+  return RB_OK;
+}
+
+// How many KV splits each attention layer takes: what a captured decode step depends on.
+int rb::layered_decode_plan(rb_model* m, int batch) {
+  int max_len = 0;
+  for (int b = 0; b < batch; ++b) max_len = std::max(max_len, m->cache->host_lens[b]);
+  uint32_t plan = 17;
+  for (const MixLayer& w : m->mix)
+    if (w.kv)
+      plan = plan * 31 + (uint32_t)attention_decode_splits(m->ctx, batch, w.c.kv_heads, attention_walk_len(max_len, w.c.window),
+                                                           w.kv->head_dim);
+  return (int)(plan & 0x7fffffffu);
+}
+
+extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out) {
+  RB_REQUIRE(ctx && cfg && layers && out, "rb_model_create_layers: null argument");
+  const rb_model_config& c = *cfg;
+  RB_REQUIRE(c.arch == RB_ARCH_MALASUN, "rb_model_create_layers: architecture %d is not described layer by layer", c.arch);
+  RB_REQUIRE(c.dtype == RB_BF16 || c.dtype == RB_F32, "rb_model_create_layers: dtype %d unsupported", c.dtype);
+  RB_REQUIRE(c.hidden_size > 0 && c.vocab_size > 0 && c.num_hidden_layers > 0, "rb_model_create_layers: bad sizes");
+  RB_REQUIRE(c.max_batch > 0 && c.max_seq > 0 && c.max_tokens >= c.max_batch, "rb_model_create_layers: bad capacities");
+  // the query / key norm runs over all heads at once, so a head-parallel split would need its sum exchanged per layer
+  if (c.tp_size > 1) return fail(RB_ERR_UNIMPLEMENTED, "rb_model_create_layers: tensor parallelism is not available for this design");
+  const int L = c.num_hidden_layers;
+  for (int l = 0; l < L; ++l) {
+    const rb_layer_config& y = layers[l];
+    RB_REQUIRE(y.mixer == RB_MIXER_ATTENTION || y.mixer == RB_MIXER_HGRN2, "layer %d: unknown mixer %d", l, y.mixer);
+    RB_REQUIRE(y.heads > 0 && y.key_dim > 0 && y.value_dim > 0 && y.mlp_size >= 0, "layer %d: bad sizes", l);
+    if (y.key_dim > 256 || y.value_dim > 256) return fail(RB_ERR_UNIMPLEMENTED, "layer %d: head sizes above 256", l);
+    if (y.mixer != RB_MIXER_ATTENTION) continue;
+    RB_REQUIRE(y.kv_heads > 0 && y.heads % y.kv_heads == 0, "layer %d: %d heads over %d key/value heads", l, y.heads, y.kv_heads);
+    RB_REQUIRE(y.conv_taps >= 1 && y.window >= 0 && y.window <= (1 << 30) && y.scale > 0.0, "layer %d: bad attention constants", l);
+    if (y.kv_from >= 0) {
+      RB_REQUIRE(y.kv_from < l && layers[y.kv_from].mixer == RB_MIXER_ATTENTION && layers[y.kv_from].kv_from < 0,
+                 "layer %d: kv_from %d is not an earlier attention layer with keys and values of its own", l, y.kv_from);
+      RB_REQUIRE(layers[y.kv_from].kv_heads == y.kv_heads && layers[y.kv_from].key_dim == y.key_dim &&
+                     layers[y.kv_from].value_dim == y.value_dim,
+                 "layer %d: its key/value heads differ from those of layer %d", l, y.kv_from);
+    }
+  }
+
+  rb_model* m = new rb_model();
+  m->ctx = ctx;
+  m->cfg = c;
+  m->cfg.tp_size = 1;
+  m->cfg.tp_rank = 0;
+  m->cfg.max_position_embeddings = 0x7fffffff;  // positions enter through distances only: no table to outgrow
+  m->layered = true;
+  m->es = dtype_size(c.dtype);
+  m->logits_dtype = RB_F32;
+  {
+    const char* g = getenv("RAI_B200_GRAPH");  // RAI_B200_GRAPH=0: plain launches for every decode step
+    m->use_graph = !(g && g[0] == '0');
+  }
+  const int W = c.hidden_size, ld = pad8(W), V = c.vocab_size;
+  m->ld = ld;
+  int st = RB_OK;
+  auto A = [&](int64_t elems, void** p) { if (st == RB_OK) st = weight_alloc(m, elems, p); };
+  auto at = [&](void* base, int64_t elem_off) { return (void*)((char*)base + elem_off * (int64_t)m->es); };
+  auto vec = [&](const std::string& name, int64_t n, void* dst) { add_param(m, name, n, 1, 1, {{0, n, 0, 1, dst, 1}}); };
+  auto num = [&](const std::string& name, void* dst) { add_param(m, name, 1, 1, 0, {{0, 1, 0, 1, dst, 1}}); };
+  auto mat = [&](const std::string& name, int64_t rows, int64_t cols, void* dst, int64_t dst_ld) {
+    add_param(m, name, rows, cols, 2, {{0, rows, 0, cols, dst, dst_ld}});
+  };
+
+  A((int64_t)V * ld, &m->embed);
+  mat("embed", V, W, m->embed, ld);
+  m->mix.resize(L);
+  std::map<std::pair<int, int>, std::vector<int>> geometry;  // (key/value heads, cache head size) -> layers with K and V of their own
+  int max_in = 8, max_q = 8, max_gate = 8, max_mix = 8, max_mlp = 8;
+  for (int l = 0; l < L && st == RB_OK; ++l) {
+    MixLayer& w = m->mix[l];
+    w.c = layers[l];
+    const rb_layer_config& y = w.c;
+    const std::string pre = "l" + std::to_string(l) + ".", mix = pre + "mix.";
+    A(8, &w.norm1);
+    num(pre + "norm1", w.norm1);
+    w.mix_k = pad8((int64_t)y.heads * y.value_dim);
+    A((int64_t)ld * w.mix_k, &w.o_w);
+    if (y.mixer == RB_MIXER_HGRN2) {
+      const int hd = y.heads * y.key_dim, p = pad8(hd);
+      w.n_in = 2 * p + w.mix_k;
+      A((int64_t)w.n_in * ld, &w.in_w);
+      A(p, &w.f_bias);
+      A(p, &w.lower);
+      A(pad8(y.value_dim), &w.out_norm);
+      if (st != RB_OK) break;
+      mat(mix + "q", hd, W, w.in_w, ld);
+      mat(mix + "f", hd, W, at(w.in_w, (int64_t)p * ld), ld);
+      vec(mix + "f.b", hd, w.f_bias);
+      vec(mix + "lower", hd, w.lower);
+      mat(mix + "v", (int64_t)y.heads * y.value_dim, W, at(w.in_w, (int64_t)2 * p * ld), ld);
+      vec(mix + "norm", y.value_dim, w.out_norm);
+      st = dev_alloc(m, (size_t)c.max_batch * y.heads * y.key_dim * y.value_dim * sizeof(float), (void**)&w.state, true);
+    } else {
+      const bool own = y.kv_from < 0;
+      const int nq = y.heads * y.key_dim, nk = own ? y.kv_heads * y.key_dim : 0, nv = own ? y.kv_heads * y.value_dim : 0;
+      const int qp = pad8(nq), kp = pad8(nk), vp = pad8(nv), C = qp + kp + vp, taps = y.conv_taps;
+      w.gate_col = C;
+      w.n_in = C + w.mix_k;
+      A((int64_t)w.n_in * ld, &w.in_w);
+      A(w.n_in, &w.in_b);
+      A((int64_t)taps * C, &w.conv);
+      A(qp, &w.q_norm);
+      if (own) A(kp, &w.k_norm);
+      if (st != RB_OK) break;
+      auto part = [&](const char* name, int n, int col, void* norm) {
+        const std::string t = mix + name;
+        mat(t, n, W, at(w.in_w, (int64_t)col * ld), ld);
+        vec(t + ".b", n, at(w.in_b, col));
+        std::vector<Piece> ps;  // [channel][tap] in the file, [tap][channel] here
+        for (int j = 0; j < taps; ++j) ps.push_back({0, n, j, 1, at(w.conv, (int64_t)j * C + col), 1});
+        add_param(m, t + ".conv", n, taps, 2, ps);
+        if (norm) vec(t + ".norm", n, norm);
+      };
+      part("q", nq, 0, w.q_norm);
+      if (own) {
+        part("k", nk, qp, w.k_norm);
+        part("v", nv, qp + kp, nullptr);
+        auto& group = geometry[{y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim)}];
+        w.kv_layer = (int)group.size();
+        group.push_back(l);
+      }
+      mat(mix + "g", (int64_t)y.heads * y.value_dim, W, at(w.in_w, (int64_t)C * ld), ld);
+      if (taps > 1) st = dev_alloc(m, (size_t)c.max_batch * (taps - 1) * C * sizeof(float), (void**)&w.state, true);
+      max_q = std::max(max_q, y.heads * cache_dim(c.dtype, y.key_dim, y.value_dim));
+      max_gate = std::max(max_gate, w.mix_k);
+    }
+    mat(mix + "o", W, (int64_t)y.heads * y.value_dim, w.o_w, w.mix_k);
+    if (y.mlp_size > 0) {
+      w.mlp_k = pad8(y.mlp_size);
+      A((int64_t)w.mlp_k * ld, &w.up);
+      A((int64_t)ld * w.mlp_k, &w.down);
+      A(8, &w.act);
+      A(8, &w.norm2);
+      if (st != RB_OK) break;
+      num(pre + "norm2", w.norm2);
+      mat(pre + "mlp.up", y.mlp_size, W, w.up, ld);
+      mat(pre + "mlp.down", W, y.mlp_size, w.down, w.mlp_k);
+      vec(pre + "mlp.act", 2, w.act);
+    }
+    max_in = std::max(max_in, w.n_in);
+    max_mix = std::max(max_mix, w.mix_k);
+    max_mlp = std::max(max_mlp, w.mlp_k);
+  }
+  A(8, &m->norm_w);
+  A((int64_t)V * ld, &m->lm_head);
+  if (st == RB_OK) {
+    num("final.norm", m->norm_w);
+    mat("head", V, W, m->lm_head, ld);
+    m->vocab_l = V;
+  }
+
+  // ---- sequence tables, one cache per attention geometry over them
+  if (st == RB_OK) st = kv_cache_create(ctx, nullptr, 0, 1, 8, c.max_batch, c.max_seq, c.dtype, &m->cache);
+  for (auto& g : geometry) {
+    rb_kv_cache* view = nullptr;
+    if (st == RB_OK) st = kv_cache_create(ctx, m->cache, (int)g.second.size(), g.first.first, g.first.second, 0, 0, c.dtype, &view);
+    if (st != RB_OK) break;
+    m->views.push_back(view);
+    for (int l : g.second) m->mix[l].kv = view;
+  }
+  if (st == RB_OK)
+    for (MixLayer& w : m->mix)
+      if (w.c.mixer == RB_MIXER_ATTENTION && w.c.kv_from >= 0) {
+        w.kv = m->mix[w.c.kv_from].kv;
+        w.kv_layer = m->mix[w.c.kv_from].kv_layer;
+      }
+  if (st == RB_OK && c.dtype == RB_BF16) {  // split-KV scratch for the worst case: a generation then never allocates
+    size_t need = 0;
+    for (const MixLayer& w : m->mix)
+      if (w.kv) need = std::max(need, (size_t)c.max_batch * w.c.heads * 32 * (w.kv->head_dim + 2) * sizeof(float));
+    st = attention_reserve_scratch(ctx, need);
+    if (st == RB_OK) st = gemm_reserve_scratch(ctx, (size_t)8 * 64 * std::max(std::max(max_in, max_mlp), ld) * sizeof(float));
+  }
+
+  // ---- workspace.  Zeroed: what lies between a row's width and its pitch is multiplied by zero weights and must be finite.
+  auto B = [&](size_t bytes, void** p) { if (st == RB_OK) st = dev_alloc(m, bytes, p, true); };
+  const size_t MT = c.max_tokens, few = std::min<size_t>(MT, 256);
+  B(MT * sizeof(uint32_t), (void**)&m->ids);
+  B(MT * ld * sizeof(float), (void**)&m->stream);
+  if (c.dtype == RB_F32) m->h = m->stream;
+  else B(MT * ld * m->es, &m->h);
+  B(MT * max_in * m->es, &m->mix_in);
+  B(MT * max_q * m->es, &m->q);
+  B(few * max_gate * m->es, &m->gate);
+  B(MT * max_mix * m->es, &m->attn);
+  B(MT * max_mlp * m->es, &m->act);
+  B(MT * ld * m->es, &m->sub_out);
+  B((size_t)c.max_batch * ld * m->es, &m->xn);
+  B((size_t)c.max_batch * V * sizeof(float), &m->logits);
+  B((size_t)c.max_batch * sizeof(uint32_t), (void**)&m->next_ids);
+  B(MT * sizeof(int32_t), (void**)&m->last_rows);
+  B((size_t)c.max_batch * sizeof(int32_t), (void**)&m->new_lens);
+  if (c.dtype == RB_BF16) {
+    m->scratch_floats = (size_t)16 * few * std::max(std::max(max_in, max_mlp), ld);
+    B(m->scratch_floats * sizeof(float), (void**)&m->scratch);
+  }
+  if (st != RB_OK) { rb_model_destroy(m); return st; }
+  RB_CUDA(cudaStreamSynchronize(ctx->stream));
+  *out = m;
+  return RB_OK;
+}

@@ -21,7 +21,7 @@
 #include <string>
 #include <vector>
 
-#include "ctx.h"
+#include "model.h"
 
 using namespace rb;
 
@@ -67,27 +67,6 @@ int nccl_load() {
     int _r = (expr);                                                                                    \
     if (_r != 0) return fail(RB_ERR_CUDA, "%s failed: %s", #expr, nccl().GetErrorString(_r));           \
   } while (0)
-
-// One rectangular piece of a reference parameter and where it lands in this rank's buffers.
-struct Piece {
-  int64_t src_row0, rows, src_col0, cols;
-  void* dst;
-  int64_t dst_ld;  // elements
-};
-struct ParamSpec {
-  int64_t rows, cols;  // full shape of the reference parameter (cols = 1 for vectors)
-  int rank;            // 1 or 2
-  std::vector<Piece> pieces;
-  bool loaded = false;
-};
-
-struct LayerW {
-  void *qkv = nullptr, *qkv_b = nullptr;
-  void *o = nullptr, *o_b = nullptr;
-  void *gate = nullptr, *up = nullptr, *fc1_b = nullptr;  // phi2: gate = fc1
-  void *down = nullptr, *down_b = nullptr;                // phi2: down = fc2
-  void *ln1_w = nullptr, *ln1_b = nullptr, *ln2_w = nullptr;
-};
 
 template <typename S, typename T>
 __global__ void copy_cast_2d_kernel(const S* __restrict__ src, int64_t src_ld, T* __restrict__ dst, int64_t dst_ld,
@@ -146,73 +125,9 @@ __global__ void unshard_logits_kernel(const T* __restrict__ g, T* __restrict__ o
   }
 }
 
-struct Pending {  // terms still to be added to the residual stream
-  const float* acc = nullptr;
-  int n_acc = 0;
-  const void* acc_bias = nullptr;
-  const void* add = nullptr;
-  bool exchange = false;  // the term is one rank's share: the norm point sums it over the tensor-parallel group
-  bool any() const { return (acc && n_acc > 0) || add || exchange; }
-};
-
 }  // namespace
 
-struct rb_model {
-  rb_ctx* ctx = nullptr;
-  rb_model_config cfg{};
-  int d = 0, nq_l = 0, nkv_l = 0, nqkv_l = 0, inter_l = 0, vocab_l = 0;
-  std::vector<int> q_head_src;  // global q head of local head j, or -1 for padding
-  int kv_head0 = 0;             // first global kv head of this rank
-  size_t es = 2;
-  std::vector<LayerW> layers;
-  void *embed = nullptr, *norm_w = nullptr, *norm_b = nullptr, *lm_head = nullptr, *lm_head_b = nullptr;
-  float *rope_cos = nullptr, *rope_sin = nullptr;
-  rb_kv_cache* cache = nullptr;
-  std::vector<void*> owned;
-  std::vector<std::string> names;
-  std::map<std::string, ParamSpec> params;
-  int64_t param_bytes = 0;
-  // workspace
-  uint32_t* ids = nullptr;
-  void *h = nullptr, *xn = nullptr, *tmp = nullptr, *qkv = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;
-  void *last_h = nullptr, *logits = nullptr, *logits_g = nullptr;
-  uint32_t* next_ids = nullptr;
-  int32_t* last_rows = nullptr;           // ragged prefill: row of each sequence's last valid token
-  std::vector<int32_t> last_rows_host;    // outlives the asynchronous upload
-  float* scratch = nullptr;  // split-K partials
-  size_t scratch_floats = 0;
-  void* comm = nullptr;
-  // peer-memory exchange for decode-sized allreduces (see TpPeers); xchg_base is this rank's region
-  TpPeers peers{};
-  void* xchg_base = nullptr;
-  int xchg_index = 0;  // exchanges launched so far in this forward pass (an even number per pass: two per layer)
-  void* peer_base[kTpMaxRanks] = {};
-  bool use_exchange = false;
-  // RAI_B200_TP_FUSED_GATE=1: a sharded gate/up GEMM sums its split-K slabs and applies activation and gating in its
-  // own epilogue.  Off by default: measured slower than split-K partials plus the small finishing kernel, whose many
-  // blocks read the slabs with far more parallelism.
-  bool fused_gate = false;
-  // Developer builds only (-DRB_DEBUG_AIDS, a library file of its own): RAI_B200_SHARD_ONLY=1 runs one rank's shard
-  // without its peers to time the per-rank kernels; its outputs are not the model's.  Always false otherwise.
-  bool shard_only = false;
-  // One decode step (advance lengths, forward of the tokens in `ids`, argmax back into `ids`)
-  // captured as a CUDA graph and replayed; re-captured when the batch or the launch plan changes.
-  cudaGraphExec_t step_graph = nullptr;
-  int graph_batch = 0, graph_plan = 0;
-  int eager_warm_batch = 0, eager_warm_plan = 0;
-  int64_t graph_launches = 0;
-  bool use_graph = true;
-  cudaEvent_t ev_in = nullptr, ev_out = nullptr;
-  // sampling of the generation entry points (rb_model_set_sampling): repeat penalty over a ring of the
-  // last `rep_last_n` tokens fed per sequence, and the end-of-sequence rule
-  float rep_penalty = 0.f;
-  int rep_last_n = 0;
-  int32_t eos = -1;
-  int32_t *hist = nullptr, *hist_count = nullptr;
-  uint8_t* finished = nullptr;
-};
-
-namespace {
+namespace rb {
 
 int dev_alloc(rb_model* m, size_t bytes, void** out, bool zero) {
   RB_TRY(rb_malloc(m->ctx, bytes, out));
@@ -232,6 +147,10 @@ void add_param(rb_model* m, const std::string& name, int64_t rows, int64_t cols,
   m->names.push_back(name);
   m->params[name] = std::move(s);
 }
+
+}  // namespace rb
+
+namespace {
 
 // The exchange is used only when every one of the `tp` ranks voted 1 (the votes arrive summed).
 bool exchange_agreed(float vote_sum, int tp) { return vote_sum > (float)tp - 0.5f; }
@@ -316,7 +235,59 @@ int linear_into_residual(rb_model* m, Pending& pend, const void* x, const void* 
   return rb_linear(m->ctx, x, w, b, m->h, m->h, rows, n, k, RB_ACT_NONE, m->cfg.dtype);
 }
 
-int forward_body(rb_model* m, const uint32_t* tokens, int batch, int seq, void* logits_out, const int32_t* last_rows = nullptr);
+// m->logits[i] for row rows_dev[i] of the residual stream (rows_dev == NULL: the last of each sequence's seq rows).
+int last_rows_logits(rb_model* m, int seq, const int32_t* rows_dev, int n) {
+  if (m->layered) return layered_logits(m, rows_dev, seq, n, (float*)m->logits);
+  const rb_model_config& c = m->cfg;
+  rb_ctx* ctx = m->ctx;
+  const int H = c.hidden_size;
+  // (qwen2.rs:356-358; phi2.rs:345-346 normalises every row first, which is the same thing for a row-wise norm)
+  const void* last = m->h;
+  if (rows_dev) {
+    RB_REQUIRE(((size_t)H * m->es) % 16 == 0, "ragged forward: hidden rows must be multiples of 16 bytes");
+    gather_rows_kernel<<<n, 128, 0, ctx->stream>>>((const uint4*)m->h, rows_dev, (uint4*)m->last_h, (int)((size_t)H * m->es / 16));
+    RB_CUDA(cudaGetLastError());
+    ctx->launches++;
+    last = m->last_h;
+  } else if (seq > 1) {
+    RB_CUDA(cudaMemcpy2DAsync(m->last_h, (size_t)H * m->es, (const char*)m->h + (size_t)(seq - 1) * H * m->es,
+                              (size_t)seq * H * m->es, (size_t)H * m->es, n, cudaMemcpyDeviceToDevice, ctx->stream));
+    last = m->last_h;
+  }
+  RB_TRY(rb_norm(ctx, norm_kind(m), last, nullptr, nullptr, 0, nullptr, m->norm_w, m->norm_b, (float)c.norm_eps, n, H,
+                 m->xn, nullptr, c.dtype));
+  void* head_w = m->lm_head ? m->lm_head : m->embed;
+  if (c.tp_size == 1) {
+    RB_TRY(rb_linear(ctx, m->xn, head_w, m->lm_head_b, nullptr, m->logits, n, m->vocab_l, H, RB_ACT_NONE, c.dtype));
+  } else {
+    RB_TRY(rb_linear(ctx, m->xn, head_w, m->lm_head_b, nullptr, m->logits_g, n, m->vocab_l, H, RB_ACT_NONE, c.dtype));
+    void* gathered = (char*)m->logits_g + (size_t)n * m->vocab_l * m->es;
+    const size_t shard_bytes = (size_t)n * m->vocab_l * m->es;
+    if (!m->shard_only) {
+      RB_NCCL(nccl().AllGather(m->logits_g, gathered, shard_bytes, kNcclUint8, m->comm, ctx->stream));
+    } else {
+      // a rank run without its peers: its own vocabulary shard in place, zeros where the others' would be
+      RB_CUDA(cudaMemsetAsync(gathered, 0, shard_bytes * c.tp_size, ctx->stream));
+      RB_CUDA(cudaMemcpyAsync((char*)gathered + shard_bytes * c.tp_rank, m->logits_g, shard_bytes, cudaMemcpyDeviceToDevice,
+                              ctx->stream));
+    }
+    const int64_t total = (int64_t)c.tp_size * n * m->vocab_l;
+    const int blocks = (int)std::min<int64_t>((total + 255) / 256, 4096);
+    if (c.dtype == RB_BF16)
+      unshard_logits_kernel<__nv_bfloat16><<<blocks, 256, 0, ctx->stream>>>((const __nv_bfloat16*)gathered,
+                                                                           (__nv_bfloat16*)m->logits, c.tp_size, n,
+                                                                           m->vocab_l);
+    else
+      unshard_logits_kernel<float><<<blocks, 256, 0, ctx->stream>>>((const float*)gathered, (float*)m->logits, c.tp_size,
+                                                                   n, m->vocab_l);
+    ctx->launches++;
+  }
+  return RB_OK;
+}
+
+int forward_body(rb_model* m, const uint32_t* tokens, int batch, int seq, void* logits_out, const int32_t* rows_dev = nullptr,
+                 int n_rows = -1, const int32_t* new_lens = nullptr);
+int finish_logits(rb_model* m, int batch, int seq, void* logits_out, const int32_t* rows_dev, int n_rows);
 
 // act = activation(x . W1^T [+ b1]) [* (x . Wup^T)]  -- the first half of MLP::fwd.  When the fused kernel
 // would leave most SMs idle (decode-sized rows and few 128-row weight tiles, i.e. small or sharded
@@ -371,7 +342,15 @@ int forward_impl(rb_model* m, const uint32_t* tokens, int batch, int seq, int po
 
 // The launches of one forward pass.  Everything position-dependent is read from device memory (the
 // cache's sequence lengths), so the same sequence of launches serves every decode step.
-int forward_body(rb_model* m, const uint32_t* tokens, int batch, int seq, void* logits_out, const int32_t* last_rows) {
+// Logits are computed for rows_dev[0..n_rows) of the call, or (rows_dev == NULL) for the last position of each sequence.
+// new_lens (device, NULL = seq each): how many of a sequence's rows are tokens; the rest is padding.
+int forward_body(rb_model* m, const uint32_t* tokens, int batch, int seq, void* logits_out, const int32_t* rows_dev, int n_rows,
+                 const int32_t* new_lens) {
+  if (!rows_dev) n_rows = batch;
+  if (m->layered) {
+    RB_TRY(layered_forward(m, tokens, batch, seq, new_lens));
+    return finish_logits(m, batch, seq, logits_out, rows_dev, n_rows);
+  }
   const rb_model_config& c = m->cfg;
   rb_ctx* ctx = m->ctx;
   RB_REQUIRE(c.tp_size == 1 || m->comm || m->shard_only,
@@ -427,51 +406,20 @@ int forward_body(rb_model* m, const uint32_t* tokens, int batch, int seq, void* 
   }
   RB_TRY(norm_point(m, pend, nullptr, nullptr, rows, nullptr));  // fold the last layer's output
 
-  // logits for the last position only (qwen2.rs:356-358; phi2.rs:345-346 normalises every row first,
-  // which is the same thing for a row-wise norm)
-  const void* last = m->h;
-  if (seq > 1 && last_rows) {
-    RB_REQUIRE(((size_t)H * m->es) % 16 == 0, "ragged forward: hidden rows must be multiples of 16 bytes");
-    gather_rows_kernel<<<batch, 128, 0, ctx->stream>>>((const uint4*)m->h, last_rows, (uint4*)m->last_h, (int)((size_t)H * m->es / 16));
-    RB_CUDA(cudaGetLastError());
-    ctx->launches++;
-    last = m->last_h;
-  } else if (seq > 1) {
-    RB_CUDA(cudaMemcpy2DAsync(m->last_h, (size_t)H * m->es, (const char*)m->h + (size_t)(seq - 1) * H * m->es,
-                              (size_t)seq * H * m->es, (size_t)H * m->es, batch, cudaMemcpyDeviceToDevice, ctx->stream));
-    last = m->last_h;
+  return finish_logits(m, batch, seq, logits_out, rows_dev, n_rows);
+}
+
+// Final norm and vocabulary product of the wanted rows, at most max_batch at a time.
+int finish_logits(rb_model* m, int batch, int seq, void* logits_out, const int32_t* rows_dev, int n_rows) {
+  const rb_model_config& c = m->cfg;
+  const size_t row_bytes = (size_t)c.vocab_size * dtype_size(m->logits_dtype);
+  for (int r0 = 0; r0 < n_rows; r0 += c.max_batch) {
+    const int n = std::min(n_rows - r0, (int)c.max_batch);
+    RB_TRY(last_rows_logits(m, seq, rows_dev ? rows_dev + r0 : nullptr, n));
+    if (logits_out && logits_out != m->logits)
+      RB_CUDA(cudaMemcpyAsync((char*)logits_out + (size_t)r0 * row_bytes, m->logits, (size_t)n * row_bytes, cudaMemcpyDeviceToDevice,
+                              m->ctx->stream));
   }
-  RB_TRY(rb_norm(ctx, norm_kind(m), last, nullptr, nullptr, 0, nullptr, m->norm_w, m->norm_b, (float)c.norm_eps, batch, H,
-                 m->xn, nullptr, c.dtype));
-  void* head_w = m->lm_head ? m->lm_head : m->embed;
-  if (c.tp_size == 1) {
-    RB_TRY(rb_linear(ctx, m->xn, head_w, m->lm_head_b, nullptr, m->logits, batch, m->vocab_l, H, RB_ACT_NONE, c.dtype));
-  } else {
-    RB_TRY(rb_linear(ctx, m->xn, head_w, m->lm_head_b, nullptr, m->logits_g, batch, m->vocab_l, H, RB_ACT_NONE, c.dtype));
-    void* gathered = (char*)m->logits_g + (size_t)batch * m->vocab_l * m->es;
-    const size_t shard_bytes = (size_t)batch * m->vocab_l * m->es;
-    if (!m->shard_only) {
-      RB_NCCL(nccl().AllGather(m->logits_g, gathered, shard_bytes, kNcclUint8, m->comm, ctx->stream));
-    } else {
-      // a rank run without its peers: its own vocabulary shard in place, zeros where the others' would be
-      RB_CUDA(cudaMemsetAsync(gathered, 0, shard_bytes * c.tp_size, ctx->stream));
-      RB_CUDA(cudaMemcpyAsync((char*)gathered + shard_bytes * c.tp_rank, m->logits_g, shard_bytes, cudaMemcpyDeviceToDevice,
-                              ctx->stream));
-    }
-    const int64_t n = (int64_t)c.tp_size * batch * m->vocab_l;
-    const int blocks = (int)std::min<int64_t>((n + 255) / 256, 4096);
-    if (c.dtype == RB_BF16)
-      unshard_logits_kernel<__nv_bfloat16><<<blocks, 256, 0, ctx->stream>>>((const __nv_bfloat16*)gathered,
-                                                                           (__nv_bfloat16*)m->logits, c.tp_size, batch,
-                                                                           m->vocab_l);
-    else
-      unshard_logits_kernel<float><<<blocks, 256, 0, ctx->stream>>>((const float*)gathered, (float*)m->logits, c.tp_size,
-                                                                   batch, m->vocab_l);
-    ctx->launches++;
-  }
-  if (logits_out && logits_out != m->logits)
-    RB_CUDA(cudaMemcpyAsync(logits_out, m->logits, (size_t)batch * c.vocab_size * m->es, cudaMemcpyDeviceToDevice,
-                            ctx->stream));
   return RB_OK;
 }
 
@@ -603,6 +551,7 @@ extern "C" int32_t rb_model_create(rb_ctx* ctx, const rb_model_config* cfg, rb_m
   }
   m->d = c.hidden_size / nq;
   m->es = dtype_size(c.dtype);
+  m->logits_dtype = c.dtype;
   const int d = m->d, H = c.hidden_size;
   // ---- head assignment
   if (tp <= nkv) {
@@ -760,7 +709,8 @@ extern "C" int32_t rb_model_create(rb_ctx* ctx, const rb_model_config* cfg, rb_m
   W((size_t)c.max_batch * V * m->es, &m->logits);
   if (tp > 1) W((size_t)c.max_batch * Vl * m->es * (tp + 1), &m->logits_g);
   W((size_t)c.max_batch * sizeof(uint32_t), (void**)&m->next_ids);
-  W((size_t)c.max_batch * sizeof(int32_t), (void**)&m->last_rows);
+  W(MT * sizeof(int32_t), (void**)&m->last_rows);
+  W((size_t)c.max_batch * sizeof(int32_t), (void**)&m->new_lens);
   if (c.dtype == RB_BF16) {
     // split-K scratch: up to 16 slabs of min(max_tokens, 256) rows of the widest split-K output
     const size_t rows = std::min<size_t>(MT, 256);
@@ -801,6 +751,7 @@ extern "C" int32_t rb_model_destroy(rb_model* m) {
   for (int r = 0; r < kTpMaxRanks; ++r)
     if (m->peer_base[r] && m->peer_base[r] != m->xchg_base) cudaIpcCloseMemHandle(m->peer_base[r]);
   if (m->comm && nccl().CommDestroy) nccl().CommDestroy(m->comm);
+  for (rb_kv_cache* v : m->views) rb_kv_cache_destroy(v);
   if (m->cache) rb_kv_cache_destroy(m->cache);
   for (void* p : m->owned) rb_free(m->ctx, p);
   delete m;
@@ -1059,40 +1010,112 @@ extern "C" int32_t rb_model_finished(rb_model* m, int32_t batch, uint8_t* flags_
   return RB_OK;
 }
 
-// Right-padded batch: sequence b has lens[b] valid tokens followed by padding.  The rectangle runs as usual
-// (under the causal mask a pad can only influence later pads), the logits come from each sequence's last
-// valid row, and the cache keeps lens[b] tokens of sequence b: the pads' K/V rows lie beyond that length,
-// are never read, and are overwritten by the tokens decoded next.
-static int forward_ragged(rb_model* m, const uint32_t* tokens, int batch, int seq, int pos, const int32_t* lens, void* logits_out) {
+// The general step: sequence b feeds lens[b] (0..seq, NULL = seq) of the tokens in its row, followed by padding.  The
+// rectangle runs as usual (under the causal mask a pad can only influence later pads, and recurrent states stop at the
+// last token), logits come from the rows asked for, and the cache keeps lens[b] more tokens of sequence b: the pads'
+// K/V rows lie beyond that length, are never read, and are overwritten by the tokens fed next.
+// pos >= 0 must be every sequence's cached length; pos < 0 continues each at its own.
+static int forward_rows(rb_model* m, const uint32_t* tokens, int batch, int seq, int pos, const int32_t* lens, const int32_t* rows,
+                        int n_rows, void* logits_out) {
   rb_ctx* ctx = m->ctx;
   rb_kv_cache* kc = m->cache;
-  for (int b = 0; b < batch; ++b)
-    RB_REQUIRE(lens[b] >= 1 && lens[b] <= seq, "ragged forward: sequence %d has %d valid tokens of %d", b, lens[b], seq);
-  m->last_rows_host.assign((size_t)batch, 0);
-  for (int b = 0; b < batch; ++b) m->last_rows_host[b] = b * seq + lens[b] - 1;
-  RB_CUDA(cudaMemcpyAsync(m->last_rows, m->last_rows_host.data(), (size_t)batch * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
   const rb_model_config& c = m->cfg;
-  const int64_t rows = (int64_t)batch * seq;
+  const int64_t total = (int64_t)batch * seq;
   RB_REQUIRE(batch > 0 && batch <= c.max_batch, "forward: batch %d exceeds max_batch %d", batch, c.max_batch);
-  RB_REQUIRE(seq > 0 && rows <= c.max_tokens, "forward: %lld tokens exceed max_tokens %d", (long long)rows, c.max_tokens);
-  RB_REQUIRE(pos >= 0 && pos + seq <= kc->max_seq && pos + seq <= c.max_position_embeddings,
-             "forward: position %d + %d exceeds the cache / rotary table capacity", pos, seq);
-  for (int b = 0; b < batch; ++b)
-    RB_REQUIRE(kc->host_lens[b] == pos, "forward: seqlen_offset %d differs from the cached length %d of sequence %d", pos,
-               kc->host_lens[b], b);
-  set_lens_kernel<<<(batch + 127) / 128, 128, 0, ctx->stream>>>(kc->seq_lens, batch, pos + seq);
-  ctx->launches++;
-  for (int b = 0; b < batch; ++b) kc->host_lens[b] = pos + seq;
-  RB_TRY(forward_body(m, tokens, batch, seq, logits_out, seq > 1 ? m->last_rows : nullptr));
-  for (int b = 0; b < batch; ++b) kc->host_lens[b] = pos + lens[b];
+  RB_REQUIRE(seq > 0 && total <= c.max_tokens, "forward: %lld tokens exceed max_tokens %d", (long long)total, c.max_tokens);
+  RB_REQUIRE(n_rows >= 0 && n_rows <= total, "forward: %d rows of logits out of %lld", n_rows, (long long)total);
+  for (int b = 0; b < batch; ++b) {
+    const int base = kc->host_lens[b];
+    RB_REQUIRE(!lens || (lens[b] >= 0 && lens[b] <= seq), "ragged forward: sequence %d has %d valid tokens of %d", b, lens[b], seq);
+    RB_REQUIRE(pos < 0 || base == pos, "forward: seqlen_offset %d differs from the cached length %d of sequence %d", pos, base, b);
+    RB_REQUIRE(base + seq <= kc->max_seq && base + seq <= c.max_position_embeddings,
+               "forward: position %d + %d exceeds the cache / rotary table capacity", base, seq);
+  }
+  for (int i = 0; i < n_rows; ++i)
+    RB_REQUIRE(rows[i] >= 0 && rows[i] < total, "forward: row %d of %lld", rows[i], (long long)total);
+  if (n_rows > 0) {
+    m->last_rows_host.assign(rows, rows + n_rows);
+    RB_CUDA(cudaMemcpyAsync(m->last_rows, m->last_rows_host.data(), (size_t)n_rows * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
+  }
+  if (lens) {
+    m->new_lens_host.assign(lens, lens + batch);
+    RB_CUDA(cudaMemcpyAsync(m->new_lens, m->new_lens_host.data(), (size_t)batch * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
+  }
+  const std::vector<int32_t> before(kc->host_lens.begin(), kc->host_lens.begin() + batch);
+  for (int b = 0; b < batch; ++b) kc->host_lens[b] = before[b] + seq;
   RB_CUDA(cudaMemcpyAsync(kc->seq_lens, kc->host_lens.data(), (size_t)batch * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
-  return RB_OK;
+  const int st = forward_body(m, tokens, batch, seq, logits_out, m->last_rows, n_rows, lens ? m->new_lens : nullptr);
+  if (lens) {
+    for (int b = 0; b < batch; ++b) kc->host_lens[b] = before[b] + lens[b];
+    RB_CUDA(cudaMemcpyAsync(kc->seq_lens, kc->host_lens.data(), (size_t)batch * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
+  }
+  return st;
+}
+
+// A right-padded batch with at least one token per sequence, logits from each sequence's last one.
+static int forward_ragged(rb_model* m, const uint32_t* tokens, int batch, int seq, int pos, const int32_t* lens, void* logits_out) {
+  RB_REQUIRE(batch > 0 && seq > 0, "ragged forward: bad sizes");
+  std::vector<int32_t> rows((size_t)batch);
+  for (int b = 0; b < batch; ++b) {
+    RB_REQUIRE(lens[b] >= 1 && lens[b] <= seq, "ragged forward: sequence %d has %d valid tokens of %d", b, lens[b], seq);
+    rows[b] = b * seq + lens[b] - 1;
+  }
+  return forward_rows(m, tokens, batch, seq, pos, lens, rows.data(), batch, logits_out);
 }
 
 extern "C" int32_t rb_model_forward_ragged(rb_model* m, const uint32_t* tokens_dev, int32_t batch, int32_t seq, int32_t pos,
                                            const int32_t* lens_host, void* logits_dev) {
   RB_REQUIRE(m && tokens_dev && lens_host, "rb_model_forward_ragged: null argument");
   return forward_ragged(m, tokens_dev, batch, seq, pos, lens_host, logits_dev);
+}
+
+extern "C" int32_t rb_model_forward_rows(rb_model* m, const uint32_t* tokens_dev, int32_t batch, int32_t seq, int32_t pos,
+                                         const int32_t* lens_host, const int32_t* rows_host, int32_t n_rows, void* logits_dev) {
+  RB_REQUIRE(m && tokens_dev && (n_rows == 0 || (rows_host && logits_dev)), "rb_model_forward_rows: null argument");
+  return forward_rows(m, tokens_dev, batch, seq, pos, lens_host, rows_host, n_rows, logits_dev);
+}
+
+extern "C" int32_t rb_model_keep_sequences(rb_model* m, const int32_t* keep, int32_t n) {
+  RB_REQUIRE(m && (keep || n == 0), "rb_model_keep_sequences: null argument");
+  const int B = m->cfg.max_batch;
+  RB_REQUIRE(n >= 0 && n <= B, "rb_model_keep_sequences: %d sequences of %d", n, B);
+  std::vector<int32_t> order;
+  std::vector<char> used((size_t)B, 0);
+  for (int i = 0; i < n; ++i) {
+    RB_REQUIRE(keep[i] >= 0 && keep[i] < B && !used[keep[i]], "rb_model_keep_sequences: sequence %d is out of range or listed twice", keep[i]);
+    used[keep[i]] = 1;
+    order.push_back(keep[i]);
+  }
+  for (int b = 0; b < B; ++b)
+    if (!used[b]) { order.push_back(b); m->cache->host_lens[b] = 0; }
+  RB_TRY(kv_cache_permute(m->cache, order));
+  if (m->hist_count) {  // the sampler's per-sequence history moves along
+    std::vector<int32_t> hist((size_t)B * 256), count(B);
+    std::vector<uint8_t> fin(B);
+    RB_CUDA(cudaMemcpy(hist.data(), m->hist, hist.size() * sizeof(int32_t), cudaMemcpyDeviceToHost));
+    RB_CUDA(cudaMemcpy(count.data(), m->hist_count, count.size() * sizeof(int32_t), cudaMemcpyDeviceToHost));
+    RB_CUDA(cudaMemcpy(fin.data(), m->finished, fin.size(), cudaMemcpyDeviceToHost));
+    std::vector<int32_t> h2(hist.size(), 0), c2(B, 0);
+    std::vector<uint8_t> f2(B, 0);
+    const size_t cap = (size_t)m->rep_last_n;
+    for (int i = 0; i < n; ++i) {
+      for (size_t j = 0; j < cap; ++j) h2[i * cap + j] = hist[order[i] * cap + j];
+      c2[i] = count[order[i]];
+      f2[i] = fin[order[i]];
+    }
+    RB_CUDA(cudaMemcpy(m->hist, h2.data(), h2.size() * sizeof(int32_t), cudaMemcpyHostToDevice));
+    RB_CUDA(cudaMemcpy(m->hist_count, c2.data(), c2.size() * sizeof(int32_t), cudaMemcpyHostToDevice));
+    RB_CUDA(cudaMemcpy(m->finished, f2.data(), f2.size(), cudaMemcpyHostToDevice));
+  }
+  return RB_OK;
+}
+
+extern "C" int32_t rb_model_logits_dtype(rb_model* m) { return m ? m->logits_dtype : RB_ERR_INVALID; }
+
+extern "C" int32_t rb_model_set_layer_trace(rb_model* m, float* dst_dev) {
+  RB_REQUIRE(m && m->layered, "rb_model_set_layer_trace: not a layered model");
+  m->layer_trace = dst_dev;
+  return RB_OK;
 }
 
 extern "C" int32_t rb_model_forward(rb_model* m, const uint32_t* tokens_dev, int32_t batch, int32_t seq, int32_t pos,
@@ -1125,14 +1148,15 @@ int history_push(rb_model* m, const uint32_t* ids, int batch, int seq, const int
 }
 
 int sample_tokens(rb_model* m, int batch, uint32_t* out) {
-  if (!sampling_on(m)) return rb_argmax_rows(m->ctx, m->logits, m->cfg.dtype, batch, m->cfg.vocab_size, out);
-  return rb_sample_greedy(m->ctx, m->logits, m->cfg.dtype, batch, m->cfg.vocab_size, m->rep_penalty, m->hist, m->rep_last_n,
+  if (!sampling_on(m)) return rb_argmax_rows(m->ctx, m->logits, m->logits_dtype, batch, m->cfg.vocab_size, out);
+  return rb_sample_greedy(m->ctx, m->logits, m->logits_dtype, batch, m->cfg.vocab_size, m->rep_penalty, m->hist, m->rep_last_n,
                           m->hist_count, m->eos, m->finished, out);
 }
 
 // Whatever host-side state shapes the launches of a decode step: a captured step is reused only
 // while this stays the same (today: how many KV splits the attention uses).
 int decode_plan(rb_model* m, int batch) {
+  if (m->layered) return layered_decode_plan(m, batch);
   int max_len = 0;
   for (int b = 0; b < batch; ++b) max_len = std::max(max_len, m->cache->host_lens[b]);
   return attention_decode_splits(m->ctx, batch, m->nkv_l, max_len, m->d);
@@ -1161,7 +1185,7 @@ int decode_step(rb_model* m, int batch) {
                "decode: position %d of sequence %d exceeds the cache / rotary table capacity", c->host_lens[b], b);
   for (int b = 0; b < batch; ++b) c->host_lens[b] += 1;
   const int plan = decode_plan(m, batch);
-  const bool graphable = m->use_graph && !ctx->profiling && !ctx->debug_simple;
+  const bool graphable = m->use_graph && !ctx->profiling && !ctx->debug_simple && !m->layer_trace;
   if (graphable && m->step_graph && m->graph_batch == batch && m->graph_plan == plan) {
     RB_CUDA(cudaGraphLaunch(m->step_graph, ctx->stream));
     ctx->launches += m->graph_launches;

@@ -10,7 +10,8 @@ namespace rb {
 template <typename T, bool GATED>
 __global__ void gemm_plain_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ w2,
                                   const T* __restrict__ bias, const T* __restrict__ residual, T* __restrict__ out,
-                                  float* __restrict__ part, int m, int n, int k, int act, int k_per_split) {
+                                  float* __restrict__ part, int m, int n, int k, int act, const T* __restrict__ act_params,
+                                  int k_per_split) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float xs[BK][BM + 1];
   __shared__ float ws[BK][BN + 1];
@@ -18,6 +19,7 @@ __global__ void gemm_plain_kernel(const T* __restrict__ x, const T* __restrict__
   const int tm = blockIdx.y * BM, tn = blockIdx.x * BN;
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
   const int k0 = blockIdx.z * k_per_split, k1 = min(k, k0 + k_per_split);
+  const float2 ac = act == RB_ACT_XIELU ? xielu_consts(act_params) : make_float2(0.f, 0.f);
   float acc[4][4] = {}, acc2[4][4] = {};
   for (int kk = k0; kk < k1; kk += BK) {
     for (int i = threadIdx.x; i < BM * BK; i += blockDim.x) {
@@ -58,7 +60,7 @@ __global__ void gemm_plain_kernel(const T* __restrict__ x, const T* __restrict__
         v = act_apply(act, v) * acc2[i][j];
       } else {
         if (bias) v += Cvt<T>::to_f(bias[c]);
-        v = act_apply(act, v);
+        v = act_apply(act, v, ac);
         if (residual) v += Cvt<T>::to_f(residual[(size_t)r * n + c]);
       }
       out[(size_t)r * n + c] = Cvt<T>::from_f(v);
@@ -72,7 +74,8 @@ template <bool GATED>
 __global__ void __launch_bounds__(256) gemv_f32_kernel(const float* __restrict__ x, const float* __restrict__ w,
                                                        const float* __restrict__ w2, const float* __restrict__ bias,
                                                        const float* __restrict__ residual, float* __restrict__ out, int m,
-                                                       int n, int k, int act, int vec) {
+                                                       int n, int k, int act, const float* __restrict__ act_params, int vec) {
+  const float2 ac = act == RB_ACT_XIELU ? xielu_consts(act_params) : make_float2(0.f, 0.f);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int col = blockIdx.x * 8 + warp;
   if (col >= n) return;
@@ -116,7 +119,7 @@ __global__ void __launch_bounds__(256) gemv_f32_kernel(const float* __restrict__
       v = act_apply(act, v) * v2;
     } else {
       if (bias) v += bias[col];
-      v = act_apply(act, v);
+      v = act_apply(act, v, ac);
       if (residual) v += residual[(size_t)r * n + col];
     }
     out[(size_t)r * n + col] = v;
@@ -131,7 +134,8 @@ template <typename T>
 __global__ void __launch_bounds__(kPlainAttnWarps * 32)
 attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                        const int32_t* __restrict__ block_table, const int32_t* __restrict__ seq_lens, int pages_per_seq,
-                       int s_new, int q_heads, int kv_heads, int d, float scale, int window, T* __restrict__ out) {
+                       int s_new, int q_heads, int kv_heads, int d, float scale, int window, T* __restrict__ out, int ext,
+                       const AttnExtra x) {
   __shared__ float sm_m[kPlainAttnWarps], sm_l[kPlainAttnWarps], sm_o[kPlainAttnWarps][256];
   const int m = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -147,9 +151,11 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
   }
   float mx = -INFINITY, l = 0.f;
   const int call_base = seq_lens[b] - s_new;  // first token of this call
-  for (int t = warp; t <= limit; t += kPlainAttnWarps) {
+  const int first = ext && x.window > 0 ? max(0, limit - x.window + 1) : 0;
+  const float slope = ext && x.alibi ? alibi_slope(h, q_heads) : 0.f;
+  for (int t = first + warp; t <= limit; t += kPlainAttnWarps) {
     // sliding window (qwen2.rs:316-334): it acts among the tokens of one call only, the cached prefix stays visible
-    if (t >= call_base && t + window < limit) continue;
+    if (!ext && t >= call_base && t + window < limit) continue;
     const int page = block_table[(size_t)b * pages_per_seq + t / kPageTokens];
     const size_t off = (((size_t)page * kv_heads + kvh) * kPageTokens + (t % kPageTokens)) * d;
     float dot = 0.f;
@@ -158,7 +164,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
       const int i = lane + 32 * j;
       if (i < d) dot += qv[j] * Cvt<T>::to_f(k_cache[off + i]);
     }
-    dot = warp_sum(dot) * scale;
+    dot = fmaf(-slope, (float)(limit - t), warp_sum(dot) * scale);
     const float mn = fmaxf(mx, dot);
     const float corr = expf(mx - mn), p = expf(dot - mn);
     l = l * corr + p;
@@ -186,7 +192,15 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
     float O = 0.f;
 #pragma unroll
     for (int w = 0; w < kPlainAttnWarps; ++w) O += (sm_m[w] == -INFINITY) ? 0.f : sm_o[w][i] * expf(sm_m[w] - M);
-    out[((size_t)m * q_heads + h) * d + i] = Cvt<T>::from_f(O / L);
+    if (ext) {
+      if (i >= x.value_dim) continue;
+      const int col = h * x.value_dim + i;
+      float y = O / L;
+      if (x.gate) y *= sigmoid_f(Cvt<T>::to_f(((const T*)x.gate)[(size_t)m * x.gate_ld + col]));
+      out[(size_t)m * x.out_ld + col] = Cvt<T>::from_f(y);
+    } else {
+      out[((size_t)m * q_heads + h) * d + i] = Cvt<T>::from_f(O / L);
+    }
   }
 }
 
@@ -197,11 +211,11 @@ static bool gemv_f32_launch(rb_ctx* ctx, const GemmArgs& a) {
   const dim3 grid((unsigned)((a.n + 7) / 8));
   if (a.w2)
     gemv_f32_kernel<true><<<grid, 256, 0, ctx->stream>>>((const float*)a.x, (const float*)a.w, (const float*)a.w2, nullptr, nullptr,
-                                                         (float*)a.out, (int)a.m, (int)a.n, (int)a.k, a.act, vec);
+                                                         (float*)a.out, (int)a.m, (int)a.n, (int)a.k, a.act, nullptr, vec);
   else
     gemv_f32_kernel<false><<<grid, 256, 0, ctx->stream>>>((const float*)a.x, (const float*)a.w, nullptr, (const float*)a.bias,
                                                           (const float*)a.residual, (float*)a.out, (int)a.m, (int)a.n, (int)a.k,
-                                                          a.act, vec);
+                                                          a.act, (const float*)a.act_params, vec);
   ctx->launches++;
   return true;
 }
@@ -215,17 +229,18 @@ static int gemm_plain_launch(rb_ctx* ctx, const GemmArgs& a) {
   if (a.w2)
     gemm_plain_kernel<T, true><<<grid, 256, 0, ctx->stream>>>((const T*)a.x, (const T*)a.w, (const T*)a.w2, nullptr,
                                                              nullptr, (T*)a.out, nullptr, (int)a.m, (int)a.n, (int)a.k,
-                                                             a.act, kps);
+                                                             a.act, nullptr, kps);
   else
     gemm_plain_kernel<T, false><<<grid, 256, 0, ctx->stream>>>(
         (const T*)a.x, (const T*)a.w, nullptr, (const T*)a.bias, (const T*)a.residual, a.partials ? nullptr : (T*)a.out,
-        a.partials ? (float*)a.out : nullptr, (int)a.m, (int)a.n, (int)a.k, a.act, kps);
+        a.partials ? (float*)a.out : nullptr, (int)a.m, (int)a.n, (int)a.k, a.act, (const T*)a.act_params, kps);
   ctx->launches++;
   return launch_status("gemm_plain");
 }
 
 int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype) {
   if (a.m == 0 || a.n == 0) return RB_OK;
+  RB_REQUIRE(a.act != RB_ACT_XIELU || (a.act_params && !a.w2), "gemm: RB_ACT_XIELU needs its parameters and an ungated product");
   if (dtype == RB_F32) {
     if (gemv_f32_launch(ctx, a)) return launch_status("gemv_f32");
     return gemm_plain_launch<float>(ctx, a);
@@ -235,18 +250,20 @@ int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype) {
 }
 
 int attention_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
-                     float scale, void* out, int dtype) {
+                     float scale, void* out, int dtype, const AttnExtra* ext) {
+  const AttnExtra x = ext ? *ext : AttnExtra();
   const size_t loff = (size_t)layer * c->layer_stride_elems();
   const int warps = kPlainAttnWarps;
   dim3 grid((unsigned)(batch * s_new), (unsigned)q_heads);
   if (dtype == RB_F32)
     attention_plain_kernel<float><<<grid, warps * 32, 0, ctx->stream>>>(
         (const float*)q, (const float*)c->k + loff, (const float*)c->v + loff, c->block_table, c->seq_lens,
-        c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (float*)out);
+        c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (float*)out, ext ? 1 : 0, x);
   else if (dtype == RB_BF16)
     attention_plain_kernel<__nv_bfloat16><<<grid, warps * 32, 0, ctx->stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)c->k + loff, (const __nv_bfloat16*)c->v + loff, c->block_table,
-        c->seq_lens, c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (__nv_bfloat16*)out);
+        c->seq_lens, c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (__nv_bfloat16*)out,
+        ext ? 1 : 0, x);
   else
     return fail(RB_ERR_DTYPE, "attention: dtype %d unsupported", dtype);
   ctx->launches++;

@@ -4,6 +4,7 @@ phi2 / phi3 / gemma twins).  torch is used for device memory of inputs and outpu
 from __future__ import annotations
 
 import ctypes
+import os
 from typing import Dict, Iterable, Optional
 
 import numpy as np
@@ -37,7 +38,8 @@ class Model:
         self._struct = configs.to_struct(cfg, dtype, max_batch, max_seq, self.max_tokens, tp_rank, tp_size)
         self._m = ctypes.c_void_p()
         device.use_torch_stream()
-        _lib.call("rb_model_create", device.ctx, ctypes.byref(self._struct), ctypes.byref(self._m))
+        configs.create_model(device.ctx, cfg, self._struct, self._m)
+        self.logits_dtype = _TORCH_DTYPE[_lib.lib().rb_model_logits_dtype(self._m)]
         self._finalized = False
 
     # ---- parameters -----------------------------------------------------------------------
@@ -49,7 +51,7 @@ class Model:
         """Tensor::update_by_name (rai-core/src/nn.rs:192-205): cast to the model dtype and copy.
         `value` is a numpy float32 array, or a torch tensor (float32 / bfloat16, host or this GPU)."""
         if isinstance(value, np.ndarray):
-            arr = np.ascontiguousarray(value, dtype=np.float32)
+            arr = np.array(value, dtype=np.float32, order="C")  # (keeps a single number's rank 0)
             _lib.call("rb_model_load_param", self._m, name.encode(), ctypes.c_void_p(arr.ctypes.data), 0, _lib.F32,
                       arr.ndim, _shape_array(arr.shape))
             return
@@ -99,7 +101,7 @@ class Model:
         ids = self._tokens_dev(tokens)
         b, s = ids.shape
         self.device.use_torch_stream()
-        logits = torch.empty((b, self.cfg["vocab_size"]), dtype=_TORCH_DTYPE[self.dtype], device=ids.device)
+        logits = torch.empty((b, self.cfg["vocab_size"]), dtype=self.logits_dtype, device=ids.device)
         _lib.call("rb_model_forward", self._m, ctypes.c_void_p(ids.data_ptr()), b, s, int(seqlen_offset),
                   ctypes.c_void_p(logits.data_ptr()))
         self.device.synchronize()
@@ -112,11 +114,43 @@ class Model:
         b, s = ids.shape
         lens_arr = np.ascontiguousarray(np.asarray(lens, dtype=np.int32))
         self.device.use_torch_stream()
-        logits = torch.empty((b, self.cfg["vocab_size"]), dtype=_TORCH_DTYPE[self.dtype], device=ids.device)
+        logits = torch.empty((b, self.cfg["vocab_size"]), dtype=self.logits_dtype, device=ids.device)
         _lib.call("rb_model_forward_ragged", self._m, ctypes.c_void_p(ids.data_ptr()), b, s, int(seqlen_offset),
                   lens_arr.ctypes.data_as(ctypes.c_void_p), ctypes.c_void_p(logits.data_ptr()))
         self.device.synchronize()
         return logits
+
+    def forward_rows(self, tokens, lens=None, rows=(), seqlen_offset: int = -1) -> torch.Tensor:
+        """The general step: tokens [B, S], lens[b] (0..S, None = S) of them real in row b, logits [len(rows), V] of the
+        positions rows[i] = b * S + s.  seqlen_offset -1 continues every sequence at its own length."""
+        ids = self._tokens_dev(tokens)
+        b, s = ids.shape
+        lens_arr = None if lens is None else np.ascontiguousarray(np.asarray(lens, dtype=np.int32))
+        rows_arr = np.ascontiguousarray(np.asarray(rows, dtype=np.int32))
+        self.device.use_torch_stream()
+        logits = torch.empty((len(rows_arr), self.cfg["vocab_size"]), dtype=self.logits_dtype, device=ids.device)
+        _lib.call("rb_model_forward_rows", self._m, ctypes.c_void_p(ids.data_ptr()), b, s, int(seqlen_offset),
+                  None if lens_arr is None else lens_arr.ctypes.data_as(ctypes.c_void_p), rows_arr.ctypes.data_as(ctypes.c_void_p),
+                  len(rows_arr), ctypes.c_void_p(logits.data_ptr()))
+        self.device.synchronize()
+        return logits
+
+    def keep_sequences(self, keep) -> None:
+        """Sequences keep[0], keep[1], ... become sequences 0, 1, ...; the others give their pages and state back."""
+        arr = np.ascontiguousarray(np.asarray(keep, dtype=np.int32))
+        self.device.use_torch_stream()
+        _lib.call("rb_model_keep_sequences", self._m, arr.ctypes.data_as(ctypes.c_void_p), len(arr))
+
+    def forward_layers(self, tokens, seqlen_offset: int = 0) -> torch.Tensor:
+        """Test hook (layer-by-layer designs): the residual stream after every layer, [layers, B * S, width] float32."""
+        ids = self._tokens_dev(tokens)
+        out = torch.zeros((len(self.cfg["layers"]), ids.numel(), self.cfg["hidden_size"]), dtype=torch.float32, device=ids.device)
+        _lib.call("rb_model_set_layer_trace", self._m, ctypes.c_void_p(out.data_ptr()))
+        try:
+            self.forward(tokens, seqlen_offset)
+        finally:
+            _lib.call("rb_model_set_layer_trace", self._m, None)
+        return out
 
     def generate_ragged(self, prompts, steps: int) -> np.ndarray:
         """Generation for prompts of different lengths in one batch (a list of 1-D token arrays): right-pad, one
@@ -166,7 +200,8 @@ class Model:
         for _ in range(steps):
             logits = self.forward(ids, pos).reshape(b, -1)
             pos += ids.shape[1]
-            _lib.call("rb_argmax_rows", self.device.ctx, ctypes.c_void_p(logits.data_ptr()), self.dtype, b,
+            _lib.call("rb_argmax_rows", self.device.ctx, ctypes.c_void_p(logits.data_ptr()),
+                      _lib.F32 if self.logits_dtype == torch.float32 else _lib.BF16, b,
                       logits.shape[1], ctypes.c_void_p(argmax.data_ptr()))
             self.device.synchronize()
             toks.append(argmax.clone())
@@ -234,6 +269,18 @@ class Model:
             safetensors_io.write_safetensors(path, {k: v.float().numpy() for k, v in named.items()}, "BF16")
         else:
             safetensors_io.write_safetensors(path, {k: v.numpy() for k, v in named.items()}, "F32")
+
+    @classmethod
+    def from_pretrained(cls, folder: str, dtype: int, device: Cuda, max_batch: int, max_seq: int,
+                        max_tokens: Optional[int] = None) -> "Model":
+        """The model in a checkpoint folder: its architecture and sizes from config.json, its weights from every
+        *.safetensors file there."""
+        files = sorted(os.path.join(folder, f) for f in os.listdir(folder) if f.endswith(".safetensors"))
+        if not files:
+            raise _lib.RaiB200Error(-8, f"no .safetensors file in {folder}")
+        m = cls(configs.from_json(folder), dtype, device, max_batch, max_seq, max_tokens)
+        m.update_by_safetensors(files)
+        return m
 
     def param_bytes(self) -> int:
         return int(_lib.lib().rb_model_param_bytes(self._m))

@@ -21,6 +21,8 @@ from . import configs
 def param_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     """[(name, shape, kind)] in checkpoint order; kind is 'matrix', 'bias', 'norm_w' or 'norm_b'."""
     a = cfg["arch"]
+    if a == "malasun":
+        return _malasun_shapes(cfg)
     H, I, V = cfg["hidden_size"], cfg["intermediate_size"], cfg["vocab_size"]
     nq = cfg["num_attention_heads"]
     nkv = cfg.get("num_key_value_heads") or nq
@@ -68,11 +70,50 @@ def param_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     return out
 
 
+def _malasun_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """Kinds beside the usual ones: 'fan_in' (a matrix that keeps its input's scale), 'gain' (one number), 'conv', 'lower'
+    (lower bounds of forget gates, in [0, 1)), 'forget_b' (their biases) and 'act' (the activation's two numbers)."""
+    W, V = cfg["hidden_size"], cfg["vocab_size"]
+    out: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        mix, mlp, p = layer["mixer"], layer["mlp"], f"l{i}."
+        H, d, e = mix["heads"], mix["dim"], mix["vdim"]
+        out.append((p + "norm1", (), "gain"))
+        if mlp:
+            out.append((p + "norm2", (), "gain"))
+        m = p + "mix."
+        if mix["type"] == "hgrn2":
+            out += [(m + "q", (H * d, W), "fan_in"), (m + "f", (H * d, W), "fan_in"), (m + "f.b", (H * d,), "forget_b"),
+                    (m + "lower", (H * d,), "lower"), (m + "v", (H * e, W), "fan_in"), (m + "norm", (e,), "norm_w")]
+        else:
+            parts = [("q", H * d)] + ([] if mix["kv_from"] is not None else [("k", mix["kv_heads"] * d), ("v", mix["kv_heads"] * e)])
+            for n, rows in parts:
+                out += [(m + n, (rows, W), "fan_in"), (m + n + ".b", (rows,), "bias"), (m + n + ".conv", (rows, mix["conv"]), "conv")]
+                if n != "v":
+                    out.append((m + n + ".norm", (rows,), "norm_w"))
+            out.append((m + "g", (H * e, W), "fan_in"))
+        out.append((m + "o", (W, H * e), "fan_in"))
+        if mlp:
+            out += [(p + "mlp.up", (mlp["ff"], W), "fan_in"), (p + "mlp.down", (W, mlp["ff"]), "fan_in"), (p + "mlp.act", (2,), "act")]
+    return out + [("final.norm", (), "gain"), ("head", (V, W), "fan_in")]
+
+
 def bf16_round(x: np.ndarray) -> np.ndarray:
     """float32 -> nearest-even bfloat16 -> float32 (so the CPU oracle and the GPU see the same values)."""
     u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
     r = ((u >> 16) & 1) + np.uint32(0x7FFF)
     return ((u + r) & np.uint32(0xFFFF0000)).view(np.float32)
+
+
+_DRAWS = {
+    "embed": lambda r, s: r.standard_normal(s),
+    "fan_in": lambda r, s: r.standard_normal(s) / np.sqrt(s[1]),
+    "gain": lambda r, s: 1.0 + 0.2 * r.standard_normal(s),
+    "conv": lambda r, s: r.standard_normal(s) / np.sqrt(s[1]),
+    "lower": lambda r, s: r.uniform(0.0, 0.9, s),
+    "forget_b": lambda r, s: r.uniform(0.0, 6.0, s),
+    "act": lambda r, s: r.uniform(-1.0, 1.0, s),
+}
 
 
 def iter_weights(cfg: dict, seed: int, round_bf16: bool = True) -> Iterator[Tuple[str, np.ndarray]]:
@@ -86,9 +127,11 @@ def iter_weights(cfg: dict, seed: int, round_bf16: bool = True) -> Iterator[Tupl
         elif kind == "norm_w":
             base = 0.0 if gemma else 1.0
             w = (base + rng.standard_normal(shape, dtype=np.float32) * np.float32(0.05)).astype(np.float32)
+        elif kind in _DRAWS:
+            w = np.asarray(_DRAWS[kind](rng, shape), dtype=np.float32)
         else:
             w = (rng.standard_normal(shape, dtype=np.float32) * np.float32(0.02)).astype(np.float32)
-        yield name, (bf16_round(w) if round_bf16 else w)
+        yield name, (bf16_round(w) if round_bf16 else w).reshape(shape)
 
 
 def weights(cfg: dict, seed: int, round_bf16: bool = True) -> Dict[str, np.ndarray]:

@@ -48,6 +48,15 @@ def test_model_config_struct_matches_header():
     assert fields == [f[0] for f in _lib.ModelConfig._fields_]
 
 
+def test_layer_config_struct_matches_header():
+    import re
+    text = _lib.HEADER.read_text()
+    body = re.search(r"typedef struct rb_layer_config \{(.*?)\} rb_layer_config;", text, flags=re.S).group(1)
+    body = re.sub(r"/\*.*?\*/", "", body, flags=re.S)
+    fields = [ln.split()[-1].rstrip(";") for ln in body.splitlines() if ln.strip().endswith(";")]
+    assert fields == [f[0] for f in _lib.LayerConfig._fields_]
+
+
 def test_no_cpu_fallback_without_gpu(library):
     """On a machine without a GPU the context cannot be created and the error says why."""
     import torch
