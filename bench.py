@@ -55,6 +55,10 @@ def parse_args():
     ap.add_argument("--skip-parity", action="store_true", help="skip the oracle comparison that follows the timed region")
     ap.add_argument("--skip-other-configs", action="store_true",
                     help="skip the short decode runs of the other benchmark configurations (single-GPU default run only)")
+    ap.add_argument("--design", default="", choices=["", "malasun"],
+                    help="instead of the headline: prefill and decode of this design at a few sizes, each beside a qwen2 "
+                         "model of equal width, heads, depth and parameter count (one JSON line)")
+    ap.add_argument("--design-sizes", default="malasun-1k,malasun-2k,malasun-4k")
     ap.add_argument("--skip-fill", action="store_true",
                     help="leave the KV cache zero-filled instead of prefilling it (same traffic; for profiler runs)")
     return ap.parse_args()
@@ -620,8 +624,144 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+# --------------------------------------------------------------------------------------------------
+# A design beside its closest relative among the reference's families, at equal size
+# --------------------------------------------------------------------------------------------------
+PROFILE_CLASSES = ["gemm", "attention", "norm", "rope_kv", "embed", "argmax", "other", "recurrence"]
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12   # FMA pipe of 148 SMs at the maximum SM clock: the recurrence's float32 peak
+
+
+def random_param(kind, shape, gen):
+    """One random tensor of a synth.param_shapes kind, on the device."""
+    import torch
+    n = lambda: torch.randn(shape, generator=gen, device="cuda")  # noqa: E731
+    u = lambda lo, hi: torch.rand(shape, generator=gen, device="cuda") * (hi - lo) + lo  # noqa: E731
+    w = {"norm_w": lambda: torch.ones(shape, device="cuda"), "gain": lambda: torch.ones(shape, device="cuda"), "embed": n,
+         "fan_in": lambda: n() / shape[1] ** 0.5, "conv": lambda: n() / shape[1] ** 0.5, "lower": lambda: u(0.0, 0.9),
+         "forget_b": lambda: u(0.0, 6.0), "act": lambda: u(-1.0, 1.0)}.get(kind, lambda: n() * 0.02)()
+    return w.to(torch.bfloat16)
+
+
+def equal_size_qwen2(cfg):
+    """qwen2 with the design's width, heads, depth and (through its gated feed-forward's size) parameter count."""
+    from rai_b200 import synth
+    import math
+    attn = [x["mixer"] for x in cfg["layers"] if x["mixer"]["type"] == "attention"][0]
+    c = dict(arch="qwen2", vocab_size=cfg["vocab_size"], hidden_size=cfg["hidden_size"], intermediate_size=128,
+             num_hidden_layers=len(cfg["layers"]), num_attention_heads=attn["heads"], num_key_value_heads=attn["kv_heads"],
+             max_position_embeddings=8192, sliding_window=1 << 30, rope_theta=1e6, rms_norm_eps=1e-6, hidden_act="silu",
+             tie_word_embeddings=False)
+    count = lambda k: sum(math.prod(s) for _, s, _ in synth.param_shapes(k))  # noqa: E731
+    missing = count(cfg) - count(c)
+    c["intermediate_size"] += max(0, round(missing / (3 * c["hidden_size"] * c["num_hidden_layers"]) / 128)) * 128
+    return c, count(cfg), count(c)
+
+
+def class_profile(dev, peaks, run):
+    """One launch-by-launch pass: per kernel class its time and how far it is from its roofline (the slower of its
+    algorithmic bytes at copy speed and its operations at the peak of the pipe it runs on)."""
+    from rai_b200 import _lib
+    _lib.call("rb_profile_start", dev.ctx)
+    run()
+    out = {}
+    for i, name in enumerate(PROFILE_CLASSES):
+        v = (ctypes.c_double * 4)()
+        _lib.call("rb_profile_read", dev.ctx, i, v)
+        if v[0] == 0:
+            continue
+        tflops = FP32_TFLOPS if name == "recurrence" else peaks["bf16_tflops"]
+        ideal_ms = max(v[2] / peaks["hbm_gbs"] / 1e6, v[3] / tflops / 1e9)
+        out[name] = {"launches": int(v[0]), "ms": round(v[1], 4), "us_per_launch": round(v[1] / v[0] * 1e3, 2),
+                     "gbs": round(v[2] / v[1] / 1e6, 1), "tflops": round(v[3] / v[1] / 1e9, 1),
+                     "of_roofline": round(ideal_ms / v[1], 3)}
+    return out
+
+
+def design_arm(cfg, args, peaks):
+    """Decode and prefill of one configuration: device-timed throughput, and the per-class profile of each."""
+    import torch
+    from rai_b200 import _lib, synth
+    from rai_b200.device import Cuda
+    from rai_b200.models import Model
+    dev = Cuda(0)
+    B, T0, K, W, PB, PS = args.decode_batch, args.context, args.steps, args.warmup, args.prefill_batch, args.prefill_len
+    model = Model(cfg, _lib.BF16, dev, max(B, PB), max(T0 + K + W + 64, PS), max(B * 256, PB * PS))
+    gen = torch.Generator(device="cuda").manual_seed(1234)
+    for name, shape, kind in synth.param_shapes(cfg):
+        model.update_param(name, random_param(kind, shape, gen))
+    model.finalize()
+    cache = ctypes.c_void_p(_lib.lib().rb_model_kv_cache(model._m))
+    ids = lambda b, s: torch.randint(0, cfg["vocab_size"], (b, s), generator=gen, device="cuda", dtype=torch.int32)  # noqa: E731
+    call = lambda t, pos: _lib.call("rb_model_forward", model._m, ctypes.c_void_p(t.data_ptr()), t.shape[0], t.shape[1], pos, None)  # noqa: E731
+
+    def timed(fn):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        dev.synchronize()
+        a.record()
+        fn()
+        b.record()
+        dev.synchronize()
+        return a.elapsed_time(b)
+
+    prompt = ids(PB, PS)
+
+    def prefill():
+        model.clear_kv_cache()
+        call(prompt, 0)
+    for _ in range(max(3, min(W, 5))):
+        prefill()
+    sampler = ClockSampler(0)
+    sampler.start()
+    t0 = sampler.mark()
+    prefill_ms = timed(lambda: [prefill() for _ in range(5)]) / 5
+    prefill_classes = class_profile(dev, peaks, prefill)
+    # decode: a filled cache, W warm-up steps (which also capture the step), then K timed ones from the same context
+    model.clear_kv_cache()
+    for pos in range(0, T0, 256):
+        call(ids(B, min(256, T0 - pos)), pos)
+    first = ids(B, 1).reshape(B)
+    rewind = lambda: _lib.call("rb_kv_cache_set_len", cache, B, T0)  # noqa: E731
+    model.decode_loop(first, T0, max(3, W))
+    dev.synchronize()
+    rewind()
+    decode_ms = timed(lambda: model.decode_loop(first, T0, K)) / K
+    graph = bool(_lib.lib().rb_model_decode_graph_active(model._m))
+    t1 = sampler.mark()
+    sampler.stop()
+    rewind()
+    decode_classes = class_profile(dev, peaks, lambda: model.decode_loop(first, T0, 1))
+    timeline = None
+    if not args.skip_timeline:
+        try:
+            timeline = decode_timeline(model, dev, lambda n: rewind(), first, T0)
+        except Exception as e:
+            timeline = {"error": f"{type(e).__name__}: {e}"}
+    model.close()
+    return {"prefill_tok_s": PB * PS / prefill_ms * 1e3, "prefill_ms": prefill_ms, "decode_tok_s": B / decode_ms * 1e3,
+            "decode_ms": decode_ms, "graph": graph, "clocks": sampler.summary(t0, t1), "prefill_classes": prefill_classes,
+            "decode_classes": decode_classes, "decode_timeline": timeline}
+
+
+def run_design(args):
+    from rai_b200 import configs
+    peaks, kind = measured_peaks()
+    rows = {}
+    for name in args.design_sizes.split(","):
+        cfg = configs.get(name)
+        other, n_ours, n_other = equal_size_qwen2(cfg)
+        rows[name] = {"layers": len(cfg["layers"]), "width": cfg["hidden_size"], "params": n_ours, "qwen2_params": n_other,
+                      "design": design_arm(cfg, args, peaks), "qwen2": design_arm(other, args, peaks)}
+    print(json.dumps({"design": args.design, "dtype": "bf16", "data": "synthetic", "peaks": peaks, "peak_kind": kind,
+                      "decode": f"batch {args.decode_batch}, context {args.context}, {args.steps} steps",
+                      "prefill": f"{args.prefill_batch} x {args.prefill_len}",
+                      "l2": "weights and cache of a step are larger than L2", "sizes": rows}), flush=True)
+
+
 def main():
     args = parse_args()
+    if args.design:
+        run_design(args)
+        return
     if args.impl == "reference":
         run_reference(args)
     else:

@@ -106,9 +106,9 @@ def _malasun_bench(vocab: int, width: int, heads: int, kv_heads: int, ff: int, p
 
 MALASUN: Dict[str, dict] = {
     # sizes that resemble a real model's layers, for throughput measurements (random weights)
-    "malasun-1k": _malasun_bench(32000, 1024, 8, 2, 4096, 2, 1024),
-    "malasun-2k": _malasun_bench(32000, 2048, 16, 4, 8192, 2, 1024),
-    "malasun-4k": _malasun_bench(32000, 4096, 32, 8, 16384, 2, 1024),
+    "malasun-1k": _malasun_bench(32000, 1024, 8, 2, 4096, 8, 1024),
+    "malasun-2k": _malasun_bench(32000, 2048, 16, 4, 8192, 6, 1024),
+    "malasun-4k": _malasun_bench(32000, 4096, 32, 8, 16384, 3, 1024),
     # small models for tests
     "tiny-malasun": _malasun(320, 160, [
         malasun_layer("attention", 4, 40, 32, 200, 2, 4, 21), malasun_layer("hgrn2", 3, 32, 48, 0),

@@ -1,7 +1,8 @@
 // Kernels of the layer-by-layer designs (layered.cu): a float32 residual stream with the norm on a sublayer's output,
-// the short causal convolution with query/key norm and cache append, and the HGRN2 recurrence.  Rows have a pitch that
+// and the short causal convolution with query/key norm and cache append.  Rows have a pitch that
 // is a multiple of 8 elements and zero padding, so every row access is a 16-byte piece; all arithmetic is float32.
 #include <algorithm>
+#include <type_traits>
 
 #include "ctx.h"
 
@@ -125,7 +126,7 @@ struct ConvArgs {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(256) conv_norm_append_kernel(const ConvArgs<T> a) {
+__global__ void __launch_bounds__(512) conv_norm_append_kernel(const ConvArgs<T> a) {
   extern __shared__ float row_s[];  // one row of q, k, v after the convolution
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -152,9 +153,10 @@ __global__ void __launch_bounds__(256) conv_norm_append_kernel(const ConvArgs<T>
     const bool is_token = !a.new_lens || s < a.new_lens[b];
     float* ring = hist > 0 ? a.ring + (size_t)a.slots[b] * hist * C : nullptr;
     float sq = 0.f, sk = 0.f;
-    for (int c = threadIdx.x * 8; c < C; c += blockDim.x * 8) {
+    for (int c = threadIdx.x * 8; c < C + (a.gate_out ? a.gp : 0); c += blockDim.x * 8) {
       float y[8], u[8], w[8];
       load_u(m, c, u);
+      if (c >= C) { store8(a.gate_out + (size_t)m * a.gp + c - C, u); continue; }
       load8(a.conv + (size_t)hist * C + c, w);
 #pragma unroll
       for (int i = 0; i < 8; ++i) y[i] = w[i] * u[i];
@@ -175,12 +177,6 @@ __global__ void __launch_bounds__(256) conv_norm_append_kernel(const ConvArgs<T>
       if (c < a.qp) sq += s2; else if (c < a.qp + a.kp) sk += s2;
       store8(row_s + c, y);
     }
-    if (a.gate_out)
-      for (int c = threadIdx.x * 8; c < a.gp; c += blockDim.x * 8) {
-        float u[8];
-        load_u(m, C + c, u);
-        store8(a.gate_out + (size_t)m * a.gp + c, u);
-      }
     sq = block_sum(sq, red);   // its barriers also publish row_s
     if (a.kv_heads > 0) sk = block_sum(sk, red);
     const float rq = a.qw ? 1.0f / sqrtf(sq / (float)(a.q_heads * a.kd) + a.eps) : 1.0f;
@@ -233,6 +229,117 @@ __global__ void __launch_bounds__(256) conv_norm_append_kernel(const ConvArgs<T>
   }
 }
 
+// The same for prompts in bf16 with head sizes that are multiples of 8 and up to four taps: one thread per 8-channel
+// piece, which keeps the last taps - 1 projected values and the outputs of four rows in registers.  One block walks
+// kRunRows rows of one sequence; the sums of squares of four rows are reduced together.
+constexpr int kRunRows = 16, kRowGroup = 4;
+template <int TAPS, int kMaxThreads>
+__global__ void __launch_bounds__(kMaxThreads) conv_norm_append_run_kernel(const ConvArgs<__nv_bfloat16> a) {
+  using T = __nv_bfloat16;
+  constexpr int H = TAPS - 1;
+  __shared__ float part[2][kRowGroup][32];
+  __shared__ float total[2][kRowGroup];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int C = a.qp + a.kp + a.vp, c = threadIdx.x * 8, b = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int base = a.seq_lens[b] - a.s_new;
+  const int s_lo = blockIdx.x * kRunRows, s_hi = min(a.s_new, s_lo + kRunRows);
+  if (base < 0 || base + a.s_new > a.max_seq) {  // block-uniform
+    if (threadIdx.x == 0) { a.status[0] = (uint32_t)(-RB_ERR_INVALID); a.status[1] = 0xC0ABu; a.status[2] = (uint32_t)base; }
+    return;
+  }
+  const bool mine = c < C, is_q = c < a.qp, is_k = !is_q && c < a.qp + a.kp;
+  const T* col = a.src + (size_t)b * a.s_new * a.ld + c;
+  // where this piece goes: its head and its place inside the head (a piece of padding columns goes nowhere)
+  const int head_size = is_q || is_k ? a.kd : a.vd;
+  const int off = is_q ? c : is_k ? c - a.qp : c - a.qp - a.kp;
+  const int head = off / head_size, i0 = off % head_size;
+  const bool real = mine && head < (is_q ? a.q_heads : a.kv_heads);
+  uint4 w[TAPS], hist[H > 0 ? H : 1], nw = make_uint4(0, 0, 0, 0);   // bf16 octets; hist[j] is j + 1 rows back
+  if (mine) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const uint4*>(a.conv + (size_t)j * C + c);
+    const T* norm = is_q ? a.qw : is_k ? a.kw : nullptr;
+    if (norm) nw = *reinterpret_cast<const uint4*>(norm + off);
+  }
+  const bool normed = is_q ? a.qw != nullptr : is_k ? a.kw != nullptr : false;
+  const float inv_n = 1.0f / (float)(is_q ? a.q_heads * a.kd : max(1, a.kv_heads * a.kd));
+#pragma unroll
+  for (int j = 0; j < H; ++j) {
+    hist[j] = make_uint4(0, 0, 0, 0);
+    const int s = s_lo - 1 - j;
+    if (!mine) continue;
+    if (s >= 0) hist[j] = *reinterpret_cast<const uint4*>(col + (size_t)s * a.ld);
+    else if (base + s >= 0) {
+      float u[8];
+      load8(a.ring + ((size_t)a.slots[b] * H + (base + s) % (H > 0 ? H : 1)) * C + c, u);
+      hist[j] = pack8_bf16(u);  // the ring holds what a tensor held, or a single-token step's value at the same precision
+    }
+  }
+  auto fma8 = [](const uint4& x, const uint4& y, float* acc) {
+    float p[8], q[8];
+    load8(reinterpret_cast<const T*>(&x), p);
+    load8(reinterpret_cast<const T*>(&y), q);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = fmaf(p[i], q[i], acc[i]);
+  };
+  for (int s0 = s_lo; s0 < s_hi; s0 += kRowGroup) {
+    uint4 u[kRowGroup];
+#pragma unroll
+    for (int r = 0; r < kRowGroup; ++r)
+      u[r] = mine && s0 + r < s_hi ? *reinterpret_cast<const uint4*>(col + (size_t)(s0 + r) * a.ld) : make_uint4(0, 0, 0, 0);
+    float y[kRowGroup][8], ss[kRowGroup];
+#pragma unroll
+    for (int r = 0; r < kRowGroup; ++r) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[r][i] = 0.f;
+      if (mine) {
+        fma8(w[H], u[r], y[r]);
+#pragma unroll
+        for (int j = 0; j < H; ++j) fma8(w[H - 1 - j], r - 1 - j >= 0 ? u[r - 1 - j >= 0 ? r - 1 - j : 0] : hist[j - r >= 0 ? j - r : 0], y[r]);
+      }
+      ss[r] = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss[r] = fmaf(y[r][i], y[r][i], ss[r]);
+    }
+#pragma unroll
+    for (int j = H - 1; j >= 0; --j) hist[j] = kRowGroup - 1 - j >= 0 ? u[kRowGroup - 1 - j >= 0 ? kRowGroup - 1 - j : 0] : hist[0];
+#pragma unroll
+    for (int r = 0; r < kRowGroup; ++r) {
+      const float q = warp_sum(is_q ? ss[r] : 0.f), k = warp_sum(is_k ? ss[r] : 0.f);
+      if (lane == 0) { part[0][r][warp] = q; part[1][r][warp] = k; }
+    }
+    __syncthreads();
+    for (int i = warp; i < 2 * kRowGroup; i += n_warps) {
+      const float t = warp_sum(lane < n_warps ? part[i / kRowGroup][i % kRowGroup][lane] : 0.f);
+      if (lane == 0) total[i / kRowGroup][i % kRowGroup] = t;
+    }
+    __syncthreads();
+    float n8[8];
+    load8(reinterpret_cast<const T*>(&nw), n8);
+#pragma unroll
+    for (int r = 0; r < kRowGroup; ++r) {
+      if (!real || s0 + r >= s_hi) continue;
+      if (normed) {
+        const float g = 1.0f / sqrtf(total[is_q ? 0 : 1][r] * inv_n + a.eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[r][i] = y[r][i] * g * n8[i];
+      }
+      if (is_q) {
+        T* dst = a.q_out + (((size_t)b * a.s_new + s0 + r) * a.q_heads + head) * a.D;
+        store8(dst + i0, y[r]);
+        if (i0 + 8 == a.kd)  // the head's last piece also writes its padding
+          for (int p = a.kd; p < a.D; p += 8) *reinterpret_cast<uint4*>(dst + p) = make_uint4(0, 0, 0, 0);
+      } else {
+        const int pos = base + s0 + r;
+        const int page = a.block_table[(size_t)b * a.pages_per_seq + pos / kPageTokens];
+        store8((is_k ? a.kc : a.vc) + (((size_t)page * a.kv_heads + head) * kPageTokens + pos % kPageTokens) * a.D + i0, y[r]);
+      }
+    }
+  }
+}
+
 // The last taps - 1 projected values of every sequence of a multi-token call, once all its rows have been convolved.
 template <typename T>
 __global__ void conv_ring_save_kernel(const ConvArgs<T> a) {
@@ -249,300 +356,7 @@ __global__ void conv_ring_save_kernel(const ConvArgs<T> a) {
     }
 }
 
-// ------------------------------------------------------------------------------------------
-// HGRN2.  One block owns a whole head's state S [key_dim][value_dim] in registers and walks tokens: a lane holds
-// kRows rows x 8 columns (16 row groups x 2 column groups per warp, 16 columns per warp), so a token costs three FMA-pipe
-// operations per state element (k v, f S + k v, S q) and o_t needs a reduction over 16 lanes.  Gates, keys and values
-// of 16 tokens at a time are prepared in shared memory.
-//
-// A prompt is cut into pieces that run side by side: pass 1 (OUT = false) runs the recurrence of each piece from zero and
-// leaves its final state and the product of its forget gates; hgrn2_carry_kernel turns these into the state in front
-// of each piece; pass 2 (OUT = true) runs the recurrence again from there.  No gate is ever divided by, so long
-// decays cannot overflow, and the arithmetic of a token does not depend on where the cuts fall.
-// ------------------------------------------------------------------------------------------
-constexpr int kTileTokens = 16;
-
-template <typename T>
-struct HgrnArgs {
-  const T* src;
-  const float* acc;
-  int n_acc;
-  size_t acc_stride;
-  int64_t ld, out_ld;
-  const T *f_bias, *lower, *norm_w;
-  float eps;
-  int heads, dim, vdim, f_off, v_off;
-  int s_new, piece, n_pieces;
-  const int32_t *seq_lens, *slots, *new_lens;
-  float* state;   // [slot][head][dim][vdim]
-  float* carry;   // [batch][head][piece][dim][vdim]
-  float* decay;   // [batch][head][piece][dim]
-  T* out;
-};
-
-template <typename T, int kRows, bool OUT, int kMaxThreads>
-__global__ void __launch_bounds__(kMaxThreads) hgrn2_kernel(const HgrnArgs<T> a) {
-  constexpr int DP = kRows * 16;
-  extern __shared__ __align__(16) float sm[];
-  const int n_warps = blockDim.x >> 5, cols = n_warps * 16;
-  float* q_s = sm;                          // [tokens][DP]
-  float* f_s = q_s + kTileTokens * DP;
-  float* k_s = f_s + kTileTokens * DP;
-  float* v_s = k_s + kTileTokens * DP;      // [tokens][cols]
-  float* o_s = v_s + kTileTokens * cols;    // [tokens][cols]
-  float* g_s = o_s + kTileTokens * cols;    // [DP] product of the gates (pass 1)
-  const int piece = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int rg = lane & 15, c0 = warp * 16 + (lane >> 4) * 8;
-  pdl_launch_dependents();
-  // A single-token step reads its lengths and state before it waits: both were left by work that a kernel without early
-  // release (the one that advances the lengths) separates from this step.
-  const bool early = a.s_new == 1;
-  if (!early) pdl_wait();
-  const int base = __ldcg(a.seq_lens + b) - a.s_new;
-  const int valid = a.new_lens ? __ldcg(a.new_lens + b) : a.s_new;
-  const int t_lo = piece * a.piece, t_hi = min(t_lo + a.piece, valid);
-  const bool last = t_hi == valid;
-  if (t_lo >= t_hi || (!OUT && last)) {
-    if (early) pdl_wait();
-    return;
-  }
-  const size_t elems = (size_t)a.dim * a.vdim;
-  float* slot_state = a.state + ((size_t)a.slots[b] * a.heads + h) * elems;
-  const size_t pc = ((size_t)b * a.heads + h) * a.n_pieces + piece;
-  float S[kRows][8];
-  const float* from = nullptr;
-  if (OUT) from = a.n_pieces > 1 ? a.carry + pc * elems : base > 0 ? slot_state : nullptr;
-  const bool vec4 = (a.vdim & 3) == 0;
-#pragma unroll
-  for (int r = 0; r < kRows; ++r) {
-    const int row = (r >> 2) * 64 + rg * 4 + (r & 3);
-#pragma unroll
-    for (int c = 0; c < 8; ++c) S[r][c] = 0.f;
-    if (from && row < a.dim) {
-      const float* p = from + (size_t)row * a.vdim + c0;
-#pragma unroll
-      for (int c = 0; c < 8; c += 4) {
-        if (vec4) {
-          if (c0 + c < a.vdim) {
-            const float4 t = __ldcg(reinterpret_cast<const float4*>(p + c));
-            S[r][c] = t.x; S[r][c + 1] = t.y; S[r][c + 2] = t.z; S[r][c + 3] = t.w;
-          }
-        } else {
-#pragma unroll
-          for (int j = 0; j < 4; ++j)
-            if (c0 + c + j < a.vdim) S[r][c + j] = __ldcg(p + c + j);
-        }
-      }
-    }
-  }
-  if (early) pdl_wait();
-  if (!OUT)
-    for (int i = threadIdx.x; i < DP; i += blockDim.x) g_s[i] = 1.f;
-
-  auto load_u = [&](size_t m, int col) {
-    float u = a.src ? Cvt<T>::to_f(a.src[m * a.ld + col]) : 0.f;
-    for (int k = 0; k < a.n_acc; ++k) u += a.acc[(size_t)k * a.acc_stride + m * a.ld + col];
-    return u;
-  };
-
-  for (int t0 = t_lo; t0 < t_hi; t0 += kTileTokens) {
-    const int nt = min(kTileTokens, t_hi - t0);
-    // ---- gates, keys, queries and values of this tile
-    for (int i = threadIdx.x; i < nt * DP; i += blockDim.x) {
-      const int t = i / DP, c = i % DP;
-      float q = 0.f, f = 0.f, k = 0.f;
-      if (c < a.dim) {
-        const size_t m = (size_t)b * a.s_new + t0 + t;
-        const int ch = h * a.dim + c;
-        if (OUT) { const float u = load_u(m, ch); q = u * sigmoid_f(u); }
-        const float z = load_u(m, a.f_off + ch) + Cvt<T>::to_f(a.f_bias[ch]);
-        const float lo = Cvt<T>::to_f(a.lower[ch]);
-        const float e = expf(-z), sg = 1.0f / (1.0f + e);
-        f = fmaf(1.0f - lo, sg, lo);
-        // 1 - f = (1 - lower) sigmoid(-z), formed without the cancellation of 1 - f
-        k = (1.0f - lo) * (z > 0.f ? e * sg : 1.0f - sg);
-      }
-      if (OUT) q_s[i] = q;
-      f_s[i] = f;
-      k_s[i] = k;
-    }
-    for (int i = threadIdx.x; i < nt * cols; i += blockDim.x) {
-      const int t = i / cols, c = i % cols;
-      v_s[i] = c < a.vdim ? load_u((size_t)b * a.s_new + t0 + t, a.v_off + h * a.vdim + c) : 0.f;
-    }
-    __syncthreads();
-    if (!OUT)
-      for (int i = threadIdx.x; i < DP; i += blockDim.x) {
-        float g = g_s[i];
-        for (int t = 0; t < nt; ++t) g *= f_s[t * DP + i];
-        g_s[i] = g;
-      }
-    // ---- the recurrence
-    for (int t = 0; t < nt; ++t) {
-      const float4 va = *reinterpret_cast<const float4*>(v_s + t * cols + c0);
-      const float4 vb = *reinterpret_cast<const float4*>(v_s + t * cols + c0 + 4);
-      const float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
-      float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-      for (int r4 = 0; r4 < kRows / 4; ++r4) {
-        const int at = t * DP + r4 * 64 + rg * 4;
-        const float4 f4 = *reinterpret_cast<const float4*>(f_s + at);
-        const float4 k4 = *reinterpret_cast<const float4*>(k_s + at);
-        float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (OUT) q4 = *reinterpret_cast<const float4*>(q_s + at);
-        const float fr[4] = {f4.x, f4.y, f4.z, f4.w}, kr[4] = {k4.x, k4.y, k4.z, k4.w}, qr[4] = {q4.x, q4.y, q4.z, q4.w};
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          float* row = S[r4 * 4 + j];
-#pragma unroll
-          for (int c = 0; c < 8; ++c) {
-            row[c] = fmaf(fr[j], row[c], kr[j] * v[c]);
-            if (OUT) o[c] = fmaf(row[c], qr[j], o[c]);
-          }
-        }
-      }
-      if (OUT) {
-        // sum over the 16 row groups; each exchange halves the columns a lane is responsible for
-        const bool b3 = lane & 8, b2 = lane & 4, b1 = lane & 2;
-        float p4[4], p2[2];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const float got = __shfl_xor_sync(0xffffffffu, b3 ? o[c] : o[c + 4], 8);
-          p4[c] = (b3 ? o[c + 4] : o[c]) + got;
-        }
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const float got = __shfl_xor_sync(0xffffffffu, b2 ? p4[c] : p4[c + 2], 4);
-          p2[c] = (b2 ? p4[c + 2] : p4[c]) + got;
-        }
-        float p1 = (b1 ? p2[1] : p2[0]) + __shfl_xor_sync(0xffffffffu, b1 ? p2[0] : p2[1], 2);
-        p1 += __shfl_xor_sync(0xffffffffu, p1, 1);
-        if ((lane & 1) == 0) o_s[t * cols + c0 + (b3 ? 4 : 0) + (b2 ? 2 : 0) + (b1 ? 1 : 0)] = p1;
-      }
-    }
-    __syncthreads();
-    if (OUT) {
-      // ---- norm over the head's values, one warp per token (the next tile's staging touches other arrays)
-      for (int t = warp; t < nt; t += n_warps) {
-        float s = 0.f;
-        for (int c = lane; c < a.vdim; c += 32) { const float y = o_s[t * cols + c]; s = fmaf(y, y, s); }
-        s = warp_sum(s);
-        const float r = 1.0f / sqrtf(s / (float)a.vdim + a.eps);
-        T* dst = a.out + ((size_t)b * a.s_new + t0 + t) * a.out_ld + (size_t)h * a.vdim;
-        for (int c = lane; c < a.vdim; c += 32) dst[c] = Cvt<T>::from_f(o_s[t * cols + c] * r * Cvt<T>::to_f(a.norm_w[c]));
-      }
-    }
-  }
-  float* to = OUT ? (last ? slot_state : nullptr) : a.carry + pc * elems;
-  if (!OUT)
-    for (int i = threadIdx.x; i < a.dim; i += blockDim.x) a.decay[pc * a.dim + i] = g_s[i];
-  if (to) {
-#pragma unroll
-    for (int r = 0; r < kRows; ++r) {
-      const int row = (r >> 2) * 64 + rg * 4 + (r & 3);
-      if (row >= a.dim) continue;
-      float* p = to + (size_t)row * a.vdim + c0;
-#pragma unroll
-      for (int c = 0; c < 8; c += 4) {
-        if (vec4) {
-          if (c0 + c < a.vdim) *reinterpret_cast<float4*>(p + c) = make_float4(S[r][c], S[r][c + 1], S[r][c + 2], S[r][c + 3]);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 4; ++j)
-            if (c0 + c + j < a.vdim) p[c + j] = S[r][c + j];
-        }
-      }
-    }
-  }
-}
-
-// carry[p] = state in front of piece p:  S_0 = the sequence's state, S_(p+1) = decay_p * S_p + (state of piece p alone)
-template <typename T>
-__global__ void hgrn2_carry_kernel(const HgrnArgs<T> a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int h = blockIdx.y, b = blockIdx.z;
-  const int valid = a.new_lens ? a.new_lens[b] : a.s_new, base = a.seq_lens[b] - a.s_new;
-  const int n = (valid + a.piece - 1) / a.piece;
-  const int elems = a.dim * a.vdim;
-  const float* state = a.state + ((size_t)a.slots[b] * a.heads + h) * elems;
-  const size_t p0 = ((size_t)b * a.heads + h) * a.n_pieces;
-  for (int e = blockIdx.x * blockDim.x + threadIdx.x; e < elems; e += gridDim.x * blockDim.x) {
-    const int row = e / a.vdim;
-    float S = base > 0 ? state[e] : 0.f;
-    constexpr int G = 8;  // loads of a group are in flight together
-    for (int p = 0; p < n; p += G) {
-      float part[G], g[G];
-#pragma unroll
-      for (int i = 0; i < G; ++i)
-        if (p + i < n - 1) { part[i] = __ldcg(a.carry + (p0 + p + i) * elems + e); g[i] = __ldcg(a.decay + (p0 + p + i) * a.dim + row); }
-#pragma unroll
-      for (int i = 0; i < G; ++i)
-        if (p + i < n) {
-          a.carry[(p0 + p + i) * elems + e] = S;
-          if (p + i < n - 1) S = fmaf(g[i], S, part[i]);
-        }
-    }
-  }
-}
-
 int round8(int v) { return (v + 7) / 8 * 8; }
-
-template <typename T, int kRows, bool OUT, int kMaxThreads>
-int hgrn2_launch_one(rb_ctx* ctx, const HgrnArgs<T>& a, int batch, int warps) {
-  auto kern = hgrn2_kernel<T, kRows, OUT, kMaxThreads>;
-  const int tokens = kTileTokens, dp = kRows * 16, cols = warps * 16;
-  const size_t smem = (size_t)(tokens * (3 * dp + 2 * cols) + dp) * sizeof(float);
-  static bool set[64] = {};  // the attribute belongs to the (kernel, device) pair
-  const int dv = ctx->device & 63;
-  if (!set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024)); set[dv] = true; }
-  RB_CUDA(launch_kernel(kern, dim3((unsigned)a.n_pieces, (unsigned)a.heads, (unsigned)batch), dim3(warps * 32), smem, ctx->stream,
-                        ctx->pdl, a));
-  ctx->launches++;
-  return RB_OK;
-}
-
-template <typename T, bool OUT>
-int hgrn2_launch(rb_ctx* ctx, const HgrnArgs<T>& a, int batch) {
-  const int warps = (a.vdim + 15) / 16;
-  if (a.dim <= 64) return hgrn2_launch_one<T, 4, OUT, 512>(ctx, a, batch, warps);
-  if (a.dim <= 128) return hgrn2_launch_one<T, 8, OUT, 512>(ctx, a, batch, warps);
-  if (warps <= 8) return hgrn2_launch_one<T, 16, OUT, 256>(ctx, a, batch, warps);
-  return hgrn2_launch_one<T, 16, OUT, 512>(ctx, a, batch, warps);
-}
-
-template <typename T>
-int hgrn2_run(rb_ctx* ctx, HgrnArgs<T> a, int batch, int chunk) {
-  // Pieces: enough blocks for about four per SM, none shorter than 64 tokens; one piece needs no second pass.
-  int piece = chunk;
-  if (piece <= 0) {
-    const int want = std::max(1, (4 * ctx->sm_count) / std::max(1, batch * a.heads));
-    piece = std::max(64, (a.s_new + want - 1) / want);
-  }
-  piece = (piece + kTileTokens - 1) / kTileTokens * kTileTokens;
-  a.piece = piece;
-  a.n_pieces = (a.s_new + piece - 1) / piece;
-  if (a.n_pieces > 1) {
-    const size_t elems = (size_t)a.dim * a.vdim, n = (size_t)batch * a.heads * a.n_pieces;
-    const size_t bytes = n * (elems + a.dim) * sizeof(float);
-    if (ctx->chunk_scratch_bytes < bytes) {
-      float* fresh = nullptr;
-      RB_CUDA(cudaMalloc(&fresh, bytes));
-      if (ctx->chunk_scratch) ctx->retired.push_back(ctx->chunk_scratch);
-      ctx->chunk_scratch = fresh;
-      ctx->chunk_scratch_bytes = bytes;
-    }
-    a.carry = ctx->chunk_scratch;
-    a.decay = ctx->chunk_scratch + n * elems;
-    RB_TRY((hgrn2_launch<T, false>(ctx, a, batch)));
-    const int blocks = (int)std::min<size_t>((elems + 255) / 256, 64);
-    RB_CUDA(launch_kernel(hgrn2_carry_kernel<T>, dim3((unsigned)blocks, (unsigned)a.heads, (unsigned)batch), dim3(256), 0, ctx->stream,
-                          ctx->pdl, a));
-    ctx->launches++;
-  }
-  return hgrn2_launch<T, true>(ctx, a, batch);
-}
 
 template <typename T>
 int conv_run(rb_ctx* ctx, ConvArgs<T> a, int batch) {
@@ -555,9 +369,26 @@ int conv_run(rb_ctx* ctx, ConvArgs<T> a, int batch) {
     RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     set[dv] = smem;
   }
-  a.per_block = a.rows >= 16 * ctx->sm_count ? 8 : 1;
-  const int blocks = (a.rows + a.per_block - 1) / a.per_block;
-  RB_CUDA(launch_kernel(kern, dim3((unsigned)blocks), dim3(256), smem, ctx->stream, ctx->pdl, a));
+  bool done = false;
+  if constexpr (sizeof(T) == 2)
+    if (a.s_new >= kRowGroup && a.src && !a.gate_out && a.taps <= 4 && (a.kd % 8) == 0 && (a.vd % 8) == 0 && C / 8 <= 1024) {
+      const dim3 grid((unsigned)((a.s_new + kRunRows - 1) / kRunRows), (unsigned)batch), block((unsigned)((C / 8 + 31) / 32 * 32));
+      auto pick = [&](auto wide) {
+        constexpr int M = decltype(wide)::value ? 1024 : 512;
+        return a.taps == 1 ? conv_norm_append_run_kernel<1, M> : a.taps == 2 ? conv_norm_append_run_kernel<2, M>
+               : a.taps == 3 ? conv_norm_append_run_kernel<3, M> : conv_norm_append_run_kernel<4, M>;
+      };
+      auto run = block.x > 512 ? pick(std::true_type()) : pick(std::false_type());
+      RB_CUDA(launch_kernel(run, grid, block, 0, ctx->stream, ctx->pdl, a));
+      done = true;
+    }
+  if (!done) {
+    a.per_block = a.rows >= 16 * ctx->sm_count ? 8 : 1;
+    const int blocks = (a.rows + a.per_block - 1) / a.per_block;
+    const int pieces = (C + (a.gate_out ? a.gp : 0)) / 8;
+    const int threads = std::min(512, std::max(64, (pieces + 31) / 32 * 32));
+    RB_CUDA(launch_kernel(kern, dim3((unsigned)blocks), dim3(threads), smem, ctx->stream, ctx->pdl, a));
+  }
   ctx->launches++;
   if (a.s_new > 1 && a.taps > 1) {
     RB_CUDA(launch_kernel(conv_ring_save_kernel<T>, dim3((unsigned)batch), dim3(256), 0, ctx->stream, ctx->pdl, a));
@@ -693,37 +524,4 @@ extern "C" int32_t rb_conv_norm_append(rb_ctx* ctx, const void* src, const float
   if (dtype == RB_BF16) return fill(__nv_bfloat16());
   if (dtype == RB_F32) return fill(float());
   return fail(RB_ERR_DTYPE, "rb_conv_norm_append: dtype %d unsupported", dtype);
-}
-
-extern "C" int32_t rb_hgrn2(rb_ctx* ctx, const void* src, const float* acc, int32_t n_acc, int64_t src_ld, const void* f_bias,
-                            const void* lower, const void* norm_w, float eps, int32_t heads, int32_t key_dim, int32_t value_dim,
-                            int32_t batch, int32_t s_new, rb_kv_cache* c, const int32_t* new_lens, float* state, int32_t chunk,
-                            void* out, int64_t out_ld, int32_t dtype) {
-  RB_REQUIRE(ctx && c && f_bias && lower && norm_w && state && out && (src || (acc && n_acc > 0)), "rb_hgrn2: null argument");
-  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0 && chunk >= 0, "rb_hgrn2: bad batch/seq");
-  RB_REQUIRE(src || s_new == 1, "rb_hgrn2: split-K partials need single-token rows");
-  RB_REQUIRE(heads > 0 && key_dim > 0 && value_dim > 0, "rb_hgrn2: bad head sizes");
-  if (key_dim > 256 || value_dim > 256) return fail(RB_ERR_UNIMPLEMENTED, "rb_hgrn2: head sizes %d x %d exceed 256", key_dim, value_dim);
-  RB_REQUIRE(aligned16(state), "rb_hgrn2: the state must be 16-byte aligned");
-  if (!acc) n_acc = 0;
-  const int64_t rows = (int64_t)batch * s_new;
-  auto fill = [&](auto tag) -> int {
-    using T = decltype(tag);
-    HgrnArgs<T> a{};
-    a.src = (const T*)src; a.acc = acc; a.n_acc = n_acc; a.acc_stride = (size_t)rows * src_ld;
-    a.ld = src_ld; a.out_ld = out_ld;
-    a.f_bias = (const T*)f_bias; a.lower = (const T*)lower; a.norm_w = (const T*)norm_w; a.eps = eps;
-    a.heads = heads; a.dim = key_dim; a.vdim = value_dim;
-    a.f_off = round8(heads * key_dim); a.v_off = 2 * a.f_off;
-    RB_REQUIRE(src_ld >= a.v_off + heads * value_dim && out_ld >= (int64_t)heads * value_dim, "rb_hgrn2: row pitches too small");
-    a.s_new = s_new; a.seq_lens = c->seq_lens; a.slots = c->slots; a.new_lens = new_lens; a.state = state; a.out = (T*)out;
-    const double sb = 4.0 * key_dim * value_dim * heads, es = sizeof(T);
-    ProfScope prof(ctx, RB_PROF_RECURRENCE,
-                   2.0 * batch * sb + rows * ((src ? es : 4.0 * n_acc) * heads * (2.0 * key_dim + value_dim) + es * heads * value_dim),
-                   5.0 * rows * heads * (double)key_dim * value_dim);
-    return hgrn2_run<T>(ctx, a, batch, chunk);
-  };
-  if (dtype == RB_BF16) return fill(__nv_bfloat16());
-  if (dtype == RB_F32) return fill(float());
-  return fail(RB_ERR_DTYPE, "rb_hgrn2: dtype %d unsupported", dtype);
 }

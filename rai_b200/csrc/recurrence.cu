@@ -1,0 +1,492 @@
+// The HGRN2 recurrence in float32.  One block owns a whole head's state [key_dim][value_dim] in registers and walks
+// tokens: a lane holds kRows rows x kCols columns (16 row groups x 2 column groups per warp), rows in pairs so that every
+// step is a packed two-lane FMA: k v, f S + k v and S q, three per pair of state elements.  o_t needs a sum over the 16
+// row groups.  Gates, keys and values of 16 tokens at a time are prepared in shared memory; the projection's rows for the
+// next 16 are on their way (cp.async) meanwhile.
+//
+// A prompt is cut into pieces that run side by side: pass 1 (OUT = false) runs the recurrence of each piece from zero and
+// leaves its final state and the product of its forget gates; hgrn2_carry_kernel turns these into the state in front of
+// each piece; pass 2 (OUT = true) runs the recurrence again from there.  No gate is ever divided by, so long decays
+// cannot overflow, and the arithmetic of a token does not depend on where the cuts fall.
+#include <algorithm>
+#include <type_traits>
+
+#include "ctx.h"
+
+namespace rb {
+
+namespace {
+
+constexpr int kTileTokens = 16;
+
+template <typename T>
+struct HgrnArgs {
+  const T* src;
+  const float* acc;
+  int n_acc;
+  size_t acc_stride;
+  int64_t ld, out_ld;
+  const T *f_bias, *lower, *norm_w;
+  float eps;
+  int heads, dim, vdim, f_off, v_off;
+  int s_new, piece, n_pieces;
+  int raw;        // rows of the projection come through cp.async (16-byte pieces line up)
+  const int32_t *seq_lens, *slots, *new_lens;
+  float* state;   // [slot][head][dim][vdim]
+  float* carry;   // [batch][head][piece][dim][vdim]
+  float* decay;   // [batch][head][piece][dim]
+  T* out;
+};
+
+// ---- pairs of float32 in one 64-bit register
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 pack2(float lo, float hi) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// keep = lower + (1 - lower) sigmoid(z), and 1 - keep formed without the cancellation.  kExact: the library's exponential
+// and division; otherwise the fast ones (still float32, a few ulp), for projections that were rounded to bf16.
+template <bool kExact>
+__device__ __forceinline__ void gates(float z, float lower, float& keep, float& take) {
+  const float e = kExact ? expf(-z) : __expf(-z);
+  const float s = kExact ? 1.0f / (1.0f + e) : __fdividef(1.0f, 1.0f + fminf(e, 1e37f));
+  keep = fmaf(1.0f - lower, s, lower);
+  take = (1.0f - lower) * (z > 0.f ? e * s : 1.0f - s);
+}
+template <bool kExact>
+__device__ __forceinline__ float silu_f(float u) {
+  return kExact ? u / (1.0f + expf(-u)) : __fdividef(u, 1.0f + fminf(__expf(-u), 1e37f));
+}
+
+__device__ __forceinline__ void load4(const float* p, float* v) {
+  const float4 t = *reinterpret_cast<const float4*>(p);
+  v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float* v) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+
+// State rows of a lane: kRows rows in groups of four neighbours, 64 rows apart; kCols neighbouring columns.
+template <int kRows, int kCols, typename F>
+__device__ __forceinline__ void load_state(f2 (&S)[kRows / 2][kCols], const float* from, int rg, int c0, F quad) {
+#pragma unroll
+  for (int p = 0; p < kRows / 2; ++p) {
+    const int row = (p >> 1) * 64 + rg * 4 + (p & 1) * 2;
+    float lo[kCols], hi[kCols];
+#pragma unroll
+    for (int c = 0; c < kCols; c += 4) {
+      quad(from, row, c0 + c, lo + c);
+      quad(from, row + 1, c0 + c, hi + c);
+    }
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) S[p][c] = pack2(lo[c], hi[c]);
+  }
+}
+
+template <typename T, int kRows, int kCols, bool OUT, int kMaxThreads>
+__global__ void __launch_bounds__(kMaxThreads) hgrn2_kernel(const HgrnArgs<T> a) {
+  constexpr int DP = kRows * 16;
+  constexpr int kPairs = kRows / 2;
+  constexpr bool kExact = sizeof(T) == 4;
+  extern __shared__ __align__(16) float sm[];
+  const int n_warps = blockDim.x >> 5, cols = n_warps * 2 * kCols, tokens = min(kTileTokens, a.s_new);
+  float* q_s = sm;                          // [tokens][DP]
+  float* f_s = q_s + tokens * DP;
+  float* k_s = f_s + tokens * DP;
+  float* v_s = k_s + tokens * DP;           // [tokens][cols]
+  float* o_s = v_s + tokens * cols;         // [tokens][cols]
+  float* g_s = o_s + tokens * cols;         // [DP] product of the gates (pass 1)
+  T* raw_q = reinterpret_cast<T*>(g_s + DP);  // the projection's rows of the next tile: [tokens][dim], [tokens][dim], [tokens][vdim]
+  T* raw_f = raw_q + tokens * a.dim;
+  T* raw_v = raw_f + tokens * a.dim;
+  const int piece = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int rg = lane & 15, c0 = (warp * 2 + (lane >> 4)) * kCols;
+  pdl_launch_dependents();
+  // A single-token step reads its lengths and state before it waits: both were left by work that a kernel without early
+  // release (the one that advances the lengths) separates from this step.
+  const bool early = a.s_new == 1;
+  if (!early) pdl_wait();
+  const int base = __ldcg(a.seq_lens + b) - a.s_new;
+  const int valid = a.new_lens ? __ldcg(a.new_lens + b) : a.s_new;
+  const int t_lo = piece * a.piece, t_hi = min(t_lo + a.piece, valid);
+  const bool last = t_hi == valid;
+  if (t_lo >= t_hi || (!OUT && last)) {
+    if (early) pdl_wait();
+    return;
+  }
+  // 16-byte pieces of the rows t .. t + nt of this head's q, f and v
+  auto fetch = [&](int t, int nt) {
+    constexpr int E = 16 / sizeof(T);
+    const int dq = a.dim / E, dv = a.vdim / E, per = 2 * dq + dv;
+    for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
+      const int r = i / per, c = i % per;
+      const T* row = a.src + ((size_t)b * a.s_new + t + r) * a.ld;
+      if (c < dq) { if (OUT) cp_async16(raw_q + r * a.dim + c * E, row + h * a.dim + c * E); }
+      else if (c < 2 * dq) cp_async16(raw_f + r * a.dim + (c - dq) * E, row + a.f_off + h * a.dim + (c - dq) * E);
+      else cp_async16(raw_v + r * a.vdim + (c - 2 * dq) * E, row + a.v_off + h * a.vdim + (c - 2 * dq) * E);
+    }
+    cp_async_commit();
+  };
+  if (a.raw) fetch(t_lo, min(kTileTokens, t_hi - t_lo));
+
+  const size_t elems = (size_t)a.dim * a.vdim;
+  float* slot_state = a.state + ((size_t)a.slots[b] * a.heads + h) * elems;
+  const size_t pc = ((size_t)b * a.heads + h) * a.n_pieces + piece;
+  const bool vec4 = (a.vdim & 3) == 0;
+  f2 S[kPairs][kCols];
+  const float* from = nullptr;
+  if (OUT) from = a.n_pieces > 1 ? a.carry + pc * elems : base > 0 ? slot_state : nullptr;
+  load_state<kRows, kCols>(S, from, rg, c0, [&](const float* p, int row, int col, float* x) {
+    x[0] = x[1] = x[2] = x[3] = 0.f;
+    if (!p || row >= a.dim) return;
+    p += (size_t)row * a.vdim + col;
+    if (vec4) {
+      if (col < a.vdim) {
+        const float4 t = __ldcg(reinterpret_cast<const float4*>(p));
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < a.vdim) x[j] = __ldcg(p + j);
+    }
+  });
+  if (early) pdl_wait();
+  if (!OUT)
+    for (int i = threadIdx.x; i < DP; i += blockDim.x) g_s[i] = 1.f;
+
+  // N columns of row m, from the tensor or summed over the split-K slabs with all loads in flight together
+  auto load_u = [&](size_t m, const int* col, float* u, auto n_const) {
+    constexpr int N = decltype(n_const)::value;
+#pragma unroll
+    for (int j = 0; j < N; ++j) u[j] = a.src ? Cvt<T>::to_f(a.src[m * a.ld + col[j]]) : 0.f;
+    for (int k0 = 0; k0 < a.n_acc; k0 += 8) {
+      float t[N][8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+#pragma unroll
+        for (int j = 0; j < N; ++j) t[j][k] = k0 + k < a.n_acc ? a.acc[(size_t)(k0 + k) * a.acc_stride + m * a.ld + col[j]] : 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+#pragma unroll
+        for (int j = 0; j < N; ++j) u[j] += t[j][k];
+    }
+  };
+
+  for (int t0 = t_lo; t0 < t_hi; t0 += kTileTokens) {
+    const int nt = min(kTileTokens, t_hi - t0);
+    // ---- queries, gates, keys and values of this tile as float32
+    if (a.raw) {
+      cp_async_wait_all();
+      __syncthreads();
+      for (int i = threadIdx.x; i < nt * (DP / 4); i += blockDim.x) {
+        const int t = i / (DP / 4), c = (i % (DP / 4)) * 4;
+        float q[4] = {0.f, 0.f, 0.f, 0.f}, f[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
+        if (c < a.dim) {
+          float uq[4], uf[4], fb[4], lo[4];
+          if (OUT) load4(raw_q + t * a.dim + c, uq);
+          load4(raw_f + t * a.dim + c, uf);
+          load4(a.f_bias + h * a.dim + c, fb);
+          load4(a.lower + h * a.dim + c, lo);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            if (OUT) q[j] = silu_f<kExact>(uq[j]);
+            gates<kExact>(uf[j] + fb[j], lo[j], f[j], k[j]);
+          }
+        }
+        if (OUT) *reinterpret_cast<float4*>(q_s + t * DP + c) = make_float4(q[0], q[1], q[2], q[3]);
+        *reinterpret_cast<float4*>(f_s + t * DP + c) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(k_s + t * DP + c) = make_float4(k[0], k[1], k[2], k[3]);
+      }
+      for (int i = threadIdx.x; i < nt * (cols / 4); i += blockDim.x) {
+        const int t = i / (cols / 4), c = (i % (cols / 4)) * 4;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (c < a.vdim) load4(raw_v + t * a.vdim + c, v);
+        *reinterpret_cast<float4*>(v_s + t * cols + c) = make_float4(v[0], v[1], v[2], v[3]);
+      }
+    } else {
+      for (int i = threadIdx.x; i < nt * (DP + cols); i += blockDim.x) {
+        const size_t m0 = (size_t)b * a.s_new + t0;
+        if (i < nt * DP) {
+          const int t = i / DP, c = i % DP;
+          float q = 0.f, f = 0.f, k = 0.f;
+          if (c < a.dim) {
+            const int ch = h * a.dim + c, col[2] = {ch, a.f_off + ch};
+            float u[2];
+            load_u(m0 + t, col, u, std::integral_constant<int, 2>());
+            q = silu_f<kExact>(u[0]);
+            gates<kExact>(u[1] + Cvt<T>::to_f(a.f_bias[ch]), Cvt<T>::to_f(a.lower[ch]), f, k);
+          }
+          q_s[i] = q;
+          f_s[i] = f;
+          k_s[i] = k;
+        } else {
+          const int j = i - nt * DP, t = j / cols, c = j % cols;
+          float u = 0.f;
+          if (c < a.vdim) {
+            const int col = a.v_off + h * a.vdim + c;
+            load_u(m0 + t, &col, &u, std::integral_constant<int, 1>());
+          }
+          v_s[j] = u;
+        }
+      }
+    }
+    __syncthreads();
+    if (a.raw && t0 + kTileTokens < t_hi) fetch(t0 + kTileTokens, min(kTileTokens, t_hi - t0 - kTileTokens));
+    if (!OUT)
+      for (int i = threadIdx.x; i < DP; i += blockDim.x) {
+        float g = g_s[i];
+        for (int t = 0; t < nt; ++t) g *= f_s[t * DP + i];
+        g_s[i] = g;
+      }
+    // ---- the recurrence
+    for (int t = 0; t < nt; ++t) {
+      f2 v[kCols], o2[kCols];
+#pragma unroll
+      for (int c = 0; c < kCols; c += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(v_s + t * cols + c0 + c);
+        v[c] = pack2(x.x, x.x); v[c + 1] = pack2(x.y, x.y); v[c + 2] = pack2(x.z, x.z); v[c + 3] = pack2(x.w, x.w);
+      }
+#pragma unroll
+      for (int c = 0; c < kCols; ++c) o2[c] = 0ull;
+#pragma unroll
+      for (int r4 = 0; r4 < kRows / 4; ++r4) {
+        const int at = t * DP + r4 * 64 + rg * 4;
+        const ulonglong2 f4 = *reinterpret_cast<const ulonglong2*>(f_s + at);
+        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(k_s + at);
+        ulonglong2 q4 = make_ulonglong2(0ull, 0ull);
+        if (OUT) q4 = *reinterpret_cast<const ulonglong2*>(q_s + at);
+#pragma unroll
+        for (int c = 0; c < kCols; ++c) {
+          S[r4 * 2][c] = fma2(f4.x, S[r4 * 2][c], mul2(k4.x, v[c]));
+          S[r4 * 2 + 1][c] = fma2(f4.y, S[r4 * 2 + 1][c], mul2(k4.y, v[c]));
+          if (OUT) {
+            o2[c] = fma2(S[r4 * 2][c], q4.x, o2[c]);
+            o2[c] = fma2(S[r4 * 2 + 1][c], q4.y, o2[c]);
+          }
+        }
+      }
+      if (OUT) {
+        // sum over the 16 row groups; each exchange halves the columns a lane is responsible for
+        float o[kCols];
+#pragma unroll
+        for (int c = 0; c < kCols; ++c) { float lo, hi; unpack2(o2[c], lo, hi); o[c] = lo + hi; }
+        int col = c0, n = kCols;
+#pragma unroll
+        for (int bit = 8; bit > 0; bit >>= 1) {
+          if (n > 1) {
+            n >>= 1;
+            const bool up = lane & bit;
+#pragma unroll
+            for (int c = 0; c < kCols / 2; ++c)
+              if (c < n) o[c] = (up ? o[c + n] : o[c]) + __shfl_xor_sync(0xffffffffu, up ? o[c] : o[c + n], bit);
+            col += up ? n : 0;
+          } else {
+            o[0] += __shfl_xor_sync(0xffffffffu, o[0], bit);
+          }
+        }
+        if (kCols == 16 || (lane & 1) == 0) o_s[t * cols + col] = o[0];
+      }
+    }
+    __syncthreads();
+    if (OUT) {
+      // ---- norm over the head's values, one warp per token (the next tile's staging touches other arrays)
+      for (int t = warp; t < nt; t += n_warps) {
+        float s = 0.f;
+        for (int c = lane; c < a.vdim; c += 32) { const float y = o_s[t * cols + c]; s = fmaf(y, y, s); }
+        s = warp_sum(s);
+        const float r = 1.0f / sqrtf(s / (float)a.vdim + a.eps);
+        T* dst = a.out + ((size_t)b * a.s_new + t0 + t) * a.out_ld + (size_t)h * a.vdim;
+        for (int c = lane; c < a.vdim; c += 32) dst[c] = Cvt<T>::from_f(o_s[t * cols + c] * r * Cvt<T>::to_f(a.norm_w[c]));
+      }
+    }
+  }
+  float* to = OUT ? (last ? slot_state : nullptr) : a.carry + pc * elems;
+  if (!OUT)
+    for (int i = threadIdx.x; i < a.dim; i += blockDim.x) a.decay[pc * a.dim + i] = g_s[i];
+  if (!to) return;
+#pragma unroll
+  for (int p = 0; p < kPairs; ++p) {
+    const int row = (p >> 1) * 64 + rg * 4 + (p & 1) * 2;
+    float x[2][kCols];
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) unpack2(S[p][c], x[0][c], x[1][c]);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      if (row + j >= a.dim) continue;
+      float* dst = to + (size_t)(row + j) * a.vdim + c0;
+#pragma unroll
+      for (int c = 0; c < kCols; c += 4) {
+        if (vec4) {
+          if (c0 + c < a.vdim) *reinterpret_cast<float4*>(dst + c) = make_float4(x[j][c], x[j][c + 1], x[j][c + 2], x[j][c + 3]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (c0 + c + i < a.vdim) dst[c + i] = x[j][c + i];
+        }
+      }
+    }
+  }
+}
+
+// carry[p] = state in front of piece p: the sequence's own state for the first; then what a piece keeps of the state in
+// front of it plus what the piece leaves on its own
+template <typename T>
+__global__ void hgrn2_carry_kernel(const HgrnArgs<T> a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int valid = a.new_lens ? a.new_lens[b] : a.s_new, base = a.seq_lens[b] - a.s_new;
+  const int n = (valid + a.piece - 1) / a.piece;
+  const int elems = a.dim * a.vdim;
+  const float* state = a.state + ((size_t)a.slots[b] * a.heads + h) * elems;
+  const size_t p0 = ((size_t)b * a.heads + h) * a.n_pieces;
+  for (int e = blockIdx.x * blockDim.x + threadIdx.x; e < elems; e += gridDim.x * blockDim.x) {
+    const int row = e / a.vdim;
+    float S = base > 0 ? state[e] : 0.f;
+    constexpr int G = 8;  // loads of a group are in flight together
+    for (int p = 0; p < n; p += G) {
+      float part[G], g[G];
+#pragma unroll
+      for (int i = 0; i < G; ++i)
+        if (p + i < n - 1) { part[i] = __ldcg(a.carry + (p0 + p + i) * elems + e); g[i] = __ldcg(a.decay + (p0 + p + i) * a.dim + row); }
+#pragma unroll
+      for (int i = 0; i < G; ++i)
+        if (p + i < n) {
+          a.carry[(p0 + p + i) * elems + e] = S;
+          if (p + i < n - 1) S = fmaf(g[i], S, part[i]);
+        }
+    }
+  }
+}
+
+int round8(int v) { return (v + 7) / 8 * 8; }
+
+template <typename T, int kRows, int kCols, bool OUT, int kMaxThreads>
+int launch_one(rb_ctx* ctx, const HgrnArgs<T>& a, int batch) {
+  auto kern = hgrn2_kernel<T, kRows, kCols, OUT, kMaxThreads>;
+  const int warps = (a.vdim + 2 * kCols - 1) / (2 * kCols);
+  const int tokens = std::min(kTileTokens, a.s_new), dp = kRows * 16, cols = warps * 2 * kCols;
+  const size_t smem = (size_t)(tokens * (3 * dp + 2 * cols) + dp) * sizeof(float) + (a.raw ? (size_t)tokens * (2 * a.dim + a.vdim) * sizeof(T) : 0);
+  static bool set[64] = {};  // the attribute belongs to the (kernel, device) pair
+  const int dv = ctx->device & 63;
+  if (!set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)); set[dv] = true; }
+  RB_CUDA(launch_kernel(kern, dim3((unsigned)a.n_pieces, (unsigned)a.heads, (unsigned)batch), dim3(warps * 32), smem, ctx->stream,
+                        ctx->pdl, a));
+  ctx->launches++;
+  return RB_OK;
+}
+
+template <typename T, bool OUT>
+int launch(rb_ctx* ctx, const HgrnArgs<T>& a, int batch) {
+  if (a.dim > 128) {
+    if (a.vdim <= 128) return launch_one<T, 16, 8, OUT, 256>(ctx, a, batch);
+    return launch_one<T, 16, 8, OUT, 512>(ctx, a, batch);
+  }
+  if constexpr (OUT)
+    if (a.s_new == 1) {  // bound by reading and writing the state: more, lighter threads
+      if (a.dim <= 64) return launch_one<T, 4, 8, true, 512>(ctx, a, batch);
+      return launch_one<T, 8, 8, true, 512>(ctx, a, batch);
+    }
+  if (a.dim <= 64) return launch_one<T, 4, 16, OUT, 256>(ctx, a, batch);
+  return launch_one<T, 8, 16, OUT, 256>(ctx, a, batch);
+}
+
+template <typename T>
+int run(rb_ctx* ctx, HgrnArgs<T> a, int batch, int chunk) {
+  // Pieces: enough blocks to fill the GPU's block slots, none shorter than 64 tokens; one piece needs no second pass.
+  int piece = chunk;
+  if (piece <= 0) {
+    const int want = std::max(1, (4 * ctx->sm_count) / std::max(1, batch * a.heads));
+    piece = std::max(64, (a.s_new + want - 1) / want);
+  }
+  piece = (piece + kTileTokens - 1) / kTileTokens * kTileTokens;
+  a.piece = piece;
+  a.n_pieces = (a.s_new + piece - 1) / piece;
+  if (a.n_pieces > 1) {
+    const size_t elems = (size_t)a.dim * a.vdim, n = (size_t)batch * a.heads * a.n_pieces;
+    const size_t bytes = n * (elems + a.dim) * sizeof(float);
+    if (ctx->chunk_scratch_bytes < bytes) {
+      float* fresh = nullptr;
+      RB_CUDA(cudaMalloc(&fresh, bytes));
+      if (ctx->chunk_scratch) ctx->retired.push_back(ctx->chunk_scratch);
+      ctx->chunk_scratch = fresh;
+      ctx->chunk_scratch_bytes = bytes;
+    }
+    a.carry = ctx->chunk_scratch;
+    a.decay = ctx->chunk_scratch + n * elems;
+    RB_TRY((launch<T, false>(ctx, a, batch)));
+    const int blocks = (int)std::min<size_t>((elems + 255) / 256, 64);
+    RB_CUDA(launch_kernel(hgrn2_carry_kernel<T>, dim3((unsigned)blocks, (unsigned)a.heads, (unsigned)batch), dim3(256), 0, ctx->stream,
+                          ctx->pdl, a));
+    ctx->launches++;
+  }
+  return launch<T, true>(ctx, a, batch);
+}
+
+bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace
+
+}  // namespace rb
+
+using namespace rb;
+
+extern "C" int32_t rb_hgrn2(rb_ctx* ctx, const void* src, const float* acc, int32_t n_acc, int64_t src_ld, const void* f_bias,
+                            const void* lower, const void* norm_w, float eps, int32_t heads, int32_t key_dim, int32_t value_dim,
+                            int32_t batch, int32_t s_new, rb_kv_cache* c, const int32_t* new_lens, float* state, int32_t chunk,
+                            void* out, int64_t out_ld, int32_t dtype) {
+  RB_REQUIRE(ctx && c && f_bias && lower && norm_w && state && out && (src || (acc && n_acc > 0)), "rb_hgrn2: null argument");
+  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0 && chunk >= 0, "rb_hgrn2: bad batch/seq");
+  RB_REQUIRE(src || s_new == 1, "rb_hgrn2: split-K partials need single-token rows");
+  RB_REQUIRE(heads > 0 && key_dim > 0 && value_dim > 0, "rb_hgrn2: bad head sizes");
+  if (key_dim > 256 || value_dim > 256) return fail(RB_ERR_UNIMPLEMENTED, "rb_hgrn2: head sizes %d x %d exceed 256", key_dim, value_dim);
+  RB_REQUIRE(aligned16(state), "rb_hgrn2: the state must be 16-byte aligned");
+  if (!acc) n_acc = 0;
+  const int64_t rows = (int64_t)batch * s_new;
+  auto fill = [&](auto tag) -> int {
+    using T = decltype(tag);
+    HgrnArgs<T> a{};
+    a.src = (const T*)src; a.acc = acc; a.n_acc = n_acc; a.acc_stride = (size_t)rows * src_ld;
+    a.ld = src_ld; a.out_ld = out_ld;
+    a.f_bias = (const T*)f_bias; a.lower = (const T*)lower; a.norm_w = (const T*)norm_w; a.eps = eps;
+    a.heads = heads; a.dim = key_dim; a.vdim = value_dim;
+    a.f_off = round8(heads * key_dim); a.v_off = 2 * a.f_off;
+    RB_REQUIRE(src_ld >= a.v_off + heads * value_dim && out_ld >= (int64_t)heads * value_dim, "rb_hgrn2: row pitches too small");
+    a.s_new = s_new; a.seq_lens = c->seq_lens; a.slots = c->slots; a.new_lens = new_lens; a.state = state; a.out = (T*)out;
+    constexpr int E = 16 / sizeof(T);
+    a.raw = src && s_new > 1 && (key_dim % E) == 0 && (value_dim % E) == 0 && (src_ld % E) == 0 && aligned16(src) && aligned16(f_bias) &&
+            aligned16(lower);
+    const double sb = 4.0 * key_dim * value_dim * heads, es = sizeof(T);
+    ProfScope prof(ctx, RB_PROF_RECURRENCE,
+                   2.0 * batch * sb + rows * ((src ? es : 4.0 * n_acc) * heads * (2.0 * key_dim + value_dim) + es * heads * value_dim),
+                   5.0 * rows * heads * (double)key_dim * value_dim);
+    return run<T>(ctx, a, batch, chunk);
+  };
+  if (dtype == RB_BF16) return fill(__nv_bfloat16());
+  if (dtype == RB_F32) return fill(float());
+  return fail(RB_ERR_DTYPE, "rb_hgrn2: dtype %d unsupported", dtype);
+}
