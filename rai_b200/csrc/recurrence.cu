@@ -352,6 +352,396 @@ __global__ void __launch_bounds__(kMaxThreads) hgrn2_kernel(const HgrnArgs<T> a)
   }
 }
 
+// ------------------------------------------------------------------------------------------
+// The same recurrence for prompts of a bf16 model, eight tokens at a time on the tensor cores.  With b_t the product of
+// a row's gates from the first of the eight to t, and z_s the product of those after s:
+//   o_t = (q_t b_t) S + sum over s <= t of A_ts v_s,   A_ts = sum over rows of q_t k_s (gates after s up to t)
+//   S  <- F S + sum over s of (k_s z_s) v_s,           F = the product of all eight gates
+// Every factor is a product of gates, never a quotient, so nothing can overflow and what has decayed is simply zero.
+//
+// A warp keeps 16 columns of S, transposed, as m16n8k8 accumulators in float32; the same registers are the A operand of
+// the product with q (the eight rows of a k-step are taken in the order the accumulator layout has them).  Operands are
+// float32 split into two tf32 parts (x = hi + lo, 21 bits and more together; v is bf16 and needs no split), and all
+// products but lo lo are summed in float32.  The gates, their products and the triangle A are made by one thread per
+// channel, from registers; a block prepares two groups of eight tokens at a time.
+// ------------------------------------------------------------------------------------------
+constexpr int kSub = 8, kIterTokens = 16;
+
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+
+// Sums each of v[0..N) over the warp.  A lane ends up with at most two of the sums, in v[0] and v[1]: the ones
+// warp_sum_owner names (-1: none).
+template <int N>
+__device__ __forceinline__ void warp_sum_many(float (&v)[N], int lane) {
+  int n = N;
+#pragma unroll
+  for (int bit = 16; bit > 0; bit >>= 1) {
+    const int h = (n + 1) / 2;
+    const bool up = lane & bit;
+#pragma unroll
+    for (int i = 0; i < (N + 1) / 2; ++i)
+      if (i < h) {
+        const float lo = v[i], hi = i + h < n ? v[i + h < N ? i + h : 0] : 0.f;
+        v[i] = (up ? hi : lo) + __shfl_xor_sync(0xffffffffu, up ? lo : hi, bit);
+      }
+    n = h;
+  }
+}
+template <int N>
+__device__ __forceinline__ int warp_sum_owner(int i, int lane) {
+  int ns[5], n = N;
+#pragma unroll
+  for (int k = 0; k < 5; ++k) { ns[k] = n; n = (n + 1) / 2; }
+  if (i >= n) return -1;
+  int pos = i;
+#pragma unroll
+  for (int k = 4; k >= 0; --k) {
+    if (lane & (16 >> k)) pos += (ns[k] + 1) / 2;
+    if (pos >= ns[k]) return -1;
+  }
+  return pos;
+}
+
+template <int kTiles, bool OUT, int kMaxThreads>
+__global__ void __launch_bounds__(kMaxThreads, kMaxThreads <= 256 ? 2 : 1) hgrn2_mma_kernel(const HgrnArgs<__nv_bfloat16> a) {
+  using T = __nv_bfloat16;
+  constexpr int DP = kTiles * 8, kPairsOf8 = kSub * (kSub + 1) / 2;  // k-steps of eight rows; (t, s) pairs with s <= t
+  constexpr int kTable = DP * kSub;                                 // floats of one operand table
+  extern __shared__ __align__(16) float sm[];
+  const int n_warps = blockDim.x >> 5, cols = n_warps * 16, o_ld = cols + 4;
+  float* qb_s = sm;                              // [2 groups][tile pairs][lane][4]: q b, as the B operand of S q
+  float* kz_s = qb_s + 2 * kTable;               // the same for k z, the B operand of the state's update
+  float* decay_s = kz_s + 2 * kTable;            // [2][DP] F
+  float* tri_s = decay_s + 2 * DP;               // [2][DP / 32][40] shares of the triangle A
+  float* g_s = tri_s + 2 * (DP / 32) * 40;       // [DP] product of all gates so far (pass 1)
+  float* o_s = g_s + DP;                         // [16][o_ld]
+  T* raw = reinterpret_cast<T*>(o_s + kIterTokens * o_ld);  // two stages of [16][dim] q, [16][dim] f, [16][vdim] v
+  const int raw_f = kIterTokens * a.dim, raw_v = 2 * raw_f, stage = raw_v + kIterTokens * a.vdim;
+  const int piece = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int base = a.seq_lens[b] - a.s_new;
+  const int valid = a.new_lens ? a.new_lens[b] : a.s_new;
+  const int t_lo = piece * a.piece, t_hi = min(t_lo + a.piece, valid);
+  const bool last = t_hi == valid;
+  if (t_lo >= t_hi || (!OUT && last)) return;
+
+  auto fetch = [&](int t, int buf) {
+    const int nt = min(kIterTokens, t_hi - t), dq = a.dim / 8, dv = a.vdim / 8, per = 2 * dq + dv;
+    T* dst = raw + buf * stage;
+    for (int i = threadIdx.x; i < kIterTokens * per; i += blockDim.x) {
+      const int r = i / per, c = i % per;
+      const T* row = a.src + ((size_t)b * a.s_new + t + r) * a.ld;
+      if (c < dq) { if (OUT && r < nt) cp_async16(dst + r * a.dim + c * 8, row + h * a.dim + c * 8); }
+      else if (c < 2 * dq) { if (r < nt) cp_async16(dst + raw_f + r * a.dim + (c - dq) * 8, row + a.f_off + h * a.dim + (c - dq) * 8); }
+      else {
+        T* v = dst + raw_v + r * a.vdim + (c - 2 * dq) * 8;
+        if (r < nt) cp_async16(v, row + a.v_off + h * a.vdim + (c - 2 * dq) * 8);
+        else *reinterpret_cast<uint4*>(v) = make_uint4(0, 0, 0, 0);   // past the end: finite, and weighed with zero
+      }
+    }
+    cp_async_commit();
+  };
+  fetch(t_lo, 0);
+
+  // ---- the state: S[r][c] for columns c = warp * 16 + g (+ 8) and rows r = 8 j + 2 t4 (+ 1)
+  const size_t elems = (size_t)a.dim * a.vdim;
+  float* slot_state = a.state + ((size_t)a.slots[b] * a.heads + h) * elems;
+  const size_t pc = ((size_t)b * a.heads + h) * a.n_pieces + piece;
+  const float* from = nullptr;
+  if (OUT) from = a.n_pieces > 1 ? a.carry + pc * elems : base > 0 ? slot_state : nullptr;
+  float S[kTiles][4];
+#pragma unroll
+  for (int j = 0; j < kTiles; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = 8 * j + 2 * t4 + (e & 1), col = warp * 16 + g + (e >> 1) * 8;
+      S[j][e] = from && row < a.dim && col < a.vdim ? __ldcg(from + (size_t)row * a.vdim + col) : 0.f;
+    }
+  if (!OUT)
+    for (int i = threadIdx.x; i < DP; i += blockDim.x) g_s[i] = 1.f;
+
+  for (int t0 = t_lo, buf = 0; t0 < t_hi; t0 += kIterTokens, buf ^= 1) {
+    const int nt = min(kIterTokens, t_hi - t0);
+    const T* now = raw + buf * stage;
+    cp_async_wait_all();
+    __syncthreads();
+    if (t0 + kIterTokens < t_hi) fetch(t0 + kIterTokens, buf ^ 1);
+    // ---- one thread per (channel, group of eight tokens): gates and their products
+    for (int item = threadIdx.x; item < 2 * DP; item += blockDim.x) {
+      const int grp = item / DP, ch = item % DP;
+      float q[kSub], f[kSub], k[kSub];
+      const bool real = ch < a.dim;
+      const float fb = real ? __bfloat162float(a.f_bias[h * a.dim + ch]) : 0.f, lo = real ? __bfloat162float(a.lower[h * a.dim + ch]) : 0.f;
+#pragma unroll
+      for (int t = 0; t < kSub; ++t) {
+        q[t] = 0.f; f[t] = 1.f; k[t] = 0.f;
+        if (real && grp * kSub + t < nt) {
+          const int at = (grp * kSub + t) * a.dim + ch;
+          if (OUT) q[t] = silu_f<false>(__bfloat162float(now[at]));
+          gates<false>(__bfloat162float(now[raw_f + at]) + fb, lo, f[t], k[t]);
+        }
+      }
+      const int j = ch >> 3, r = ch & 7;
+      float* qb = qb_s + grp * kTable + (j >> 1) * 128 + (r >> 1) * 4 + (j & 1) * 2 + (r & 1);   // + token * 16
+      float* kz = kz_s + grp * kTable + (j >> 1) * 128 + r * 16 + (j & 1) * 2;                   // + (token % 4) * 4 + token / 4
+      float p = 1.f;
+#pragma unroll
+      for (int t = 0; t < kSub; ++t) { p *= f[t]; if (OUT) qb[t * 16] = q[t] * p; }
+      decay_s[grp * DP + ch] = p;
+      float z[kSub];
+      z[kSub - 1] = 1.f;
+#pragma unroll
+      for (int t = kSub - 2; t >= 0; --t) z[t] = z[t + 1] * f[t + 1];
+#pragma unroll
+      for (int t = 0; t < 4; ++t) *reinterpret_cast<float2*>(kz + t * 4) = make_float2(k[t] * z[t], k[t + 4] * z[t + 4]);
+      if (OUT) {
+        float pair[kPairsOf8];
+#pragma unroll
+        for (int s = 0; s < kSub; ++s) {
+          float w = k[s];
+#pragma unroll
+          for (int t = s; t < kSub; ++t) {
+            if (t > s) w *= f[t];
+            pair[t * (t + 1) / 2 + s] = q[t] * w;
+          }
+        }
+        warp_sum_many<kPairsOf8>(pair, lane);
+        float* tri = tri_s + (grp * (DP / 32) + (ch >> 5)) * 40;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int e = warp_sum_owner<kPairsOf8>(i, lane);
+          if (e >= 0) tri[e] = pair[i];
+        }
+      }
+    }
+    __syncthreads();
+    if (!OUT)
+      for (int i = threadIdx.x; i < DP; i += blockDim.x) g_s[i] *= decay_s[i] * decay_s[DP + i];
+    // ---- two groups of eight tokens through the tensor cores
+#pragma unroll 1
+    for (int grp = 0; grp < 2; ++grp) {
+      const int n = nt - grp * kSub;
+      if (n <= 0) break;
+      const T* v = now + raw_v + grp * kSub * a.vdim;
+      uint32_t va[4];   // v transposed: columns g, g + 8; tokens t4, t4 + 4
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int col = warp * 16 + g + (e & 1) * 8;
+        va[e] = col < a.vdim ? (uint32_t)*reinterpret_cast<const uint16_t*>(v + (t4 + (e >> 1) * 4) * a.vdim + col) << 16 : 0u;
+      }
+      if (OUT) {
+        float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};   // two chains
+        const float* qb = qb_s + grp * kTable + lane * 4;
+#pragma unroll
+        for (int j = 0; j < kTiles; j += 2) {
+          const float4 x = *reinterpret_cast<const float4*>(qb + (j >> 1) * 128);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            uint32_t sh[4], sl[4], b0h, b0l, b1h, b1l;
+            split_tf32(S[j + i][0], sh[0], sl[0]);
+            split_tf32(S[j + i][2], sh[1], sl[1]);
+            split_tf32(S[j + i][1], sh[2], sl[2]);
+            split_tf32(S[j + i][3], sh[3], sl[3]);
+            split_tf32(i ? x.z : x.x, b0h, b0l);
+            split_tf32(i ? x.w : x.y, b1h, b1l);
+            mma_tf32(o[i], sl, b0h, b1h);
+            mma_tf32(o[i], sh, b0l, b1l);
+            mma_tf32(o[i], sh, b0h, b1h);
+          }
+        }
+        // what the group's own tokens add: A is the B operand (token g, source tokens t4 and t4 + 4)
+        float a0 = 0.f, a1 = 0.f;
+        const float* tri = tri_s + grp * (DP / 32) * 40 + g * (g + 1) / 2;
+#pragma unroll
+        for (int w = 0; w < DP / 32; ++w) {
+          if (t4 <= g) a0 += tri[w * 40 + t4];
+          if (t4 + 4 <= g) a1 += tri[w * 40 + t4 + 4];
+        }
+        uint32_t a0h, a0l, a1h, a1l;
+        split_tf32(a0, a0h, a0l);
+        split_tf32(a1, a1h, a1l);
+        mma_tf32(o[0], va, a0l, a1l);
+        mma_tf32(o[1], va, a0h, a1h);
+        float* dst = o_s + (grp * kSub + 2 * t4) * o_ld + warp * 16 + g;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dst[(e & 1) * o_ld + (e >> 1) * 8] = o[0][e] + o[1][e];
+      }
+      const float* kz = kz_s + grp * kTable + lane * 4;
+      const float* dec = decay_s + grp * DP + 2 * t4;
+#pragma unroll
+      for (int j = 0; j < kTiles; j += 2) {
+        const float4 x = *reinterpret_cast<const float4*>(kz + (j >> 1) * 128);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float2 d = *reinterpret_cast<const float2*>(dec + 8 * (j + i));
+          uint32_t b0h, b0l, b1h, b1l;
+          split_tf32(i ? x.z : x.x, b0h, b0l);
+          split_tf32(i ? x.w : x.y, b1h, b1l);
+          S[j + i][0] *= d.x; S[j + i][1] *= d.y; S[j + i][2] *= d.x; S[j + i][3] *= d.y;
+          mma_tf32(S[j + i], va, b0l, b1l);
+          mma_tf32(S[j + i], va, b0h, b1h);
+        }
+      }
+    }
+    if (!OUT) continue;
+    __syncthreads();
+    // ---- norm over the head's values, one warp per token (the next tokens' tables are other arrays)
+    for (int t = warp; t < nt; t += n_warps) {
+      float s = 0.f;
+      for (int c = lane * 4; c < a.vdim; c += 128) {
+        float y[4];
+        load4(o_s + t * o_ld + c, y);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s = fmaf(y[i], y[i], s);
+      }
+      s = warp_sum(s);
+      const float r = 1.0f / sqrtf(s / (float)a.vdim + a.eps);
+      T* dst = a.out + ((size_t)b * a.s_new + t0 + t) * a.out_ld + (size_t)h * a.vdim;
+      for (int c = lane * 4; c < a.vdim; c += 128) {
+        float y[4], w[4];
+        load4(o_s + t * o_ld + c, y);
+        load4(a.norm_w + c, w);
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(y[0] * r * w[0], y[1] * r * w[1]), p1 = __floats2bfloat162_rn(y[2] * r * w[2], y[3] * r * w[3]);
+        *reinterpret_cast<uint2*>(dst + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&p0), *reinterpret_cast<const uint32_t*>(&p1));
+      }
+    }
+  }
+  float* to = OUT ? (last ? slot_state : nullptr) : a.carry + pc * elems;
+  if (!OUT) {
+    __syncthreads();
+    for (int i = threadIdx.x; i < a.dim; i += blockDim.x) a.decay[pc * a.dim + i] = g_s[i];
+  }
+  if (!to) return;
+#pragma unroll
+  for (int j = 0; j < kTiles; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = 8 * j + 2 * t4 + (e & 1), col = warp * 16 + g + (e >> 1) * 8;
+      if (row < a.dim && col < a.vdim) to[(size_t)row * a.vdim + col] = S[j][e];
+    }
+}
+
+// ------------------------------------------------------------------------------------------
+// A single-token step, bound by reading and writing the state.  One block per (sequence, head) streams it through
+// registers, eight rows per thread at a time, kLanes lanes x 4 kWide columns per row; the first rows are requested before
+// the projection that feeds the step has finished.
+// ------------------------------------------------------------------------------------------
+constexpr int kStepWarps = 8, kStepBatch = 8;
+
+template <typename T, int kLanes, int kWide>
+__global__ void __launch_bounds__(kStepWarps * 32, kWide == 1 ? 4 : 2) hgrn2_step_kernel(const HgrnArgs<T> a) {
+  constexpr bool kExact = sizeof(T) == 4;
+  constexpr int kRowsAtOnce = kStepWarps * (32 / kLanes);   // rows the block touches per turn
+  __shared__ float q_s[256], f_s[256], k_s[256], v_s[256];
+  __shared__ float o_s[kStepWarps * (32 / kLanes)][kLanes * 4 * kWide];
+  __shared__ float red[32];
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31;
+  const int r0 = (threadIdx.x >> 5) * (32 / kLanes) + lane / kLanes, c0 = (lane % kLanes) * 4;
+  pdl_launch_dependents();
+  // Read before the wait: lengths and states were left by work that a kernel without early release (the one that advances
+  // the lengths) separates from this step.
+  const int base = __ldcg(a.seq_lens + b) - 1;
+  const bool token = !a.new_lens || __ldcg(a.new_lens + b) > 0;
+  float* state = a.state + ((size_t)a.slots[b] * a.heads + h) * a.dim * a.vdim;
+  float4 S[kStepBatch][kWide];
+  auto request = [&](int i0) {
+#pragma unroll
+    for (int i = 0; i < kStepBatch; ++i)
+#pragma unroll
+      for (int w = 0; w < kWide; ++w) {
+        const int row = r0 + (i0 + i) * kRowsAtOnce, c = c0 + w * kLanes * 4;
+        S[i][w] = base > 0 && row < a.dim && c < a.vdim ? __ldcs(reinterpret_cast<const float4*>(state + (size_t)row * a.vdim + c))
+                                                       : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+  };
+  if (token) request(0);
+  pdl_wait();
+  if (!token) return;
+  auto load_u = [&](int c1, int c2, float& u1, float& u2) {  // two columns of the projection's row
+    u1 = a.src ? Cvt<T>::to_f(a.src[(size_t)b * a.ld + c1]) : 0.f;
+    u2 = a.src ? Cvt<T>::to_f(a.src[(size_t)b * a.ld + c2]) : 0.f;
+    const float* p = a.acc + (size_t)b * a.ld;
+    for (int k0 = 0; k0 < a.n_acc; k0 += 8) {
+      float t1[8], t2[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const bool have = k0 + k < a.n_acc;
+        t1[k] = have ? p[(size_t)(k0 + k) * a.acc_stride + c1] : 0.f;
+        t2[k] = have ? p[(size_t)(k0 + k) * a.acc_stride + c2] : 0.f;
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) { u1 += t1[k]; u2 += t2[k]; }
+    }
+  };
+  // items: one per channel (its q and f), one per pair of values
+  const int v_items = (a.vdim + 1) / 2;
+  for (int i = threadIdx.x; i < a.dim + v_items; i += blockDim.x) {
+    float u1, u2;
+    if (i < a.dim) {
+      const int ch = h * a.dim + i;
+      load_u(ch, a.f_off + ch, u1, u2);
+      q_s[i] = silu_f<kExact>(u1);
+      gates<kExact>(u2 + Cvt<T>::to_f(a.f_bias[ch]), Cvt<T>::to_f(a.lower[ch]), f_s[i], k_s[i]);
+    } else {
+      const int c = (i - a.dim) * 2, at = a.v_off + h * a.vdim + c, at2 = c + 1 < a.vdim ? at + 1 : at;
+      load_u(at, at2, u1, u2);
+      v_s[c] = u1;
+      if (c + 1 < a.vdim) v_s[c + 1] = u2;
+    }
+  }
+  __syncthreads();
+  float v[kWide][4], o[kWide][4];
+#pragma unroll
+  for (int w = 0; w < kWide; ++w)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int col = c0 + w * kLanes * 4 + c;
+      v[w][c] = col < a.vdim ? v_s[col] : 0.f;
+      o[w][c] = 0.f;
+    }
+  for (int i0 = 0; r0 + i0 * kRowsAtOnce < a.dim; i0 += kStepBatch) {
+    if (i0 > 0) request(i0);
+#pragma unroll
+    for (int i = 0; i < kStepBatch; ++i) {
+      const int row = r0 + (i0 + i) * kRowsAtOnce;
+      if (row >= a.dim) break;
+      const float f = f_s[row], k = k_s[row], q = q_s[row];
+#pragma unroll
+      for (int w = 0; w < kWide; ++w) {
+        float4& x = S[i][w];
+        x.x = fmaf(f, x.x, k * v[w][0]); x.y = fmaf(f, x.y, k * v[w][1]);
+        x.z = fmaf(f, x.z, k * v[w][2]); x.w = fmaf(f, x.w, k * v[w][3]);
+        o[w][0] = fmaf(x.x, q, o[w][0]); o[w][1] = fmaf(x.y, q, o[w][1]);
+        o[w][2] = fmaf(x.z, q, o[w][2]); o[w][3] = fmaf(x.w, q, o[w][3]);
+        const int c = c0 + w * kLanes * 4;
+        if (c < a.vdim) __stcs(reinterpret_cast<float4*>(state + (size_t)row * a.vdim + c), x);
+      }
+    }
+  }
+#pragma unroll
+  for (int w = 0; w < kWide; ++w) *reinterpret_cast<float4*>(&o_s[r0][c0 + w * kLanes * 4]) = make_float4(o[w][0], o[w][1], o[w][2], o[w][3]);
+  __syncthreads();
+  float y = 0.f;
+  if ((int)threadIdx.x < a.vdim) {
+#pragma unroll
+    for (int r = 0; r < kRowsAtOnce; ++r) y += o_s[r][threadIdx.x];
+  }
+  const float s = block_sum(y * y, red);
+  const float r = 1.0f / sqrtf(s / (float)a.vdim + a.eps);
+  if ((int)threadIdx.x < a.vdim)
+    a.out[(size_t)b * a.out_ld + (size_t)h * a.vdim + threadIdx.x] = Cvt<T>::from_f(y * r * Cvt<T>::to_f(a.norm_w[threadIdx.x]));
+}
+
 // carry[p] = state in front of piece p: the sequence's own state for the first; then what a piece keeps of the state in
 // front of it plus what the piece leaves on its own
 template <typename T>
@@ -400,28 +790,63 @@ int launch_one(rb_ctx* ctx, const HgrnArgs<T>& a, int batch) {
   return RB_OK;
 }
 
+template <int kTiles, bool OUT, int kMaxThreads>
+int launch_mma(rb_ctx* ctx, const HgrnArgs<__nv_bfloat16>& a, int batch) {
+  auto kern = hgrn2_mma_kernel<kTiles, OUT, kMaxThreads>;
+  const int warps = (a.vdim + 15) / 16, dp = kTiles * 8;
+  const size_t floats = 4 * dp * kSub + 2 * dp + 2 * (dp / 32) * 40 + dp + (size_t)kIterTokens * (warps * 16 + 4);
+  const size_t smem = floats * sizeof(float) + (size_t)2 * kIterTokens * (2 * a.dim + a.vdim) * sizeof(__nv_bfloat16);
+  static bool set[64] = {};
+  const int dv = ctx->device & 63;
+  if (!set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024)); set[dv] = true; }
+  RB_CUDA(launch_kernel(kern, dim3((unsigned)a.n_pieces, (unsigned)a.heads, (unsigned)batch), dim3(warps * 32), smem, ctx->stream,
+                        ctx->pdl, a));
+  ctx->launches++;
+  return RB_OK;
+}
+
 template <typename T, bool OUT>
 int launch(rb_ctx* ctx, const HgrnArgs<T>& a, int batch) {
+  if constexpr (OUT)
+    if (a.s_new == 1 && (a.vdim & 3) == 0) {
+      auto kern = a.vdim <= 64 ? hgrn2_step_kernel<T, 16, 1> : a.vdim <= 128 ? hgrn2_step_kernel<T, 32, 1> : hgrn2_step_kernel<T, 32, 2>;
+      RB_CUDA(launch_kernel(kern, dim3((unsigned)a.heads, (unsigned)batch), dim3(kStepWarps * 32), 0, ctx->stream, ctx->pdl, a));
+      ctx->launches++;
+      return RB_OK;
+    }
+  if constexpr (sizeof(T) == 2)
+    if (a.raw && a.dim <= 128) {
+      const bool wide = a.vdim > 128;
+      if (a.dim <= 64) return wide ? launch_mma<8, OUT, 512>(ctx, a, batch) : launch_mma<8, OUT, 256>(ctx, a, batch);
+      return wide ? launch_mma<16, OUT, 512>(ctx, a, batch) : launch_mma<16, OUT, 256>(ctx, a, batch);
+    }
   if (a.dim > 128) {
     if (a.vdim <= 128) return launch_one<T, 16, 8, OUT, 256>(ctx, a, batch);
     return launch_one<T, 16, 8, OUT, 512>(ctx, a, batch);
   }
-  if constexpr (OUT)
-    if (a.s_new == 1) {  // bound by reading and writing the state: more, lighter threads
-      if (a.dim <= 64) return launch_one<T, 4, 8, true, 512>(ctx, a, batch);
-      return launch_one<T, 8, 8, true, 512>(ctx, a, batch);
-    }
   if (a.dim <= 64) return launch_one<T, 4, 16, OUT, 256>(ctx, a, batch);
   return launch_one<T, 8, 16, OUT, 256>(ctx, a, batch);
 }
 
 template <typename T>
 int run(rb_ctx* ctx, HgrnArgs<T> a, int batch, int chunk) {
-  // Pieces: enough blocks to fill the GPU's block slots, none shorter than 64 tokens; one piece needs no second pass.
+  // Pieces, when the caller does not say.  A pass runs in waves of 16 warps per SM; a wave that leaves half of that is
+  // about a third faster per token, a pass without outputs takes about 0.45 of one with (measured at 128 x 128 heads).
   int piece = chunk;
   if (piece <= 0) {
-    const int want = std::max(1, (4 * ctx->sm_count) / std::max(1, batch * a.heads));
-    piece = std::max(64, (a.s_new + want - 1) / want);
+    const int64_t heads = (int64_t)batch * a.heads;
+    const int64_t slots = (int64_t)std::max(1, 16 / ((a.vdim + 15) / 16)) * ctx->sm_count;
+    auto waves = [&](int64_t blocks) {
+      const int64_t full = blocks / slots, rest = blocks % slots;
+      return (double)full + (rest == 0 ? 0.0 : rest <= slots / 2 ? 0.68 : 1.0);
+    };
+    double best = 1e30;
+    for (int n = 1; n <= 64; ++n) {
+      const int len = ((a.s_new + n - 1) / n + kTileTokens - 1) / kTileTokens * kTileTokens;
+      if (n > 1 && len < 64) break;
+      const double cost = len * (waves(heads * n) + 0.45 * waves(heads * (n - 1))) + 1e-2 * heads * (n - 1);
+      if (cost < best) { best = cost; piece = len; }
+    }
   }
   piece = (piece + kTileTokens - 1) / kTileTokens * kTileTokens;
   a.piece = piece;
