@@ -127,3 +127,16 @@ def test_shared_keys_and_prefixes():
     changed = dict(w, **{"l0.mix.k": w["l0.mix.k"] * 1.5})
     a, b = ref.residual_streams(cfg, w, toks), ref.residual_streams(cfg, changed, toks)
     assert np.abs(a[2] - b[2]).max() > np.abs(a[1] - b[1]).max() * 0.1 > 0
+
+
+def test_benchmark_compares_models_of_equal_size():
+    import os
+    import sys
+    sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    import bench
+    for name in ("malasun-1k", "malasun-2k", "malasun-4k"):
+        cfg = configs.get(name)
+        other, ours, theirs = bench.equal_size_qwen2(cfg)
+        assert abs(ours - theirs) < 0.02 * ours
+        assert other["num_hidden_layers"] == len(cfg["layers"]) and other["hidden_size"] == cfg["hidden_size"]
+        assert configs.head_dim(other) == 128
