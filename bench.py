@@ -748,6 +748,8 @@ def run_design(args):
     rows = {}
     for name in args.design_sizes.split(","):
         cfg = configs.get(name)
+        if args.layers:
+            cfg["layers"] = cfg["layers"][:args.layers]
         other, n_ours, n_other = equal_size_qwen2(cfg)
         rows[name] = {"layers": len(cfg["layers"]), "width": cfg["hidden_size"], "params": n_ours, "qwen2_params": n_other,
                       "design": design_arm(cfg, args, peaks), "qwen2": design_arm(other, args, peaks)}
