@@ -627,7 +627,7 @@ def run_ours(args):
 # --------------------------------------------------------------------------------------------------
 # A design beside its closest relative among the reference's families, at equal size
 # --------------------------------------------------------------------------------------------------
-PROFILE_CLASSES = ["gemm", "attention", "norm", "rope_kv", "embed", "argmax", "other", "recurrence"]
+PROFILE_CLASSES = ["gemm", "attention", "norm", "rope_kv", "embed", "argmax", "other", "recurrence", "experts"]
 FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12   # FMA pipe of 148 SMs at the maximum SM clock: the recurrence's float32 peak
 
 

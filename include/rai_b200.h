@@ -57,10 +57,16 @@ enum {
 
 /* ---- decoder families, rai-models/src/llm/{qwen2,phi2,phi3,gemma}.rs ---- */
 enum { RB_ARCH_QWEN2 = 0, RB_ARCH_PHI2 = 1, RB_ARCH_PHI3 = 2, RB_ARCH_GEMMA = 3,
-       RB_ARCH_MALASUN = 4 /* described layer by layer (rb_model_create_layers); no counterpart in the reference */ };
+       RB_ARCH_MALASUN = 4, RB_ARCH_VOTAPEL = 5 /* described layer by layer (rb_model_create_layers); no counterpart in
+                                                   the reference */ };
 
 /* ---- sequence mixers of a layer-by-layer design (rb_layer_config) ---- */
 enum { RB_MIXER_ATTENTION = 0, RB_MIXER_HGRN2 = 1 };
+/* ---- its feed-forwards, and how a layer joins its sublayers to the residual stream ---- */
+enum { RB_MLP_DENSE = 0,    /* one up projection with RB_ACT_XIELU */
+       RB_MLP_EXPERTS = 1   /* routed gated experts (see rb_moe_route) plus an optional shared one */ };
+enum { RB_BLOCK_POST_NORM = 0,  /* x += norm(sublayer(x)), sublayer by sublayer */
+       RB_BLOCK_PARALLEL = 1    /* h = norm(x); x += residual_mult (mixer(h) + feed_forward(h)) */ };
 
 /* ---- elementwise / reduce op tags of the primitive set (rai-core/src/dispatch.rs:41-157) ---- */
 enum {
@@ -170,6 +176,10 @@ int32_t rb_kv_cache_create(rb_ctx* ctx, int32_t layers, int32_t kv_heads, int32_
 int32_t rb_kv_cache_destroy(rb_kv_cache* c);
 /* clear_kv_cache, rai-models/src/llm/qwen2.rs:361-365: every sequence length back to 0. */
 int32_t rb_kv_cache_reset(rb_kv_cache* c);
+/* A cache of a design whose values are its keys: one set of pages serves as both (half the memory, and attention reads
+ * each page once). */
+int32_t rb_kv_cache_create_shared(rb_ctx* ctx, int32_t layers, int32_t kv_heads, int32_t head_dim, int32_t max_batch,
+                                  int32_t max_seq, int32_t dtype, rb_kv_cache** out);
 /* The sliding-window term of qwen2's mask (rai-models/src/llm/qwen2.rs:316-334): attention over this cache hides
  * key j from query i when both belong to the tokens of the same call and j + window < i (the reference's mask
  * leaves the cached prefix visible, and builds no mask for a single-token call).  Default: no window. */
@@ -278,6 +288,65 @@ int32_t rb_conv_norm_append(rb_ctx* ctx, const void* src_dev, const float* acc_d
 int32_t rb_attention_window(rb_ctx* ctx, const void* q_dev, rb_kv_cache* cache, int32_t layer, int32_t batch, int32_t s_new,
                             int32_t q_heads, int32_t value_dim, float scale, int32_t window, int32_t alibi, const void* gate_dev,
                             int64_t gate_ld, void* out_dev, int64_t out_ld, int32_t dtype);
+/* What attention may have beyond the causal softmax; a zeroed structure asks for nothing. */
+typedef struct rb_attention_options {
+  int32_t window;                  /* see rb_attention_window */
+  int32_t alibi;
+  int32_t temp_every;              /* > 0: the row at position p has its score multiplied by
+                                      1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) */
+  float temp_coef;
+  float softcap;                   /* > 0: score <- softcap * tanh(score / softcap), after scale and temperature */
+  int32_t value_dim;               /* columns of a head that are stored (<= the cache's head_dim); 0 = all */
+  const void* gate;                /* see rb_attention_window */
+  int64_t gate_ld;
+  const void* sink;                /* [q_heads], model dtype: exp(sink[h]) joins the softmax denominator of head h and
+                                      nothing else; it is neither scaled nor capped */
+  int64_t out_ld;                  /* row pitch of the output, a multiple of 8; 0 = q_heads * value_dim */
+} rb_attention_options;
+int32_t rb_attention_general(rb_ctx* ctx, const void* q_dev, rb_kv_cache* cache, int32_t layer, int32_t batch, int32_t s_new,
+                             int32_t q_heads, float scale, const rb_attention_options* options, void* out_dev, int32_t dtype);
+/* Embedding plus a learned position vector into a float32 residual stream: row i holds token i % s_new of sequence
+ * i / s_new, at position seq_len - s_new + i % s_new of its sequence (lengths from `cache`, the new tokens counted);
+ *   h[i, :] = table[ids[i], :] + positions[position, :].
+ * new_lens_dev as in rb_conv_norm_append: a row of padding takes the last position of the table when it lies beyond it. */
+int32_t rb_embed_positions(rb_ctx* ctx, const void* table_dev, const void* positions_dev, int32_t n_positions, int32_t dtype,
+                           int64_t vocab, int64_t width, int64_t ld, const uint32_t* ids_dev, int32_t batch, int32_t s_new,
+                           rb_kv_cache* cache, const int32_t* new_lens_dev, float* h_dev);
+/* The joint of a pre-norm block: with y = y_dev + sum_s acc[s] + sum_{j < top} weight[i, j] part[i * top + j, :] (each may
+ * be NULL; part rows have pitch ld, weights are float32),
+ *   h += mult * y,   out = h / sqrt(eps + mean(h^2)) * (1 + gain)   in the model dtype (out NULL: no norm).  */
+int32_t rb_add_then_norm(rb_ctx* ctx, const void* y_dev, const float* acc_dev, int32_t n_acc, const void* part_dev,
+                         const float* weight_dev, int32_t top, float mult, const void* gain_dev, float eps, int64_t rows,
+                         int64_t width, int64_t ld, float* h_dev, void* out_dev, int32_t dtype);
+/* rb_scalar_norm_rows with a gain per channel, stored as its difference from one. */
+int32_t rb_one_plus_norm_rows(rb_ctx* ctx, const float* h_dev, const int32_t* rows_dev, int64_t row_step, const void* gain_dev,
+                              float eps, int64_t n_rows, int64_t width, int64_t ld, void* out_dev, int32_t dtype);
+/* One fused input projection of a parallel block taken apart.  u = src + sum_s acc[s] + bias (acc needs s_new == 1, and
+ * bias counts only with acc: a finished tensor has its bias) has columns [q | k | gate | up], each part padded to a
+ * multiple of 8.  q goes to q_out [rows, q_heads, cache head_dim], k to the cache (which holds keys that are also the
+ * values), each head padded with zeros; silu(gate) * up, glu_size padded columns, goes to glu_out (pitch glu_ld). */
+int32_t rb_split_append(rb_ctx* ctx, const void* src_dev, const float* acc_dev, int32_t n_acc, const void* bias_dev, int64_t src_ld,
+                        int32_t batch, int32_t s_new, int32_t q_heads, int32_t kv_heads, int32_t dim, int32_t glu_size,
+                        rb_kv_cache* cache, int32_t layer, void* q_out_dev, void* glu_out_dev, int64_t glu_ld, int32_t dtype);
+/* Routing of tokens to experts.  z = sum_s acc[s] are float32 router logits: row i's experts at acc + i * z_ld, slabs
+ * acc_stride apart.  Scores are sigmoid(z).  Experts form `groups` equal runs of neighbours; a run's strength is the sum
+ * of its two largest scores; the `top` largest scores (ties: the lower index) among the `keep` strongest runs are taken.
+ *   weight[i, j] = scale * score of the j-th expert of row i          (not renormalised)
+ *   list[e * cap + t] = i * top + j                                    for every row that chose expert e, in any order
+ *   count[e] += how many                                               (zero it first; cap >= rows) */
+int32_t rb_moe_route(rb_ctx* ctx, const float* acc_dev, int32_t n_acc, int64_t acc_stride, int64_t z_ld, int64_t rows,
+                     int32_t experts, int32_t top, int32_t groups, int32_t keep, float scale, float* weight_dev,
+                     int32_t* list_dev, int32_t* count_dev, int64_t cap);
+/* The experts' two products over the lists that rb_moe_route made.  Weights are stacked by expert, wg, wu [experts][n][k]
+ * and wd [experts][n][k]; n and k are multiples of 8.  The first writes act(x Wg^T) * (x Wu^T) of each listed row (row
+ * list / top of x) to compact rows of `out` (expert after expert, [rows * top, n]); the second multiplies those rows and
+ * writes each result to row list[...] of out [rows * top, n]. */
+int32_t rb_moe_gated(rb_ctx* ctx, const void* x_dev, const void* wg_dev, const void* wu_dev, void* out_dev, int64_t rows,
+                     int32_t top, int32_t experts, const int32_t* list_dev, const int32_t* count_dev, int64_t cap, int64_t n,
+                     int64_t k, int32_t act, int32_t dtype);
+int32_t rb_moe_down(rb_ctx* ctx, const void* x_dev, const void* wd_dev, void* out_dev, int64_t rows, int32_t top,
+                    int32_t experts, const int32_t* list_dev, const int32_t* count_dev, int64_t cap, int64_t n, int64_t k,
+                    int32_t dtype);
 /* The HGRN2 recurrence: a head's state is a key_dim x value_dim matrix, and what a row forgets makes room for what it
  * takes in.  One fused projection u = src + sum_s acc[s] (with acc, s_new must be 1) has columns [q | f | v], each padded
  * to a multiple of 8.  Per token and head, for state row r with keep = lower + (1 - lower) sigmoid(u_f + f_bias):
@@ -422,19 +491,31 @@ typedef struct rb_layer_config {
   int32_t conv_taps;               /* attention: taps of the short convolution on q, k and v */
   int32_t window;                  /* attention: how many keys, its own included, a token sees; 0 = all of them */
   int32_t kv_from;                 /* attention: the earlier layer whose keys and values this one reads; -1 = its own */
-  int32_t mlp_size;                /* dense feed-forward, RB_ACT_XIELU; 0 = the layer has none */
-  int32_t reserved0;               /* set to 0 */
+  int32_t mlp_size;                /* feed-forward: inner size (of one expert, with RB_MLP_EXPERTS); 0 = the layer has none */
+  int32_t block;                   /* RB_BLOCK_* */
+  int32_t mlp_kind;                /* RB_MLP_* */
+  int32_t experts;                 /* RB_MLP_EXPERTS: how many, how many a token uses, */
+  int32_t top;
+  int32_t groups;                  /* into how many runs of neighbours they fall, and from how many a token may choose */
+  int32_t keep_groups;
+  int32_t shared_size;             /* inner size of the expert every token uses; 0 = none */
+  int32_t temp_every;              /* RB_BLOCK_PARALLEL attention: see rb_attention_options; the values are the keys */
   double scale;                    /* attention: factor on q.k */
+  double temp_coef;
+  double softcap;                  /* 0 = none */
+  double router_scale;
+  double residual_mult;            /* RB_BLOCK_PARALLEL: factor on what a layer adds to the stream */
 } rb_layer_config;
 
-/* A model of RB_ARCH_MALASUN: `layers` has cfg->num_hidden_layers entries.  Of cfg, the fields arch, dtype, vocab_size,
- * hidden_size, num_hidden_layers, norm_eps and the capacities are read.  The residual stream and the logits are float32
+/* A model of RB_ARCH_MALASUN (post-norm blocks) or RB_ARCH_VOTAPEL (parallel blocks of attention and experts, learned
+ * positions): `layers` has cfg->num_hidden_layers entries.  Of cfg, the fields arch, dtype, vocab_size, hidden_size,
+ * num_hidden_layers, norm_eps, max_position_embeddings (learned positions only) and the capacities are read.  The residual stream and the logits are float32
  * whatever the model dtype; every other rb_model_* entry point works as for the other families.  Single GPU. */
 int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out);
 /* RB_F32 or RB_BF16: the type in which rb_model_forward* return logits (the model dtype for the reference's families). */
 int32_t rb_model_logits_dtype(rb_model* m);
 /* Test hook: from now on every forward call copies the residual stream after each layer to dst_dev
- * [layers][batch * seq][hidden_size] (float32); NULL stops it.  RB_ARCH_MALASUN only; not with the captured decode step. */
+ * [layers][batch * seq][hidden_size] (float32); NULL stops it.  Layer-by-layer designs only; not with the captured decode step. */
 int32_t rb_model_set_layer_trace(rb_model* m, float* dst_dev);
 int32_t rb_model_destroy(rb_model* m);
 /* Tensor::update_by_name, rai-core/src/nn.rs:192-205: copies (and casts to the model dtype) one named
@@ -539,7 +620,7 @@ int64_t rb_launch_count(rb_ctx* ctx);
  * and fills out4 = {launches, total milliseconds, algorithmic bytes, floating-point operations} for
  * one kernel class (RB_PROF_*). */
 enum { RB_PROF_GEMM = 0, RB_PROF_ATTENTION = 1, RB_PROF_NORM = 2, RB_PROF_ROPE_KV = 3, RB_PROF_EMBED = 4,
-       RB_PROF_ARGMAX = 5, RB_PROF_OTHER = 6, RB_PROF_RECURRENCE = 7, RB_PROF_CLASSES = 8 };
+       RB_PROF_ARGMAX = 5, RB_PROF_OTHER = 6, RB_PROF_RECURRENCE = 7, RB_PROF_EXPERTS = 8, RB_PROF_CLASSES = 9 };
 int32_t rb_profile_start(rb_ctx* ctx);
 int32_t rb_profile_read(rb_ctx* ctx, int32_t kernel_class, double* out4);
 /* Bytes of device memory the model holds for parameters (after sharding). */

@@ -78,8 +78,35 @@ pub struct rb_layer_config {
     pub window: i32,
     pub kv_from: i32,
     pub mlp_size: i32,
-    pub reserved0: i32,
+    pub block: i32,
+    pub mlp_kind: i32,
+    pub experts: i32,
+    pub top: i32,
+    pub groups: i32,
+    pub keep_groups: i32,
+    pub shared_size: i32,
+    pub temp_every: i32,
     pub scale: f64,
+    pub temp_coef: f64,
+    pub softcap: f64,
+    pub router_scale: f64,
+    pub residual_mult: f64,
+}
+
+/// `struct rb_attention_options` of include/rai_b200.h, field for field.
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct rb_attention_options {
+    pub window: i32,
+    pub alibi: i32,
+    pub temp_every: i32,
+    pub temp_coef: f32,
+    pub softcap: f32,
+    pub value_dim: i32,
+    pub gate: *const c_void,
+    pub gate_ld: i64,
+    pub sink: *const c_void,
+    pub out_ld: i64,
 }
 
 /// `struct rb_model_config` of include/rai_b200.h, field for field.
@@ -137,6 +164,7 @@ extern "C" {
     pub fn rb_kv_cache_create(ctx: *mut rb_ctx, layers: i32, kv_heads: i32, head_dim: i32, max_batch: i32, max_seq: i32, dtype: i32, out: *mut *mut rb_kv_cache) -> i32;
     pub fn rb_kv_cache_destroy(c: *mut rb_kv_cache) -> i32;
     pub fn rb_kv_cache_reset(c: *mut rb_kv_cache) -> i32;
+    pub fn rb_kv_cache_create_shared(ctx: *mut rb_ctx, layers: i32, kv_heads: i32, head_dim: i32, max_batch: i32, max_seq: i32, dtype: i32, out: *mut *mut rb_kv_cache) -> i32;
     pub fn rb_kv_cache_set_window(c: *mut rb_kv_cache, window: i32) -> i32;
     pub fn rb_kv_cache_set_len(c: *mut rb_kv_cache, batch: i32, len: i32) -> i32;
     pub fn rb_kv_cache_read(c: *mut rb_kv_cache, layer: i32, seq: i32, kv_head: i32, t0: i32, n: i32, k_host: *mut c_void, v_host: *mut c_void) -> i32;
@@ -151,6 +179,14 @@ extern "C" {
     pub fn rb_scalar_norm_rows(ctx: *mut rb_ctx, h_dev: *const f32, rows_dev: *const i32, row_step: i64, gain_dev: *const c_void, eps: f32, n_rows: i64, width: i64, ld: i64, out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_conv_norm_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, conv_dev: *const c_void, taps: i32, q_weight_dev: *const c_void, k_weight_dev: *const c_void, eps: f32, batch: i32, s_new: i32, q_heads: i32, kv_heads: i32, key_dim: i32, value_dim: i32, src_ld: i64, cache: *mut rb_kv_cache, layer: i32, ring_dev: *mut f32, new_lens_dev: *const i32, q_out_dev: *mut c_void, gate_out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_attention_window(ctx: *mut rb_ctx, q_dev: *const c_void, cache: *mut rb_kv_cache, layer: i32, batch: i32, s_new: i32, q_heads: i32, value_dim: i32, scale: f32, window: i32, alibi: i32, gate_dev: *const c_void, gate_ld: i64, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
+    pub fn rb_attention_general(ctx: *mut rb_ctx, q_dev: *const c_void, cache: *mut rb_kv_cache, layer: i32, batch: i32, s_new: i32, q_heads: i32, scale: f32, options: *const rb_attention_options, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_embed_positions(ctx: *mut rb_ctx, table_dev: *const c_void, positions_dev: *const c_void, n_positions: i32, dtype: i32, vocab: i64, width: i64, ld: i64, ids_dev: *const u32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, new_lens_dev: *const i32, h_dev: *mut f32) -> i32;
+    pub fn rb_add_then_norm(ctx: *mut rb_ctx, y_dev: *const c_void, acc_dev: *const f32, n_acc: i32, part_dev: *const c_void, weight_dev: *const f32, top: i32, mult: f32, gain_dev: *const c_void, eps: f32, rows: i64, width: i64, ld: i64, h_dev: *mut f32, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_one_plus_norm_rows(ctx: *mut rb_ctx, h_dev: *const f32, rows_dev: *const i32, row_step: i64, gain_dev: *const c_void, eps: f32, n_rows: i64, width: i64, ld: i64, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_split_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, src_ld: i64, batch: i32, s_new: i32, q_heads: i32, kv_heads: i32, dim: i32, glu_size: i32, cache: *mut rb_kv_cache, layer: i32, q_out_dev: *mut c_void, glu_out_dev: *mut c_void, glu_ld: i64, dtype: i32) -> i32;
+    pub fn rb_moe_route(ctx: *mut rb_ctx, acc_dev: *const f32, n_acc: i32, acc_stride: i64, z_ld: i64, rows: i64, experts: i32, top: i32, groups: i32, keep: i32, scale: f32, weight_dev: *mut f32, list_dev: *mut i32, count_dev: *mut i32, cap: i64) -> i32;
+    pub fn rb_moe_gated(ctx: *mut rb_ctx, x_dev: *const c_void, wg_dev: *const c_void, wu_dev: *const c_void, out_dev: *mut c_void, rows: i64, top: i32, experts: i32, list_dev: *const i32, count_dev: *const i32, cap: i64, n: i64, k: i64, act: i32, dtype: i32) -> i32;
+    pub fn rb_moe_down(ctx: *mut rb_ctx, x_dev: *const c_void, wd_dev: *const c_void, out_dev: *mut c_void, rows: i64, top: i32, experts: i32, list_dev: *const i32, count_dev: *const i32, cap: i64, n: i64, k: i64, dtype: i32) -> i32;
     pub fn rb_hgrn2(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, f_bias_dev: *const c_void, lower_dev: *const c_void, norm_weight_dev: *const c_void, eps: f32, heads: i32, key_dim: i32, value_dim: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, new_lens_dev: *const i32, state_dev: *mut f32, chunk: i32, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
     pub fn rb_argmax_rows(ctx: *mut rb_ctx, logits_dev: *const c_void, dtype: i32, rows: i64, cols: i64, out_dev: *mut u32) -> i32;
     pub fn rb_sample_greedy(ctx: *mut rb_ctx, logits_dev: *const c_void, dtype: i32, rows: i64, cols: i64, penalty: f32, context_dev: *const i32, context_stride: i32, context_count_dev: *const i32, eos_token: i32, finished_dev: *mut u8, out_dev: *mut u32) -> i32;

@@ -22,8 +22,10 @@ RB_OK = 0
 U8, U32, I64, F16, BF16, F32, F64 = range(7)
 ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF, ACT_RELU, ACT_XIELU = range(6)
 NORM_RMS, NORM_RMS_ONE_PLUS, NORM_LAYER = range(3)
-ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA, ARCH_MALASUN = range(5)
+ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA, ARCH_MALASUN, ARCH_VOTAPEL = range(6)
 MIXER_ATTENTION, MIXER_HGRN2 = range(2)
+MLP_DENSE, MLP_EXPERTS = range(2)
+BLOCK_POST_NORM, BLOCK_PARALLEL = range(2)
 (UN_NEG, UN_EXP, UN_SQRT, UN_RSQRT, UN_SQUARE, UN_TANH, UN_ERF, UN_SIN, UN_COS, UN_POWF, UN_SILU, UN_GELU_TANH,
  UN_GELU_ERF, UN_RELU, UN_LOG, UN_ABS, UN_RECIP, UN_ADD_SCALAR, UN_MUL_SCALAR, UN_SIGN, UN_LOG2, UN_LOG10) = range(22)
 CMP_EQ, CMP_NE, CMP_GT, CMP_GE, CMP_LT, CMP_LE = range(6)
@@ -53,7 +55,15 @@ class LayerConfig(ctypes.Structure):
     """struct rb_layer_config of include/rai_b200.h."""
     _fields_ = [(n, ctypes.c_int32) for n in (
         "mixer", "heads", "kv_heads", "key_dim", "value_dim", "conv_taps", "window", "kv_from", "mlp_size",
-        "reserved0")] + [("scale", ctypes.c_double)]
+        "block", "mlp_kind", "experts", "top", "groups", "keep_groups", "shared_size", "temp_every")] + [
+        (n, ctypes.c_double) for n in ("scale", "temp_coef", "softcap", "router_scale", "residual_mult")]
+
+
+class AttentionOptions(ctypes.Structure):
+    """struct rb_attention_options of include/rai_b200.h."""
+    _fields_ = [("window", ctypes.c_int32), ("alibi", ctypes.c_int32), ("temp_every", ctypes.c_int32),
+                ("temp_coef", ctypes.c_float), ("softcap", ctypes.c_float), ("value_dim", ctypes.c_int32),
+                ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64), ("sink", ctypes.c_void_p), ("out_ld", ctypes.c_int64)]
 
 
 _SCALARS = {"int32_t": ctypes.c_int32, "int64_t": ctypes.c_int64, "size_t": ctypes.c_size_t, "float": ctypes.c_float,

@@ -1,7 +1,7 @@
 """Decoder configurations.
 
-Malasun, a design described layer by layer (no counterpart in the reference), has a configuration of its own shape: see
-`malasun_config`.  For the others, field names follow the reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24,
+Malasun and Votapel, designs described layer by layer (no counterpart in the reference), have configurations of their own
+shape: see `malasun_config` and `votapel_config`.  For the others, field names follow the reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24,
 phi3.rs:9-24, gemma.rs:12-27) as they appear in a Hugging Face config.json, plus `arch`.
 `BASELINE` holds the five benchmark configurations; `TINY` holds small models of the same four
 architectures for parity tests.
@@ -17,7 +17,8 @@ from typing import Dict
 from . import _lib
 
 ARCH_IDS = {"qwen2": _lib.ARCH_QWEN2, "phi2": _lib.ARCH_PHI2, "phi3": _lib.ARCH_PHI3, "gemma": _lib.ARCH_GEMMA,
-            "malasun": _lib.ARCH_MALASUN}
+            "malasun": _lib.ARCH_MALASUN, "votapel": _lib.ARCH_VOTAPEL}
+LAYERED = ("malasun", "votapel")   # described layer by layer: rb_model_create_layers
 MIXER_IDS = {"attention": _lib.MIXER_ATTENTION, "hgrn2": _lib.MIXER_HGRN2}
 # serde names of rai-nn/src/activations.rs:5-17
 ACT_IDS = {"silu": _lib.ACT_SILU, "gelu_new": _lib.ACT_GELU_TANH, "newgelu": _lib.ACT_GELU_TANH,
@@ -137,6 +138,65 @@ def malasun_config(raw: dict) -> dict:
     return _malasun(int(raw["vocab"]), int(raw["width"]), layers, float(raw["norm"]["eps"]))
 
 
+def votapel_layer(heads: int, kv_heads: int, dim: int, ff: int = 0, experts: int = 0, top: int = 0, groups: int = 1,
+                  keep: int = 1, router_scale: float = 1.0, shared_ff: int = 0, scale: float = 0.0, softcap: float = 0.0,
+                  temp_coef: float = 0.0, temp_every: int = 0) -> dict:
+    """One entry of a Votapel configuration's `layers`: attention whose values are its keys beside routed experts of inner size
+    ff (0 leaves the feed-forward out) and a shared one (shared_ff).  softcap = 0 and temp_every = 0 leave those out."""
+    mixer = dict(type="attention", heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=scale or dim ** -0.5, softcap=softcap,
+                 temp_coef=temp_coef, temp_every=temp_every)
+    mlp = dict(kind="moe", ff=ff, experts=experts, top=top, groups=groups, keep=keep, router_scale=router_scale,
+               shared_ff=shared_ff) if ff else None
+    return dict(mixer=mixer, mlp=mlp)
+
+
+def _votapel(vocab: int, width: int, layers, max_positions: int, eps: float = 1e-6, residual_mult: float = 1.0) -> dict:
+    return dict(arch="votapel", vocab_size=vocab, hidden_size=width, norm_eps=eps, max_positions=max_positions,
+                residual_mult=residual_mult, layers=layers)
+
+
+VOTAPEL: Dict[str, dict] = {
+    # sizes that resemble a real model's layers, for throughput measurements (random weights)
+    "votapel-1k": _votapel(32000, 1024, [votapel_layer(8, 2, 128, 512, 64, 4, 8, 4, 2.0, 1024, softcap=30.0, temp_coef=0.1,
+                                                       temp_every=1024)] * 16, 8192, residual_mult=0.7),
+    "votapel-2k": _votapel(32000, 2048, [votapel_layer(16, 4, 128, 1024, 32, 4, 4, 2, 2.0, 2048, softcap=30.0, temp_coef=0.1,
+                                                       temp_every=1024)] * 12, 8192, residual_mult=0.7),
+    "votapel-4k": _votapel(32000, 4096, [votapel_layer(32, 8, 128, 2048, 16, 2, 4, 2, 2.0, 4096, softcap=30.0, temp_coef=0.1,
+                                                       temp_every=1024)] * 6, 8192, residual_mult=0.7),
+    # a small model for tests
+    "tiny-votapel": _votapel(352, 144, [
+        votapel_layer(4, 2, 40, 56, 8, 2, 4, 2, 1.7, 72, softcap=9.0, temp_coef=0.3, temp_every=19),
+        votapel_layer(6, 2, 64, 96, 15, 4, 5, 3, 0.8, 0, 0.11, temp_coef=0.6, temp_every=7),
+        votapel_layer(3, 3, 24, softcap=20.0)], 400, 1e-5, 0.6),
+}
+
+
+def votapel_config(raw: dict) -> dict:
+    """A Votapel config.json -> the configuration the library takes."""
+    layers = []
+    for i, entry in enumerate(raw["layers"]):
+        kind, mix, mlp = entry["type"], entry["mixer"], entry.get("mlp")
+        if kind != "attention":
+            raise _lib.RaiB200Error(-7, f"layer {i}: mixer {kind!r} is not implemented")
+        if int(mix["vdim"]) != int(mix["dim"]):
+            raise _lib.RaiB200Error(-7, f"layer {i}: the values are the keys, so vdim must be dim")
+        ff = {}
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise _lib.RaiB200Error(-7, f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented")
+            router, groups, shared = mlp["router"], mlp["router"].get("groups") or {}, mlp.get("shared") or {}
+            ff = dict(ff=int(mlp["expert"]["ff"]), experts=int(router["experts"]), top=int(router["top"]),
+                      groups=int(groups.get("count", 1)), keep=int(groups.get("keep", 1)),
+                      router_scale=float(router.get("scale", 1.0)), shared_ff=int(shared.get("ff", 0)))
+        temp = mix.get("q_temp") or {}
+        layers.append(votapel_layer(int(mix["heads"]), int(mix["kv_heads"]), int(mix["dim"]), scale=float(mix["scale"]),
+                                    softcap=float(mix.get("softcap") or 0.0), temp_coef=float(temp.get("coef", 0.0)),
+                                    temp_every=int(temp.get("every", 0)), **ff))
+    return _votapel(int(raw["vocab"]), int(raw["width"]), layers, int(raw["max_positions"]), float(raw["norm"]["eps"]),
+                    float(raw.get("residual_mult", 1.0)))
+
+
+_CONFIG_READERS = {"Malasun": malasun_config, "Votapel": votapel_config}   # by config.json's `architecture`
 _MODEL_TYPES = {"qwen2": "qwen2", "phi": "phi2", "phi2": "phi2", "phi3": "phi3", "gemma": "gemma"}
 
 
@@ -146,16 +206,17 @@ def from_json(path: str) -> dict:
         path = os.path.join(path, "config.json")
     with open(path) as f:
         raw = json.load(f)
-    if raw.get("architecture") == "Malasun":
-        return malasun_config(raw)
+    reader = _CONFIG_READERS.get(raw.get("architecture"))
+    if reader:
+        return reader(raw)
     name = raw.get("arch") or _MODEL_TYPES.get(raw.get("model_type"))
-    if name not in ARCH_IDS or name == "malasun":
+    if name not in ARCH_IDS or name in LAYERED:
         raise _lib.RaiB200Error(-7, f"{path}: architecture {raw.get('architecture') or raw.get('model_type')!r} is not implemented")
     return dict(raw, arch=name)
 
 
 def get(name: str) -> dict:
-    src = BASELINE.get(name) or TINY.get(name) or MALASUN.get(name)
+    src = BASELINE.get(name) or TINY.get(name) or MALASUN.get(name) or VOTAPEL.get(name)
     if src is None:
         raise KeyError(f"unknown configuration {name!r}")
     return copy.deepcopy(src)
@@ -187,7 +248,15 @@ def layer_structs(cfg: dict):
         s.heads, s.key_dim, s.value_dim = mix["heads"], mix["dim"], mix["vdim"]
         s.kv_from = -1
         s.mlp_size = mlp["ff"] if mlp else 0
-        if mix["type"] == "attention":
+        if cfg["arch"] == "votapel":
+            s.block, s.residual_mult = _lib.BLOCK_PARALLEL, cfg["residual_mult"]
+            s.kv_heads, s.scale, s.softcap = mix["kv_heads"], mix["scale"], mix["softcap"]
+            s.temp_coef, s.temp_every = mix["temp_coef"], mix["temp_every"]
+            if mlp:
+                s.mlp_kind, s.experts, s.top = _lib.MLP_EXPERTS, mlp["experts"], mlp["top"]
+                s.groups, s.keep_groups = mlp["groups"], mlp["keep"]
+                s.router_scale, s.shared_size = mlp["router_scale"], mlp["shared_ff"]
+        elif mix["type"] == "attention":
             s.kv_heads, s.conv_taps, s.window, s.scale = mix["kv_heads"], mix["conv"], mix["window"], mix["scale"]
             s.kv_from = -1 if mix["kv_from"] is None else mix["kv_from"]
     return arr
@@ -195,7 +264,7 @@ def layer_structs(cfg: dict):
 
 def create_model(ctx, cfg: dict, struct, out) -> None:
     """rb_model_create or rb_model_create_layers, by architecture."""
-    if cfg["arch"] == "malasun":
+    if cfg["arch"] in LAYERED:
         _lib.call("rb_model_create_layers", ctx, ctypes.byref(struct), ctypes.byref(layer_structs(cfg)), ctypes.byref(out))
     else:
         _lib.call("rb_model_create", ctx, ctypes.byref(struct), ctypes.byref(out))
@@ -210,8 +279,9 @@ def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: i
     s.dtype = dtype
     s.max_batch, s.max_seq, s.max_tokens = int(max_batch), int(max_seq), int(max_tokens)
     s.tp_rank, s.tp_size = int(tp_rank), int(tp_size)
-    if cfg["arch"] == "malasun":
+    if cfg["arch"] in LAYERED:
         s.vocab_size, s.hidden_size, s.num_hidden_layers = cfg["vocab_size"], cfg["hidden_size"], len(cfg["layers"])
+        s.max_position_embeddings = cfg.get("max_positions", 0)
         s.norm_eps = cfg["norm_eps"]
         return s
     for k in ("vocab_size", "hidden_size", "intermediate_size", "num_hidden_layers", "num_attention_heads",

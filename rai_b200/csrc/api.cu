@@ -249,7 +249,7 @@ extern "C" int32_t rb_download(rb_ctx* ctx, void* dst, const void* src, size_t b
 
 // ------------------------------------------------------------------------------------------ KV cache
 int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_heads, int head_dim, int max_batch, int max_seq,
-                        int dtype, rb_kv_cache** out) {
+                        int dtype, rb_kv_cache** out, bool values_are_keys) {
   rb_kv_cache* c = new rb_kv_cache(shared);
   c->ctx = ctx;
   c->layers = layers; c->kv_heads = kv_heads; c->head_dim = head_dim;
@@ -260,7 +260,8 @@ int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_hea
   c->num_pages = c->pages_per_seq * c->max_batch;
   const size_t bytes = (size_t)layers * c->layer_stride_elems() * dtype_size(dtype);
   int st = rb_malloc(ctx, bytes, &c->k);
-  if (st == RB_OK) st = rb_malloc(ctx, bytes, &c->v);
+  if (st == RB_OK && values_are_keys) c->v = c->k;
+  else if (st == RB_OK) st = rb_malloc(ctx, bytes, &c->v);
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->num_pages * sizeof(int32_t), (void**)&c->block_table);
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->seq_lens);
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->slots);
@@ -269,7 +270,7 @@ int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_hea
   // Zero the pages: the tail of a sequence's last page is read (and masked) by the attention
   // kernels, so it must hold finite values.
   if (bytes) RB_CUDA(cudaMemsetAsync(c->k, 0, bytes, ctx->stream));
-  if (bytes) RB_CUDA(cudaMemsetAsync(c->v, 0, bytes, ctx->stream));
+  if (bytes && !values_are_keys) RB_CUDA(cudaMemsetAsync(c->v, 0, bytes, ctx->stream));
   if (shared) {
     c->block_table = shared->block_table;
     c->seq_lens = shared->seq_lens;
@@ -302,6 +303,15 @@ extern "C" int32_t rb_kv_cache_create(rb_ctx* ctx, int32_t layers, int32_t kv_he
   return kv_cache_create(ctx, nullptr, layers, kv_heads, head_dim, max_batch, max_seq, dtype, out);
 }
 
+extern "C" int32_t rb_kv_cache_create_shared(rb_ctx* ctx, int32_t layers, int32_t kv_heads, int32_t head_dim, int32_t max_batch,
+                                             int32_t max_seq, int32_t dtype, rb_kv_cache** out) {
+  RB_REQUIRE(ctx && out, "rb_kv_cache_create_shared: null argument");
+  RB_REQUIRE(layers > 0 && kv_heads > 0 && head_dim > 0 && max_batch > 0 && max_seq > 0, "rb_kv_cache_create_shared: bad sizes");
+  RB_REQUIRE(dtype == RB_BF16 || dtype == RB_F32, "rb_kv_cache_create_shared: dtype %d unsupported", dtype);
+  RB_REQUIRE(head_dim % 8 == 0 && head_dim <= 256, "rb_kv_cache_create_shared: head_dim %d unsupported", head_dim);
+  return kv_cache_create(ctx, nullptr, layers, kv_heads, head_dim, max_batch, max_seq, dtype, out, true);
+}
+
 int rb::kv_cache_permute(rb_kv_cache* c, const std::vector<int32_t>& order) {
   const size_t pp = (size_t)c->pages_per_seq;
   std::vector<int32_t> table(c->host_table.size()), slots(c->host_slots.size()), lens(c->host_lens.size());
@@ -326,7 +336,7 @@ extern "C" int32_t rb_kv_cache_destroy(rb_kv_cache* c) {
   for (auto it = c->ctx->caches.begin(); it != c->ctx->caches.end(); ++it)
     if (*it == c) { c->ctx->caches.erase(it); break; }
   if (c->k) cudaFree(c->k);
-  if (c->v) cudaFree(c->v);
+  if (c->v && c->v != c->k) cudaFree(c->v);
   if (!c->tables) {
     if (c->block_table) cudaFree(c->block_table);
     if (c->seq_lens) cudaFree(c->seq_lens);
@@ -429,7 +439,8 @@ extern "C" int32_t rb_gated_linear(rb_ctx* ctx, const void* x, const void* wg, c
 extern "C" int32_t rb_linear_partials(rb_ctx* ctx, const void* x, const void* w, float* part, int64_t m, int64_t n,
                                       int64_t k, int32_t n_split) {
   RB_REQUIRE(ctx && x && w && part, "rb_linear_partials: null argument");
-  RB_REQUIRE(m > 0 && m <= 256 && n > 0 && k > 0 && n_split >= 1, "rb_linear_partials: bad sizes (M must be <= 256)");
+  RB_REQUIRE(m > 0 && n > 0 && k > 0 && n_split >= 1 && (m <= 256 || n_split == 1),
+             "rb_linear_partials: bad sizes (above 256 rows: one slab)");
   GemmArgs a;
   a.x = x; a.w = w; a.out = part;
   a.m = m; a.n = n; a.k = k;
@@ -502,32 +513,45 @@ extern "C" int32_t rb_attention(rb_ctx* ctx, const void* q, rb_kv_cache* c, int3
 extern "C" int32_t rb_attention_window(rb_ctx* ctx, const void* q, rb_kv_cache* c, int32_t layer, int32_t batch, int32_t s_new,
                                        int32_t q_heads, int32_t value_dim, float scale, int32_t window, int32_t alibi,
                                        const void* gate, int64_t gate_ld, void* out, int64_t out_ld, int32_t dtype) {
-  RB_REQUIRE(ctx && q && c && out, "rb_attention_window: null argument");
-  RB_REQUIRE(dtype == c->dtype, "rb_attention_window: cache dtype differs");
-  RB_REQUIRE(layer >= 0 && layer < c->layers, "rb_attention_window: layer %d out of range", layer);
-  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0, "rb_attention_window: bad batch/seq");
-  RB_REQUIRE(q_heads > 0 && q_heads % c->kv_heads == 0, "rb_attention_window: %d query heads over %d KV heads", q_heads, c->kv_heads);
-  RB_REQUIRE(value_dim > 0 && value_dim <= c->head_dim, "rb_attention_window: value size %d of a %d-wide cache", value_dim, c->head_dim);
-  RB_REQUIRE(window >= 0 && window <= (1 << 30), "rb_attention_window: bad window %d", window);
-  RB_REQUIRE(scale > 0.f, "rb_attention_window: the scale must be positive");
-  RB_REQUIRE(out_ld >= (int64_t)q_heads * value_dim && (out_ld % 8) == 0 && (!gate || (gate_ld % 8) == 0),
-             "rb_attention_window: row pitches must be multiples of 8 and hold every head");
+  rb_attention_options o{};
+  o.window = window; o.alibi = alibi; o.gate = gate; o.gate_ld = gate_ld; o.value_dim = value_dim; o.out_ld = out_ld;
+  return rb_attention_general(ctx, q, c, layer, batch, s_new, q_heads, scale, &o, out, dtype);
+}
+
+extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache* c, int32_t layer, int32_t batch, int32_t s_new,
+                                        int32_t q_heads, float scale, const rb_attention_options* o, void* out, int32_t dtype) {
+  RB_REQUIRE(ctx && q && c && o && out, "rb_attention_general: null argument");
+  RB_REQUIRE(dtype == c->dtype, "rb_attention_general: cache dtype differs");
+  RB_REQUIRE(layer >= 0 && layer < c->layers, "rb_attention_general: layer %d out of range", layer);
+  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0, "rb_attention_general: bad batch/seq");
+  RB_REQUIRE(q_heads > 0 && q_heads % c->kv_heads == 0, "rb_attention_general: %d query heads over %d KV heads", q_heads, c->kv_heads);
+  AttnExtra x;
+  x.window = o->window; x.alibi = o->alibi != 0; x.gate = o->gate; x.gate_ld = o->gate_ld;
+  x.value_dim = o->value_dim ? o->value_dim : c->head_dim;
+  x.out_ld = o->out_ld ? o->out_ld : (int64_t)q_heads * x.value_dim;
+  x.temp_every = o->temp_every; x.temp_coef = o->temp_coef; x.softcap = o->softcap; x.sink = o->sink;
+  RB_REQUIRE(x.value_dim > 0 && x.value_dim <= c->head_dim, "rb_attention_general: value size %d of a %d-wide cache", x.value_dim,
+             c->head_dim);
+  RB_REQUIRE(x.window >= 0 && x.window <= (1 << 30), "rb_attention_general: bad window %d", x.window);
+  RB_REQUIRE(scale > 0.f, "rb_attention_general: the scale must be positive");
+  RB_REQUIRE(x.temp_every >= 0 && x.softcap >= 0.f, "rb_attention_general: bad temperature or cap");
+  RB_REQUIRE(x.out_ld >= (int64_t)q_heads * x.value_dim && (x.out_ld % 8) == 0 && (!x.gate || (x.gate_ld % 8) == 0),
+             "rb_attention_general: row pitches must be multiples of 8 and hold every head");
   double kv_tokens = 0.0, pairs = 0.0;  // keys read; visible (query, key) pairs
   for (int b = 0; b < batch; ++b) {
-    RB_REQUIRE(c->host_lens[b] >= s_new, "rb_attention_window: sequence %d holds %d tokens, fewer than the %d new ones", b,
+    RB_REQUIRE(c->host_lens[b] >= s_new, "rb_attention_general: sequence %d holds %d tokens, fewer than the %d new ones", b,
                c->host_lens[b], s_new);
-    const double len = c->host_lens[b], base = len - s_new, w = window > 0 ? window : 1e18;
-    kv_tokens += window > 0 ? (len < w + s_new - 1 ? len : w + s_new - 1) : len;
+    const double len = c->host_lens[b], base = len - s_new, w = x.window > 0 ? x.window : 1e18;
+    kv_tokens += x.window > 0 ? (len < w + s_new - 1 ? len : w + s_new - 1) : len;
     // sum over the new rows i of min(i + 1, w)
     const double full = base + 1 >= w ? s_new : (len <= w ? 0.0 : len - w);
     const double grow = s_new - full;
     pairs += (full > 0 ? full * w : 0.0) + grow * (base + 1) + 0.5 * grow * (grow - 1.0);
   }
-  AttnExtra x;
-  x.window = window; x.alibi = alibi != 0; x.gate = gate; x.gate_ld = gate_ld; x.value_dim = value_dim; x.out_ld = out_ld;
   const double es = (double)dtype_size(dtype), d = c->head_dim;
   ProfScope prof(ctx, RB_PROF_ATTENTION,
-                 es * (2.0 * kv_tokens * c->kv_heads * d + (gate ? 3.0 : 2.0) * batch * s_new * q_heads * d), 4.0 * pairs * q_heads * d);
+                 es * ((c->shared() ? 1.0 : 2.0) * kv_tokens * c->kv_heads * d + (x.gate ? 3.0 : 2.0) * batch * s_new * q_heads * d),
+                 4.0 * pairs * q_heads * d);
   if (!ctx->debug_simple_attn && attention_mma_takes(c, q_heads))
     return attention_mma_bf16(ctx, q, c, layer, batch, s_new, q_heads, scale, out, &x);
   return attention_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, &x);

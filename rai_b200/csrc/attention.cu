@@ -76,14 +76,16 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // in the 128-byte-swizzled layout [D/64 column blocks][64 keys][128 bytes]; the copy engine keeps
 // far more bytes in flight than 16-byte cp.async requests through the load/store unit can.
 // TMA = false: padded rows filled with cp.async (head sizes that are not a multiple of 64).
-template <int D, bool DECODE, bool TMA = false>
+// SHARED: the values are the keys, so a stage is one tile and the ring is twice as deep.
+template <int D, bool DECODE, bool TMA = false, bool SHARED = false>
 struct ACfg {
   static constexpr int kDP = D + 8;                      // padded row: conflict-free ldmatrix
   static constexpr int kRowBytes = kDP * 2;              // Q rows always, K/V rows when !TMA
-  static constexpr int kStages = (DECODE && D <= 128) ? 3 : 2;
+  static constexpr int kStages = ((DECODE && D <= 128) ? 3 : 2) * (SHARED ? 2 : 1);
   static constexpr int kQRows = DECODE ? 16 : 64;
   static constexpr int kTileBytes = TMA ? kTile * D * 2 : kTile * kRowBytes;   // one of K or V
-  static constexpr int kStageBytes = 2 * kTileBytes;
+  static constexpr int kStageBytes = (SHARED ? 1 : 2) * kTileBytes;
+  static constexpr int kVOffset = SHARED ? 0 : kTileBytes;
   static constexpr int kQBytes = kQRows * kRowBytes;
   static constexpr int kMergeBytes = DECODE ? (4 * 16 * D + 2 * 4 * 16) * 4 : 0;
   static constexpr int kPipeBytes = kStages * kStageBytes + kQBytes + (TMA ? 1024 : 0);
@@ -113,6 +115,10 @@ struct AParams {
   int x_window, x_alibi, x_value_dim;  // x_window: 2^30 = none
   const bf16* x_gate;
   int64_t x_gate_ld, x_out_ld;
+  int x_temp_every;
+  float x_temp_coef, x_softcap;
+  const bf16* x_sink;
+  float scale;
   // Fused single-token step (decode, tiled-copy path): the new token's q, k and v are taken straight from
   // the q/k/v projection's output (bf16 rows and/or float32 split-K partials, plus bias), rotated, and the
   // k/v rows appended to the cache by this kernel, which then needs no separate RoPE/append launch and
@@ -138,10 +144,12 @@ __device__ __forceinline__ void store_ext(const AParams& p, size_t row, int head
   p.out[row * p.x_out_ld + col] = __float2bfloat16_rn(v);
 }
 
-template <int D, bool DECODE, bool TMA, bool EXT>
+// EXT: 0 = plain causal, 1 = with what AttnExtra names, 2 = that over a cache whose values are its keys
+template <int D, bool DECODE, bool TMA, int EXT>
 __global__ void __launch_bounds__(128, (D <= 128) ? 2 : 1)
 attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v) {
-  using C = ACfg<D, DECODE, TMA>;
+  constexpr bool SHARED = EXT == 2;
+  using C = ACfg<D, DECODE, TMA, SHARED>;
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ __align__(8) uint64_t full_bar[C::kStages];
   __shared__ volatile uint32_t abort_flag;
@@ -211,12 +219,12 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
         const int page = p.block_table[(size_t)b * p.pages_per_seq + tile];
         const int y = (page * p.kv_heads + kvh) * kTile;  // first row of this (page, KV head) in the layer
         uint8_t* ks = kv_s + stage * C::kStageBytes;
-        uint8_t* vs = ks + C::kTileBytes;
+        uint8_t* vs = ks + C::kVOffset;
         ptx::mbar_expect_tx(&full_bar[stage], C::kStageBytes);
 #pragma unroll
         for (int cb = 0; cb < D / 64; ++cb) {
           ptx::tma_load_2d(ks + cb * (kTile * 128), &tm_k, &full_bar[stage], cb * 64, y);
-          ptx::tma_load_2d(vs + cb * (kTile * 128), &tm_v, &full_bar[stage], cb * 64, y);
+          if (!SHARED) ptx::tma_load_2d(vs + cb * (kTile * 128), &tm_v, &full_bar[stage], cb * 64, y);
         }
       }
       return;
@@ -226,12 +234,12 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     const bf16* ksrc = p.k + off;
     const bf16* vsrc = p.v + off;
     uint8_t* ks = kv_s + stage * C::kStageBytes;
-    uint8_t* vs = ks + C::kTileBytes;
+    uint8_t* vs = ks + C::kVOffset;
     constexpr int chunks_per_row = D / 8;
     for (int i = threadIdx.x; i < kTile * chunks_per_row; i += blockDim.x) {
       const int r = i / chunks_per_row, c = i % chunks_per_row;
       cp_async16(s_u32(ks + r * C::kRowBytes + c * 16), ksrc + (size_t)r * D + c * 8);
-      cp_async16(s_u32(vs + r * C::kRowBytes + c * 16), vsrc + (size_t)r * D + c * 8);
+      if (!SHARED) cp_async16(s_u32(vs + r * C::kRowBytes + c * 16), vsrc + (size_t)r * D + c * 8);
     }
   };
   // byte offset of the 16-byte chunk holding (key, dcol..dcol+8) inside a K or V tile
@@ -358,6 +366,14 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     slope2[0] = alibi_slope(DECODE ? head + g : head, p.q_heads) * kLog2e;
     slope2[1] = DECODE ? alibi_slope(head + g + 8, p.q_heads) * kLog2e : slope2[0];
   }
+  // what a raw score is multiplied with (row temperature included): up to log2 units, or up to the cap's argument
+  float row_unit[2] = {p.scale_log2, p.scale_log2};
+  const float cap2 = EXT ? p.x_softcap * kLog2e : 0.f;
+  if (EXT) {
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf)
+      row_unit[hf] = p.scale * query_temperature(lim[hf], p.x_temp_every, p.x_temp_coef) * (cap2 > 0.f ? 1.0f / p.x_softcap : kLog2e);
+  }
   bool q_loaded = false;
   bool aborted = false;
   for (int tile = tile_lo; tile < tile_hi; ++tile) {
@@ -380,7 +396,7 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
       uint8_t* ks_w = kv_s + (it % C::kStages) * C::kStageBytes;
       for (int i = threadIdx.x; i < 2 * (D / 8); i += blockDim.x) {
         const int is_v = i / (D / 8), c = i % (D / 8);
-        *reinterpret_cast<uint4*>(ks_w + is_v * C::kTileBytes + tile_off(new_slot, c * 8)) =
+        *reinterpret_cast<uint4*>(ks_w + is_v * C::kVOffset + tile_off(new_slot, c * 8)) =
             *reinterpret_cast<const uint4*>(new_kv + is_v * D + c * 8);
       }
       __syncthreads();
@@ -392,7 +408,7 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
       q_loaded = true;
     }
     const uint8_t* ks = kv_s + (it % C::kStages) * C::kStageBytes;
-    const uint8_t* vs = ks + C::kTileBytes;
+    const uint8_t* vs = ks + C::kVOffset;
     const int tile_start = tile * kTile;
     // a warp whose rows all precede this tile has nothing to do (prefill, diagonal tiles only)
     // (warp-uniform by construction: mma.sync and ldmatrix need every lane)
@@ -426,10 +442,11 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
           const int hf = e >> 1;
           // causal limit (lim is the row's own position) and, among the new tokens only, the sliding window
           bool seen;
-          float score = s[nt][e] * p.scale_log2;
+          float score = s[nt][e] * row_unit[hf];
           if (EXT) {  // rolling window, in prompts and single-token steps alike; then the distance bias
             const int dist = lim[hf] - key_abs;
             seen = dist >= 0 && dist < p.x_window;
+            if (cap2 > 0.f) score = cap2 * tanh_sfu(score);
             score = fmaf(-slope2[hf], (float)dist, score);
           } else {
             seen = key_abs <= lim[hf] && (DECODE || key_abs < base || key_abs + p.window >= lim[hf]);
@@ -503,6 +520,7 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     for (int hf = 0; hf < 2; ++hf) {
       const int row = q0 + qrow0 + g + hf * 8;
       if (row >= p.s_new) continue;
+      if (EXT && p.x_sink) l_run[hf] += exp2f(__bfloat162float(p.x_sink[head]) * kLog2e - m_run[hf]);
       const float inv = 1.0f / l_run[hf];
       if (EXT) {
 #pragma unroll
@@ -551,6 +569,7 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     }
     const size_t bh = (size_t)b * p.q_heads + head + row;
     if (p.n_splits == 1) {
+      if (EXT && p.x_sink) L += exp2f(__bfloat162float(p.x_sink[head + row]) * kLog2e - Mu);
       if (EXT) store_ext(p, b, head + row, dd, O / L);
       else p.out[bh * D + dd] = __float2bfloat16_rn(O / L);
     } else {
@@ -593,6 +612,7 @@ attention_kernel(const AParams p, const __grid_constant__ CUtensorMap tm_k, cons
     float L = 0.f;
     for (int sp = 0; sp < ns; ++sp) L += w_s[512 + row * 32 + sp] * exp2f(w_s[row * 32 + sp] - Mu);
     for (int sp = 0; sp < ns; ++sp) w_s[row * 32 + sp] = exp2f(w_s[row * 32 + sp] - Mu);
+    if (EXT && p.x_sink) L += exp2f(__bfloat162float(p.x_sink[head + row]) * kLog2e - Mu);  // once, not per split
     w_s[1024 + row] = L;
   }
   __syncthreads();
@@ -634,10 +654,10 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
 }
 
 // Launches attention_kernel<D, DECODE> with tiled-copy loading when the head size allows it.
-template <int D, bool DECODE, bool EXT = false>
+template <int D, bool DECODE, int EXT = 0>
 int launch_attn_kernel(rb_ctx* ctx, rb_kv_cache* c, const AParams& p, dim3 grid) {
   constexpr bool kTma = (D % 64) == 0;
-  using C = ACfg<D, DECODE, kTma>;
+  using C = ACfg<D, DECODE, kTma, EXT == 2>;
   auto kern = attention_kernel<D, DECODE, kTma, EXT>;
   static bool set[64] = {};  // the attribute belongs to the (kernel, device) pair
   const int dv = ctx->device & 63;
@@ -654,7 +674,7 @@ int launch_attn_kernel(rb_ctx* ctx, rb_kv_cache* c, const AParams& p, dim3 grid)
   return RB_OK;
 }
 
-template <int D, bool EXT = false>
+template <int D, int EXT = 0>
 int launch_attention(rb_ctx* ctx, rb_kv_cache* c, AParams& p, int batch, int max_len) {
   if (p.s_new > 1) {
     dim3 grid((unsigned)((p.s_new + 63) / 64), (unsigned)p.q_heads, (unsigned)batch);
@@ -785,13 +805,19 @@ int attention_mma_bf16(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, in
     p.x_gate = (const bf16*)ext->gate;
     p.x_gate_ld = ext->gate_ld;
     p.x_out_ld = ext->out_ld;
+    p.x_temp_every = ext->temp_every;
+    p.x_temp_coef = ext->temp_coef;
+    p.x_softcap = ext->softcap;
+    p.x_sink = (const bf16*)ext->sink;
+    p.scale = scale;
     max_len = attention_walk_len(max_len, ext->window);
+    const bool sh = c->shared();
     switch (c->head_dim) {
-      case 64: return launch_attention<64, true>(ctx, c, p, batch, max_len);
-      case 80: return launch_attention<80, true>(ctx, c, p, batch, max_len);
-      case 96: return launch_attention<96, true>(ctx, c, p, batch, max_len);
-      case 128: return launch_attention<128, true>(ctx, c, p, batch, max_len);
-      case 256: return launch_attention<256, true>(ctx, c, p, batch, max_len);
+      case 64: return sh ? launch_attention<64, 2>(ctx, c, p, batch, max_len) : launch_attention<64, 1>(ctx, c, p, batch, max_len);
+      case 80: return sh ? launch_attention<80, 2>(ctx, c, p, batch, max_len) : launch_attention<80, 1>(ctx, c, p, batch, max_len);
+      case 96: return sh ? launch_attention<96, 2>(ctx, c, p, batch, max_len) : launch_attention<96, 1>(ctx, c, p, batch, max_len);
+      case 128: return sh ? launch_attention<128, 2>(ctx, c, p, batch, max_len) : launch_attention<128, 1>(ctx, c, p, batch, max_len);
+      case 256: return sh ? launch_attention<256, 2>(ctx, c, p, batch, max_len) : launch_attention<256, 1>(ctx, c, p, batch, max_len);
     }
     return fail(RB_ERR_UNIMPLEMENTED, "attention: head_dim %d has no tensor-core kernel (64, 80, 96, 128, 256)", c->head_dim);
   }

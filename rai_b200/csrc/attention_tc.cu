@@ -40,8 +40,10 @@ constexpr int kBN = 64;   // keys per tile = tokens per cache page
 constexpr int kThreads = 192;
 constexpr float kLog2e = 1.4426950408889634f;
 
-template <int D>
+template <int D, bool SHARED = false>
 struct TCfg {
+  // the values are the keys: one ring over the space of both, a tile is released once both products have read it
+  static constexpr int kRing = SHARED ? 4 : 2;
   static constexpr int kQBytes = kBM * D * 2;   // [D/64 column blocks][128 rows][128 bytes]
   static constexpr int kKBytes = kBN * D * 2;   // [D/64][64 keys][128 bytes]
   static constexpr int kVBytes = kBN * D * 2;
@@ -73,6 +75,9 @@ struct TParams {
   int x_window, x_alibi, x_value_dim;
   const bf16* x_gate;
   int64_t x_gate_ld, x_out_ld;
+  int x_temp_every;
+  float x_temp_coef, x_softcap, scale;
+  const bf16* x_sink;
 #ifdef RB_DEBUG_AIDS
   unsigned long long* trace;  // developer build: cycles per phase of one softmax thread (see launch_tc)
 #endif
@@ -85,18 +90,40 @@ struct TParams {
 #endif
 
 struct Ctrl {  // lives in dynamic shared memory behind the tiles
-  uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], s_empty[2], p_full, o_done;
+  uint64_t q_full, k_full[4], k_empty[4], v_full[2], v_empty[2], s_full[2], s_empty[2], p_full, o_done;
   uint32_t tmem_base;
   uint32_t abort_flag;
   uint32_t k_issued, v_issued;
 };
 static_assert(sizeof(Ctrl) <= 256, "control block exceeds its reservation");
 
-template <int D, bool EXT>
+// tanh(x) = x (c0 + c1 x^2 + ... + c4 x^8) for |x| <= 1/2: a least-maximum fit of the relative error (1.3e-8)
+constexpr float kTanhPolyLimit = 0.5f;
+constexpr float kTanhC0 = 0.99999999f, kTanhC1 = -0.33333076f, kTanhC2 = 0.13324908f, kTanhC3 = -0.05299429f, kTanhC4 = 0.01715141f;
+
+// two float32 operations in one instruction
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+  return r;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)),
+        "l"(reinterpret_cast<unsigned long long&>(c)));
+  return r;
+}
+
+// EXT: 0 = plain causal, 1 = with what AttnExtra names, 2 = that over a cache whose values are its keys
+template <int D, int EXT>
 __global__ void __launch_bounds__(kThreads, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                             const __grid_constant__ CUtensorMap tm_v, const TParams p) {
-  using C = TCfg<D>;
+  constexpr bool SHARED = EXT == 2;
+  using C = TCfg<D, SHARED>;
+  constexpr int KR = C::kRing;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* q_s = smem;
   uint8_t* k_s = q_s + C::kQBytes;
@@ -108,8 +135,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
 
   if (threadIdx.x == 0) {
     ptx::mbar_init(&ctl->q_full, 1);
+    for (int i = 0; i < KR; ++i) { ptx::mbar_init(&ctl->k_full[i], 1); ptx::mbar_init(&ctl->k_empty[i], 1); }
     for (int i = 0; i < 2; ++i) {
-      ptx::mbar_init(&ctl->k_full[i], 1); ptx::mbar_init(&ctl->k_empty[i], 1);
       ptx::mbar_init(&ctl->v_full[i], 1); ptx::mbar_init(&ctl->v_empty[i], 1);
       ptx::mbar_init(&ctl->s_full[i], 1); ptx::mbar_init(&ctl->s_empty[i], 4);
     }
@@ -156,16 +183,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         ptx::tma_load_2d(q_s + cb * (kBM * 128), &tm_q, &ctl->q_full, head * D + cb * 64, b * p.s_new + q0);
       bool ok = true;
       for (int j = 0; j < n && ok; ++j) {
-        const int st = j & 1;
-        const uint32_t ph = (uint32_t)(j >> 1) & 1u;
+        const int st = j & 1, kst = j % KR;
+        const uint32_t ph = (uint32_t)(j >> 1) & 1u, kph = (uint32_t)(j / KR) & 1u;
         const int page = p.block_table[(size_t)b * p.pages_per_seq + tile_lo + j];
         const int y = (page * p.kv_heads + kvh) * kBN;  // first row of this (page, KV head) in the layer
-        if (!ptx::mbar_wait(&ctl->k_empty[st], ph ^ 1u, abort_flag, p.wait_cycles)) { ok = false; break; }
-        ptx::mbar_expect_tx(&ctl->k_full[st], C::kKBytes);
+        if (!ptx::mbar_wait(&ctl->k_empty[kst], kph ^ 1u, abort_flag, p.wait_cycles)) { ok = false; break; }
+        ptx::mbar_expect_tx(&ctl->k_full[kst], C::kKBytes);
 #pragma unroll
         for (int cb = 0; cb < D / 64; ++cb)
-          ptx::tma_load_2d(k_s + st * C::kKBytes + cb * (kBN * 128), &tm_k, &ctl->k_full[st], cb * 64, y);
+          ptx::tma_load_2d(k_s + kst * C::kKBytes + cb * (kBN * 128), &tm_k, &ctl->k_full[kst], cb * 64, y);
         ctl->k_issued = (uint32_t)(j + 1);
+        if (SHARED) continue;
         if (!ptx::mbar_wait(&ctl->v_empty[st], ph ^ 1u, abort_flag, p.wait_cycles)) { ok = false; break; }
         ptx::mbar_expect_tx(&ctl->v_full[st], C::kVBytes);
 #pragma unroll
@@ -183,20 +211,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       const uint32_t qa = ptx::smem_u32(q_s), ka = ptx::smem_u32(k_s), va = ptx::smem_u32(v_s), pa = ptx::smem_u32(p_s);
       bool ok = ptx::mbar_wait(&ctl->q_full, 0u, abort_flag, p.wait_cycles);
       auto issue_scores = [&](int j) -> bool {
-        const int st = j & 1;
+        const int st = j & 1, kst = j % KR;
         const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-        if (!ptx::mbar_wait(&ctl->k_full[st], ph, abort_flag, p.wait_cycles)) return false;
+        if (!ptx::mbar_wait(&ctl->k_full[kst], (uint32_t)(j / KR) & 1u, abort_flag, p.wait_cycles)) return false;
         if (!ptx::mbar_wait(&ctl->s_empty[st], ph ^ 1u, abort_flag, p.wait_cycles)) return false;
         ptx::tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
           const uint32_t a = qa + (kk >> 2) * (kBM * 128) + (kk & 3) * 32;
-          const uint32_t bb = ka + st * C::kKBytes + (kk >> 2) * (kBN * 128) + (kk & 3) * 32;
+          const uint32_t bb = ka + kst * C::kKBytes + (kk >> 2) * (kBN * 128) + (kk & 3) * 32;
           ptx::umma_bf16(tmem_base + (uint32_t)(st * kBN), ptx::umma_desc_k_sw128(a), ptx::umma_desc_k_sw128(bb), idesc_s,
                          kk > 0 ? 1u : 0u);
         }
         ptx::umma_commit(&ctl->s_full[st]);
-        ptx::umma_commit(&ctl->k_empty[st]);
+        if (!SHARED) ptx::umma_commit(&ctl->k_empty[kst]);
         return true;
       };
       if (ok) ok = issue_scores(0);
@@ -204,7 +232,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         if (j + 1 < n && !issue_scores(j + 1)) { ok = false; break; }
         const int st = j & 1;
         const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-        if (!ptx::mbar_wait(&ctl->v_full[st], ph, abort_flag, p.wait_cycles)) { ok = false; break; }
+        if (!SHARED && !ptx::mbar_wait(&ctl->v_full[st], ph, abort_flag, p.wait_cycles)) { ok = false; break; }
+        const uint32_t vt = SHARED ? ka + (j % KR) * C::kKBytes : va + st * C::kVBytes;
         if (!ptx::mbar_wait(&ctl->p_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles)) { ok = false; break; }
         ptx::tc_fence_after();
 #pragma unroll
@@ -212,11 +241,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           // A = P: K-major, 16 keys = 32 bytes further along the 128-byte row.  B = V: MN-major, 16 keys = 16 rows of
           // 128 bytes further; the second 64 columns of head_dim follow one [64 keys][128 B] block later.
           const uint64_t da = ptx::umma_desc_k_sw128(pa + ks * 32);
-          const uint64_t db = ptx::umma_desc_mn_sw128(va + st * C::kVBytes + ks * (16 * 128), kBN * 128, 1024);
+          const uint64_t db = ptx::umma_desc_mn_sw128(vt + ks * (16 * 128), kBN * 128, 1024);
           ptx::umma_bf16(tmem_base + C::kOCol, da, db, idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
         }
         ptx::umma_commit(&ctl->o_done);
-        ptx::umma_commit(&ctl->v_empty[st]);
+        ptx::umma_commit(SHARED ? &ctl->k_empty[j % KR] : &ctl->v_empty[st]);
       }
       if (!ok) { p.status[0] = (uint32_t)(-RB_ERR_TIMEOUT); p.status[1] = 0xA7C2u; p.status[2] = blockIdx.x; p.status[3] = blockIdx.z; }
     }
@@ -228,6 +257,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     const uint32_t t_row = tmem_base + ((uint32_t)(quarter * 32) << 16);
     const bool windowed = EXT ? p.x_window < (1 << 30) : p.window < (1 << 30);
     const float slope2 = EXT && p.x_alibi ? alibi_slope(head, p.q_heads) * kLog2e : 0.f;
+    const bool capped = EXT && p.x_softcap > 0.f;
+    // what a raw score of this row is multiplied with: up to log2 units, or up to the cap's argument
+    const float row_unit = EXT ? p.scale * query_temperature(row_abs, p.x_temp_every, p.x_temp_coef) * (capped ? 1.0f / p.x_softcap : kLog2e) : 0.f;
+    const float cap2 = EXT ? p.x_softcap * kLog2e : 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
 #ifdef RB_DEBUG_AIDS
@@ -262,9 +295,44 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       const bool window_edge = EXT ? windowed && base + q0 + kBM - 1 - key0 >= p.x_window
                                    : windowed && key0 + kBN > base && base + q0 + kBM - 1 - p.window > key0;
       if (EXT) {  // log2-scaled score less the distance bias; what follows then needs no scale of its own
-        const float b0 = slope2 * (float)(key0 - row_abs);
+        if (capped) {
+          // cap * tanh(score / cap), in log2 units.  Scores are mostly small against the cap: an odd polynomial on the FMA
+          // pipe covers them and leaves the special-function unit to the exponentials; a warp with a larger one takes
+          // the general form for its whole tile.
+          float top4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < kBN; ++i) s[i] = fmaf(s[i], p.scale_log2, fmaf(slope2, (float)i, b0));
+          for (int i = 0; i < kBN; i += 4) {
+            top4[0] = fmaxf(top4[0], fabsf(s[i])); top4[1] = fmaxf(top4[1], fabsf(s[i + 1]));
+            top4[2] = fmaxf(top4[2], fabsf(s[i + 2])); top4[3] = fmaxf(top4[3], fabsf(s[i + 3]));
+          }
+          const float top = fmaxf(fmaxf(top4[0], top4[1]), fmaxf(top4[2], top4[3])) * row_unit;
+          if (__any_sync(0xffffffffu, top > kTanhPolyLimit)) {
+#pragma unroll
+            for (int i = 0; i < kBN; ++i) s[i] = cap2 * tanh_sfu(s[i] * row_unit);
+          } else {
+            // in x = score / cap: cap2 (c0 x + c1 x^3 + ...) with the powers of row_unit folded into the coefficients
+            const float r2 = row_unit * row_unit;
+            const float c0 = cap2 * row_unit * kTanhC0, c1 = c0 * r2 * (kTanhC1 / kTanhC0), c2 = c0 * r2 * r2 * (kTanhC2 / kTanhC0);
+            const float c3 = c0 * r2 * r2 * r2 * (kTanhC3 / kTanhC0), c4 = c0 * r2 * r2 * r2 * r2 * (kTanhC4 / kTanhC0);
+            const float2 d0 = make_float2(c0, c0), d1 = make_float2(c1, c1), d2 = make_float2(c2, c2), d3 = make_float2(c3, c3),
+                         d4 = make_float2(c4, c4);
+#pragma unroll
+            for (int i = 0; i < kBN; i += 2) {
+              const float2 x = make_float2(s[i], s[i + 1]), u = mul2(x, x);
+              const float2 y = mul2(x, fma2(u, fma2(u, fma2(u, fma2(u, d4, d3), d2), d1), d0));
+              s[i] = y.x;
+              s[i + 1] = y.y;
+            }
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < kBN; ++i) s[i] *= row_unit;
+        }
+        if (p.x_alibi) {
+          const float b0 = slope2 * (float)(key0 - row_abs);
+#pragma unroll
+          for (int i = 0; i < kBN; ++i) s[i] += fmaf(slope2, (float)i, b0);
+        }
       }
       if (causal_edge || window_edge) {
 #pragma unroll
@@ -346,6 +414,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     if (ok) ok = __all_sync(0xffffffffu, ptx::mbar_wait(&ctl->o_done, (uint32_t)(n - 1) & 1u, abort_flag, p.wait_cycles));
     if (ok) {
       ptx::tc_fence_after();
+      if (EXT && p.x_sink) l_run += ex2_fast(fmaf(__bfloat162float(p.x_sink[head]), kLog2e, -m_run));
       const float inv = 1.0f / l_run;
       const bool store = q0 + row < p.s_new;
       bf16* dst = p.out + (((size_t)b * p.s_new + q0 + row) * p.q_heads + head) * D;
@@ -405,8 +474,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     // copies already handed to the copy engine get a bounded chance to land before the shared memory is released
     volatile uint32_t never = 0;
     ptx::mbar_wait(&ctl->q_full, 0u, &never, p.wait_cycles);
-    for (uint32_t i = (ctl->k_issued > 2 ? ctl->k_issued - 2 : 0); i < ctl->k_issued; ++i)
-      ptx::mbar_wait(&ctl->k_full[i & 1], (i >> 1) & 1u, &never, p.wait_cycles);
+    for (uint32_t i = (ctl->k_issued > KR ? ctl->k_issued - KR : 0); i < ctl->k_issued; ++i)
+      ptx::mbar_wait(&ctl->k_full[i % KR], (i / KR) & 1u, &never, p.wait_cycles);
     for (uint32_t i = (ctl->v_issued > 2 ? ctl->v_issued - 2 : 0); i < ctl->v_issued; ++i)
       ptx::mbar_wait(&ctl->v_full[i & 1], (i >> 1) & 1u, &never, p.wait_cycles);
   }
@@ -418,10 +487,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   }
 }
 
-template <int D, bool EXT>
+template <int D, int EXT>
 int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
               const AttnExtra* ext) {
-  using C = TCfg<D>;
+  using C = TCfg<D, EXT == 2>;
   const size_t loff = (size_t)layer * c->layer_stride_elems();
   const bf16* kbase = (const bf16*)c->k + loff;
   const bf16* vbase = (const bf16*)c->v + loff;
@@ -456,6 +525,11 @@ int launch_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, 
     p.x_gate = (const bf16*)ext->gate;
     p.x_gate_ld = ext->gate_ld;
     p.x_out_ld = ext->out_ld;
+    p.x_temp_every = ext->temp_every;
+    p.x_temp_coef = ext->temp_coef;
+    p.x_softcap = ext->softcap;
+    p.x_sink = (const bf16*)ext->sink;
+    p.scale = scale;
   }
   dim3 grid((unsigned)((s_new + kBM - 1) / kBM), (unsigned)q_heads, (unsigned)batch);
 #ifdef RB_DEBUG_AIDS
@@ -495,10 +569,12 @@ bool attention_prefill_tc_supported(const rb_kv_cache* c, int s_new, int q_heads
 
 int attention_prefill_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
                          void* out, const AttnExtra* ext) {
-  if (ext && c->head_dim == 64) return launch_tc<64, true>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
-  if (ext && c->head_dim == 128) return launch_tc<128, true>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
-  if (c->head_dim == 64) return launch_tc<64, false>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, nullptr);
-  if (c->head_dim == 128) return launch_tc<128, false>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, nullptr);
+  const int kind = !ext ? 0 : c->shared() ? 2 : 1;
+  auto go = [&](auto plain, auto extra, auto shared) {
+    return (kind == 0 ? plain : kind == 1 ? extra : shared)(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
+  };
+  if (c->head_dim == 64) return go(launch_tc<64, 0>, launch_tc<64, 1>, launch_tc<64, 2>);
+  if (c->head_dim == 128) return go(launch_tc<128, 0>, launch_tc<128, 1>, launch_tc<128, 2>);
   return fail(RB_ERR_UNIMPLEMENTED, "tensor-core prefill attention: head_dim %d unsupported (64, 128)", c->head_dim);
 }
 

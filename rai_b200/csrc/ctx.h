@@ -68,7 +68,8 @@ struct rb_kv_cache {
   int pages_per_seq = 0, num_pages = 0;
   int window = 1 << 30;  // sliding-window width of the attention mask (rb_kv_cache_set_window); 2^30 = none
   void* k = nullptr;
-  void* v = nullptr;
+  void* v = nullptr;               // == k: the values are the keys
+  bool shared() const { return k == v; }
   int32_t* block_table = nullptr;  // device [max_batch][pages_per_seq]
   int32_t* seq_lens = nullptr;     // device [max_batch]
   int32_t* slots = nullptr;        // device [max_batch]: where sequence b keeps its recurrent and convolution state
@@ -110,8 +111,9 @@ struct TpPeers {
 
 namespace rb {
 // api.cu: layers >= 0; `shared` makes a view over another cache's sequences (max_batch and max_seq are then its)
+// (values_are_keys: one set of pages for both)
 int kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_heads, int head_dim, int max_batch, int max_seq, int dtype,
-                    rb_kv_cache** out);
+                    rb_kv_cache** out, bool values_are_keys = false);
 // sequences order[0 .. max_batch) (a permutation) become 0, 1, ...: pages, slots and lengths move with them
 int kv_cache_permute(rb_kv_cache* c, const std::vector<int32_t>& order);
 constexpr int kPageTokens = 64;
@@ -151,12 +153,62 @@ struct GemmArgs {
   const void* act_params = nullptr;  // RB_ACT_XIELU: its two numbers, model dtype
   int n_split = 1;              // > 1: write float partials, no epilogue
   bool partials = false;
+  // Grouped form: the rows of x are shared out among `experts` weight matrices stacked in w (and w2), see rb_moe_gated.
+  const int32_t *list = nullptr, *count = nullptr;
+  int64_t cap = 0;
+  int experts = 0, top = 1;
   bool reduce = false;            // M <= 64: if K is split, sum the splits inside the kernel and apply the epilogue
 };
 int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a);
+constexpr int kMaxExperts = 256;
+int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a);
 int gemm_tc_pick_splits(rb_ctx* ctx, int64_t m, int64_t n, int64_t k);
 int gemm_reserve_scratch(rb_ctx* ctx, size_t bytes);
 int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype);
+
+// moe.cu: rb_split_append and rb_moe_route in one launch (route NULL: the first alone)
+struct SplitSpec {
+  const void* src = nullptr;
+  const float* acc = nullptr;
+  int n_acc = 0;
+  const void* bias = nullptr;
+  int64_t src_ld = 0;
+  int batch = 0, s_new = 0, q_heads = 0, kv_heads = 0, dim = 0, glu_size = 0;
+  rb_kv_cache* cache = nullptr;
+  int layer = 0;
+  void *q_out = nullptr, *glu_out = nullptr;
+  int64_t glu_ld = 0;
+};
+struct RouteSpec {
+  const float* acc = nullptr;
+  int n_acc = 0;
+  int64_t acc_stride = 0, z_ld = 0;
+  int experts = 0, top = 0, groups = 1, keep = 1;
+  float scale = 1.f;
+  float* weight = nullptr;
+  int32_t *list = nullptr, *count = nullptr;
+  int64_t cap = 0;
+};
+int split_and_route(rb_ctx* ctx, const SplitSpec& split, const RouteSpec* route, int dtype);
+// mixer_kernels.cu: rb_add_then_norm, and the experts' row counters back to zero for the next layer
+struct JoinSpec {
+  const void* y = nullptr;
+  const float* acc = nullptr;
+  int n_acc = 0;
+  const void* part = nullptr;
+  const float* weight = nullptr;
+  int top = 0;
+  float mult = 1.f;
+  const void* gain = nullptr;
+  float eps = 0.f;
+  int64_t rows = 0;
+  int width = 0, ld = 0;
+  float* h = nullptr;
+  void* out = nullptr;
+  int32_t* zero = nullptr;
+  int n_zero = 0;
+};
+int add_then_norm(rb_ctx* ctx, const JoinSpec& s, int dtype);
 
 // What an attention layer may have beyond the plain causal form.
 struct AttnExtra {
@@ -166,7 +218,21 @@ struct AttnExtra {
   int64_t gate_ld = 0;
   int value_dim = 0;           // columns of a head that are stored (the cache may hold padded heads)
   int64_t out_ld = 0;          // row pitch of the output
+  int temp_every = 0;          // > 0: scores of the row at position p grow by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+  float temp_coef = 0.f;
+  float softcap = 0.f;         // > 0: score <- softcap tanh(score / softcap)
+  const void* sink = nullptr;  // [q_heads], cache dtype: exp(sink) joins the softmax denominator
 };
+// factor on the scores of the row at position `pos`
+__device__ __forceinline__ float query_temperature(int pos, int every, float coef) {
+  return every > 0 ? fmaf(coef, logf((float)((pos + 1) / every + 1)), 1.0f) : 1.0f;
+}
+// tanh to about 1e-7 absolute from two special-function operations; saturates without a NaN
+__device__ __forceinline__ float tanh_sfu(float x) {
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
+  return 1.0f - __fdividef(2.0f, 1.0f + e);
+}
 // slope of the distance bias, 2^(-8 (h + 1) / heads)
 __device__ __forceinline__ float alibi_slope(int head, int heads) { return exp2f(-8.0f * (float)(head + 1) / (float)heads); }
 

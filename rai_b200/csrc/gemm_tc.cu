@@ -29,6 +29,10 @@
 //            `reduce`, an epilogue that pushes the finished slice straight into the tensor-parallel peers'
 //            exchange buffers - 9 us per launch against 8 us for the separate publishing kernel, whose many
 //            small blocks read the slabs with far more parallelism than one CTA per tile slice can.)
+// GROUP (swapped form only) is the same product for a mixture of experts: a stack of weight matrices, each applied to the
+// rows that chose it.  The work items are (expert, weight tile, tile of its rows), counted on the device from the experts'
+// row counts; rows of X are fetched by index with gather copies, so no sorted copy of X is made, and a tile fetches only
+// the rows it has.  GROUP 1 reads listed rows of X and writes compact rows, GROUP 2 reads those and writes listed rows.
 // GATED computes act(X.Wg^T) * (X.Wu^T) with two accumulators per stage (qwen2.rs:100-103).
 //
 // Every barrier wait is bounded; a give-up is recorded in the context's status word and the CTA
@@ -36,6 +40,7 @@
 #include <stdlib.h>
 
 #include <algorithm>
+#include <type_traits>
 #include <vector>
 
 #include "ctx.h"
@@ -84,11 +89,15 @@ struct Params {
   float* part;
   int act;
   const bf16* act_params;  // RB_ACT_XIELU
+  const int32_t *list, *count;  // GROUP: [experts][cap] entries row * top + choice, and how many each expert has
+  int64_t cap;
+  int experts, top;
   int stages;           // ring depth of this launch, 2..Cfg::kStages
   int reduce;           // split-K reduced inside the kernel: the splits of a tile wait for one another (see the epilogue)
   uint32_t* tile_count; // reduce: arrivals per tile, and readers done per tile; both self-resetting
   uint32_t* tile_done;
   long long wait_cycles;  // give-up budget of every bounded wait
+  int stream_weights;   // GROUP: every weight byte is read about once, keep them from displacing the rest of L2
   uint32_t* status;
 };
 
@@ -115,6 +124,48 @@ __device__ __forceinline__ void decode_item(const Params& p, int item, bool swap
     pt = first + in_group % gsz;
     qt = in_group / gsz;
   }
+}
+
+// GROUP: where each expert's work items and compact rows start
+struct Groups {
+  int item[kMaxExperts + 1], row[kMaxExperts + 1];
+};
+// by the whole block; E experts, tiles of BN rows, n_p weight tiles each
+template <int BN>
+__device__ __forceinline__ void make_groups(Groups& g, const int32_t* count, int E, int n_p) {
+  for (int e = threadIdx.x; e < E; e += blockDim.x) g.row[e + 1] = __ldcg(count + e);
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    int items = 0, rows = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + (int)threadIdx.x;
+      const int c = e < E ? g.row[e + 1] : 0;
+      int ri = c, ti = (c + BN - 1) / BN * n_p;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, ri, o), b = __shfl_up_sync(0xffffffffu, ti, o);
+        if ((int)threadIdx.x >= o) { ri += a; ti += b; }
+      }
+      if (e < E) { g.row[e + 1] = rows + ri; g.item[e + 1] = items + ti; }
+      rows += __shfl_sync(0xffffffffu, ri, 31);
+      items += __shfl_sync(0xffffffffu, ti, 31);
+    }
+    if (threadIdx.x == 0) { g.row[0] = 0; g.item[0] = 0; }
+  }
+  __syncthreads();
+}
+// the expert, weight tile and row tile of an item; rows of neighbouring items share a weight tile
+template <int BN>
+__device__ __forceinline__ void group_item(const Groups& g, int E, int item, int& e, int& pt, int& qt) {
+  int lo = 0, hi = E;  // item[lo] <= item < item[hi]
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (g.item[mid] <= item) lo = mid; else hi = mid;
+  }
+  e = lo;
+  const int n_q = (g.row[e + 1] - g.row[e] + BN - 1) / BN, at = item - g.item[e];
+  pt = at / n_q;
+  qt = at % n_q;
 }
 
 __device__ __forceinline__ uint4 pack8(const float* v) {
@@ -179,10 +230,13 @@ __device__ __forceinline__ void act_inplace(int act, float (&v)[N], float2 ac) {
   }
 }
 
-template <int BN, bool SWAP, bool GATED>
+template <int BN, bool SWAP, bool GATED, int GROUP>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__ CUtensorMap tm_p2,
                const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_q2, const Params p) {
+  static_assert(GROUP == 0 || SWAP, "the grouped form is a swapped one");
+  constexpr bool kGather = GROUP == 1 || (GROUP == 2 && BN <= 64);  // rows by index; else one copy of BN rows
+  static_assert(!kGather || BN <= 128, "one gather per lane");
   using C = Cfg<BN, SWAP, GATED>;
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t full_bar[C::kStages];
@@ -194,6 +248,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
   __shared__ uint32_t issued_count;  // stages the producer has handed to the copy engine
   __shared__ volatile uint32_t epi_ok[4];
   __shared__ __align__(16) bf16 epi_tile[32 * kEpiPitch];  // 32 output rows x 128 columns, padded
+  __shared__ typename std::conditional<GROUP != 0, Groups, int>::type groups;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n_stages = p.stages;
@@ -219,7 +274,66 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
   const uint32_t tmem_base = tmem_base_slot;
 
   pdl_launch_dependents();
-  if (warp == 0) {
+  int n_items = p.n_items;
+  if constexpr (GROUP != 0) {
+    pdl_wait();  // the counts come from a kernel before this one
+    make_groups<BN>(groups, p.count, p.experts, p.n_p);
+    n_items = groups.item[p.experts];
+  }
+  if (GROUP != 0 && warp == 0) {
+    if constexpr (GROUP != 0) {
+      // ---------------------------------------------------------------- TMA producer of the grouped form (whole warp)
+      const uint64_t stream_policy = ptx::policy_evict_first();
+      int stage = 0;
+      uint32_t phase = 0, issued = 0;
+      bool ok = true;
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
+        int e, pt, qt;
+        group_item<BN>(groups, p.experts, item, e, pt, qt);
+        const int first = groups.row[e], have = min(BN, groups.row[e + 1] - first - qt * BN);
+        const int n_gather = (have + 3) / 4;
+        int r[4] = {0, 0, 0, 0};
+        if (kGather && lane < n_gather) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int at = qt * BN + min(lane * 4 + i, have - 1);
+            r[i] = GROUP == 1 ? p.list[(size_t)e * p.cap + at] / p.top : first + at;
+          }
+        }
+        const uint32_t bytes = C::kPTiles * C::kPBytes + (kGather ? (uint32_t)n_gather * 512u : (uint32_t)C::kQBytes);
+        const int wy = e * p.p_rows + pt * kBM;
+        for (int kb = 0; kb < p.num_kb; ++kb) {
+          uint8_t* st = tiles + (size_t)stage * C::kStageBytes;
+          uint8_t* qs = st + C::kPTiles * C::kPBytes;
+          int mine = 1;
+          if (lane == 0) {
+            mine = ptx::mbar_wait(&empty_bar[stage], phase ^ 1u, &abort_flag, p.wait_cycles) ? 1 : 0;
+            if (mine) {
+              ptx::mbar_expect_tx(&full_bar[stage], bytes);
+              if (p.stream_weights) {
+                ptx::tma_load_2d_hint(st, &tm_p, &full_bar[stage], kb * kBK, wy, stream_policy);
+                if (C::kPTiles == 2) ptx::tma_load_2d_hint(st + C::kPBytes, &tm_p2, &full_bar[stage], kb * kBK, wy, stream_policy);
+              } else {
+                ptx::tma_load_2d(st, &tm_p, &full_bar[stage], kb * kBK, wy);
+                if (C::kPTiles == 2) ptx::tma_load_2d(st + C::kPBytes, &tm_p2, &full_bar[stage], kb * kBK, wy);
+              }
+              if (!kGather) ptx::tma_load_2d(qs, &tm_q, &full_bar[stage], kb * kBK, first + qt * BN);
+            }
+          }
+          mine = __shfl_sync(0xffffffffu, mine, 0);  // also orders the expected byte count before the gathers
+          if (!mine) { ok = false; break; }
+          if (kGather && lane < n_gather)
+            ptx::tma_gather4(qs + lane * 512, &tm_q, &full_bar[stage], kb * kBK, r[0], r[1], r[2], r[3]);
+          ++issued;
+          if (++stage == n_stages) { stage = 0; phase ^= 1u; }
+        }
+      }
+      if (lane == 0) {
+        issued_count = issued;
+        if (!ok) { p.status[0] = (uint32_t)(-RB_ERR_TIMEOUT); p.status[1] = 0x6E05u; p.status[2] = blockIdx.x; }
+      }
+    }
+  } else if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       // The weight operand does not depend on the kernel before this one: its first ring of
@@ -287,9 +401,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
       int as = 0;
       uint32_t aphase = 0;
       bool ok = true;
-      for (int item = blockIdx.x; item < p.n_items && ok; item += gridDim.x) {
-        int pt, qt, split;
-        decode_item(p, item, SWAP, pt, qt, split);
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
+        int pt, qt, split = 0;
+        if (GROUP == 0) decode_item(p, item, SWAP, pt, qt, split);
         const int kb0 = split * p.kb_per_split, kb1 = min(p.num_kb, kb0 + p.kb_per_split);
         if (kb0 >= kb1) continue;  // empty split: the epilogue writes zeros on its own
         if (!ptx::mbar_wait(&acc_empty[as], aphase ^ 1u, &abort_flag, p.wait_cycles)) { ok = false; break; }
@@ -327,9 +441,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
     int as = 0;
     uint32_t aphase = 0;
     bool ok = true;
-    for (int item = blockIdx.x; item < p.n_items && ok; item += gridDim.x) {
-      int pt, qt, split;
-      decode_item(p, item, SWAP, pt, qt, split);
+    for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
+      int pt, qt, split = 0;
+      int m_lim = p.m, row0 = 0;            // rows of this item's group, and where they go
+      const int32_t* scatter = nullptr;
+      if constexpr (GROUP != 0) {
+        int e;
+        group_item<BN>(groups, p.experts, item, e, pt, qt);
+        row0 = groups.row[e];
+        m_lim = groups.row[e + 1] - row0;
+        if (GROUP == 2) scatter = p.list + (size_t)e * p.cap;
+      } else {
+        decode_item(p, item, SWAP, pt, qt, split);
+      }
       if (split * p.kb_per_split >= p.num_kb) {  // empty split (only with partials): zero slab, no accumulator
         const int gn = pt * kBM + lane_row;
         if (p.part && gn < p.n)
@@ -348,6 +472,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
       constexpr int CH = BN >= 32 ? 32 : 16;  // columns per TMEM load
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += CH) {
+        if (GROUP != 0 && qt * BN + c0 >= m_lim) break;
         float v[CH], g[GATED ? CH : 1];
         {
           uint32_t r[CH];
@@ -412,9 +537,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
             for (int id = et; id < CH * (kBM / 8); id += 128) {
               const int j = id / (kBM / 8), c8 = (id % (kBM / 8)) * 8;
               const int gm = qt * BN + c0 + j, gn8 = pt * kBM + c8;
-              if (gm >= p.m || gn8 >= p.n) continue;
+              if (gm >= m_lim || gn8 >= p.n) continue;
               uint4 u = *reinterpret_cast<const uint4*>(epi_tile + j * kEpiPitch + c8);
-              bf16* dst = p.out + (size_t)gm * p.n + gn8;
+              bf16* dst = p.out + (size_t)(GROUP == 0 ? gm : GROUP == 1 ? row0 + gm : scatter[gm]) * p.n + gn8;
               if (vec_ok) {
                 if (!GATED && p.residual) {
                   float a8[8], r8[8];
@@ -628,7 +753,7 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-template <int BN, bool SWAP, bool GATED>
+template <int BN, bool SWAP, bool GATED, int GROUP = 0>
 int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
   using C = Cfg<BN, SWAP, GATED>;
   const void* pbase = SWAP ? a.w : a.x;
@@ -636,13 +761,15 @@ int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
   const void* qbase = SWAP ? a.x : a.w;
   const void* q2base = SWAP ? a.x : a.w2;
   CUtensorMap tp, tp2, tq, tq2;
-  RB_TRY(tmap_2d_bf16(ctx, pbase, p.p_rows, a.k, a.k, kBM, &tp));
-  RB_TRY(tmap_2d_bf16(ctx, (GATED && SWAP) ? p2base : pbase, p.p_rows, a.k, a.k, kBM, &tp2));
-  RB_TRY(tmap_2d_bf16(ctx, qbase, p.q_rows, a.k, a.k, BN, &tq));
-  RB_TRY(tmap_2d_bf16(ctx, (GATED && !SWAP) ? q2base : qbase, p.q_rows, a.k, a.k, BN, &tq2));
+  const int64_t stacked = (int64_t)p.p_rows * (GROUP != 0 ? p.experts : 1);
+  constexpr int q_box = GROUP == 1 || (GROUP == 2 && BN <= 64) ? 1 : BN;  // gather copies take a box of one row
+  RB_TRY(tmap_2d_bf16(ctx, pbase, stacked, a.k, a.k, kBM, &tp));
+  RB_TRY(tmap_2d_bf16(ctx, (GATED && SWAP) ? p2base : pbase, stacked, a.k, a.k, kBM, &tp2));
+  RB_TRY(tmap_2d_bf16(ctx, qbase, p.q_rows, a.k, a.k, q_box, &tq));
+  RB_TRY(tmap_2d_bf16(ctx, (GATED && !SWAP) ? q2base : qbase, p.q_rows, a.k, a.k, q_box, &tq2));
   p.n_p = (p.p_rows + kBM - 1) / kBM;
   p.n_q = (p.q_rows + BN - 1) / BN;
-  auto kern = gemm_tc_kernel<BN, SWAP, GATED>;
+  auto kern = gemm_tc_kernel<BN, SWAP, GATED, GROUP>;
   static bool attr_set[64] = {};  // the attribute belongs to the (kernel, device) pair
   const int dv = ctx->device & 63;
   if (!attr_set[dv]) {
@@ -652,6 +779,11 @@ int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
   // Ring depth: as deep as the shared-memory budget allows (decode-sized launches are bound by the bytes they
   // keep in flight; a shallower ring measured slower even where it lets two kernels share an SM).
   int stages = C::kStages;
+  if (GROUP != 0) {
+    // at most this many row tiles: each expert ends in a partial one
+    const int64_t pairs = (int64_t)p.m;
+    p.n_q = (int)(pairs / BN + std::min<int64_t>(p.experts, pairs));
+  }
   if (SWAP) stages = std::max(2, std::min(C::kStages, (int)(ctx->gemm_ring_bytes / C::kStageBytes)));
   p.stages = stages;
   const size_t smem = (size_t)stages * C::kStageBytes + 1024;
@@ -771,10 +903,10 @@ int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a) {
   p.act_params = (const bf16*)a.act_params;
   RB_REQUIRE(a.act != RB_ACT_XIELU || (a.act_params && !gated), "GEMM: RB_ACT_XIELU needs its parameters and an ungated product");
   p.status = ctx->status_dev;
-  const bool swap = a.m <= 256 && !(gated && a.m > 128);
+  const bool swap = a.partials || (a.m <= 256 && !(gated && a.m > 128));
   if (a.partials) {
-    RB_REQUIRE(swap, "GEMM: split-K partials need M <= 256");
     const int s = std::max(1, a.n_split);
+    RB_REQUIRE(a.m <= 256 || s == 1, "GEMM: split-K partials need M <= 256");
     p.kb_per_split = (p.num_kb + s - 1) / s;
     p.n_split = s;
   }
@@ -794,6 +926,32 @@ int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a) {
   p.p_rows = (int)a.m; p.q_rows = (int)a.n;
   if (gated) return launch<128, false, true>(ctx, a, p);
   return launch<256, false, false>(ctx, a, p);
+}
+
+// The grouped form: a.m is the number of (row, choice) pairs, a.x has a.m / a.top rows (gated) or a.m compact rows.
+int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a) {
+  if (a.m == 0) return RB_OK;
+  RB_REQUIRE(a.k > 0 && (a.k % 8) == 0 && a.n > 0 && (a.n % 8) == 0, "grouped GEMM: N = %lld and K = %lld must be multiples of 8",
+             (long long)a.n, (long long)a.k);
+  RB_REQUIRE(a.experts > 0 && a.experts <= kMaxExperts, "grouped GEMM: %d experts (1..%d)", a.experts, kMaxExperts);
+  const bool gated = a.w2 != nullptr;
+  Params p{};
+  p.m = (int)a.m; p.n = (int)a.n; p.k = (int)a.k;
+  p.p_rows = (int)a.n;
+  p.q_rows = (int)(gated ? a.m / a.top : a.m);
+  p.num_kb = (int)((a.k + kBK - 1) / kBK);
+  p.n_split = 1;
+  p.kb_per_split = p.num_kb;
+  p.out = (bf16*)a.out;
+  p.act = a.act;
+  p.list = a.list; p.count = a.count; p.cap = a.cap; p.experts = a.experts; p.top = a.top;
+  p.status = ctx->status_dev;
+  const int64_t rows = a.m / a.top;
+  const double mean = (double)a.m / a.experts;  // rows per expert, if they spread evenly
+  p.stream_weights = mean <= 48.0;
+  if (rows <= 16) return gated ? launch<16, true, true, 1>(ctx, a, p) : launch<16, true, false, 2>(ctx, a, p);
+  if (mean <= 48.0) return gated ? launch<64, true, true, 1>(ctx, a, p) : launch<64, true, false, 2>(ctx, a, p);
+  return gated ? launch<128, true, true, 1>(ctx, a, p) : launch<256, true, false, 2>(ctx, a, p);
 }
 
 }  // namespace rb

@@ -6,6 +6,13 @@
 //   hgrn2       x -> [q|f|v] GEMM -> recurrence (+ per-head norm) -> output GEMM -> x += norm(.)
 //   feed-forward  x -> up GEMM (+ xIELU) -> down GEMM -> x += norm(.)
 //
+// or, with one norm ahead of a mixer and a feed-forward that both read it (parallel block), attention whose values are its
+// keys beside routed experts:
+//
+//   h -> [q|k|shared gate|shared up|router] GEMM -> head split + key append + gated activation + routing
+//     -> experts' gated GEMM -> experts' down GEMM;  attention;  output GEMM over [heads | shared expert]
+//     -> x += m (.), h = norm(x)
+//
 // Single-token GEMMs leave float32 split-K slabs that the next kernel sums, as in the other families.  The driver around
 // this walk (lengths, the captured decode step, sampling, loading) is model.cu's.
 #include <algorithm>
@@ -93,21 +100,96 @@ int mlp_up(rb_model* m, const MixLayer& w, int64_t rows) {
   return rb_linear_act(ctx, m->h, w.up, nullptr, m->act, rows, w.mlp_k, m->ld, RB_ACT_XIELU, w.act, m->cfg.dtype);
 }
 
+// A parallel block on m->h (the stream, normalised): the stream moves on, and m->h is what the next block (gain, or NULL after
+// the last) reads.
+int parallel_block(rb_model* m, const MixLayer& w, int batch, int seq, const void* next_gain) {
+  rb_ctx* ctx = m->ctx;
+  const int dt = m->cfg.dtype;
+  const int64_t rows = (int64_t)batch * seq;
+  const rb_layer_config& c = w.c;
+  const bool experts = c.mlp_size > 0;
+  // input projection: one set of slabs, router logits included, at single-token steps; otherwise a tensor and float32 logits
+  const int s = seq == 1 ? slab_count(m, rows, w.n_in, m->ld) : 0;
+  SplitSpec f;
+  f.batch = batch; f.s_new = seq; f.q_heads = c.heads; f.kv_heads = c.kv_heads; f.dim = c.key_dim; f.glu_size = c.shared_size;
+  f.cache = w.kv; f.layer = w.kv_layer; f.q_out = m->q; f.glu_ld = w.mix_k;
+  f.glu_out = c.shared_size > 0 ? (char*)m->attn + (size_t)w.attn_cols * m->es : nullptr;
+  RouteSpec r;
+  r.experts = c.experts; r.top = c.top; r.groups = c.groups; r.keep = c.keep_groups; r.scale = (float)c.router_scale;
+  r.weight = m->route_w; r.list = m->route_list; r.count = m->route_count; r.cap = m->cfg.max_tokens;
+  if (s > 0) {
+    RB_TRY(rb_linear_partials(ctx, m->h, w.in_w, m->scratch, rows, w.n_in, m->ld, s));
+    f.acc = m->scratch; f.n_acc = s; f.bias = w.in_b; f.src_ld = w.n_in;
+    r.acc = m->scratch + w.n_main; r.n_acc = s; r.acc_stride = rows * w.n_in; r.z_ld = w.n_in;
+  } else {
+    RB_TRY(rb_linear(ctx, m->h, w.in_w, w.in_b, nullptr, m->mix_in, rows, w.n_main, m->ld, RB_ACT_NONE, dt));
+    f.src = m->mix_in; f.src_ld = w.n_main;
+    if (experts) {
+      const void* router = (const char*)w.in_w + (size_t)w.n_main * m->ld * m->es;
+      const int n = w.n_in - w.n_main;
+      if (dt == RB_F32) RB_TRY(rb_linear(ctx, m->h, router, nullptr, nullptr, m->route_z, rows, n, m->ld, RB_ACT_NONE, dt));
+      else RB_TRY(rb_linear_partials(ctx, m->h, router, m->route_z, rows, n, m->ld, 1));
+      r.acc = m->route_z; r.n_acc = 1; r.z_ld = n;
+    }
+  }
+  RB_TRY(split_and_route(ctx, f, experts ? &r : nullptr, dt));
+  if (experts) {
+    RB_TRY(rb_moe_gated(ctx, m->h, w.gate, w.up, m->expert_act, rows, c.top, c.experts, r.list, r.count, r.cap, w.ff_p, m->ld, RB_ACT_SILU, dt));
+    RB_TRY(rb_moe_down(ctx, m->expert_act, w.down, m->expert_out, rows, c.top, c.experts, r.list, r.count, r.cap, m->ld, w.ff_p, dt));
+  }
+  rb_attention_options o{};
+  o.temp_every = c.temp_every; o.temp_coef = (float)c.temp_coef; o.softcap = (float)c.softcap; o.value_dim = c.value_dim;
+  o.sink = w.sink; o.out_ld = w.mix_k;
+  RB_TRY(rb_attention_general(ctx, m->q, w.kv, w.kv_layer, batch, seq, c.heads, (float)c.scale, &o, m->attn, dt));
+  JoinSpec j;
+  const int so = slab_count(m, rows, m->ld, w.mix_k);
+  if (so > 0) {
+    RB_TRY(rb_linear_partials(ctx, m->attn, w.o_w, m->scratch, rows, m->ld, w.mix_k, so));
+    j.acc = m->scratch; j.n_acc = so;
+  } else {
+    RB_TRY(rb_linear(ctx, m->attn, w.o_w, nullptr, nullptr, m->sub_out, rows, m->ld, w.mix_k, RB_ACT_NONE, dt));
+    j.y = m->sub_out;
+  }
+  if (experts) { j.part = m->expert_out; j.weight = m->route_w; j.top = c.top; j.zero = m->route_count; j.n_zero = c.experts; }
+  j.mult = (float)c.residual_mult; j.gain = next_gain; j.eps = (float)m->cfg.norm_eps; j.rows = rows; j.width = m->cfg.hidden_size;
+  j.ld = m->ld; j.h = m->stream; j.out = next_gain ? m->h : nullptr;
+  return add_then_norm(ctx, j, dt);
+}
+
+// The stream's first value and the first block's input
+int parallel_embed(rb_model* m, const uint32_t* tokens, int batch, int seq, const int32_t* new_lens) {
+  const rb_model_config& c = m->cfg;
+  RB_TRY(rb_embed_positions(m->ctx, m->embed, m->pos, c.max_position_embeddings, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens,
+                            batch, seq, m->cache, new_lens, m->stream));
+  JoinSpec j;
+  j.gain = m->mix[0].norm1; j.eps = (float)c.norm_eps; j.rows = (int64_t)batch * seq; j.width = c.hidden_size; j.ld = m->ld;
+  j.h = m->stream; j.out = m->h;
+  j.zero = m->route_count; j.n_zero = kMaxExperts;  // (a call that failed half-way may have left them)
+  return add_then_norm(m->ctx, j, c.dtype);
+}
+
 }  // namespace
 
 int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq, const int32_t* new_lens) {
   const rb_model_config& c = m->cfg;
   rb_ctx* ctx = m->ctx;
   const int64_t rows = (int64_t)batch * seq;
-  RB_TRY(rb_embed_stream(ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->stream,
-                         c.dtype == RB_F32 ? nullptr : m->h));
+  const bool parallel = c.arch == RB_ARCH_VOTAPEL;
+  if (parallel) RB_TRY(parallel_embed(m, tokens, batch, seq, new_lens));
+  else
+    RB_TRY(rb_embed_stream(ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->stream,
+                           c.dtype == RB_F32 ? nullptr : m->h));
   for (size_t l = 0; l < m->mix.size(); ++l) {
     const MixLayer& w = m->mix[l];
-    RB_TRY(mixer(m, w, batch, seq, new_lens));
-    RB_TRY(sublayer_out(m, m->attn, w.o_w, w.mix_k, w.norm1, rows));
-    if (w.c.mlp_size > 0) {
-      RB_TRY(mlp_up(m, w, rows));
-      RB_TRY(sublayer_out(m, m->act, w.down, w.mlp_k, w.norm2, rows));
+    if (parallel) {
+      RB_TRY(parallel_block(m, w, batch, seq, l + 1 < m->mix.size() ? m->mix[l + 1].norm1 : nullptr));
+    } else {
+      RB_TRY(mixer(m, w, batch, seq, new_lens));
+      RB_TRY(sublayer_out(m, m->attn, w.o_w, w.mix_k, w.norm1, rows));
+      if (w.c.mlp_size > 0) {
+        RB_TRY(mlp_up(m, w, rows));
+        RB_TRY(sublayer_out(m, m->act, w.down, w.mlp_k, w.norm2, rows));
+      }
     }
     if (m->layer_trace)
       RB_CUDA(cudaMemcpy2DAsync(m->layer_trace + (size_t)l * rows * c.hidden_size, (size_t)c.hidden_size * 4, m->stream, (size_t)m->ld * 4,
@@ -118,7 +200,8 @@ int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq,
 
 int rb::layered_logits(rb_model* m, const int32_t* rows, int seq, int n, float* out) {
   const rb_model_config& c = m->cfg;
-  RB_TRY(rb_scalar_norm_rows(m->ctx, m->stream, rows, seq, m->norm_w, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
+  const auto norm = c.arch == RB_ARCH_VOTAPEL ? rb_one_plus_norm_rows : rb_scalar_norm_rows;
+  RB_TRY(norm(m->ctx, m->stream, rows, seq, m->norm_w, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
   if (c.dtype == RB_F32)
     return rb_linear(m->ctx, m->xn, m->lm_head, nullptr, nullptr, out, n, c.vocab_size, m->ld, RB_ACT_NONE, RB_F32);
   for (int r = 0; r < n; r += 256)  // one float32 slab is a float32 product
@@ -142,21 +225,38 @@ int rb::layered_decode_plan(rb_model* m, int batch) {
 extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out) {
   RB_REQUIRE(ctx && cfg && layers && out, "rb_model_create_layers: null argument");
   const rb_model_config& c = *cfg;
-  RB_REQUIRE(c.arch == RB_ARCH_MALASUN, "rb_model_create_layers: architecture %d is not described layer by layer", c.arch);
+  const bool parallel = c.arch == RB_ARCH_VOTAPEL;
+  RB_REQUIRE(c.arch == RB_ARCH_MALASUN || parallel, "rb_model_create_layers: architecture %d is not described layer by layer", c.arch);
   RB_REQUIRE(c.dtype == RB_BF16 || c.dtype == RB_F32, "rb_model_create_layers: dtype %d unsupported", c.dtype);
   RB_REQUIRE(c.hidden_size > 0 && c.vocab_size > 0 && c.num_hidden_layers > 0, "rb_model_create_layers: bad sizes");
   RB_REQUIRE(c.max_batch > 0 && c.max_seq > 0 && c.max_tokens >= c.max_batch, "rb_model_create_layers: bad capacities");
   // the query / key norm runs over all heads at once, so a head-parallel split would need its sum exchanged per layer
   if (c.tp_size > 1) return fail(RB_ERR_UNIMPLEMENTED, "rb_model_create_layers: tensor parallelism is not available for this design");
+  RB_REQUIRE(!parallel || c.max_position_embeddings > 0, "rb_model_create_layers: learned positions need their number");
   const int L = c.num_hidden_layers;
   for (int l = 0; l < L; ++l) {
     const rb_layer_config& y = layers[l];
+    RB_REQUIRE(y.block == (parallel ? RB_BLOCK_PARALLEL : RB_BLOCK_POST_NORM) &&
+                   (y.mlp_size == 0 || y.mlp_kind == (parallel ? RB_MLP_EXPERTS : RB_MLP_DENSE)),
+               "layer %d: block or feed-forward kind does not belong to this architecture", l);
+    if (parallel) {
+      RB_REQUIRE(y.mixer == RB_MIXER_ATTENTION && y.kv_from < 0 && y.window == 0 && y.key_dim == y.value_dim,
+                 "layer %d: a parallel block has attention over every earlier key, whose values are the keys", l);
+      RB_REQUIRE(y.temp_every >= 0 && y.softcap >= 0.0 && y.shared_size >= 0, "layer %d: bad constants", l);
+      RB_REQUIRE(y.mlp_size > 0 || y.shared_size == 0, "layer %d: a shared expert without experts", l);
+      if (y.mlp_size > 0) {
+        RB_REQUIRE(y.experts > 0 && y.groups > 0 && y.experts % y.groups == 0 && y.keep_groups > 0 && y.keep_groups <= y.groups &&
+                       y.top > 0 && y.top <= y.experts / y.groups * y.keep_groups,
+                   "layer %d: top %d of %d experts in %d groups of which %d stay", l, y.top, y.experts, y.groups, y.keep_groups);
+        if (y.experts > kMaxExperts || y.top > 32) return fail(RB_ERR_UNIMPLEMENTED, "layer %d: more than %d experts or top 32", l, kMaxExperts);
+      }
+    }
     RB_REQUIRE(y.mixer == RB_MIXER_ATTENTION || y.mixer == RB_MIXER_HGRN2, "layer %d: unknown mixer %d", l, y.mixer);
     RB_REQUIRE(y.heads > 0 && y.key_dim > 0 && y.value_dim > 0 && y.mlp_size >= 0, "layer %d: bad sizes", l);
     if (y.key_dim > 256 || y.value_dim > 256) return fail(RB_ERR_UNIMPLEMENTED, "layer %d: head sizes above 256", l);
     if (y.mixer != RB_MIXER_ATTENTION) continue;
     RB_REQUIRE(y.kv_heads > 0 && y.heads % y.kv_heads == 0, "layer %d: %d heads over %d key/value heads", l, y.heads, y.kv_heads);
-    RB_REQUIRE(y.conv_taps >= 1 && y.window >= 0 && y.window <= (1 << 30) && y.scale > 0.0, "layer %d: bad attention constants", l);
+    RB_REQUIRE((parallel || y.conv_taps >= 1) && y.window >= 0 && y.window <= (1 << 30) && y.scale > 0.0, "layer %d: bad attention constants", l);
     if (y.kv_from >= 0) {
       RB_REQUIRE(y.kv_from < l && layers[y.kv_from].mixer == RB_MIXER_ATTENTION && layers[y.kv_from].kv_from < 0,
                  "layer %d: kv_from %d is not an earlier attention layer with keys and values of its own", l, y.kv_from);
@@ -171,7 +271,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   m->cfg = c;
   m->cfg.tp_size = 1;
   m->cfg.tp_rank = 0;
-  m->cfg.max_position_embeddings = 0x7fffffff;  // positions enter through distances only: no table to outgrow
+  if (!parallel) m->cfg.max_position_embeddings = 0x7fffffff;  // positions enter through distances only: no table to outgrow
   m->layered = true;
   m->es = dtype_size(c.dtype);
   m->logits_dtype = RB_F32;
@@ -192,14 +292,72 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
 
   A((int64_t)V * ld, &m->embed);
   mat("embed", V, W, m->embed, ld);
+  if (parallel) {
+    A((int64_t)c.max_position_embeddings * ld, &m->pos);
+    mat("pos", c.max_position_embeddings, W, m->pos, ld);
+  }
   m->mix.resize(L);
   std::map<std::pair<int, int>, std::vector<int>> geometry;  // (key/value heads, cache head size) -> layers with K and V of their own
-  int max_in = 8, max_q = 8, max_gate = 8, max_mix = 8, max_mlp = 8;
+  int max_in = 8, max_q = 8, max_gate = 8, max_mix = 8, max_mlp = 8, max_experts = 0, max_top = 0, max_ff = 8;
   for (int l = 0; l < L && st == RB_OK; ++l) {
     MixLayer& w = m->mix[l];
     w.c = layers[l];
     const rb_layer_config& y = w.c;
     const std::string pre = "l" + std::to_string(l) + ".", mix = pre + "mix.";
+    if (parallel) {
+      const int nq = y.heads * y.key_dim, nk = y.kv_heads * y.key_dim, qp = pad8(nq), kp = pad8(nk);
+      w.glu_p = pad8(y.shared_size);
+      w.ff_p = pad8(y.mlp_size);
+      w.n_main = qp + kp + 2 * w.glu_p;
+      w.n_in = w.n_main + (y.mlp_size > 0 ? pad8(y.experts) : 0);
+      w.attn_cols = pad8((int64_t)y.heads * y.value_dim);
+      w.mix_k = w.attn_cols + w.glu_p;
+      A(ld, &w.norm1);
+      A((int64_t)w.n_in * ld, &w.in_w);
+      A(w.n_in, &w.in_b);
+      A(pad8(y.heads), &w.sink);
+      A((int64_t)ld * w.mix_k, &w.o_w);
+      if (y.mlp_size > 0) {
+        A((int64_t)y.experts * w.ff_p * ld, &w.gate);
+        A((int64_t)y.experts * w.ff_p * ld, &w.up);
+        A((int64_t)y.experts * ld * w.ff_p, &w.down);
+      }
+      if (st != RB_OK) break;
+      const std::string mlp = pre + "mlp.";
+      vec(pre + "norm1", W, w.norm1);
+      mat(mix + "q", nq, W, w.in_w, ld);
+      vec(mix + "q.b", nq, w.in_b);
+      mat(mix + "k", nk, W, at(w.in_w, (int64_t)qp * ld), ld);
+      vec(mix + "k.b", nk, at(w.in_b, qp));
+      vec(mix + "sink", y.heads, w.sink);
+      mat(mix + "o", W, nq, w.o_w, w.mix_k);
+      if (y.mlp_size > 0) {
+        for (int e = 0; e < y.experts; ++e) {
+          const std::string x = mlp + "e" + std::to_string(e) + ".";
+          mat(x + "gate", y.mlp_size, W, at(w.gate, (int64_t)e * w.ff_p * ld), ld);
+          mat(x + "up", y.mlp_size, W, at(w.up, (int64_t)e * w.ff_p * ld), ld);
+          mat(x + "down", W, y.mlp_size, at(w.down, (int64_t)e * ld * w.ff_p), w.ff_p);
+        }
+        mat(mlp + "router", y.experts, W, at(w.in_w, (int64_t)w.n_main * ld), ld);
+      }
+      if (y.shared_size > 0) {
+        mat(mlp + "shared.gate", y.shared_size, W, at(w.in_w, (int64_t)(qp + kp) * ld), ld);
+        mat(mlp + "shared.up", y.shared_size, W, at(w.in_w, (int64_t)(qp + kp + w.glu_p) * ld), ld);
+        mat(mlp + "shared.down", W, y.shared_size, at(w.o_w, w.attn_cols), w.mix_k);
+      }
+      auto& group = geometry[{y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim)}];
+      w.kv_layer = (int)group.size();
+      group.push_back(l);
+      max_q = std::max(max_q, y.heads * cache_dim(c.dtype, y.key_dim, y.value_dim));
+      max_in = std::max(max_in, w.n_in);
+      max_mix = std::max(max_mix, w.mix_k);
+      if (y.mlp_size > 0) {
+        max_experts = std::max(max_experts, pad8(y.experts));
+        max_top = std::max(max_top, y.top);
+        max_ff = std::max(max_ff, w.ff_p);
+      }
+      continue;
+    }
     A(8, &w.norm1);
     num(pre + "norm1", w.norm1);
     w.mix_k = pad8((int64_t)y.heads * y.value_dim);
@@ -270,10 +428,11 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
     max_mix = std::max(max_mix, w.mix_k);
     max_mlp = std::max(max_mlp, w.mlp_k);
   }
-  A(8, &m->norm_w);
+  A(parallel ? ld : 8, &m->norm_w);
   A((int64_t)V * ld, &m->lm_head);
   if (st == RB_OK) {
-    num("final.norm", m->norm_w);
+    if (parallel) vec("final.norm", W, m->norm_w);
+    else num("final.norm", m->norm_w);
     mat("head", V, W, m->lm_head, ld);
     m->vocab_l = V;
   }
@@ -282,7 +441,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   if (st == RB_OK) st = kv_cache_create(ctx, nullptr, 0, 1, 8, c.max_batch, c.max_seq, c.dtype, &m->cache);
   for (auto& g : geometry) {
     rb_kv_cache* view = nullptr;
-    if (st == RB_OK) st = kv_cache_create(ctx, m->cache, (int)g.second.size(), g.first.first, g.first.second, 0, 0, c.dtype, &view);
+    if (st == RB_OK) st = kv_cache_create(ctx, m->cache, (int)g.second.size(), g.first.first, g.first.second, 0, 0, c.dtype, &view, parallel);
     if (st != RB_OK) break;
     m->views.push_back(view);
     for (int l : g.second) m->mix[l].kv = view;
@@ -306,7 +465,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   const size_t MT = c.max_tokens, few = std::min<size_t>(MT, 256);
   B(MT * sizeof(uint32_t), (void**)&m->ids);
   B(MT * ld * sizeof(float), (void**)&m->stream);
-  if (c.dtype == RB_F32) m->h = m->stream;
+  if (c.dtype == RB_F32 && !parallel) m->h = m->stream;
   else B(MT * ld * m->es, &m->h);
   B(MT * max_in * m->es, &m->mix_in);
   B(MT * max_q * m->es, &m->q);
@@ -318,6 +477,14 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   B((size_t)c.max_batch * V * sizeof(float), &m->logits);
   B((size_t)c.max_batch * sizeof(uint32_t), (void**)&m->next_ids);
   B(MT * sizeof(int32_t), (void**)&m->last_rows);
+  if (parallel) B(kMaxExperts * sizeof(int32_t), (void**)&m->route_count);
+  if (max_experts > 0) {
+    B(MT * max_experts * sizeof(float), (void**)&m->route_z);
+    B(MT * max_top * sizeof(float), (void**)&m->route_w);
+    B(MT * max_experts * sizeof(int32_t), (void**)&m->route_list);
+    B(MT * max_top * max_ff * m->es, &m->expert_act);
+    B(MT * max_top * ld * m->es, &m->expert_out);
+  }
   B((size_t)c.max_batch * sizeof(int32_t), (void**)&m->new_lens);
   if (c.dtype == RB_BF16) {
     m->scratch_floats = (size_t)16 * few * std::max(std::max(max_in, max_mlp), ld);

@@ -32,6 +32,36 @@ __global__ void embed_stream_kernel(const T* __restrict__ table, const uint32_t*
   }
 }
 
+// The same plus a learned vector of the row's position in its sequence.
+template <typename T>
+__global__ void embed_positions_kernel(const T* __restrict__ table, const T* __restrict__ positions, int n_pos,
+                                       const uint32_t* __restrict__ ids, int64_t vocab, int ld, int s_new,
+                                       const int32_t* __restrict__ seq_lens, const int32_t* __restrict__ new_lens, float* __restrict__ h,
+                                       uint32_t* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, b = row / s_new, s = row % s_new;
+  uint32_t id = ids[row];
+  if (id >= (uint64_t)vocab) {
+    if (threadIdx.x == 0) { status[0] = (uint32_t)(-RB_ERR_INVALID); status[1] = 0xE3BEDu; status[2] = id; }
+    id = (uint32_t)(vocab - 1);
+  }
+  int pos = seq_lens[b] - s_new + s;
+  if (pos < 0 || pos >= n_pos) {  // a row of padding may lie beyond the table, a token may not
+    const bool is_token = !new_lens || s < new_lens[b];
+    if (is_token && threadIdx.x == 0) { status[0] = (uint32_t)(-RB_ERR_INVALID); status[1] = 0xE3B05u; status[2] = (uint32_t)pos; }
+    pos = min(max(pos, 0), n_pos - 1);
+  }
+  for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
+    float v[8], p[8];
+    load8(table + (size_t)id * ld + c, v);
+    load8(positions + (size_t)pos * ld + c, p);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] += p[i];
+    store8(h + (size_t)row * ld + c, v);
+  }
+}
+
 // ------------------------------------------------------------------------------------------
 // h += y / rms(y) * gain, x = h in the model dtype; y = tensor and/or split-K slabs.  One block per row (several rows
 // per block at prefill sizes); the row stays in registers between the sum of squares and the scaling.
@@ -75,8 +105,98 @@ __global__ void __launch_bounds__(512) add_scaled_norm_kernel(const T* __restric
   }
 }
 
+// ------------------------------------------------------------------------------------------
+// The joint of a pre-norm block: h += mult * (tensor + split-K slabs + weighted rows of experts), then the norm of the sum
+// as the next block's input.  Rows as above.
+// ------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(512) scalar_norm_rows_kernel(const float* __restrict__ h, const int32_t* __restrict__ rows,
+struct JoinArgs {
+  const T* y;
+  const float* acc;
+  int n_acc;
+  size_t acc_stride;
+  const T* part;
+  const float* weight;
+  int top;
+  float mult;
+  const T* gain;
+  float eps;
+  int width, ld;
+  float* h;
+  T* out;
+  int64_t n_rows;
+  int32_t* zero;
+  int n_zero;
+};
+
+template <typename T, int kChunks, bool kSlabs>
+__global__ void __launch_bounds__(512) add_then_norm_kernel(const JoinArgs<T> a) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  const int nchunk = a.ld >> 3;
+  pdl_wait();
+  if (blockIdx.x == 0)
+    for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
+  const bool adds = a.y || kSlabs || a.part;
+  for (int64_t row = blockIdx.x; row < a.n_rows; row += gridDim.x) {
+    const size_t base = (size_t)row * a.ld;
+    float hv[kChunks][8];
+    float s = 0.f;
+#pragma unroll
+    for (int c = 0; c < kChunks; ++c) {
+      const int ch = threadIdx.x + c * blockDim.x;
+      if (ch >= nchunk) continue;
+      load8(a.h + base + ch * 8, hv[c]);
+      if (adds) {
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = 0.f;
+        if (a.y) load8(a.y + base + ch * 8, v);
+        if (kSlabs) add_slabs<(kChunks > 1 ? 4 : 8)>(a.acc, a.n_acc, a.acc_stride, base + ch * 8, v);
+        if (a.part) {
+          const T* p = a.part + (size_t)row * a.top * a.ld + ch * 8;
+          const float* w = a.weight + row * a.top;
+          for (int j0 = 0; j0 < a.top; j0 += 4) {   // four experts' rows in flight
+            float t[4][8], wj[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              wj[j] = 0.f;
+              if (j0 + j < a.top) { wj[j] = w[j0 + j]; load8(p + (size_t)(j0 + j) * a.ld, t[j]); }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              if (j0 + j < a.top) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) v[i] = fmaf(wj[j], t[j][i], v[i]);
+              }
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) hv[c][i] = fmaf(a.mult, v[i], hv[c][i]);
+        store8(a.h + base + ch * 8, hv[c]);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s += hv[c][i] * hv[c][i];
+    }
+    if (!a.out) continue;
+    s = block_sum(s, red);
+    const float r = 1.0f / sqrtf(s / (float)a.width + a.eps);
+#pragma unroll
+    for (int c = 0; c < kChunks; ++c) {
+      const int ch = threadIdx.x + c * blockDim.x;
+      if (ch >= nchunk) continue;
+      float g[8];
+      load8(a.gain + ch * 8, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) g[i] = hv[c][i] * r * (1.0f + g[i]);
+      store8(a.out + base + ch * 8, g);
+    }
+  }
+}
+
+// kVector: a gain per channel, stored as its difference from one; otherwise one number
+template <typename T, bool kVector>
+__global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict__ h, const int32_t* __restrict__ rows,
                                                                int64_t row_step, const T* __restrict__ gain, float eps, int width,
                                                                int ld, T* __restrict__ out) {
   __shared__ float red[32];
@@ -92,12 +212,13 @@ __global__ void __launch_bounds__(512) scalar_norm_rows_kernel(const float* __re
     for (int i = 0; i < 8; ++i) s += v[i] * v[i];
   }
   s = block_sum(s, red);
-  const float r = Cvt<T>::to_f(gain[0]) / sqrtf(s / (float)width + eps);
+  const float r = (kVector ? 1.0f : Cvt<T>::to_f(gain[0])) / sqrtf(s / (float)width + eps);
   for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
-    float v[8];
+    float v[8], g[8];
     load8(p + c, v);
+    if (kVector) load8(gain + c, g);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] *= r;
+    for (int i = 0; i < 8; ++i) v[i] *= kVector ? r * (1.0f + g[i]) : r;
     store8(out + (size_t)blockIdx.x * ld + c, v);
   }
 }
@@ -420,7 +541,44 @@ int add_norm_run(rb_ctx* ctx, const void* y, const float* acc, int n_acc, const 
   return fail(RB_ERR_UNIMPLEMENTED, "rb_add_scaled_norm: width %d exceeds 16384", width);
 }
 
+template <typename T>
+int join_run(rb_ctx* ctx, const JoinSpec& s) {
+  const int nchunk = s.ld / 8;
+  const int threads = std::min(512, (nchunk + 31) / 32 * 32);
+  const int chunks = (nchunk + threads - 1) / threads;
+  const bool slabs = s.acc && s.n_acc > 0;
+  const int64_t grid = std::min<int64_t>(s.rows, (int64_t)ctx->sm_count * (slabs ? 16 : std::max(4, 2048 / threads * 2)));
+  JoinArgs<T> a{};
+  a.y = (const T*)s.y; a.acc = s.acc; a.n_acc = slabs ? s.n_acc : 0; a.acc_stride = (size_t)s.rows * s.ld; a.part = (const T*)s.part;
+  a.weight = s.weight; a.top = s.top; a.mult = s.mult; a.gain = (const T*)s.gain; a.eps = s.eps; a.width = s.width; a.ld = s.ld; a.h = s.h;
+  a.out = (T*)s.out; a.n_rows = s.rows; a.zero = s.zero; a.n_zero = s.zero ? s.n_zero : 0;
+  auto go = [&](auto kern) -> int {
+    RB_CUDA(launch_kernel(kern, dim3((unsigned)grid), dim3(threads), 0, ctx->stream, ctx->pdl, a));
+    ctx->launches++;
+    return RB_OK;
+  };
+  if (chunks <= 1) return slabs ? go(add_then_norm_kernel<T, 1, true>) : go(add_then_norm_kernel<T, 1, false>);
+  if (chunks <= 2) return slabs ? go(add_then_norm_kernel<T, 2, true>) : go(add_then_norm_kernel<T, 2, false>);
+  if (chunks <= 4) return slabs ? go(add_then_norm_kernel<T, 4, true>) : go(add_then_norm_kernel<T, 4, false>);
+  return fail(RB_ERR_UNIMPLEMENTED, "rb_add_then_norm: width %d exceeds 16384", s.width);
+}
+
 }  // namespace
+
+int add_then_norm(rb_ctx* ctx, const JoinSpec& s, int dtype) {
+  RB_REQUIRE(ctx && s.h && (!s.out || s.gain) && (!s.part || (s.weight && s.top > 0)), "rb_add_then_norm: null argument");
+  RB_REQUIRE(s.rows >= 0 && s.width > 0 && s.ld >= s.width && (s.ld % 8) == 0, "rb_add_then_norm: bad sizes");
+  RB_REQUIRE(aligned16(s.y) && aligned16(s.acc) && aligned16(s.part) && aligned16(s.h) && aligned16(s.out) && aligned16(s.gain),
+             "rb_add_then_norm: buffers must be 16-byte aligned");
+  if (s.rows == 0) return RB_OK;
+  const double es = (double)dtype_size(dtype);
+  ProfScope prof(ctx, RB_PROF_NORM,
+                 (double)s.rows * s.width * ((s.y ? es : 0.0) + (s.acc ? 4.0 * s.n_acc : 0.0) + (s.part ? es * s.top : 0.0) + 8.0 +
+                                             (s.out ? es : 0.0)), 0.0);
+  if (dtype == RB_BF16) return join_run<__nv_bfloat16>(ctx, s);
+  if (dtype == RB_F32) return join_run<float>(ctx, s);
+  return fail(RB_ERR_DTYPE, "rb_add_then_norm: dtype %d unsupported", dtype);
+}
 
 }  // namespace rb
 
@@ -461,25 +619,68 @@ extern "C" int32_t rb_add_scaled_norm(rb_ctx* ctx, const void* y, const float* a
   return fail(RB_ERR_DTYPE, "rb_add_scaled_norm: dtype %d unsupported", dtype);
 }
 
-extern "C" int32_t rb_scalar_norm_rows(rb_ctx* ctx, const float* h, const int32_t* rows, int64_t row_step, const void* gain, float eps,
-                                       int64_t n_rows, int64_t width, int64_t ld, void* out, int32_t dtype) {
-  RB_REQUIRE(ctx && h && gain && out, "rb_scalar_norm_rows: null argument");
-  RB_REQUIRE(n_rows >= 0 && width > 0 && ld >= width && (ld % 8) == 0 && (rows || row_step >= 1), "rb_scalar_norm_rows: bad sizes");
-  RB_REQUIRE(aligned16(h) && aligned16(out), "rb_scalar_norm_rows: buffers must be 16-byte aligned");
+template <bool kVector>
+static int norm_rows(rb_ctx* ctx, const float* h, const int32_t* rows, int64_t row_step, const void* gain, float eps, int64_t n_rows,
+                     int64_t width, int64_t ld, void* out, int32_t dtype) {
+  RB_REQUIRE(ctx && h && gain && out, "norm of rows: null argument");
+  RB_REQUIRE(n_rows >= 0 && width > 0 && ld >= width && (ld % 8) == 0 && (rows || row_step >= 1), "norm of rows: bad sizes");
+  RB_REQUIRE(aligned16(h) && aligned16(out) && aligned16(gain), "norm of rows: buffers must be 16-byte aligned");
   if (n_rows == 0) return RB_OK;
   const double es = (double)dtype_size(dtype);
   ProfScope prof(ctx, RB_PROF_NORM, (double)n_rows * width * (4.0 + es), 0.0);
   const int threads = (int)std::min<int64_t>(512, (ld / 8 + 31) / 32 * 32);
   if (dtype == RB_BF16)
-    RB_CUDA(launch_kernel(scalar_norm_rows_kernel<__nv_bfloat16>, dim3((unsigned)n_rows), dim3(threads), 0, ctx->stream, ctx->pdl, h,
+    RB_CUDA(launch_kernel(norm_rows_kernel<__nv_bfloat16, kVector>, dim3((unsigned)n_rows), dim3(threads), 0, ctx->stream, ctx->pdl, h,
                           rows, row_step, (const __nv_bfloat16*)gain, eps, (int)width, (int)ld, (__nv_bfloat16*)out));
   else if (dtype == RB_F32)
-    RB_CUDA(launch_kernel(scalar_norm_rows_kernel<float>, dim3((unsigned)n_rows), dim3(threads), 0, ctx->stream, ctx->pdl, h, rows,
+    RB_CUDA(launch_kernel(norm_rows_kernel<float, kVector>, dim3((unsigned)n_rows), dim3(threads), 0, ctx->stream, ctx->pdl, h, rows,
                           row_step, (const float*)gain, eps, (int)width, (int)ld, (float*)out));
   else
-    return fail(RB_ERR_DTYPE, "rb_scalar_norm_rows: dtype %d unsupported", dtype);
+    return fail(RB_ERR_DTYPE, "norm of rows: dtype %d unsupported", dtype);
   ctx->launches++;
   return RB_OK;
+}
+
+extern "C" int32_t rb_scalar_norm_rows(rb_ctx* ctx, const float* h, const int32_t* rows, int64_t row_step, const void* gain, float eps,
+                                       int64_t n_rows, int64_t width, int64_t ld, void* out, int32_t dtype) {
+  return norm_rows<false>(ctx, h, rows, row_step, gain, eps, n_rows, width, ld, out, dtype);
+}
+
+extern "C" int32_t rb_one_plus_norm_rows(rb_ctx* ctx, const float* h, const int32_t* rows, int64_t row_step, const void* gain, float eps,
+                                         int64_t n_rows, int64_t width, int64_t ld, void* out, int32_t dtype) {
+  return norm_rows<true>(ctx, h, rows, row_step, gain, eps, n_rows, width, ld, out, dtype);
+}
+
+extern "C" int32_t rb_add_then_norm(rb_ctx* ctx, const void* y, const float* acc, int32_t n_acc, const void* part, const float* weight,
+                                    int32_t top, float mult, const void* gain, float eps, int64_t rows, int64_t width, int64_t ld,
+                                    float* h, void* out, int32_t dtype) {
+  JoinSpec s;
+  s.y = y; s.acc = acc; s.n_acc = acc ? n_acc : 0; s.part = part; s.weight = weight; s.top = top; s.mult = mult; s.gain = gain; s.eps = eps;
+  s.rows = rows; s.width = (int)width; s.ld = (int)ld; s.h = h; s.out = out;
+  return add_then_norm(ctx, s, dtype);
+}
+
+extern "C" int32_t rb_embed_positions(rb_ctx* ctx, const void* table, const void* positions, int32_t n_positions, int32_t dtype,
+                                      int64_t vocab, int64_t width, int64_t ld, const uint32_t* ids, int32_t batch, int32_t s_new,
+                                      rb_kv_cache* c, const int32_t* new_lens, float* h) {
+  RB_REQUIRE(ctx && table && positions && ids && c && h, "rb_embed_positions: null argument");
+  RB_REQUIRE(vocab > 0 && n_positions > 0 && width > 0 && ld >= width && (ld % 8) == 0, "rb_embed_positions: bad sizes");
+  RB_REQUIRE(batch > 0 && batch <= c->max_batch && s_new > 0, "rb_embed_positions: bad batch/seq");
+  RB_REQUIRE(aligned16(table) && aligned16(positions) && aligned16(h), "rb_embed_positions: buffers must be 16-byte aligned");
+  const int64_t rows = (int64_t)batch * s_new;
+  ProfScope prof(ctx, RB_PROF_EMBED, (double)rows * width * (2.0 * dtype_size(dtype) + 4.0), 0.0);
+  const int threads = (int)std::min<int64_t>(256, (ld / 8 + 31) / 32 * 32);
+  auto go = [&](auto tag) -> int {
+    using T = decltype(tag);
+    RB_CUDA(launch_kernel(embed_positions_kernel<T>, dim3((unsigned)rows), dim3(threads), 0, ctx->stream, ctx->pdl, (const T*)table,
+                          (const T*)positions, n_positions, ids, vocab, (int)ld, s_new, (const int32_t*)c->seq_lens, new_lens, h,
+                          ctx->status_dev));
+    ctx->launches++;
+    return RB_OK;
+  };
+  if (dtype == RB_BF16) return go(__nv_bfloat16());
+  if (dtype == RB_F32) return go(float());
+  return fail(RB_ERR_DTYPE, "rb_embed_positions: dtype %d unsupported", dtype);
 }
 
 extern "C" int32_t rb_conv_norm_append(rb_ctx* ctx, const void* src, const float* acc, int32_t n_acc, const void* bias,

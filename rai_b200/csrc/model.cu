@@ -1028,8 +1028,9 @@ static int forward_rows(rb_model* m, const uint32_t* tokens, int batch, int seq,
     const int base = kc->host_lens[b];
     RB_REQUIRE(!lens || (lens[b] >= 0 && lens[b] <= seq), "ragged forward: sequence %d has %d valid tokens of %d", b, lens[b], seq);
     RB_REQUIRE(pos < 0 || base == pos, "forward: seqlen_offset %d differs from the cached length %d of sequence %d", pos, base, b);
-    RB_REQUIRE(base + seq <= kc->max_seq && base + seq <= c.max_position_embeddings,
-               "forward: position %d + %d exceeds the cache / rotary table capacity", base, seq);
+    // (padding may lie beyond a layered design's position table, not beyond a rotary table)
+    RB_REQUIRE(base + seq <= kc->max_seq && base + (m->layered && lens ? lens[b] : seq) <= c.max_position_embeddings,
+               "forward: position %d + %d exceeds the cache / position table capacity", base, seq);
   }
   for (int i = 0; i < n_rows; ++i)
     RB_REQUIRE(rows[i] >= 0 && rows[i] < total, "forward: row %d of %lld", rows[i], (long long)total);

@@ -49,6 +49,10 @@ struct MixLayer {
   void *conv = nullptr, *q_norm = nullptr, *k_norm = nullptr;         // attention
   void *f_bias = nullptr, *lower = nullptr, *out_norm = nullptr;      // hgrn2
   void *up = nullptr, *down = nullptr, *act = nullptr;
+  // parallel block (one fused input projection [q | k | shared gate | shared up | router], one fused output projection over
+  // [heads | shared expert's inner row]) with experts stacked in gate, up and down
+  int n_main = 0, attn_cols = 0, glu_p = 0, ff_p = 0;  // columns before the router's; of the heads; padded inner sizes
+  void *sink = nullptr, *gate = nullptr;
   rb_kv_cache* kv = nullptr;   // the cache (of this layer's geometry) its keys and values are in, and the layer there
   int kv_layer = 0;
   float* state = nullptr;      // attention: ring of projected values [slot][taps - 1][channels]; hgrn2: [slot][head][key][value]
@@ -116,6 +120,11 @@ struct rb_model {
   int ld = 0;                             // pitch of the residual stream (hidden_size padded to a multiple of 8)
   float* stream = nullptr;                // float32 residual stream [max_tokens][ld]
   void *mix_in = nullptr, *gate = nullptr, *sub_out = nullptr;
+  void *pos = nullptr;                    // learned position vectors
+  // routing of a call's rows to experts: logits, weights of the choices, each expert's list of them, and their rows
+  float *route_z = nullptr, *route_w = nullptr;
+  int32_t *route_list = nullptr, *route_count = nullptr;
+  void *expert_act = nullptr, *expert_out = nullptr;
   float* layer_trace = nullptr;
   int logits_dtype = RB_BF16;
   int32_t* new_lens = nullptr;            // device [max_batch]: tokens each sequence feeds in this call

@@ -1,0 +1,436 @@
+// Kernels of a parallel block with routed experts (layered.cu): what follows the fused input projection (head split, key
+// append, gated activation of the shared expert, and the routing of tokens to experts), the experts' products on CUDA
+// cores (float32 models), and the entry points of the tensor-core form (gemm_tc.cu, grouped).
+#include <algorithm>
+
+#include "ctx.h"
+
+namespace rb {
+
+namespace {
+
+// ------------------------------------------------------------------------------------------
+// Routing: one warp per row.
+// ------------------------------------------------------------------------------------------
+constexpr int kRouteWarps = 8;       // rows per block
+constexpr int kMaxTop = 32;          // one lane per choice
+constexpr int kPerLane = kMaxExperts / 32;
+
+struct RouteArgs {
+  const float* acc;                  // logits: slab s of row r, expert e at acc[s * stride + r * ld + e]
+  int n_acc;
+  size_t stride;
+  int64_t ld;
+  int rows, experts, top, groups, keep;
+  float scale;
+  float* weight;                     // [rows][top]
+  int32_t *list, *count;
+  int64_t cap;
+};
+
+__device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* sc) {  // sc: kMaxExperts floats of this warp
+  const int lane = threadIdx.x & 31;
+  float s[kPerLane];
+#pragma unroll
+  for (int i = 0; i < kPerLane; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = -1.f;
+    if (e < a.experts) {
+      float z = 0.f;
+      for (int k0 = 0; k0 < a.n_acc; k0 += 8) {   // slab order; the loads of up to eight slabs in flight together
+        float t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = k0 + k < a.n_acc ? __ldg(a.acc + (size_t)(k0 + k) * a.stride + (size_t)row * a.ld + e) : 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) z += t[k];
+      }
+      s[i] = sigmoid_f(z);
+      sc[e] = s[i];
+    }
+  }
+  __syncwarp();
+  const int n = a.experts / a.groups;
+  if (a.keep < a.groups) {
+    // a run's strength: its two largest scores.  Lane g has run g (and g + 32, ...); a run stays if fewer than `keep` beat it.
+    float strength[kPerLane];
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const int g = lane + 32 * i;
+      float b1 = 0.f, b2 = 0.f;
+      if (g < a.groups)
+        for (int j = 0; j < n; ++j) {
+          const float v = sc[g * n + j];
+          if (v > b1) { b2 = b1; b1 = v; } else b2 = fmaxf(b2, v);
+        }
+      strength[i] = b1 + b2;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i)
+      if (lane + 32 * i < a.groups) sc[lane + 32 * i] = strength[i];  // groups <= experts
+    __syncwarp();
+    uint32_t kept = 0;  // bit i: run lane + 32 i
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const int g = lane + 32 * i;
+      if (g >= a.groups) continue;
+      int better = 0;
+      for (int o = 0; o < a.groups; ++o) better += sc[o] > strength[i] || (sc[o] == strength[i] && o < g);
+      if (better < a.keep) kept |= 1u << i;
+    }
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const int e = lane + 32 * i, g = e < a.experts ? e / n : 0;
+      const uint32_t of_owner = __shfl_sync(0xffffffffu, kept, g & 31);
+      if (!(of_owner >> (g >> 5) & 1u)) s[i] = -1.f;
+    }
+  }
+  // the largest scores, one at a time (positive floats order like their bits); lane j keeps the j-th choice
+  int chosen = -1;
+  float weight = 0.f;
+  for (int j = 0; j < a.top; ++j) {
+    uint32_t best = 0;
+    int at = 0;
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) {
+      const uint32_t b = s[i] < 0.f ? 0u : __float_as_uint(s[i]) + 1u;
+      if (b > best) { best = b; at = i; }
+    }
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    const uint32_t e = __reduce_min_sync(0xffffffffu, best == top ? (uint32_t)(lane + 32 * at) : 0xffffffffu);
+    if ((e & 31u) == (uint32_t)lane) {
+#pragma unroll
+      for (int i = 0; i < kPerLane; ++i)
+        if (i == (int)(e >> 5)) s[i] = -1.f;
+    }
+    if (lane == j) { chosen = (int)e; weight = __uint_as_float(top - 1u); }
+  }
+  if (lane < a.top) {
+    a.weight[(size_t)row * a.top + lane] = weight * a.scale;
+    const int at = atomicAdd(a.count + chosen, 1);
+    if (at < a.cap) a.list[(size_t)chosen * a.cap + at] = row * a.top + lane;
+  }
+}
+
+// ------------------------------------------------------------------------------------------
+// Head split, key append and gated activation, one block per row (or several); then, in the blocks after those, routing.
+// ------------------------------------------------------------------------------------------
+template <typename T>
+struct SplitArgs {
+  const T* src;
+  const float* acc;
+  int n_acc;
+  size_t acc_stride;
+  const T* bias;
+  int64_t ld;
+  int s_new, q_heads, kv_heads, dim, D, qp, kp, gp;   // padded widths of q, k and of gate (= up)
+  T* kc;
+  const int32_t *block_table, *seq_lens;
+  int pages_per_seq, max_seq, rows, blocks;
+  T *q_out, *glu_out;
+  int64_t glu_ld;
+  uint32_t* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(512) split_route_kernel(const SplitArgs<T> a, const RouteArgs r) {
+  __shared__ float scores[kRouteWarps][kMaxExperts];
+  pdl_launch_dependents();
+  pdl_wait();
+  if ((int)blockIdx.x >= a.blocks) {
+    const int warp = threadIdx.x >> 5;
+    const int row = ((int)blockIdx.x - a.blocks) * kRouteWarps + warp;
+    if (warp < kRouteWarps && row < r.rows) route_row(r, row, scores[warp]);
+    return;
+  }
+  auto load_u = [&](size_t m, int c, float* u) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) u[i] = 0.f;
+    if (a.src) { load8(a.src + m * a.ld + c, u); return; }
+    add_slabs<4>(a.acc, a.n_acc, a.acc_stride, m * a.ld + c, u);
+    if (a.bias) {
+      float t[8];
+      load8(a.bias + c, t);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) u[i] += t[i];
+    }
+  };
+  for (int m = blockIdx.x; m < a.rows; m += a.blocks) {
+    const int b = m / a.s_new, pos = a.seq_lens[b] - a.s_new + m % a.s_new;
+    if (pos < 0 || pos >= a.max_seq) {  // block-uniform
+      if (threadIdx.x == 0) { a.status[0] = (uint32_t)(-RB_ERR_INVALID); a.status[1] = 0x5A11u; a.status[2] = (uint32_t)pos; }
+      continue;
+    }
+    T* q_row = a.q_out + (size_t)m * a.q_heads * a.D;
+    const int page = a.kv_heads > 0 ? a.block_table[(size_t)b * a.pages_per_seq + pos / kPageTokens] : 0;
+    T* k_row = a.kc + ((size_t)page * a.kv_heads * kPageTokens + pos % kPageTokens) * a.D;  // head g: g pages of one head further
+    const size_t k_step = (size_t)kPageTokens * a.D;
+    const int n_glu = a.gp / 8;
+    if ((a.dim & 7) == 0) {
+      const int dq = a.D / 8, n_q = a.q_heads * dq, n_k = a.kv_heads * dq;
+      for (int it = threadIdx.x; it < n_q + n_k; it += blockDim.x) {
+        const int j = it < n_q ? it : it - n_q, h = j / dq, i0 = (j % dq) * 8;
+        float u[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] = 0.f;
+        if (i0 < a.dim) load_u(m, (it < n_q ? 0 : a.qp) + h * a.dim + i0, u);
+        store8((it < n_q ? q_row + h * a.D : k_row + h * k_step) + i0, u);
+      }
+    } else {
+      for (int it = threadIdx.x; it < (a.qp + a.kp) / 8; it += blockDim.x) {
+        float u[8];
+        load_u(m, it * 8, u);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int c = it * 8 + i;
+          if (c < a.q_heads * a.dim) q_row[c / a.dim * a.D + c % a.dim] = Cvt<T>::from_f(u[i]);
+          const int ck = c - a.qp;
+          if (ck >= 0 && ck < a.kv_heads * a.dim) k_row[ck / a.dim * k_step + ck % a.dim] = Cvt<T>::from_f(u[i]);
+        }
+      }
+      const int pad = a.D - a.dim;
+      for (int it = threadIdx.x; it < (a.q_heads + a.kv_heads) * pad; it += blockDim.x) {
+        const int h = it / pad, i = a.dim + it % pad;
+        (h < a.q_heads ? q_row + h * a.D : k_row + (h - a.q_heads) * k_step)[i] = Cvt<T>::from_f(0.f);
+      }
+    }
+    for (int it = threadIdx.x; it < n_glu; it += blockDim.x) {
+      float g[8], u[8];
+      load_u(m, a.qp + a.kp + it * 8, g);
+      load_u(m, a.qp + a.kp + a.gp + it * 8, u);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) g[i] = act_apply(RB_ACT_SILU, g[i]) * u[i];
+      store8(a.glu_out + (size_t)m * a.glu_ld + it * 8, g);
+    }
+  }
+}
+
+template <typename T>
+int split_route_run(rb_ctx* ctx, SplitArgs<T> a, const RouteArgs& r) {
+  // enough blocks to fill the GPU several times over; a prompt's rows share them
+  a.blocks = a.rows > 0 ? (int)std::min<int64_t>(a.rows, (int64_t)ctx->sm_count * 32) : 0;
+  const int pieces = a.rows > 0 ? (a.q_heads + a.kv_heads) * a.D / 8 : 0;
+  int threads = std::min(512, std::max(64, (pieces + 31) / 32 * 32));
+  int route_blocks = 0;
+  if (r.rows > 0) {
+    threads = std::max(threads, kRouteWarps * 32);
+    route_blocks = (r.rows + kRouteWarps - 1) / kRouteWarps;
+  }
+  if (a.blocks + route_blocks == 0) return RB_OK;
+  RB_CUDA(launch_kernel(split_route_kernel<T>, dim3((unsigned)(a.blocks + route_blocks)), dim3(threads), 0, ctx->stream, ctx->pdl, a, r));
+  ctx->launches++;
+  return RB_OK;
+}
+
+int route_check(const RouteArgs& r) {
+  RB_REQUIRE(r.acc && r.n_acc >= 1 && r.weight && r.list && r.count, "rb_moe_route: null argument");
+  RB_REQUIRE(r.experts > 0 && r.experts <= kMaxExperts, "rb_moe_route: %d experts (1..%d)", r.experts, kMaxExperts);
+  RB_REQUIRE(r.groups > 0 && r.experts % r.groups == 0 && r.keep > 0 && r.keep <= r.groups,
+             "rb_moe_route: %d experts in %d groups of which %d stay", r.experts, r.groups, r.keep);
+  RB_REQUIRE(r.top > 0 && r.top <= kMaxTop && r.top <= r.experts / r.groups * r.keep, "rb_moe_route: top %d of %d experts", r.top,
+             r.experts / r.groups * r.keep);
+  RB_REQUIRE(r.cap >= r.rows && r.ld >= r.experts, "rb_moe_route: the lists hold %lld rows, %d given", (long long)r.cap, r.rows);
+  return RB_OK;
+}
+
+// ------------------------------------------------------------------------------------------
+// The experts' products without tensor cores: 64 x 64 tiles as in gemm_plain_kernel, rows by list.
+// ------------------------------------------------------------------------------------------
+template <typename T, bool GATED>
+__global__ void __launch_bounds__(256) moe_plain_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ w2,
+                                                        T* __restrict__ out, const int32_t* __restrict__ list,
+                                                        const int32_t* __restrict__ count, int64_t cap, int experts, int top, int n,
+                                                        int k, int act) {
+  constexpr int BM = 64, BN = 64, BK = 16;
+  __shared__ float xs[BK][BM + 1];
+  __shared__ float ws[BK][BN + 1];
+  __shared__ float ws2[GATED ? BK : 1][BN + 1];
+  __shared__ int where[4];       // expert, first row of the tile inside it, its rows, its first compact row
+  __shared__ int src[BM], dst[BM];
+  if (threadIdx.x == 0) {
+    int tile = blockIdx.y, row = 0;
+    where[0] = -1;
+    for (int e = 0; e < experts; ++e) {
+      const int c = count[e], t = (c + BM - 1) / BM;
+      if (tile < t) { where[0] = e; where[1] = tile * BM; where[2] = c; where[3] = row; break; }
+      tile -= t;
+      row += c;
+    }
+  }
+  __syncthreads();
+  const int e = where[0];
+  if (e < 0) return;
+  const int r0 = where[1], have = min(BM, where[2] - r0);
+  if (threadIdx.x < BM) {
+    const int at = r0 + min((int)threadIdx.x, have - 1);
+    const int entry = list[(size_t)e * cap + at], compact = where[3] + at;
+    src[threadIdx.x] = GATED ? entry / top : compact;
+    dst[threadIdx.x] = GATED ? compact : entry;
+  }
+  __syncthreads();
+  const int tn = blockIdx.x * BN, tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+  const T* we = w + (size_t)e * n * k;
+  const T* we2 = GATED ? w2 + (size_t)e * n * k : nullptr;
+  float acc[4][4] = {}, acc2[4][4] = {};
+  for (int kk = 0; kk < k; kk += BK) {
+    for (int i = threadIdx.x; i < BM * BK; i += blockDim.x) {
+      const int r = i / BK, c = i % BK;
+      xs[c][r] = kk + c < k ? Cvt<T>::to_f(x[(size_t)src[r] * k + kk + c]) : 0.f;
+      const bool ok = tn + r < n && kk + c < k;
+      ws[c][r] = ok ? Cvt<T>::to_f(we[(size_t)(tn + r) * k + kk + c]) : 0.f;
+      if (GATED) ws2[c][r] = ok ? Cvt<T>::to_f(we2[(size_t)(tn + r) * k + kk + c]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < BK; ++c)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          acc[i][j] = fmaf(xs[c][ty * 4 + i], ws[c][tx * 4 + j], acc[i][j]);
+          if (GATED) acc2[i][j] = fmaf(xs[c][ty * 4 + i], ws2[c][tx * 4 + j], acc2[i][j]);
+        }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = ty * 4 + i, c = tn + tx * 4 + j;
+      if (r >= have || c >= n) continue;
+      out[(size_t)dst[r] * n + c] = Cvt<T>::from_f(GATED ? act_apply(act, acc[i][j]) * acc2[i][j] : acc[i][j]);
+    }
+}
+
+template <typename T>
+int moe_plain(rb_ctx* ctx, const GemmArgs& a) {
+  const int64_t tiles = a.m / 64 + std::min<int64_t>(a.experts, a.m);
+  RB_REQUIRE(tiles <= 65535, "moe: %lld row tiles", (long long)tiles);
+  const dim3 grid((unsigned)((a.n + 63) / 64), (unsigned)tiles);
+  if (a.w2)
+    moe_plain_kernel<T, true><<<grid, 256, 0, ctx->stream>>>((const T*)a.x, (const T*)a.w, (const T*)a.w2, (T*)a.out, a.list, a.count,
+                                                            a.cap, a.experts, a.top, (int)a.n, (int)a.k, a.act);
+  else
+    moe_plain_kernel<T, false><<<grid, 256, 0, ctx->stream>>>((const T*)a.x, (const T*)a.w, nullptr, (T*)a.out, a.list, a.count, a.cap,
+                                                             a.experts, a.top, (int)a.n, (int)a.k, a.act);
+  ctx->launches++;
+  return launch_status("moe_plain");
+}
+
+int moe_product(rb_ctx* ctx, const GemmArgs& a, int dtype) {
+  if (a.m == 0) return RB_OK;
+  // experts that some row is expected to choose, if the choices spread evenly
+  double untouched = 1.0;
+  for (int64_t r = 0; r < a.m / a.top && untouched > 1e-9; ++r) untouched *= 1.0 - (double)a.top / a.experts;
+  const double es = (double)dtype_size(dtype), mats = a.w2 ? 2.0 : 1.0;
+  const double in_rows = a.w2 ? (double)a.m / a.top : (double)a.m;
+  ProfScope prof(ctx, RB_PROF_EXPERTS, es * (mats * (1.0 - untouched) * a.experts * a.n * a.k + in_rows * a.k + (double)a.m * a.n),
+                 2.0 * mats * a.m * a.n * a.k);
+  if (dtype == RB_BF16 && !ctx->debug_simple_gemm) return gemm_tc_grouped(ctx, a);
+  if (dtype == RB_BF16) return moe_plain<__nv_bfloat16>(ctx, a);
+  if (dtype == RB_F32) return moe_plain<float>(ctx, a);
+  return fail(RB_ERR_DTYPE, "moe: dtype %d unsupported", dtype);
+}
+
+bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+int round8(int v) { return (v + 7) / 8 * 8; }
+
+}  // namespace
+
+int split_and_route(rb_ctx* ctx, const SplitSpec& f, const RouteSpec* route, int dtype) {
+  rb_kv_cache* c = f.cache;
+  RB_REQUIRE(ctx && c && f.q_out && (f.src || (f.acc && f.n_acc > 0)), "rb_split_append: null argument");
+  RB_REQUIRE(f.batch > 0 && f.batch <= c->max_batch && f.s_new > 0, "rb_split_append: bad batch/seq");
+  RB_REQUIRE(f.src || f.s_new == 1, "rb_split_append: split-K partials need single-token rows");
+  RB_REQUIRE(f.q_heads > 0 && f.kv_heads == c->kv_heads && f.dim > 0 && f.dim <= c->head_dim && f.layer >= 0 && f.layer < c->layers &&
+                 dtype == c->dtype && c->shared(),
+             "rb_split_append: the cache does not fit the layer");
+  RB_REQUIRE(f.glu_size >= 0 && (f.glu_size == 0 || (f.glu_out && f.glu_ld >= round8(f.glu_size) && f.glu_ld % 8 == 0)),
+             "rb_split_append: bad gated part");
+  RB_REQUIRE(aligned16(f.src) && aligned16(f.acc) && aligned16(f.bias) && aligned16(f.q_out) && aligned16(f.glu_out),
+             "rb_split_append: buffers must be 16-byte aligned");
+  const int64_t rows = (int64_t)f.batch * f.s_new;
+  RouteArgs r{};
+  if (route) {
+    r.acc = route->acc; r.n_acc = route->n_acc; r.stride = (size_t)route->acc_stride; r.ld = route->z_ld; r.rows = (int)rows;
+    r.experts = route->experts; r.top = route->top; r.groups = route->groups; r.keep = route->keep; r.scale = route->scale;
+    r.weight = route->weight; r.list = route->list; r.count = route->count; r.cap = route->cap;
+    RB_TRY(route_check(r));
+  }
+  auto fill = [&](auto tag) -> int {
+    using T = decltype(tag);
+    SplitArgs<T> a{};
+    a.src = (const T*)f.src; a.acc = f.acc; a.n_acc = f.acc ? f.n_acc : 0; a.acc_stride = (size_t)rows * f.src_ld;
+    a.bias = (const T*)f.bias; a.ld = f.src_ld; a.s_new = f.s_new; a.q_heads = f.q_heads; a.kv_heads = f.kv_heads; a.dim = f.dim;
+    a.D = c->head_dim; a.qp = round8(f.q_heads * f.dim); a.kp = round8(f.kv_heads * f.dim); a.gp = round8(f.glu_size);
+    RB_REQUIRE(f.src_ld % 8 == 0 && f.src_ld >= a.qp + a.kp + 2 * a.gp, "rb_split_append: row pitch %lld does not hold the parts",
+               (long long)f.src_ld);
+    a.kc = (T*)c->k + (size_t)f.layer * c->layer_stride_elems();
+    a.block_table = c->block_table; a.seq_lens = c->seq_lens; a.pages_per_seq = c->pages_per_seq; a.max_seq = c->max_seq;
+    a.rows = (int)rows; a.q_out = (T*)f.q_out; a.glu_out = (T*)f.glu_out; a.glu_ld = f.glu_ld; a.status = ctx->status_dev;
+    const double C = a.qp + a.kp + 2.0 * a.gp, es = sizeof(T);
+    ProfScope prof(ctx, RB_PROF_ROPE_KV,
+                   (double)rows * ((f.src ? es : 4.0 * f.n_acc) * C + es * (a.qp + a.kp + a.gp)) +
+                       (route ? 4.0 * rows * (route->n_acc * (double)route->experts + 2.0 * route->top) : 0.0), 0.0);
+    return split_route_run<T>(ctx, a, r);
+  };
+  if (dtype == RB_BF16) return fill(__nv_bfloat16());
+  if (dtype == RB_F32) return fill(float());
+  return fail(RB_ERR_DTYPE, "rb_split_append: dtype %d unsupported", dtype);
+}
+
+}  // namespace rb
+
+using namespace rb;
+
+extern "C" int32_t rb_split_append(rb_ctx* ctx, const void* src, const float* acc, int32_t n_acc, const void* bias, int64_t src_ld,
+                                   int32_t batch, int32_t s_new, int32_t q_heads, int32_t kv_heads, int32_t dim, int32_t glu_size,
+                                   rb_kv_cache* c, int32_t layer, void* q_out, void* glu_out, int64_t glu_ld, int32_t dtype) {
+  SplitSpec f;
+  f.src = src; f.acc = acc; f.n_acc = n_acc; f.bias = bias; f.src_ld = src_ld; f.batch = batch; f.s_new = s_new; f.q_heads = q_heads;
+  f.kv_heads = kv_heads; f.dim = dim; f.glu_size = glu_size; f.cache = c; f.layer = layer; f.q_out = q_out; f.glu_out = glu_out;
+  f.glu_ld = glu_ld;
+  return split_and_route(ctx, f, nullptr, dtype);
+}
+
+extern "C" int32_t rb_moe_route(rb_ctx* ctx, const float* acc, int32_t n_acc, int64_t acc_stride, int64_t z_ld, int64_t rows,
+                                int32_t experts, int32_t top, int32_t groups, int32_t keep, float scale, float* weight,
+                                int32_t* list, int32_t* count, int64_t cap) {
+  RB_REQUIRE(ctx && rows >= 0, "rb_moe_route: null argument");
+  RouteArgs r{};
+  r.acc = acc; r.n_acc = n_acc; r.stride = (size_t)acc_stride; r.ld = z_ld; r.rows = (int)rows; r.experts = experts; r.top = top;
+  r.groups = groups; r.keep = keep; r.scale = scale; r.weight = weight; r.list = list; r.count = count; r.cap = cap;
+  RB_TRY(route_check(r));
+  ProfScope prof(ctx, RB_PROF_OTHER, 4.0 * rows * (n_acc * (double)experts + 2.0 * top), 0.0);
+  return split_route_run<float>(ctx, SplitArgs<float>{}, r);
+}
+
+static int moe_args(GemmArgs& a, const void* x, const void* w, const void* w2, void* out, int64_t rows, int32_t top, int32_t experts,
+                    const int32_t* list, const int32_t* count, int64_t cap, int64_t n, int64_t k, int act) {
+  RB_REQUIRE(x && w && out && list && count, "rb_moe: null argument");
+  RB_REQUIRE(rows >= 0 && top > 0 && experts > 0 && experts <= kMaxExperts && cap >= rows && n > 0 && k > 0 && n % 8 == 0 && k % 8 == 0,
+             "rb_moe: bad sizes");
+  RB_REQUIRE(rows * top <= 0x7fffffff && (int64_t)experts * n <= 0x7fffffff, "rb_moe: too many rows");
+  RB_REQUIRE(aligned16(x) && aligned16(w) && aligned16(w2) && aligned16(out), "rb_moe: buffers must be 16-byte aligned");
+  a.x = x; a.w = w; a.w2 = w2; a.out = out; a.m = rows * top; a.n = n; a.k = k; a.act = act;
+  a.list = list; a.count = count; a.cap = cap; a.experts = experts; a.top = top;
+  return RB_OK;
+}
+
+extern "C" int32_t rb_moe_gated(rb_ctx* ctx, const void* x, const void* wg, const void* wu, void* out, int64_t rows, int32_t top,
+                                int32_t experts, const int32_t* list, const int32_t* count, int64_t cap, int64_t n, int64_t k,
+                                int32_t act, int32_t dtype) {
+  RB_REQUIRE(ctx && wu, "rb_moe_gated: null argument");
+  RB_REQUIRE(act != RB_ACT_XIELU, "rb_moe_gated: the activation needs parameters");
+  GemmArgs a;
+  RB_TRY(moe_args(a, x, wg, wu, out, rows, top, experts, list, count, cap, n, k, act));
+  return moe_product(ctx, a, dtype);
+}
+
+extern "C" int32_t rb_moe_down(rb_ctx* ctx, const void* x, const void* wd, void* out, int64_t rows, int32_t top, int32_t experts,
+                               const int32_t* list, const int32_t* count, int64_t cap, int64_t n, int64_t k, int32_t dtype) {
+  RB_REQUIRE(ctx, "rb_moe_down: null argument");
+  GemmArgs a;
+  RB_TRY(moe_args(a, x, wd, nullptr, out, rows, top, experts, list, count, cap, n, k, RB_ACT_NONE));
+  return moe_product(ctx, a, dtype);
+}

@@ -153,6 +153,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
   const int call_base = seq_lens[b] - s_new;  // first token of this call
   const int first = ext && x.window > 0 ? max(0, limit - x.window + 1) : 0;
   const float slope = ext && x.alibi ? alibi_slope(h, q_heads) : 0.f;
+  if (ext) scale *= query_temperature(limit, x.temp_every, x.temp_coef);
   for (int t = first + warp; t <= limit; t += kPlainAttnWarps) {
     // sliding window (qwen2.rs:316-334): it acts among the tokens of one call only, the cached prefix stays visible
     if (!ext && t >= call_base && t + window < limit) continue;
@@ -164,7 +165,9 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
       const int i = lane + 32 * j;
       if (i < d) dot += qv[j] * Cvt<T>::to_f(k_cache[off + i]);
     }
-    dot = fmaf(-slope, (float)(limit - t), warp_sum(dot) * scale);
+    dot = warp_sum(dot) * scale;
+    if (ext && x.softcap > 0.f) dot = x.softcap * tanhf(dot / x.softcap);
+    dot = fmaf(-slope, (float)(limit - t), dot);
     const float mn = fmaxf(mx, dot);
     const float corr = expf(mx - mn), p = expf(dot - mn);
     l = l * corr + p;
@@ -188,6 +191,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
   float L = 0.f;
 #pragma unroll
   for (int w = 0; w < kPlainAttnWarps; ++w) L += (sm_m[w] == -INFINITY) ? 0.f : sm_l[w] * expf(sm_m[w] - M);
+  if (ext && x.sink) L += expf(Cvt<T>::to_f(((const T*)x.sink)[h]) - M);
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float O = 0.f;
 #pragma unroll

@@ -23,6 +23,8 @@ def param_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     a = cfg["arch"]
     if a == "malasun":
         return _malasun_shapes(cfg)
+    if a == "votapel":
+        return _votapel_shapes(cfg)
     H, I, V = cfg["hidden_size"], cfg["intermediate_size"], cfg["vocab_size"]
     nq = cfg["num_attention_heads"]
     nkv = cfg.get("num_key_value_heads") or nq
@@ -98,6 +100,26 @@ def _malasun_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     return out + [("final.norm", (), "gain"), ("head", (V, W), "fan_in")]
 
 
+def _votapel_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """Kinds as in _malasun_shapes; 'delta' is a norm weight stored as its difference from one, 'sink' a score."""
+    W, V = cfg["hidden_size"], cfg["vocab_size"]
+    out: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed"), ("pos", (cfg["max_positions"], W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        mix, mlp, p = layer["mixer"], layer["mlp"], f"l{i}."
+        q, k = mix["heads"] * mix["dim"], mix["kv_heads"] * mix["dim"]
+        out += [(p + "norm1", (W,), "delta"), (p + "mix.q", (q, W), "fan_in"), (p + "mix.q.b", (q,), "bias"),
+                (p + "mix.k", (k, W), "fan_in"), (p + "mix.k.b", (k,), "bias"), (p + "mix.sink", (mix["heads"],), "sink"),
+                (p + "mix.o", (W, q), "fan_in")]
+        if not mlp:
+            continue
+        parts = [(f"e{e}", mlp["ff"]) for e in range(mlp["experts"])] + ([("shared", mlp["shared_ff"])] if mlp["shared_ff"] else [])
+        for name, ff in parts:
+            m = f"{p}mlp.{name}."
+            out += [(m + "gate", (ff, W), "fan_in"), (m + "up", (ff, W), "fan_in"), (m + "down", (W, ff), "fan_in")]
+        out.append((p + "mlp.router", (mlp["experts"], W), "fan_in"))
+    return out + [("final.norm", (W,), "delta"), ("head", (V, W), "fan_in")]
+
+
 def bf16_round(x: np.ndarray) -> np.ndarray:
     """float32 -> nearest-even bfloat16 -> float32 (so the CPU oracle and the GPU see the same values)."""
     u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
@@ -112,6 +134,8 @@ _DRAWS = {
     "conv": lambda r, s: r.standard_normal(s) / np.sqrt(s[1]),
     "lower": lambda r, s: r.uniform(0.0, 0.9, s),
     "forget_b": lambda r, s: r.uniform(0.0, 6.0, s),
+    "delta": lambda r, s: 0.2 * r.standard_normal(s),
+    "sink": lambda r, s: r.standard_normal(s),
     "act": lambda r, s: r.uniform(-1.0, 1.0, s),
 }
 
