@@ -55,10 +55,10 @@ def parse_args():
     ap.add_argument("--skip-parity", action="store_true", help="skip the oracle comparison that follows the timed region")
     ap.add_argument("--skip-other-configs", action="store_true",
                     help="skip the short decode runs of the other benchmark configurations (single-GPU default run only)")
-    ap.add_argument("--design", default="", choices=["", "malasun"],
+    ap.add_argument("--design", default="", choices=["", "malasun", "votapel"],
                     help="instead of the headline: prefill and decode of this design at a few sizes, each beside a qwen2 "
                          "model of equal width, heads, depth and parameter count (one JSON line)")
-    ap.add_argument("--design-sizes", default="malasun-1k,malasun-2k,malasun-4k")
+    ap.add_argument("--design-sizes", default="", help="comma-separated configurations (default: the design's 1k, 2k and 4k)")
     ap.add_argument("--skip-fill", action="store_true",
                     help="leave the KV cache zero-filled instead of prefilling it (same traffic; for profiler runs)")
     return ap.parse_args()
@@ -638,7 +638,7 @@ def random_param(kind, shape, gen):
     u = lambda lo, hi: torch.rand(shape, generator=gen, device="cuda") * (hi - lo) + lo  # noqa: E731
     w = {"norm_w": lambda: torch.ones(shape, device="cuda"), "gain": lambda: torch.ones(shape, device="cuda"), "embed": n,
          "fan_in": lambda: n() / shape[1] ** 0.5, "conv": lambda: n() / shape[1] ** 0.5, "lower": lambda: u(0.0, 0.9),
-         "forget_b": lambda: u(0.0, 6.0), "act": lambda: u(-1.0, 1.0)}.get(kind, lambda: n() * 0.02)()
+         "forget_b": lambda: u(0.0, 6.0), "delta": lambda: n() * 0.2, "sink": n, "act": lambda: u(-1.0, 1.0)}.get(kind, lambda: n() * 0.02)()
     return w.to(torch.bfloat16)
 
 
@@ -746,7 +746,7 @@ def run_design(args):
     from rai_b200 import configs
     peaks, kind = measured_peaks()
     rows = {}
-    for name in args.design_sizes.split(","):
+    for name in (args.design_sizes or ",".join(f"{args.design}-{k}" for k in ("1k", "2k", "4k"))).split(","):
         cfg = configs.get(name)
         if args.layers:
             cfg["layers"] = cfg["layers"][:args.layers]
