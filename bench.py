@@ -57,7 +57,8 @@ def parse_args():
                     help="skip the short decode runs of the other benchmark configurations (single-GPU default run only)")
     ap.add_argument("--design", default="", choices=["", "malasun", "votapel"],
                     help="instead of the headline: prefill and decode of this design at a few sizes, each beside a qwen2 "
-                         "model of equal width, heads, depth and parameter count (one JSON line)")
+                         "model of equal width, heads, depth and parameter count; with routed experts also beside one with as "
+                         "many parameters as a token uses (one JSON line)")
     ap.add_argument("--design-sizes", default="", help="comma-separated configurations (default: the design's 1k, 2k and 4k)")
     ap.add_argument("--skip-fill", action="store_true",
                     help="leave the KV cache zero-filled instead of prefilling it (same traffic; for profiler runs)")
@@ -642,8 +643,9 @@ def random_param(kind, shape, gen):
     return w.to(torch.bfloat16)
 
 
-def equal_size_qwen2(cfg):
-    """qwen2 with the design's width, heads, depth and (through its gated feed-forward's size) parameter count."""
+def equal_size_qwen2(cfg, active=False):
+    """qwen2 with the design's width, heads, depth and (through its gated feed-forward's size) parameter count; active: as
+    many parameters as one token uses, which counts a design's routed experts only as often as they are chosen."""
     from rai_b200 import synth
     import math
     attn = [x["mixer"] for x in cfg["layers"] if x["mixer"]["type"] == "attention"][0]
@@ -652,9 +654,14 @@ def equal_size_qwen2(cfg):
              max_position_embeddings=8192, sliding_window=1 << 30, rope_theta=1e6, rms_norm_eps=1e-6, hidden_act="silu",
              tie_word_embeddings=False)
     count = lambda k: sum(math.prod(s) for _, s, _ in synth.param_shapes(k))  # noqa: E731
-    missing = count(cfg) - count(c)
+    idle = 0
+    if active:
+        for x in cfg["layers"]:
+            mlp = x["mlp"] or {}
+            idle += 3 * c["hidden_size"] * mlp.get("ff", 0) * (mlp.get("experts", 0) - mlp.get("top", 0))
+    missing = count(cfg) - idle - count(c)
     c["intermediate_size"] += max(0, round(missing / (3 * c["hidden_size"] * c["num_hidden_layers"]) / 128)) * 128
-    return c, count(cfg), count(c)
+    return c, count(cfg) - idle, count(c)
 
 
 def class_profile(dev, peaks, run):
@@ -753,6 +760,9 @@ def run_design(args):
         other, n_ours, n_other = equal_size_qwen2(cfg)
         rows[name] = {"layers": len(cfg["layers"]), "width": cfg["hidden_size"], "params": n_ours, "qwen2_params": n_other,
                       "design": design_arm(cfg, args, peaks), "qwen2": design_arm(other, args, peaks)}
+        if any((x["mlp"] or {}).get("experts") for x in cfg["layers"]):
+            lean, n_active, n_lean = equal_size_qwen2(cfg, active=True)
+            rows[name].update(active_params=n_active, qwen2_active_params=n_lean, qwen2_active=design_arm(lean, args, peaks))
     print(json.dumps({"design": args.design, "dtype": "bf16", "data": "synthetic", "peaks": peaks, "peak_kind": kind,
                       "decode": f"batch {args.decode_batch}, context {args.context}, {args.steps} steps",
                       "prefill": f"{args.prefill_batch} x {args.prefill_len}",

@@ -340,10 +340,11 @@ int32_t rb_moe_route(rb_ctx* ctx, const float* acc_dev, int32_t n_acc, int64_t a
 /* The experts' two products over the lists that rb_moe_route made.  Weights are stacked by expert, wg, wu [experts][n][k]
  * and wd [experts][n][k]; n and k are multiples of 8.  The first writes act(x Wg^T) * (x Wu^T) of each listed row (row
  * list / top of x) to compact rows of `out` (expert after expert, [rows * top, n]); the second multiplies those rows and
- * writes each result to row list[...] of out [rows * top, n]. */
+ * writes each result to row list[...] of out [rows * top, n].  sorted_dev, [rows * top, k], is space for a copy of x in the
+ * order of the lists, which makes the products of many rows faster; NULL = do without. */
 int32_t rb_moe_gated(rb_ctx* ctx, const void* x_dev, const void* wg_dev, const void* wu_dev, void* out_dev, int64_t rows,
                      int32_t top, int32_t experts, const int32_t* list_dev, const int32_t* count_dev, int64_t cap, int64_t n,
-                     int64_t k, int32_t act, int32_t dtype);
+                     int64_t k, int32_t act, void* sorted_dev, int32_t dtype);
 int32_t rb_moe_down(rb_ctx* ctx, const void* x_dev, const void* wd_dev, void* out_dev, int64_t rows, int32_t top,
                     int32_t experts, const int32_t* list_dev, const int32_t* count_dev, int64_t cap, int64_t n, int64_t k,
                     int32_t dtype);

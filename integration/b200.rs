@@ -185,7 +185,7 @@ extern "C" {
     pub fn rb_one_plus_norm_rows(ctx: *mut rb_ctx, h_dev: *const f32, rows_dev: *const i32, row_step: i64, gain_dev: *const c_void, eps: f32, n_rows: i64, width: i64, ld: i64, out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_split_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, src_ld: i64, batch: i32, s_new: i32, q_heads: i32, kv_heads: i32, dim: i32, glu_size: i32, cache: *mut rb_kv_cache, layer: i32, q_out_dev: *mut c_void, glu_out_dev: *mut c_void, glu_ld: i64, dtype: i32) -> i32;
     pub fn rb_moe_route(ctx: *mut rb_ctx, acc_dev: *const f32, n_acc: i32, acc_stride: i64, z_ld: i64, rows: i64, experts: i32, top: i32, groups: i32, keep: i32, scale: f32, weight_dev: *mut f32, list_dev: *mut i32, count_dev: *mut i32, cap: i64) -> i32;
-    pub fn rb_moe_gated(ctx: *mut rb_ctx, x_dev: *const c_void, wg_dev: *const c_void, wu_dev: *const c_void, out_dev: *mut c_void, rows: i64, top: i32, experts: i32, list_dev: *const i32, count_dev: *const i32, cap: i64, n: i64, k: i64, act: i32, dtype: i32) -> i32;
+    pub fn rb_moe_gated(ctx: *mut rb_ctx, x_dev: *const c_void, wg_dev: *const c_void, wu_dev: *const c_void, out_dev: *mut c_void, rows: i64, top: i32, experts: i32, list_dev: *const i32, count_dev: *const i32, cap: i64, n: i64, k: i64, act: i32, sorted_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_moe_down(ctx: *mut rb_ctx, x_dev: *const c_void, wd_dev: *const c_void, out_dev: *mut c_void, rows: i64, top: i32, experts: i32, list_dev: *const i32, count_dev: *const i32, cap: i64, n: i64, k: i64, dtype: i32) -> i32;
     pub fn rb_hgrn2(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, f_bias_dev: *const c_void, lower_dev: *const c_void, norm_weight_dev: *const c_void, eps: f32, heads: i32, key_dim: i32, value_dim: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, new_lens_dev: *const i32, state_dev: *mut f32, chunk: i32, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
     pub fn rb_argmax_rows(ctx: *mut rb_ctx, logits_dev: *const c_void, dtype: i32, rows: i64, cols: i64, out_dev: *mut u32) -> i32;

@@ -25,7 +25,7 @@ namespace rb {
 
 using bf16 = __nv_bfloat16;
 
-int attention_decode_splits(rb_ctx* ctx, int batch, int kv_heads, int max_len, int head_dim);
+
 
 // Split-KV scratch of the context, grow-only.  A captured decode step has the buffer's address baked in, and other
 // models or direct calls on the same context may need more later: a buffer that has been handed out is therefore

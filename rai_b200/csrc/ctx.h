@@ -157,16 +157,18 @@ struct GemmArgs {
   const int32_t *list = nullptr, *count = nullptr;
   int64_t cap = 0;
   int experts = 0, top = 1;
+  bool sorted = false;  // gated: x is already in the order of the lists
   bool reduce = false;            // M <= 64: if K is split, sum the splits inside the kernel and apply the epilogue
 };
 int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a);
 constexpr int kMaxExperts = 256;
 int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a);
+bool grouped_wants_sorted(int64_t rows, int top, int experts);
 int gemm_tc_pick_splits(rb_ctx* ctx, int64_t m, int64_t n, int64_t k);
 int gemm_reserve_scratch(rb_ctx* ctx, size_t bytes);
 int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype);
 
-// moe.cu: rb_split_append and rb_moe_route in one launch (route NULL: the first alone)
+// moe.cu: rb_split_append and rb_moe_route, in one launch at single-token steps (route NULL: the first alone)
 struct SplitSpec {
   const void* src = nullptr;
   const float* acc = nullptr;

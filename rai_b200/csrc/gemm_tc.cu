@@ -29,10 +29,12 @@
 //            `reduce`, an epilogue that pushes the finished slice straight into the tensor-parallel peers'
 //            exchange buffers - 9 us per launch against 8 us for the separate publishing kernel, whose many
 //            small blocks read the slabs with far more parallelism than one CTA per tile slice can.)
-// GROUP (swapped form only) is the same product for a mixture of experts: a stack of weight matrices, each applied to the
-// rows that chose it.  The work items are (expert, weight tile, tile of its rows), counted on the device from the experts'
-// row counts; rows of X are fetched by index with gather copies, so no sorted copy of X is made, and a tile fetches only
-// the rows it has.  GROUP 1 reads listed rows of X and writes compact rows, GROUP 2 reads those and writes listed rows.
+// GROUP is the same product for a mixture of experts: a stack of weight matrices, each applied to the rows that chose it.
+// The work items are (expert, weight tile, tile of its rows), counted on the device from the experts' row counts.  GROUP 1
+// writes compact rows (expert after expert), GROUP 2 reads those and writes listed rows.  With few rows per expert
+// (swapped) rows are fetched by index with gather copies, so no sorted copy of X is made and a tile fetches only the rows it
+// has; such a copy moves about one row in twenty cycles, too slow to feed the tensor cores a full tile, so with many rows
+// (normal form) GROUP 1 reads a sorted copy.
 // GATED computes act(X.Wg^T) * (X.Wu^T) with two accumulators per stage (qwen2.rs:100-103).
 //
 // Every barrier wait is bounded; a give-up is recorded in the context's status word and the CTA
@@ -44,6 +46,7 @@
 #include <vector>
 
 #include "ctx.h"
+#include "groups.cuh"
 #include "ptx.cuh"
 
 namespace rb {
@@ -97,7 +100,6 @@ struct Params {
   uint32_t* tile_count; // reduce: arrivals per tile, and readers done per tile; both self-resetting
   uint32_t* tile_done;
   long long wait_cycles;  // give-up budget of every bounded wait
-  int stream_weights;   // GROUP: every weight byte is read about once, keep them from displacing the rest of L2
   uint32_t* status;
 };
 
@@ -126,46 +128,12 @@ __device__ __forceinline__ void decode_item(const Params& p, int item, bool swap
   }
 }
 
-// GROUP: where each expert's work items and compact rows start
-struct Groups {
-  int item[kMaxExperts + 1], row[kMaxExperts + 1];
-};
-// by the whole block; E experts, tiles of BN rows, n_p weight tiles each
-template <int BN>
-__device__ __forceinline__ void make_groups(Groups& g, const int32_t* count, int E, int n_p) {
-  for (int e = threadIdx.x; e < E; e += blockDim.x) g.row[e + 1] = __ldcg(count + e);
-  __syncthreads();
-  if (threadIdx.x < 32) {
-    int items = 0, rows = 0;
-    for (int e0 = 0; e0 < E; e0 += 32) {
-      const int e = e0 + (int)threadIdx.x;
-      const int c = e < E ? g.row[e + 1] : 0;
-      int ri = c, ti = (c + BN - 1) / BN * n_p;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int a = __shfl_up_sync(0xffffffffu, ri, o), b = __shfl_up_sync(0xffffffffu, ti, o);
-        if ((int)threadIdx.x >= o) { ri += a; ti += b; }
-      }
-      if (e < E) { g.row[e + 1] = rows + ri; g.item[e + 1] = items + ti; }
-      rows += __shfl_sync(0xffffffffu, ri, 31);
-      items += __shfl_sync(0xffffffffu, ti, 31);
-    }
-    if (threadIdx.x == 0) { g.row[0] = 0; g.item[0] = 0; }
-  }
-  __syncthreads();
-}
-// the expert, weight tile and row tile of an item; rows of neighbouring items share a weight tile
-template <int BN>
-__device__ __forceinline__ void group_item(const Groups& g, int E, int item, int& e, int& pt, int& qt) {
-  int lo = 0, hi = E;  // item[lo] <= item < item[hi]
-  while (hi - lo > 1) {
-    const int mid = (lo + hi) >> 1;
-    if (g.item[mid] <= item) lo = mid; else hi = mid;
-  }
-  e = lo;
-  const int n_q = (g.row[e + 1] - g.row[e] + BN - 1) / BN, at = item - g.item[e];
-  pt = at / n_q;
-  qt = at % n_q;
+// GROUP: the expert, weight tile and row tile (of `tile` rows) of an item; neighbouring items share a weight tile
+__device__ __forceinline__ void group_item(const Groups& g, int E, int item, int tile, int& e, int& wt, int& rt) {
+  e = group_of(g.item, E, item);
+  const int n_rt = (g.row[e + 1] - g.row[e] + tile - 1) / tile, at = item - g.item[e];
+  wt = at / n_rt;
+  rt = at % n_rt;
 }
 
 __device__ __forceinline__ uint4 pack8(const float* v) {
@@ -234,9 +202,9 @@ template <int BN, bool SWAP, bool GATED, int GROUP>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__ CUtensorMap tm_p2,
                const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_q2, const Params p) {
-  static_assert(GROUP == 0 || SWAP, "the grouped form is a swapped one");
-  constexpr bool kGather = GROUP == 1 || (GROUP == 2 && BN <= 64);  // rows by index; else one copy of BN rows
+  constexpr bool kGather = GROUP != 0 && SWAP;  // rows by index
   static_assert(!kGather || BN <= 128, "one gather per lane");
+  constexpr int kRowTile = SWAP ? BN : kBM;
   using C = Cfg<BN, SWAP, GATED>;
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t full_bar[C::kStages];
@@ -277,7 +245,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
   int n_items = p.n_items;
   if constexpr (GROUP != 0) {
     pdl_wait();  // the counts come from a kernel before this one
-    make_groups<BN>(groups, p.count, p.experts, p.n_p);
+    make_groups(groups, p.count, p.experts, kRowTile, SWAP ? p.n_p : p.n_q);
     n_items = groups.item[p.experts];
   }
   if (GROUP != 0 && warp == 0) {
@@ -288,20 +256,20 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
       uint32_t phase = 0, issued = 0;
       bool ok = true;
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
-        int e, pt, qt;
-        group_item<BN>(groups, p.experts, item, e, pt, qt);
-        const int first = groups.row[e], have = min(BN, groups.row[e + 1] - first - qt * BN);
+        int e, wt, rt;
+        group_item(groups, p.experts, item, kRowTile, e, wt, rt);
+        const int first = groups.row[e], have = min(kRowTile, groups.row[e + 1] - first - rt * kRowTile);
         const int n_gather = (have + 3) / 4;
         int r[4] = {0, 0, 0, 0};
         if (kGather && lane < n_gather) {
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            const int at = qt * BN + min(lane * 4 + i, have - 1);
+            const int at = rt * BN + min(lane * 4 + i, have - 1);
             r[i] = GROUP == 1 ? p.list[(size_t)e * p.cap + at] / p.top : first + at;
           }
         }
-        const uint32_t bytes = C::kPTiles * C::kPBytes + (kGather ? (uint32_t)n_gather * 512u : (uint32_t)C::kQBytes);
-        const int wy = e * p.p_rows + pt * kBM;
+        const uint32_t bytes = kGather ? C::kPTiles * C::kPBytes + (uint32_t)n_gather * 512u : (uint32_t)C::kStageBytes;
+        const int wy = e * p.n + wt * (SWAP ? kBM : BN);
         for (int kb = 0; kb < p.num_kb; ++kb) {
           uint8_t* st = tiles + (size_t)stage * C::kStageBytes;
           uint8_t* qs = st + C::kPTiles * C::kPBytes;
@@ -310,14 +278,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
             mine = ptx::mbar_wait(&empty_bar[stage], phase ^ 1u, &abort_flag, p.wait_cycles) ? 1 : 0;
             if (mine) {
               ptx::mbar_expect_tx(&full_bar[stage], bytes);
-              if (p.stream_weights) {
+              if (SWAP) {
                 ptx::tma_load_2d_hint(st, &tm_p, &full_bar[stage], kb * kBK, wy, stream_policy);
                 if (C::kPTiles == 2) ptx::tma_load_2d_hint(st + C::kPBytes, &tm_p2, &full_bar[stage], kb * kBK, wy, stream_policy);
               } else {
-                ptx::tma_load_2d(st, &tm_p, &full_bar[stage], kb * kBK, wy);
-                if (C::kPTiles == 2) ptx::tma_load_2d(st + C::kPBytes, &tm_p2, &full_bar[stage], kb * kBK, wy);
+                ptx::tma_load_2d(st, &tm_p, &full_bar[stage], kb * kBK, first + rt * kBM);
+                ptx::tma_load_2d(qs, &tm_q, &full_bar[stage], kb * kBK, wy);
+                if (C::kQTiles == 2) ptx::tma_load_2d(qs + C::kQBytes, &tm_q2, &full_bar[stage], kb * kBK, wy);
               }
-              if (!kGather) ptx::tma_load_2d(qs, &tm_q, &full_bar[stage], kb * kBK, first + qt * BN);
             }
           }
           mine = __shfl_sync(0xffffffffu, mine, 0);  // also orders the expected byte count before the gathers
@@ -446,8 +414,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
       int m_lim = p.m, row0 = 0;            // rows of this item's group, and where they go
       const int32_t* scatter = nullptr;
       if constexpr (GROUP != 0) {
-        int e;
-        group_item<BN>(groups, p.experts, item, e, pt, qt);
+        int e, wt, rt;
+        group_item(groups, p.experts, item, kRowTile, e, wt, rt);
+        pt = SWAP ? wt : rt;
+        qt = SWAP ? rt : wt;
         row0 = groups.row[e];
         m_lim = groups.row[e + 1] - row0;
         if (GROUP == 2) scatter = p.list + (size_t)e * p.cap;
@@ -472,7 +442,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
       constexpr int CH = BN >= 32 ? 32 : 16;  // columns per TMEM load
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += CH) {
-        if (GROUP != 0 && qt * BN + c0 >= m_lim) break;
+        if (GROUP != 0 && SWAP && qt * BN + c0 >= m_lim) break;
         float v[CH], g[GATED ? CH : 1];
         {
           uint32_t r[CH];
@@ -565,8 +535,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
           const int gm = pt * kBM + lane_row;
           const int gn0 = qt * BN + c0;
           if (GATED) act_inplace(p.act, g, ac);
-          if (gm < p.m) {
+          if (gm < m_lim) {
             const bool vec_ok = (p.n % 8) == 0;
+            const size_t o_row = GROUP == 0 ? gm : GROUP == 1 ? row0 + gm : scatter[gm];
 #pragma unroll
             for (int j8 = 0; j8 < CH; j8 += 8) {
               const int gn = gn0 + j8;
@@ -602,7 +573,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_p, const __grid_constant__
                 }
               }
               if (vec_ok) {
-                *reinterpret_cast<uint4*>(p.out + (size_t)gm * p.n + gn) = pack8(y);
+                *reinterpret_cast<uint4*>(p.out + o_row * p.n + gn) = pack8(y);
               } else {
                 for (int j = 0; j < 8 && gn + j < p.n; ++j) p.out[(size_t)gm * p.n + gn + j] = __float2bfloat16_rn(y[j]);
               }
@@ -761,12 +732,13 @@ int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
   const void* qbase = SWAP ? a.x : a.w;
   const void* q2base = SWAP ? a.x : a.w2;
   CUtensorMap tp, tp2, tq, tq2;
-  const int64_t stacked = (int64_t)p.p_rows * (GROUP != 0 ? p.experts : 1);
-  constexpr int q_box = GROUP == 1 || (GROUP == 2 && BN <= 64) ? 1 : BN;  // gather copies take a box of one row
-  RB_TRY(tmap_2d_bf16(ctx, pbase, stacked, a.k, a.k, kBM, &tp));
-  RB_TRY(tmap_2d_bf16(ctx, (GATED && SWAP) ? p2base : pbase, stacked, a.k, a.k, kBM, &tp2));
-  RB_TRY(tmap_2d_bf16(ctx, qbase, p.q_rows, a.k, a.k, q_box, &tq));
-  RB_TRY(tmap_2d_bf16(ctx, (GATED && !SWAP) ? q2base : qbase, p.q_rows, a.k, a.k, q_box, &tq2));
+  const int64_t stack = GROUP != 0 ? p.experts : 1;  // weight matrices one below the other
+  const int64_t p_all = p.p_rows * (SWAP ? stack : 1), q_all = p.q_rows * (SWAP ? 1 : stack);
+  constexpr int q_box = GROUP != 0 && SWAP ? 1 : BN;  // gather copies take a box of one row
+  RB_TRY(tmap_2d_bf16(ctx, pbase, p_all, a.k, a.k, kBM, &tp));
+  RB_TRY(tmap_2d_bf16(ctx, (GATED && SWAP) ? p2base : pbase, p_all, a.k, a.k, kBM, &tp2));
+  RB_TRY(tmap_2d_bf16(ctx, qbase, q_all, a.k, a.k, q_box, &tq));
+  RB_TRY(tmap_2d_bf16(ctx, (GATED && !SWAP) ? q2base : qbase, q_all, a.k, a.k, q_box, &tq2));
   p.n_p = (p.p_rows + kBM - 1) / kBM;
   p.n_q = (p.q_rows + BN - 1) / BN;
   auto kern = gemm_tc_kernel<BN, SWAP, GATED, GROUP>;
@@ -779,11 +751,9 @@ int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
   // Ring depth: as deep as the shared-memory budget allows (decode-sized launches are bound by the bytes they
   // keep in flight; a shallower ring measured slower even where it lets two kernels share an SM).
   int stages = C::kStages;
-  if (GROUP != 0) {
-    // at most this many row tiles: each expert ends in a partial one
-    const int64_t pairs = (int64_t)p.m;
-    p.n_q = (int)(pairs / BN + std::min<int64_t>(p.experts, pairs));
-  }
+  int64_t items = (int64_t)p.n_p * p.n_q * p.n_split;
+  if (GROUP != 0)  // at most: each expert ends in a partial row tile
+    items = (p.m / (SWAP ? BN : kBM) + std::min<int64_t>(p.experts, p.m)) * (SWAP ? p.n_p : p.n_q);
   if (SWAP) stages = std::max(2, std::min(C::kStages, (int)(ctx->gemm_ring_bytes / C::kStageBytes)));
   p.stages = stages;
   const size_t smem = (size_t)stages * C::kStageBytes + 1024;
@@ -811,8 +781,8 @@ int launch(rb_ctx* ctx, const GemmArgs& a, Params& p, int want_split = 0) {
     ctx->launches++;
     return RB_OK;
   }
-  p.n_items = p.n_p * p.n_q * p.n_split;
-  const int grid = std::min(p.n_items, ctx->sm_count);
+  p.n_items = (int)items;
+  const int grid = (int)std::min<int64_t>(items, ctx->sm_count);
   RB_CUDA(launch_kernel(kern, dim3((unsigned)grid), dim3(kThreads), smem, ctx->stream, ctx->pdl, tp, tp2, tq, tq2, p));
   ctx->launches++;
   return RB_OK;
@@ -928,7 +898,8 @@ int gemm_tc_bf16(rb_ctx* ctx, const GemmArgs& a) {
   return launch<256, false, false>(ctx, a, p);
 }
 
-// The grouped form: a.m is the number of (row, choice) pairs, a.x has a.m / a.top rows (gated) or a.m compact rows.
+// The grouped form: a.m is the number of (row, choice) pairs.  a.x has a.m / a.top rows (gated), or a.m compact rows (down,
+// or gated with a.sorted).
 int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a) {
   if (a.m == 0) return RB_OK;
   RB_REQUIRE(a.k > 0 && (a.k % 8) == 0 && a.n > 0 && (a.n % 8) == 0, "grouped GEMM: N = %lld and K = %lld must be multiples of 8",
@@ -937,8 +908,6 @@ int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a) {
   const bool gated = a.w2 != nullptr;
   Params p{};
   p.m = (int)a.m; p.n = (int)a.n; p.k = (int)a.k;
-  p.p_rows = (int)a.n;
-  p.q_rows = (int)(gated ? a.m / a.top : a.m);
   p.num_kb = (int)((a.k + kBK - 1) / kBK);
   p.n_split = 1;
   p.kb_per_split = p.num_kb;
@@ -947,11 +916,20 @@ int gemm_tc_grouped(rb_ctx* ctx, const GemmArgs& a) {
   p.list = a.list; p.count = a.count; p.cap = a.cap; p.experts = a.experts; p.top = a.top;
   p.status = ctx->status_dev;
   const int64_t rows = a.m / a.top;
-  const double mean = (double)a.m / a.experts;  // rows per expert, if they spread evenly
-  p.stream_weights = mean <= 48.0;
+  const int x_rows = (int)(gated && !a.sorted ? rows : a.m);
+  if (grouped_wants_sorted(rows, a.top, a.experts) && (!gated || a.sorted)) {
+    p.p_rows = x_rows;
+    p.q_rows = (int)a.n;
+    return gated ? launch<128, false, true, 1>(ctx, a, p) : launch<256, false, false, 2>(ctx, a, p);
+  }
+  RB_REQUIRE(!gated || !a.sorted, "grouped GEMM: sorted rows are for many rows per expert");
+  p.p_rows = (int)a.n;
+  p.q_rows = x_rows;
   if (rows <= 16) return gated ? launch<16, true, true, 1>(ctx, a, p) : launch<16, true, false, 2>(ctx, a, p);
-  if (mean <= 48.0) return gated ? launch<64, true, true, 1>(ctx, a, p) : launch<64, true, false, 2>(ctx, a, p);
-  return gated ? launch<128, true, true, 1>(ctx, a, p) : launch<256, true, false, 2>(ctx, a, p);
+  return gated ? launch<64, true, true, 1>(ctx, a, p) : launch<64, true, false, 2>(ctx, a, p);
 }
+
+// Enough rows per expert (if they spread evenly) for full tiles, and so for a sorted copy of the rows?
+bool grouped_wants_sorted(int64_t rows, int top, int experts) { return rows * top > (int64_t)48 * experts && rows > 64; }
 
 }  // namespace rb

@@ -134,7 +134,8 @@ int parallel_block(rb_model* m, const MixLayer& w, int batch, int seq, const voi
   }
   RB_TRY(split_and_route(ctx, f, experts ? &r : nullptr, dt));
   if (experts) {
-    RB_TRY(rb_moe_gated(ctx, m->h, w.gate, w.up, m->expert_act, rows, c.top, c.experts, r.list, r.count, r.cap, w.ff_p, m->ld, RB_ACT_SILU, dt));
+    RB_TRY(rb_moe_gated(ctx, m->h, w.gate, w.up, m->expert_act, rows, c.top, c.experts, r.list, r.count, r.cap, w.ff_p, m->ld, RB_ACT_SILU,
+                        m->expert_out, dt));  // (the second product's output is free until then)
     RB_TRY(rb_moe_down(ctx, m->expert_act, w.down, m->expert_out, rows, c.top, c.experts, r.list, r.count, r.cap, m->ld, w.ff_p, dt));
   }
   rb_attention_options o{};

@@ -4,17 +4,18 @@
 #include <algorithm>
 
 #include "ctx.h"
+#include "groups.cuh"
 
 namespace rb {
 
 namespace {
 
 // ------------------------------------------------------------------------------------------
-// Routing: one warp per row.
+// Routing: one warp per row.  A block counts its rows' choices in shared memory and takes its places in the experts' lists
+// with one addition per expert: counters that lie side by side would otherwise serve a prompt's choices one after the other.
 // ------------------------------------------------------------------------------------------
-constexpr int kRouteWarps = 8;       // rows per block
+constexpr int kRouteWarps = 8;
 constexpr int kMaxTop = 32;          // one lane per choice
-constexpr int kPerLane = kMaxExperts / 32;
 
 struct RouteArgs {
   const float* acc;                  // logits: slab s of row r, expert e at acc[s * stride + r * ld + e]
@@ -28,7 +29,10 @@ struct RouteArgs {
   int64_t cap;
 };
 
-__device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* sc) {  // sc: kMaxExperts floats of this warp
+// kPerLane: experts per lane (32 kPerLane of them at most)
+template <int kPerLane>
+// lane j gets the row's j-th choice and its weight; sc: 32 kPerLane floats of this warp
+__device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* sc, int& chosen, float& weight) {
   const int lane = threadIdx.x & 31;
   float s[kPerLane];
 #pragma unroll
@@ -86,8 +90,6 @@ __device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* sc
     }
   }
   // the largest scores, one at a time (positive floats order like their bits); lane j keeps the j-th choice
-  int chosen = -1;
-  float weight = 0.f;
   for (int j = 0; j < a.top; ++j) {
     uint32_t best = 0;
     int at = 0;
@@ -105,15 +107,49 @@ __device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* sc
     }
     if (lane == j) { chosen = (int)e; weight = __uint_as_float(top - 1u); }
   }
-  if (lane < a.top) {
-    a.weight[(size_t)row * a.top + lane] = weight * a.scale;
-    const int at = atomicAdd(a.count + chosen, 1);
-    if (at < a.cap) a.list[(size_t)chosen * a.cap + at] = row * a.top + lane;
+}
+
+template <int kPerLane>
+struct RouteSmem {
+  float scores[kRouteWarps][32 * kPerLane];
+  int have[32 * kPerLane], base[32 * kPerLane];
+};
+// a whole block (kRouteWarps warps): kRows rows per warp from `first` on
+template <int kPerLane, int kRows>
+__device__ __forceinline__ void route_block(const RouteArgs& a, int first, RouteSmem<kPerLane>& sm) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e = threadIdx.x; e < a.experts; e += blockDim.x) sm.have[e] = 0;
+  __syncthreads();
+  int chosen[kRows], place[kRows];
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {
+    const int row = first + i * kRouteWarps + warp;
+    chosen[i] = -1;
+    place[i] = 0;
+    if (row >= a.rows) continue;
+    float weight = 0.f;
+    route_row<kPerLane>(a, row, sm.scores[warp], chosen[i], weight);
+    if (lane < a.top) {
+      a.weight[(size_t)row * a.top + lane] = weight * a.scale;
+      place[i] = atomicAdd(&sm.have[chosen[i]], 1);
+    }
+    __syncwarp();  // the scores are rewritten by the next row
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < a.experts; e += blockDim.x) sm.base[e] = sm.have[e] > 0 ? atomicAdd(a.count + e, sm.have[e]) : 0;
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {
+    const int row = first + i * kRouteWarps + warp;
+    if (row >= a.rows || lane >= a.top) continue;
+    const int at = sm.base[chosen[i]] + place[i];
+    if (at < a.cap) a.list[(size_t)chosen[i] * a.cap + at] = row * a.top + lane;
   }
 }
 
 // ------------------------------------------------------------------------------------------
-// Head split, key append and gated activation, one block per row (or several); then, in the blocks after those, routing.
+// Head split, key append and gated activation: a thread keeps to one 8-column piece of the output (of a query head, a key
+// head or the gated part) and walks rows; then, in the blocks after those, routing.
 // ------------------------------------------------------------------------------------------
 template <typename T>
 struct SplitArgs {
@@ -126,27 +162,45 @@ struct SplitArgs {
   int s_new, q_heads, kv_heads, dim, D, qp, kp, gp;   // padded widths of q, k and of gate (= up)
   T* kc;
   const int32_t *block_table, *seq_lens;
-  int pages_per_seq, max_seq, rows, blocks;
+  int pages_per_seq, max_seq, rows;
+  int pieces, row_groups, blocks;                     // output pieces of a row; rows that are worked on at once; blocks for them
   T *q_out, *glu_out;
   int64_t glu_ld;
   uint32_t* status;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(512) split_route_kernel(const SplitArgs<T> a, const RouteArgs r) {
-  __shared__ float scores[kRouteWarps][kMaxExperts];
+constexpr int kSplitThreads = 256;
+static_assert(kSplitThreads == kRouteWarps * 32, "the blocks of both parts are one launch");
+
+template <typename T, bool kSlabs, int kPerLane>
+__global__ void __launch_bounds__(kSplitThreads) split_route_kernel(const SplitArgs<T> a, const RouteArgs r) {
+  __shared__ RouteSmem<kPerLane> sm;
   pdl_launch_dependents();
   pdl_wait();
   if ((int)blockIdx.x >= a.blocks) {
-    const int warp = threadIdx.x >> 5;
-    const int row = ((int)blockIdx.x - a.blocks) * kRouteWarps + warp;
-    if (warp < kRouteWarps && row < r.rows) route_row(r, row, scores[warp]);
+    route_block<kPerLane, 1>(r, ((int)blockIdx.x - a.blocks) * kRouteWarps, sm);
     return;
   }
-  auto load_u = [&](size_t m, int c, float* u) {
+  const int id = (int)blockIdx.x * kSplitThreads + (int)threadIdx.x;
+  if (id >= a.row_groups * a.pieces) return;
+  const int piece = id % a.pieces;
+  // what this piece is
+  const int dq = a.D / 8, n_q = a.q_heads * dq, n_k = a.kv_heads * dq;
+  const bool is_q = piece < n_q, is_k = !is_q && piece < n_q + n_k;
+  const int j = is_q ? piece : is_k ? piece - n_q : piece - n_q - n_k;
+  const int head = is_q || is_k ? j / dq : 0, i0 = is_q || is_k ? (j % dq) * 8 : j * 8;
+  const int col = is_q ? head * a.dim + i0 : is_k ? a.qp + head * a.dim + i0 : a.qp + a.kp + i0;
+  const int live = is_q || is_k ? max(0, min(8, a.dim - i0)) : 8;   // columns of the piece that exist; the rest is zero
+  const bool vec = live == 8 && (col & 7) == 0;
+  auto load_one = [&](size_t m, int c) -> float {   // a head whose size is no multiple of 8
+    if (!kSlabs) return Cvt<T>::to_f(a.src[m * a.ld + c]);
+    float v = 0.f;
+    for (int s = 0; s < a.n_acc; ++s) v += a.acc[(size_t)s * a.acc_stride + m * a.ld + c];
+    return a.bias ? v + Cvt<T>::to_f(a.bias[c]) : v;
+  };
+  auto load_sum = [&](size_t m, int c, float* u) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) u[i] = 0.f;
-    if (a.src) { load8(a.src + m * a.ld + c, u); return; }
     add_slabs<4>(a.acc, a.n_acc, a.acc_stride, m * a.ld + c, u);
     if (a.bias) {
       float t[8];
@@ -155,71 +209,116 @@ __global__ void __launch_bounds__(512) split_route_kernel(const SplitArgs<T> a, 
       for (int i = 0; i < 8; ++i) u[i] += t[i];
     }
   };
-  for (int m = blockIdx.x; m < a.rows; m += a.blocks) {
-    const int b = m / a.s_new, pos = a.seq_lens[b] - a.s_new + m % a.s_new;
-    if (pos < 0 || pos >= a.max_seq) {  // block-uniform
-      if (threadIdx.x == 0) { a.status[0] = (uint32_t)(-RB_ERR_INVALID); a.status[1] = 0x5A11u; a.status[2] = (uint32_t)pos; }
-      continue;
-    }
-    T* q_row = a.q_out + (size_t)m * a.q_heads * a.D;
-    const int page = a.kv_heads > 0 ? a.block_table[(size_t)b * a.pages_per_seq + pos / kPageTokens] : 0;
-    T* k_row = a.kc + ((size_t)page * a.kv_heads * kPageTokens + pos % kPageTokens) * a.D;  // head g: g pages of one head further
-    const size_t k_step = (size_t)kPageTokens * a.D;
-    const int n_glu = a.gp / 8;
-    if ((a.dim & 7) == 0) {
-      const int dq = a.D / 8, n_q = a.q_heads * dq, n_k = a.kv_heads * dq;
-      for (int it = threadIdx.x; it < n_q + n_k; it += blockDim.x) {
-        const int j = it < n_q ? it : it - n_q, h = j / dq, i0 = (j % dq) * 8;
-        float u[8];
+  constexpr int R = kSlabs ? 1 : 4;   // rows in flight
+  constexpr int kWords = sizeof(T) / 2;
+  const int step = a.row_groups;
+  const bool paired = !is_q && !is_k;
+  for (int m0 = id / a.pieces; m0 < a.rows; m0 += R * step) {
+    uint4 x[kSlabs ? 1 : R][kWords], y[kSlabs ? 1 : R][kWords];   // raw pieces of the tensor: every load is issued before the first is used
+    if (!kSlabs && vec) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) u[i] = 0.f;
-        if (i0 < a.dim) load_u(m, (it < n_q ? 0 : a.qp) + h * a.dim + i0, u);
-        store8((it < n_q ? q_row + h * a.D : k_row + h * k_step) + i0, u);
-      }
-    } else {
-      for (int it = threadIdx.x; it < (a.qp + a.kp) / 8; it += blockDim.x) {
-        float u[8];
-        load_u(m, it * 8, u);
+      for (int t = 0; t < R; ++t) {
+        const T* p = a.src + (size_t)min(m0 + t * step, a.rows - 1) * a.ld + col;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const int c = it * 8 + i;
-          if (c < a.q_heads * a.dim) q_row[c / a.dim * a.D + c % a.dim] = Cvt<T>::from_f(u[i]);
-          const int ck = c - a.qp;
-          if (ck >= 0 && ck < a.kv_heads * a.dim) k_row[ck / a.dim * k_step + ck % a.dim] = Cvt<T>::from_f(u[i]);
+        for (int w = 0; w < kWords; ++w) {
+          x[t][w] = reinterpret_cast<const uint4*>(p)[w];
+          if (paired) y[t][w] = reinterpret_cast<const uint4*>(p + a.gp)[w];
         }
       }
-      const int pad = a.D - a.dim;
-      for (int it = threadIdx.x; it < (a.q_heads + a.kv_heads) * pad; it += blockDim.x) {
-        const int h = it / pad, i = a.dim + it % pad;
-        (h < a.q_heads ? q_row + h * a.D : k_row + (h - a.q_heads) * k_step)[i] = Cvt<T>::from_f(0.f);
-      }
     }
-    for (int it = threadIdx.x; it < n_glu; it += blockDim.x) {
-      float g[8], u[8];
-      load_u(m, a.qp + a.kp + it * 8, g);
-      load_u(m, a.qp + a.kp + a.gp + it * 8, u);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) g[i] = act_apply(RB_ACT_SILU, g[i]) * u[i];
-      store8(a.glu_out + (size_t)m * a.glu_ld + it * 8, g);
+    for (int t = 0; t < R; ++t) {
+      const int m = m0 + t * step;
+      if (m >= a.rows) break;
+      float u[8], g[8];
+      if (kSlabs && vec) {
+        load_sum(m, col, u);
+        if (paired) load_sum(m, col + a.gp, g);
+      } else if (vec) {
+        load8(reinterpret_cast<const T*>(x[t]), u);
+        if (paired) load8(reinterpret_cast<const T*>(y[t]), g);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] = i < live ? load_one(m, col + i) : 0.f;
+      }
+      if (is_q) {
+        store8(a.q_out + ((size_t)m * a.q_heads + head) * a.D + i0, u);
+      } else if (is_k) {
+        const int b = m / a.s_new, pos = a.seq_lens[b] - a.s_new + (m - b * a.s_new);
+        if (pos < 0 || pos >= a.max_seq) {
+          a.status[0] = (uint32_t)(-RB_ERR_INVALID); a.status[1] = 0x5A11u; a.status[2] = (uint32_t)pos;
+          continue;
+        }
+        const int page = a.block_table[(size_t)b * a.pages_per_seq + pos / kPageTokens];
+        store8(a.kc + (((size_t)page * a.kv_heads + head) * kPageTokens + pos % kPageTokens) * a.D + i0, u);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] = act_apply(RB_ACT_SILU, u[i]) * g[i];
+        store8(a.glu_out + (size_t)m * a.glu_ld + i0, u);
+      }
     }
   }
 }
 
-template <typename T>
-int split_route_run(rb_ctx* ctx, SplitArgs<T> a, const RouteArgs& r) {
-  // enough blocks to fill the GPU several times over; a prompt's rows share them
-  a.blocks = a.rows > 0 ? (int)std::min<int64_t>(a.rows, (int64_t)ctx->sm_count * 32) : 0;
-  const int pieces = a.rows > 0 ? (a.q_heads + a.kv_heads) * a.D / 8 : 0;
-  int threads = std::min(512, std::max(64, (pieces + 31) / 32 * 32));
-  int route_blocks = 0;
-  if (r.rows > 0) {
-    threads = std::max(threads, kRouteWarps * 32);
-    route_blocks = (r.rows + kRouteWarps - 1) / kRouteWarps;
-  }
-  if (a.blocks + route_blocks == 0) return RB_OK;
-  RB_CUDA(launch_kernel(split_route_kernel<T>, dim3((unsigned)(a.blocks + route_blocks)), dim3(threads), 0, ctx->stream, ctx->pdl, a, r));
+constexpr int kRouteRows = 4;  // rows per warp of a prompt's routing
+template <int kPerLane>
+__global__ void __launch_bounds__(kRouteWarps * 32) route_kernel(const RouteArgs r) {
+  __shared__ RouteSmem<kPerLane> sm;
+  pdl_launch_dependents();
+  pdl_wait();
+  route_block<kPerLane, kRouteRows>(r, (int)blockIdx.x * kRouteWarps * kRouteRows, sm);
+}
+
+int route_run(rb_ctx* ctx, const RouteArgs& r) {
+  if (r.rows == 0) return RB_OK;
+  const auto kern = r.experts <= 64 ? route_kernel<2> : route_kernel<kMaxExperts / 32>;
+  RB_CUDA(launch_kernel(kern, dim3((unsigned)((r.rows + kRouteWarps * kRouteRows - 1) / (kRouteWarps * kRouteRows))),
+                        dim3(kRouteWarps * 32), 0, ctx->stream, ctx->pdl, r));
   ctx->launches++;
   return RB_OK;
+}
+
+// Both in one launch at single-token steps, where each is latency; a prompt's routing wants more warps than the split leaves room for.
+template <typename T>
+int split_route_run(rb_ctx* ctx, SplitArgs<T> a, RouteArgs r) {
+  const bool together = a.acc != nullptr;
+  const RouteArgs apart = r;
+  if (!together) r.rows = 0;
+  a.pieces = (a.q_heads + a.kv_heads) * a.D / 8 + a.gp / 8;
+  // enough threads to fill the GPU several times over; a prompt's rows share them
+  a.row_groups = (int)std::min<int64_t>(a.rows, std::max<int64_t>(1, (int64_t)ctx->sm_count * 16 * kSplitThreads / a.pieces));
+  a.blocks = (int)(((int64_t)a.row_groups * a.pieces + kSplitThreads - 1) / kSplitThreads);
+  const int blocks = a.blocks + (r.rows + kRouteWarps - 1) / kRouteWarps;
+  const auto kern = !together ? split_route_kernel<T, false, 2> : r.experts <= 64 ? split_route_kernel<T, true, 2>
+                                                                                 : split_route_kernel<T, true, kMaxExperts / 32>;
+  RB_CUDA(launch_kernel(kern, dim3((unsigned)blocks), dim3(kSplitThreads), 0, ctx->stream, ctx->pdl, a, r));
+  ctx->launches++;
+  return together ? RB_OK : route_run(ctx, apart);
+}
+
+// dst[i, :] = src[list[i] / top, :] in the order of the lists, expert after expert; one warp per row
+__global__ void __launch_bounds__(256) sort_rows_kernel(const uint4* __restrict__ src, const int32_t* __restrict__ list,
+                                                        const int32_t* __restrict__ count, int64_t cap, int experts, int top, int pieces,
+                                                        uint4* __restrict__ dst) {
+  __shared__ Groups g;
+  pdl_launch_dependents();
+  pdl_wait();
+  make_groups(g, count, experts, 1, 0);
+  const int total = g.row[experts], lane = threadIdx.x & 31;
+  for (int i = (int)blockIdx.x * 8 + (threadIdx.x >> 5); i < total; i += (int)gridDim.x * 8) {
+    const int e = group_of(g.row, experts, i);
+    const uint4* s = src + (size_t)(list[(size_t)e * cap + i - g.row[e]] / top) * pieces;
+    uint4* d = dst + (size_t)i * pieces;
+    for (int p = lane; p < pieces; p += 128) {
+      uint4 v[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (p + 32 * k < pieces) v[k] = __ldg(s + p + 32 * k);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (p + 32 * k < pieces) d[p + 32 * k] = v[k];
+    }
+  }
 }
 
 int route_check(const RouteArgs& r) {
@@ -317,14 +416,22 @@ int moe_plain(rb_ctx* ctx, const GemmArgs& a) {
   return launch_status("moe_plain");
 }
 
-int moe_product(rb_ctx* ctx, const GemmArgs& a, int dtype) {
+int moe_product(rb_ctx* ctx, GemmArgs a, void* sorted, int dtype) {
   if (a.m == 0) return RB_OK;
   // experts that some row is expected to choose, if the choices spread evenly
   double untouched = 1.0;
   for (int64_t r = 0; r < a.m / a.top && untouched > 1e-9; ++r) untouched *= 1.0 - (double)a.top / a.experts;
   const double es = (double)dtype_size(dtype), mats = a.w2 ? 2.0 : 1.0;
-  const double in_rows = a.w2 ? (double)a.m / a.top : (double)a.m;
-  ProfScope prof(ctx, RB_PROF_EXPERTS, es * (mats * (1.0 - untouched) * a.experts * a.n * a.k + in_rows * a.k + (double)a.m * a.n),
+  if (dtype == RB_BF16 && !ctx->debug_simple_gemm && sorted && grouped_wants_sorted(a.m / a.top, a.top, a.experts)) {
+    ProfScope prof(ctx, RB_PROF_OTHER, 2.0 * a.k * ((double)a.m / a.top + a.m), 0.0);
+    const int64_t blocks = std::min<int64_t>((a.m + 7) / 8, (int64_t)ctx->sm_count * 8);
+    RB_CUDA(launch_kernel(sort_rows_kernel, dim3((unsigned)blocks), dim3(256), 0, ctx->stream, ctx->pdl, (const uint4*)a.x, a.list, a.count,
+                          a.cap, a.experts, a.top, (int)(a.k / 8), (uint4*)sorted));
+    ctx->launches++;
+    a.x = sorted;
+    a.sorted = true;
+  }
+  ProfScope prof(ctx, RB_PROF_EXPERTS, es * (mats * (1.0 - untouched) * a.experts * a.n * a.k + (a.w2 && !a.sorted ? (double)a.m / a.top : (double)a.m) * a.k + (double)a.m * a.n),
                  2.0 * mats * a.m * a.n * a.k);
   if (dtype == RB_BF16 && !ctx->debug_simple_gemm) return gemm_tc_grouped(ctx, a);
   if (dtype == RB_BF16) return moe_plain<__nv_bfloat16>(ctx, a);
@@ -402,7 +509,7 @@ extern "C" int32_t rb_moe_route(rb_ctx* ctx, const float* acc, int32_t n_acc, in
   r.groups = groups; r.keep = keep; r.scale = scale; r.weight = weight; r.list = list; r.count = count; r.cap = cap;
   RB_TRY(route_check(r));
   ProfScope prof(ctx, RB_PROF_OTHER, 4.0 * rows * (n_acc * (double)experts + 2.0 * top), 0.0);
-  return split_route_run<float>(ctx, SplitArgs<float>{}, r);
+  return route_run(ctx, r);
 }
 
 static int moe_args(GemmArgs& a, const void* x, const void* w, const void* w2, void* out, int64_t rows, int32_t top, int32_t experts,
@@ -419,12 +526,12 @@ static int moe_args(GemmArgs& a, const void* x, const void* w, const void* w2, v
 
 extern "C" int32_t rb_moe_gated(rb_ctx* ctx, const void* x, const void* wg, const void* wu, void* out, int64_t rows, int32_t top,
                                 int32_t experts, const int32_t* list, const int32_t* count, int64_t cap, int64_t n, int64_t k,
-                                int32_t act, int32_t dtype) {
-  RB_REQUIRE(ctx && wu, "rb_moe_gated: null argument");
+                                int32_t act, void* sorted, int32_t dtype) {
+  RB_REQUIRE(ctx && wu && aligned16(sorted), "rb_moe_gated: null argument");
   RB_REQUIRE(act != RB_ACT_XIELU, "rb_moe_gated: the activation needs parameters");
   GemmArgs a;
   RB_TRY(moe_args(a, x, wg, wu, out, rows, top, experts, list, count, cap, n, k, act));
-  return moe_product(ctx, a, dtype);
+  return moe_product(ctx, a, sorted, dtype);
 }
 
 extern "C" int32_t rb_moe_down(rb_ctx* ctx, const void* x, const void* wd, void* out, int64_t rows, int32_t top, int32_t experts,
@@ -432,5 +539,5 @@ extern "C" int32_t rb_moe_down(rb_ctx* ctx, const void* x, const void* wd, void*
   RB_REQUIRE(ctx, "rb_moe_down: null argument");
   GemmArgs a;
   RB_TRY(moe_args(a, x, wd, nullptr, out, rows, top, experts, list, count, cap, n, k, RB_ACT_NONE));
-  return moe_product(ctx, a, dtype);
+  return moe_product(ctx, a, nullptr, dtype);
 }

@@ -193,7 +193,8 @@ def routed(rng, rows, E, top, hot=None):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("rows,E,top,W,F", [(1, 4, 2, 72, 40), (9, 12, 3, 136, 200), (40, 6, 2, 256, 136), (150, 200, 3, 64, 72),
                                             (300, 5, 2, 320, 264), (700, 7, 3, 144, 128)])
-def test_expert_products(cuda, dtype, rows, E, top, W, F):
+@pytest.mark.parametrize("with_sorted_copy", [False, True])
+def test_expert_products(cuda, dtype, with_sorted_copy, rows, E, top, W, F):
     """Experts with no row, with one, and with more rows than a tile; sizes that are no multiple of any tile."""
     rng = np.random.default_rng(rows)
     pick, lists, count = routed(rng, rows, E, top, hot=1)
@@ -201,7 +202,9 @@ def test_expert_products(cuda, dtype, rows, E, top, W, F):
     wd = rounded(rng.standard_normal((E, W, F)) * F ** -0.5, dtype)
     xd, gd, ud, dd, ld, cd = dev(x, dtype), dev(wg, dtype), dev(wu, dtype), dev(wd, dtype), torch.from_numpy(lists).cuda(), torch.from_numpy(count).cuda()
     act, out = zeros((rows * top, F), dtype), zeros((rows * top, W), dtype)
-    _lib.call("rb_moe_gated", cuda.ctx, ptr(xd), ptr(gd), ptr(ud), ptr(act), rows, top, E, ptr(ld), ptr(cd), rows, F, W, _lib.ACT_SILU, dtype)
+    space = zeros((rows * top, W), dtype) if with_sorted_copy else None
+    _lib.call("rb_moe_gated", cuda.ctx, ptr(xd), ptr(gd), ptr(ud), ptr(act), rows, top, E, ptr(ld), ptr(cd), rows, F, W, _lib.ACT_SILU,
+              ptr(space), dtype)
     _lib.call("rb_moe_down", cuda.ctx, ptr(act), ptr(dd), ptr(out), rows, top, E, ptr(ld), ptr(cd), rows, W, F, dtype)
     cuda.synchronize()
     inner = ref.silu(np.einsum("rw,rjfw->rjf", x, wg[pick])) * np.einsum("rw,rjfw->rjf", x, wu[pick])

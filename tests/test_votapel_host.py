@@ -125,3 +125,5 @@ def test_benchmark_compares_models_of_equal_size():
         assert abs(ours - theirs) < 0.03 * ours
         assert other["num_hidden_layers"] == len(cfg["layers"]) and other["hidden_size"] == cfg["hidden_size"]
         assert configs.head_dim(other) == 128
+        lean, active, theirs = bench.equal_size_qwen2(cfg, active=True)
+        assert abs(active - theirs) < 0.03 * active and active < 0.5 * ours and lean["intermediate_size"] < other["intermediate_size"]
