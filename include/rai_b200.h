@@ -162,7 +162,8 @@ int32_t rb_gated_linear(rb_ctx* ctx, const void* x_dev, const void* wg_dev, cons
 
 /* Split-K form of rb_linear for skinny M (decode): writes `n_split` float32 partial products
  * part[s][m][n]; the consumer (rb_norm / rb_rope_kv_append) sums them in a fixed order, so results
- * are deterministic.  bf16 only.  Needs n_split * m * n * 4 bytes at part_dev (scratch memory). */
+ * are deterministic.  bf16 only.  Needs n_split * m * n * 4 bytes at part_dev (scratch memory).  With one slab M is
+ * not limited: a float32 product of bf16 operands. */
 int32_t rb_linear_partials(rb_ctx* ctx, const void* x_dev, const void* w_dev, float* part_dev, int64_t m, int64_t n,
                            int64_t k, int32_t n_split);
 /* The split count the library would pick for this shape on this GPU (>= 1). */

@@ -19,6 +19,8 @@
 // The score MMA of tile j+1 is issued before the P.V MMA of tile j, so the tensor pipe computes the next scores while
 // the softmax warps work on the current ones; two CTAs fit per SM (112 KB of shared memory, 256 TMEM columns
 // each), which overlaps one CTA's softmax with the other's MMAs.
+// Where the values are the keys (EXT == 2) a tile is loaded once, serves both products from a ring of four, and is released
+// after P.V.
 //
 // Every wait is bounded; a give-up is recorded in the context's status word, in-flight copies are drained, the TMEM
 // allocation is freed and the CTA returns without writing output.
