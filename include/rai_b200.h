@@ -58,20 +58,23 @@ enum {
 
 /* ---- decoder families, rai-models/src/llm/{qwen2,phi2,phi3,gemma}.rs ---- */
 enum { RB_ARCH_QWEN2 = 0, RB_ARCH_PHI2 = 1, RB_ARCH_PHI3 = 2, RB_ARCH_GEMMA = 3,
-       RB_ARCH_MALASUN = 4, RB_ARCH_VOTAPEL = 5, RB_ARCH_KUFULIX = 6 /* described layer by layer (rb_model_create_layers);
-                                                                        no counterpart in the reference */ };
+       RB_ARCH_MALASUN = 4, RB_ARCH_VOTAPEL = 5, RB_ARCH_KUFULIX = 6,
+       RB_ARCH_FIZADRA = 7 /* these four are described layer by layer (rb_model_create_layers); no counterpart in the reference */ };
 
 /* ---- sequence mixers of a layer-by-layer design (rb_layer_config) ---- */
 enum { RB_MIXER_ATTENTION = 0, RB_MIXER_HGRN2 = 1,
-       RB_MIXER_ATTENTION_SSD = 2 /* attention beside a Mamba-2 recurrence (rb_ssd) on the same input */ };
+       RB_MIXER_ATTENTION_SSD = 2, /* attention beside a Mamba-2 recurrence (rb_ssd) on the same input */
+       RB_MIXER_LATENT = 3 /* attention over a cached latent of all heads' keys and values (rb_latent_append) */ };
 /* ---- its feed-forwards, and how a layer joins its sublayers to the residual stream ---- */
 enum { RB_MLP_DENSE = 0,    /* one up projection with RB_ACT_XIELU */
        RB_MLP_EXPERTS = 1,  /* routed gated experts (see rb_moe_route) plus an optional shared one */
-       RB_MLP_EXPERTS_RELU2 = 2 /* routed experts of two products with RB_ACT_RELU2 between them; softmax scores, a
-                                   correction of the choice, renormalised weights, identity experts (rb_moe_route_general) */ };
+       RB_MLP_EXPERTS_RELU2 = 2, /* routed experts of two products with RB_ACT_RELU2 between them; softmax scores, a
+                                   correction of the choice, renormalised weights, identity experts (rb_moe_route_general) */
+       RB_MLP_DENSE_RELU2 = 3 /* one up projection with RB_ACT_RELU2 */ };
 enum { RB_BLOCK_POST_NORM = 0,  /* x += norm(sublayer(x)), sublayer by sublayer */
        RB_BLOCK_PARALLEL = 1,   /* h = norm(x); x += residual_mult (mixer(h) + feed_forward(h)) */
-       RB_BLOCK_PRE_NORM = 2    /* x += sublayer(norm(x)), sublayer by sublayer */ };
+       RB_BLOCK_PRE_NORM = 2,   /* x += sublayer(norm(x)), sublayer by sublayer */
+       RB_BLOCK_SANDWICH = 3    /* x += norm(sublayer(norm(x))), sublayer by sublayer; then the depth average of rb_sandwich_join */ };
 
 /* ---- elementwise / reduce op tags of the primitive set (rai-core/src/dispatch.rs:41-157) ---- */
 enum {
@@ -312,6 +315,8 @@ typedef struct rb_attention_options {
   int32_t head_gate;               /* gate has one number per head: out[row, h, :] *= sigmoid(gate[row, h]) */
   float out_scale;                 /* factor on the output, after the gate; 0 = 1 */
   int32_t reserved0;
+  const void* talk;                /* [q_heads][q_heads], model dtype: score[h] <- sum over g of talk[h][g] * score[g], after scale and
+                                      before mask and softmax; goes with window, chunk, sink and value_dim only */
 } rb_attention_options;
 int32_t rb_attention_general(rb_ctx* ctx, const void* q_dev, rb_kv_cache* cache, int32_t layer, int32_t batch, int32_t s_new,
                              int32_t q_heads, float scale, const rb_attention_options* options, void* out_dev, int32_t dtype);
@@ -390,6 +395,61 @@ int32_t rb_soft_cap(rb_ctx* ctx, float* x_dev, int64_t n, float cap);
  * them (1 - s) f_i / factor + s f_i with s = (t - low) / (high - low). */
 int32_t rb_rotary_tables(rb_ctx* ctx, int32_t dims, int32_t max_pos, double base, double factor, double low, double high,
                          double original, float* cos_dev, float* sin_dev);
+/* The same tables for YaRN: with index(t) = dims ln(original / (2 pi t)) / (2 ln base), pair i has f_i below
+ * max(floor(index(fast)), 0), f_i / factor from min(ceil(index(slow)), dims - 1) on and a linear passage between, and every entry
+ * is multiplied by 0.1 ln(factor) + 1. */
+int32_t rb_rotary_tables_yarn(rb_ctx* ctx, int32_t dims, int32_t max_pos, double base, double factor, double fast, double slow,
+                              double original, float* cos_dev, float* sin_dev);
+/* A joint of a block with a norm on both sides of its sublayers.  rms_g(x) divides each of `groups` equal parts of a row by its own
+ * root mean square.  With y = y_dev + sum_s acc[s] (both NULL: no y),
+ *   x = h_in + rms_g(y) * post_gain;   with depth weights: history[n_depth - 1] = x, x = sum over j < n_depth of depth[j] history[j];
+ *   h_out = x (NULL: not stored);   out = rms_g(x) * gain   in the model dtype (NULL: no norm).
+ * The stream and its history (slices of history_stride floats, rows of pitch ld) are float32; h_out may be h_in. */
+int32_t rb_sandwich_join(rb_ctx* ctx, const void* y_dev, const float* acc_dev, int32_t n_acc, const void* post_gain_dev,
+                         int32_t groups, float eps, int64_t rows, int64_t width, int64_t ld, const float* h_in_dev, float* h_out_dev,
+                         const void* depth_dev, int32_t n_depth, float* history_dev, int64_t history_stride, const void* gain_dev,
+                         void* out_dev, int32_t dtype);
+/* rb_scalar_norm_rows with a gain per channel and rms_g as above. */
+int32_t rb_group_norm_rows(rb_ctx* ctx, const float* h_dev, const int32_t* rows_dev, int64_t row_step, const void* gain_dev,
+                           int32_t groups, float eps, int64_t n_rows, int64_t width, int64_t ld, void* out_dev, int32_t dtype);
+/* Latent attention: what a token leaves in the cache is one vector for all heads, its normed latent of kv_rank numbers and, behind
+ * it, a key part of rot_dim numbers that turns with the position; head h has the key [Uk_h latent | turned part] and the value
+ * Uv_h latent.  The cache holds keys that are also the values (one head, head_dim >= kv_rank + rot_dim, the rest zero).
+ *
+ * rb_latent_append takes one fused projection u = src + sum_s acc[s] (acc needs s_new == 1) with columns
+ * [query latent: q_rank | latent: kv_rank, key part: rot_dim | gate], each of the three padded to a multiple of 8:
+ *   q_latent_out = rms(query latent) * q_weight, pitch q_rank padded to 8;   cache <- [rms(latent) * kv_weight | turned key part]
+ * kv_rank == 0: the columns are [query latent | gate] (a layer that reads another layer's latent).  latent_out (may be NULL): the
+ * same latent once more, pitch kv_rank padded to 8.  gate_out (may be NULL): the first gate_size gate columns, pitch padded to 8.
+ * rot_dims of the key part's numbers turn, neighbours paired (interleaved) or the two halves. */
+int32_t rb_latent_append(rb_ctx* ctx, const void* src_dev, const float* acc_dev, int32_t n_acc, int64_t src_ld, int32_t q_rank,
+                         int32_t kv_rank, int32_t rot_dim, const void* q_weight_dev, const void* kv_weight_dev, float eps,
+                         const float* cos_dev, const float* sin_dev, int32_t rot_dims, int32_t interleaved, int32_t batch, int32_t s_new,
+                         rb_kv_cache* cache, int32_t layer, void* q_latent_out_dev, void* latent_out_dev, void* gate_out_dev,
+                         int32_t gate_size, int32_t dtype);
+/* The latents of the last s_new tokens of each sequence out of the cache, pitch kv_rank padded to 8. */
+int32_t rb_latent_gather(rb_ctx* ctx, rb_kv_cache* cache, int32_t layer, int32_t kv_rank, int32_t batch, int32_t s_new, void* out_dev,
+                         int32_t dtype);
+/* Queries in the latent's space: u = src + sum_s acc[s] has columns [head][dim | rot_dim]; with uk [heads * dim][kv_rank padded
+ * to 8],   out[row, h, :] = [uk_h^T u_dim | turned u_rot | zeros], head pitch the cache's head_dim.  rb_attention_general over
+ * the cache, with value_dim = kv_rank padded to 8, then gives each head's weighted latent. */
+int32_t rb_latent_query(rb_ctx* ctx, const void* src_dev, const float* acc_dev, int32_t n_acc, int64_t src_ld, const void* uk_dev,
+                        int32_t heads, int32_t dim, int32_t rot_dim, int32_t kv_rank, const float* cos_dev, const float* sin_dev,
+                        int32_t rot_dims, int32_t interleaved, int32_t batch, int32_t s_new, rb_kv_cache* cache, void* out_dev,
+                        int32_t dtype);
+/* Back out of it: out[row, h * value_dim + e] = (uv_h x[row, h, :])[e] * sigmoid(gate), x with head pitch kv_rank padded to 8, uv
+ * [heads * value_dim][kv_rank padded to 8]; gate as in rb_attention_options (NULL: none). */
+int32_t rb_latent_output(rb_ctx* ctx, const void* x_dev, const void* uv_dev, int32_t heads, int32_t kv_rank, int32_t value_dim,
+                         const void* gate_dev, int64_t gate_ld, int32_t head_gate, int64_t rows, void* out_dev, int64_t out_ld,
+                         int32_t dtype);
+/* Prompts from their first token multiply the latents out instead: q has columns [head][dim | rot_dim], kv the columns
+ * [head][dim] keys and, from column v_col on, [head][value_dim] values.  Queries (turned) go to q_out [rows, heads, head_dim of
+ * prompt_kv], keys [dim | the cache's turned part] and values to prompt_kv, each padded with zeros: a cache of `heads` key/value
+ * heads for the tokens of this call. */
+int32_t rb_latent_heads(rb_ctx* ctx, const void* q_dev, int64_t q_ld, const void* kv_dev, int64_t kv_ld, int32_t v_col, int32_t heads,
+                        int32_t dim, int32_t rot_dim, int32_t value_dim, int32_t kv_rank, const float* cos_dev, const float* sin_dev,
+                        int32_t rot_dims, int32_t interleaved, int32_t batch, int32_t s_new, rb_kv_cache* cache, int32_t layer,
+                        rb_kv_cache* prompt_kv, void* q_out_dev, int32_t dtype);
 /* Head split, RMS norm of each query and key head, rotary positions and cache append, for one fused projection
  * u = src + sum_s acc[s] + bias (acc needs s_new == 1, and bias counts only with acc: a finished tensor has its bias) whose
  * columns [q | k | v | gate ...] start with the three parts, each padded to a multiple of 8.
@@ -550,7 +610,7 @@ typedef struct rb_model_config {
                                       key j is masked for query i when j + sliding_window < i; cached tokens stay
                                       visible and a single-token call has no mask, exactly as the reference builds it.
                                       Honoured for RB_ARCH_QWEN2 (the one family whose mask has the term); 0 = none */
-  int32_t reserved0;               /* keeps the doubles 8-byte aligned; set to 0 */
+  int32_t norm_groups;             /* RB_ARCH_FIZADRA: equal parts of a row that are normed each by itself */
   double rope_theta;
   double norm_eps;
   double logit_softcap;            /* RB_ARCH_KUFULIX: logits <- cap * tanh(logits / cap); 0 = none */
@@ -567,7 +627,7 @@ typedef struct rb_layer_config {
   int32_t value_dim;               /* per-head value size */
   int32_t conv_taps;               /* attention: taps of the short convolution on q, k and v */
   int32_t window;                  /* attention: how many keys, its own included, a token sees; 0 = all of them */
-  int32_t kv_from;                 /* attention: the earlier layer whose keys and values this one reads; -1 = its own */
+  int32_t kv_from;                 /* attention: the earlier layer whose keys and values (or latent) this one reads; -1 = its own */
   int32_t mlp_size;                /* feed-forward: inner size (of one expert, with RB_MLP_EXPERTS); 0 = the layer has none */
   int32_t block;                   /* RB_BLOCK_* */
   int32_t mlp_kind;                /* RB_MLP_* */
@@ -581,7 +641,8 @@ typedef struct rb_layer_config {
                                       that layer's; cache and state are its own); -1 = its own */
   int32_t chunk;                   /* RB_BLOCK_PRE_NORM attention: see rb_attention_options */
   int32_t qk_norm;                 /* RB_BLOCK_PRE_NORM attention: RMS norm of each query and key head */
-  int32_t head_gate;               /* RB_BLOCK_PRE_NORM attention: one output gate per head */
+  int32_t head_gate;               /* RB_BLOCK_PRE_NORM attention, RB_MIXER_LATENT: one output gate per head (a latent mixer without
+                                      it has one per output element) */
   int32_t rot_dims;                /* rotary positions on that many dimensions of a head (even; 0 = none), see rb_rotary_tables */
   int32_t rot_original;            /* 0 = frequencies as they are */
   int32_t ssd_heads;               /* RB_MIXER_ATTENTION_SSD: see rb_ssd (conv_taps are its taps) */
@@ -590,6 +651,14 @@ typedef struct rb_layer_config {
   int32_t ssd_groups;
   int32_t ssd_norm_groups;         /* see rb_gated_group_norm */
   int32_t identity;                /* RB_MLP_EXPERTS_RELU2: identity experts beside the `experts` */
+  int32_t talk;                    /* RB_BLOCK_SANDWICH attention: the heads' scores are mixed (rb_attention_options.talk) */
+  int32_t softmax_one;             /* RB_BLOCK_SANDWICH attention: one is added to the softmax denominator */
+  int32_t sink;                    /* RB_MIXER_LATENT: a learned sink per head */
+  int32_t rot_interleaved;         /* RB_MIXER_LATENT: neighbours turn together instead of the halves */
+  int32_t rot_yarn;                /* rb_rotary_tables_yarn, rot_high and rot_low being its fast and slow */
+  int32_t rot_dim;                 /* RB_MIXER_LATENT: size of the key part that all heads share (key_dim does not count it) */
+  int32_t q_rank;                  /* RB_MIXER_LATENT: sizes of the query's and the cached latent (kv_from names the earlier layer */
+  int32_t kv_rank;                 /* whose cached latent this one reads) */
   int32_t reserved0;
   double scale;                    /* attention: factor on q.k */
   double temp_coef;
@@ -605,8 +674,9 @@ typedef struct rb_layer_config {
 } rb_layer_config;
 
 /* A model of RB_ARCH_MALASUN (post-norm blocks), RB_ARCH_VOTAPEL (parallel blocks of attention and experts, learned
- * positions) or RB_ARCH_KUFULIX (pre-norm blocks, rotary positions): `layers` has cfg->num_hidden_layers entries.  Of cfg, the
- * fields arch, dtype, vocab_size, hidden_size, num_hidden_layers, norm_eps, max_position_embeddings (learned positions only),
+ * positions), RB_ARCH_KUFULIX (pre-norm blocks, rotary positions) or RB_ARCH_FIZADRA (sandwich blocks of latent and of
+ * head-mixing attention, depth averages): `layers` has cfg->num_hidden_layers entries.  Of cfg, the fields arch, dtype,
+ * vocab_size, hidden_size, num_hidden_layers, norm_eps, norm_groups, max_position_embeddings (learned positions only),
  * logit_softcap and the capacities are read.  The residual stream and the logits are float32 whatever the model dtype; every other rb_model_* entry point works as for the other families.  Single GPU. */
 int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out);
 /* RB_F32 or RB_BF16: the type in which rb_model_forward* return logits (the model dtype for the reference's families). */

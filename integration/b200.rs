@@ -98,6 +98,14 @@ pub struct rb_layer_config {
     pub ssd_groups: i32,
     pub ssd_norm_groups: i32,
     pub identity: i32,
+    pub talk: i32,
+    pub softmax_one: i32,
+    pub sink: i32,
+    pub rot_interleaved: i32,
+    pub rot_yarn: i32,
+    pub rot_dim: i32,
+    pub q_rank: i32,
+    pub kv_rank: i32,
     pub reserved0: i32,
     pub scale: f64,
     pub temp_coef: f64,
@@ -130,6 +138,7 @@ pub struct rb_attention_options {
     pub head_gate: i32,
     pub out_scale: f32,
     pub reserved0: i32,
+    pub talk: *const c_void,
 }
 
 /// `struct rb_route_options` of include/rai_b200.h, field for field.
@@ -166,7 +175,7 @@ pub struct rb_model_config {
     pub tp_rank: i32,
     pub tp_size: i32,
     pub sliding_window: i32,
-    pub reserved0: i32,
+    pub norm_groups: i32,
     pub rope_theta: f64,
     pub norm_eps: f64,
     pub logit_softcap: f64,
@@ -229,6 +238,14 @@ extern "C" {
     pub fn rb_embed_norm_stream(ctx: *mut rb_ctx, table_dev: *const c_void, dtype: i32, vocab: i64, width: i64, ld: i64, ids_dev: *const u32, n_ids: i64, gain_dev: *const c_void, eps: f32, h_dev: *mut f32) -> i32;
     pub fn rb_soft_cap(ctx: *mut rb_ctx, x_dev: *mut f32, n: i64, cap: f32) -> i32;
     pub fn rb_rotary_tables(ctx: *mut rb_ctx, dims: i32, max_pos: i32, base: f64, factor: f64, low: f64, high: f64, original: f64, cos_dev: *mut f32, sin_dev: *mut f32) -> i32;
+    pub fn rb_rotary_tables_yarn(ctx: *mut rb_ctx, dims: i32, max_pos: i32, base: f64, factor: f64, fast: f64, slow: f64, original: f64, cos_dev: *mut f32, sin_dev: *mut f32) -> i32;
+    pub fn rb_sandwich_join(ctx: *mut rb_ctx, y_dev: *const c_void, acc_dev: *const f32, n_acc: i32, post_gain_dev: *const c_void, groups: i32, eps: f32, rows: i64, width: i64, ld: i64, h_in_dev: *const f32, h_out_dev: *mut f32, depth_dev: *const c_void, n_depth: i32, history_dev: *mut f32, history_stride: i64, gain_dev: *const c_void, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_group_norm_rows(ctx: *mut rb_ctx, h_dev: *const f32, rows_dev: *const i32, row_step: i64, gain_dev: *const c_void, groups: i32, eps: f32, n_rows: i64, width: i64, ld: i64, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_latent_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, q_rank: i32, kv_rank: i32, rot_dim: i32, q_weight_dev: *const c_void, kv_weight_dev: *const c_void, eps: f32, cos_dev: *const f32, sin_dev: *const f32, rot_dims: i32, interleaved: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, layer: i32, q_latent_out_dev: *mut c_void, latent_out_dev: *mut c_void, gate_out_dev: *mut c_void, gate_size: i32, dtype: i32) -> i32;
+    pub fn rb_latent_gather(ctx: *mut rb_ctx, cache: *mut rb_kv_cache, layer: i32, kv_rank: i32, batch: i32, s_new: i32, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_latent_query(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, uk_dev: *const c_void, heads: i32, dim: i32, rot_dim: i32, kv_rank: i32, cos_dev: *const f32, sin_dev: *const f32, rot_dims: i32, interleaved: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, out_dev: *mut c_void, dtype: i32) -> i32;
+    pub fn rb_latent_output(ctx: *mut rb_ctx, x_dev: *const c_void, uv_dev: *const c_void, heads: i32, kv_rank: i32, value_dim: i32, gate_dev: *const c_void, gate_ld: i64, head_gate: i32, rows: i64, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
+    pub fn rb_latent_heads(ctx: *mut rb_ctx, q_dev: *const c_void, q_ld: i64, kv_dev: *const c_void, kv_ld: i64, v_col: i32, heads: i32, dim: i32, rot_dim: i32, value_dim: i32, kv_rank: i32, cos_dev: *const f32, sin_dev: *const f32, rot_dims: i32, interleaved: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, layer: i32, prompt_kv: *mut rb_kv_cache, q_out_dev: *mut c_void, dtype: i32) -> i32;
     pub fn rb_head_norm_rope_append(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, bias_dev: *const c_void, src_ld: i64, q_weight_dev: *const c_void, k_weight_dev: *const c_void, eps: f32, cos_dev: *const f32, sin_dev: *const f32, rot_dims: i32, batch: i32, s_new: i32, q_heads: i32, kv_heads: i32, key_dim: i32, value_dim: i32, cache: *mut rb_kv_cache, layer: i32, q_out_dev: *mut c_void, gate_out_dev: *mut c_void, gate_size: i32, dtype: i32) -> i32;
     pub fn rb_ssd(ctx: *mut rb_ctx, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, col: i32, conv_dev: *const c_void, conv_bias_dev: *const c_void, taps: i32, dt_bias_dev: *const c_void, a_log_dev: *const c_void, d_dev: *const c_void, heads: i32, value_dim: i32, state_dim: i32, groups: i32, batch: i32, s_new: i32, cache: *mut rb_kv_cache, new_lens_dev: *const i32, ring_dev: *mut f32, state_dev: *mut f32, chunk: i32, conv_space_dev: *mut c_void, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;
     pub fn rb_gated_group_norm(ctx: *mut rb_ctx, y_dev: *const c_void, y_ld: i64, src_dev: *const c_void, acc_dev: *const f32, n_acc: i32, src_ld: i64, col: i32, weight_dev: *const c_void, groups: i32, eps: f32, scale: f32, rows: i64, width: i64, out_dev: *mut c_void, out_ld: i64, dtype: i32) -> i32;

@@ -22,10 +22,10 @@ RB_OK = 0
 U8, U32, I64, F16, BF16, F32, F64 = range(7)
 ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF, ACT_RELU, ACT_XIELU, ACT_RELU2 = range(7)
 NORM_RMS, NORM_RMS_ONE_PLUS, NORM_LAYER = range(3)
-ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA, ARCH_MALASUN, ARCH_VOTAPEL, ARCH_KUFULIX = range(7)
-MIXER_ATTENTION, MIXER_HGRN2, MIXER_ATTENTION_SSD = range(3)
-MLP_DENSE, MLP_EXPERTS, MLP_EXPERTS_RELU2 = range(3)
-BLOCK_POST_NORM, BLOCK_PARALLEL, BLOCK_PRE_NORM = range(3)
+ARCH_QWEN2, ARCH_PHI2, ARCH_PHI3, ARCH_GEMMA, ARCH_MALASUN, ARCH_VOTAPEL, ARCH_KUFULIX, ARCH_FIZADRA = range(8)
+MIXER_ATTENTION, MIXER_HGRN2, MIXER_ATTENTION_SSD, MIXER_LATENT = range(4)
+MLP_DENSE, MLP_EXPERTS, MLP_EXPERTS_RELU2, MLP_DENSE_RELU2 = range(4)
+BLOCK_POST_NORM, BLOCK_PARALLEL, BLOCK_PRE_NORM, BLOCK_SANDWICH = range(4)
 (UN_NEG, UN_EXP, UN_SQRT, UN_RSQRT, UN_SQUARE, UN_TANH, UN_ERF, UN_SIN, UN_COS, UN_POWF, UN_SILU, UN_GELU_TANH,
  UN_GELU_ERF, UN_RELU, UN_LOG, UN_ABS, UN_RECIP, UN_ADD_SCALAR, UN_MUL_SCALAR, UN_SIGN, UN_LOG2, UN_LOG10) = range(22)
 CMP_EQ, CMP_NE, CMP_GT, CMP_GE, CMP_LT, CMP_LE = range(6)
@@ -47,7 +47,7 @@ class ModelConfig(ctypes.Structure):
     _fields_ = [(n, ctypes.c_int32) for n in (
         "arch", "dtype", "vocab_size", "hidden_size", "intermediate_size", "num_hidden_layers",
         "num_attention_heads", "num_key_value_heads", "max_position_embeddings", "rotary_dim", "hidden_act",
-        "tie_word_embeddings", "max_batch", "max_seq", "max_tokens", "tp_rank", "tp_size", "sliding_window", "reserved0")] + [
+        "tie_word_embeddings", "max_batch", "max_seq", "max_tokens", "tp_rank", "tp_size", "sliding_window", "norm_groups")] + [
         ("rope_theta", ctypes.c_double), ("norm_eps", ctypes.c_double), ("logit_softcap", ctypes.c_double)]
 
 
@@ -57,7 +57,8 @@ class LayerConfig(ctypes.Structure):
         "mixer", "heads", "kv_heads", "key_dim", "value_dim", "conv_taps", "window", "kv_from", "mlp_size",
         "block", "mlp_kind", "experts", "top", "groups", "keep_groups", "shared_size", "temp_every",
         "weights_of", "chunk", "qk_norm", "head_gate", "rot_dims", "rot_original", "ssd_heads", "ssd_value_dim", "ssd_state",
-        "ssd_groups", "ssd_norm_groups", "identity", "reserved0")] + [
+        "ssd_groups", "ssd_norm_groups", "identity", "talk", "softmax_one", "sink", "rot_interleaved", "rot_yarn", "rot_dim", "q_rank",
+        "kv_rank", "reserved0")] + [
         (n, ctypes.c_double) for n in ("scale", "temp_coef", "softcap", "router_scale", "residual_mult", "rot_base", "rot_factor",
                                        "rot_low", "rot_high", "mixer_scale", "ssd_scale")]
 
@@ -67,7 +68,8 @@ class AttentionOptions(ctypes.Structure):
     _fields_ = [("window", ctypes.c_int32), ("alibi", ctypes.c_int32), ("temp_every", ctypes.c_int32),
                 ("temp_coef", ctypes.c_float), ("softcap", ctypes.c_float), ("value_dim", ctypes.c_int32),
                 ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64), ("sink", ctypes.c_void_p), ("out_ld", ctypes.c_int64),
-                ("chunk", ctypes.c_int32), ("head_gate", ctypes.c_int32), ("out_scale", ctypes.c_float), ("reserved0", ctypes.c_int32)]
+                ("chunk", ctypes.c_int32), ("head_gate", ctypes.c_int32), ("out_scale", ctypes.c_float), ("reserved0", ctypes.c_int32),
+                ("talk", ctypes.c_void_p)]
 
 
 class RouteOptions(ctypes.Structure):

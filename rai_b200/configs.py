@@ -1,9 +1,9 @@
 """Decoder configurations.
 
-Malasun, Votapel and Kufulix, designs described layer by layer (no counterpart in the reference), have configurations of
-their own shape: see `malasun_config`, `votapel_config` and `kufulix_config`.  For the others, field names follow the
-reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24, phi3.rs:9-24, gemma.rs:12-27) as they appear in a
-Hugging Face config.json, plus `arch`.
+Malasun, Votapel, Kufulix and Fizadra, designs described layer by layer (no counterpart in the reference), have configurations
+of their own shape: see `malasun_config`, `votapel_config`, `kufulix_config` and `fizadra_config`.  For the others, field names
+follow the reference `Config` structs (rai-models/src/llm/qwen2.rs:8-24, phi2.rs:9-24, phi3.rs:9-24, gemma.rs:12-27) as they
+appear in a Hugging Face config.json, plus `arch`.
 `BASELINE` holds the five benchmark configurations; `TINY` holds small models of the same four
 architectures for parity tests.
 """
@@ -18,9 +18,11 @@ from typing import Dict
 from . import _lib
 
 ARCH_IDS = {"qwen2": _lib.ARCH_QWEN2, "phi2": _lib.ARCH_PHI2, "phi3": _lib.ARCH_PHI3, "gemma": _lib.ARCH_GEMMA,
-            "malasun": _lib.ARCH_MALASUN, "votapel": _lib.ARCH_VOTAPEL, "kufulix": _lib.ARCH_KUFULIX}
-LAYERED = ("malasun", "votapel", "kufulix")   # described layer by layer: rb_model_create_layers
-MIXER_IDS = {"attention": _lib.MIXER_ATTENTION, "hgrn2": _lib.MIXER_HGRN2, "attention_ssd": _lib.MIXER_ATTENTION_SSD}
+            "malasun": _lib.ARCH_MALASUN, "votapel": _lib.ARCH_VOTAPEL, "kufulix": _lib.ARCH_KUFULIX,
+            "fizadra": _lib.ARCH_FIZADRA}
+LAYERED = ("malasun", "votapel", "kufulix", "fizadra")   # described layer by layer: rb_model_create_layers
+MIXER_IDS = {"attention": _lib.MIXER_ATTENTION, "hgrn2": _lib.MIXER_HGRN2, "attention_ssd": _lib.MIXER_ATTENTION_SSD,
+             "latent_attention": _lib.MIXER_LATENT}
 # serde names of rai-nn/src/activations.rs:5-17
 ACT_IDS = {"silu": _lib.ACT_SILU, "gelu_new": _lib.ACT_GELU_TANH, "newgelu": _lib.ACT_GELU_TANH,
            "gelu": _lib.ACT_GELU_ERF, "relu": _lib.ACT_RELU}
@@ -295,7 +297,97 @@ def kufulix_config(raw: dict) -> dict:
     return _kufulix(int(raw["vocab"]), int(raw["width"]), layers, float(raw["norm"]["eps"]), float(raw.get("logit_softcap") or 0.0))
 
 
-_CONFIG_READERS = {"Malasun": malasun_config, "Votapel": votapel_config, "Kufulix": kufulix_config}   # by config.json's `architecture`
+def yarn_rotation(dims: int, base: float, factor: float = 0.0, fast: float = 32.0, slow: float = 1.0, original: int = 0,
+                  interleaved: bool = False) -> dict:
+    """Rotary positions on the first `dims` dimensions, neighbours paired (interleaved) or halves.  original > 0: pairs that turn
+    fewer than about `slow` times over that many positions have their frequency divided by `factor`, those that turn more than
+    about `fast` times keep it, and the turned vectors grow by 0.1 ln(factor) + 1 (YaRN)."""
+    scaling = dict(factor=factor, fast=fast, slow=slow, original=original) if original else None
+    return dict(dims=dims, base=base, scaling=scaling, interleaved=interleaved)
+
+
+def fizadra_attention(heads: int, kv_heads: int, dim: int, vdim: int = 0, rot=None, scale: float = 0.0) -> dict:
+    """Causal attention whose heads' scores are mixed before a softmax with one added to its denominator."""
+    return dict(type="attention", heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim or dim, rot=rot, scale=scale or dim ** -0.5)
+
+
+def fizadra_latent(heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, rot=None, scale: float = 0.0,
+                   sink: bool = False, gate: str = "heads", kv_from=None) -> dict:
+    """Causal attention over a cached latent; gate: one number per output element ("elements") or per head ("heads"); kv_from
+    names the earlier layer whose latent it reads."""
+    return dict(type="latent_attention", heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank,
+                rot=rot or yarn_rotation(rot_dim, 1e4), scale=scale or (dim + rot_dim) ** -0.5, sink=sink, gate=gate, kv_from=kv_from)
+
+
+def fizadra_layer(mixer: dict, ff: int = 0) -> dict:
+    """One entry of a Fizadra configuration's `layers`; ff = 0 leaves the feed-forward out."""
+    return dict(mixer=mixer, mlp=dict(kind="dense", ff=ff) if ff else None)
+
+
+def _fizadra(vocab: int, width: int, layers, groups: int = 1, eps: float = 1e-6) -> dict:
+    return dict(arch="fizadra", vocab_size=vocab, hidden_size=width, norm_eps=eps, norm_groups=groups, layers=layers)
+
+
+def _fizadra_bench(vocab: int, width: int, heads: int, kv_heads: int, kv_rank: int, ff: int, quads: int) -> dict:
+    """Layers in fours: latent attention with sinks, attention with mixed heads, and two of latent attention with a gate per head;
+    the sinks' layer of every second four reads the latent of the one before it."""
+    layers = []
+    for n in range(quads):
+        rot = yarn_rotation(32, 1e4, 8.0, original=4096, interleaved=True)
+        layers.append(fizadra_latent(heads, 96, 32, 128, width // 2, kv_rank, rot, sink=True, gate="elements",
+                                     kv_from=4 * n - 4 if n % 2 else None))
+        layers.append(fizadra_attention(heads, kv_heads, 128, rot=yarn_rotation(128, 5e5)))
+        layers += [fizadra_latent(heads, 96, 32, 128, width // 2, kv_rank, yarn_rotation(32, 5e5))] * 2
+    return _fizadra(vocab, width, [fizadra_layer(m, ff) for m in layers], 4)
+
+
+FIZADRA: Dict[str, dict] = {
+    # sizes that resemble a real model's layers, for throughput measurements (random weights)
+    "fizadra-1k": _fizadra_bench(32000, 1024, 8, 2, 256, 4096, 4),
+    "fizadra-2k": _fizadra_bench(32000, 2048, 16, 4, 512, 8192, 3),
+    "fizadra-4k": _fizadra_bench(32000, 4096, 32, 8, 512, 16384, 2),
+    # a small model for tests
+    "tiny-fizadra": _fizadra(328, 168, [
+        fizadra_layer(fizadra_latent(3, 24, 16, 40, 56, 72, yarn_rotation(16, 700.0, 5.0, 9.0, 0.5, 90, True), 0.19, True, "elements"), 104),
+        fizadra_layer(fizadra_attention(6, 2, 40, 56, yarn_rotation(24, 2e3), 0.21), 96),
+        fizadra_layer(fizadra_latent(5, 32, 8, 24, 48, 40, yarn_rotation(8, 3e3)), 72),
+        fizadra_layer(fizadra_latent(4, 16, 16, 32, 40, 72, yarn_rotation(16, 700.0, 5.0, 9.0, 0.5, 90, True), 0.25, True, "elements", 0)),
+        fizadra_layer(fizadra_attention(4, 4, 24, 24, yarn_rotation(24, 1e4)), 88)], 3, 1e-5),
+}
+
+
+def _fizadra_rotation(rot, interleaved: bool):
+    if not rot:
+        return None
+    s = rot.get("scaling")
+    return yarn_rotation(int(rot["dims"]), float(rot["base"]), *((float(s["factor"]), float(s["fast"]), float(s["slow"]),
+                                                                  int(s["original"])) if s else ()), interleaved=interleaved)
+
+
+def fizadra_config(raw: dict) -> dict:
+    """A Fizadra config.json -> the configuration the library takes."""
+    layers = []
+    for i, entry in enumerate(raw["layers"]):
+        kind, mix, mlp = entry["type"], entry["mixer"], entry.get("mlp")
+        if kind == "attention":
+            mixer = fizadra_attention(int(mix["heads"]), int(mix["kv_heads"]), int(mix["dim"]), int(mix["vdim"]),
+                                      _fizadra_rotation(mix.get("rot"), False), float(mix["scale"]))
+        elif kind in ("latent_attention", "latent_attention_2"):
+            first, src = kind == "latent_attention", mix.get("kv_from")   # the first kind: neighbours turn, sinks, a gate per element
+            mixer = fizadra_latent(int(mix["heads"]), int(mix["dim"]), int(mix["rot_dim"]), int(mix["vdim"]), int(mix["q_rank"]),
+                                   int(mix["kv_rank"]), _fizadra_rotation(mix["rot"], first), float(mix["scale"]), first,
+                                   "elements" if first else "heads", None if src is None else int(src))
+        else:
+            raise _lib.RaiB200Error(-7, f"layer {i}: mixer {kind!r} is not implemented")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise _lib.RaiB200Error(-7, f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented")
+        layers.append(fizadra_layer(mixer, int(mlp["ff"]) if mlp is not None else 0))
+    norm = raw["norm"]
+    return _fizadra(int(raw["vocab"]), int(raw["width"]), layers, int(norm.get("groups") or 1), float(norm["eps"]))
+
+
+# by config.json's `architecture`
+_CONFIG_READERS = {"Malasun": malasun_config, "Votapel": votapel_config, "Kufulix": kufulix_config, "Fizadra": fizadra_config}
 _MODEL_TYPES = {"qwen2": "qwen2", "phi": "phi2", "phi2": "phi2", "phi3": "phi3", "gemma": "gemma"}
 
 
@@ -315,7 +407,7 @@ def from_json(path: str) -> dict:
 
 
 def get(name: str) -> dict:
-    src = BASELINE.get(name) or TINY.get(name) or MALASUN.get(name) or VOTAPEL.get(name) or KUFULIX.get(name)
+    src = BASELINE.get(name) or TINY.get(name) or MALASUN.get(name) or VOTAPEL.get(name) or KUFULIX.get(name) or FIZADRA.get(name)
     if src is None:
         raise KeyError(f"unknown configuration {name!r}")
     return copy.deepcopy(src)
@@ -347,7 +439,21 @@ def layer_structs(cfg: dict):
         s.heads, s.key_dim, s.value_dim = mix["heads"], mix["dim"], mix["vdim"]
         s.kv_from = s.weights_of = -1
         s.mlp_size = mlp["ff"] if mlp else 0
-        if cfg["arch"] == "kufulix":
+        if cfg["arch"] == "fizadra":
+            s.block, s.scale, s.mlp_kind = _lib.BLOCK_SANDWICH, mix["scale"], _lib.MLP_DENSE_RELU2
+            r = mix["rot"]
+            if r:
+                s.rot_dims, s.rot_base, s.rot_interleaved = r["dims"], r["base"], int(r["interleaved"])
+                if r["scaling"]:
+                    r = r["scaling"]
+                    s.rot_yarn, s.rot_original, s.rot_factor, s.rot_low, s.rot_high = 1, r["original"], r["factor"], r["slow"], r["fast"]
+            if mix["type"] == "attention":
+                s.kv_heads, s.qk_norm, s.talk, s.softmax_one = mix["kv_heads"], 1, 1, 1
+            else:
+                s.kv_heads, s.rot_dim, s.q_rank, s.kv_rank = 1, mix["rot_dim"], mix["q_rank"], mix["kv_rank"]
+                s.sink, s.head_gate = int(mix["sink"]), int(mix["gate"] == "heads")
+                s.kv_from = -1 if mix["kv_from"] is None else mix["kv_from"]
+        elif cfg["arch"] == "kufulix":
             s.block = _lib.BLOCK_PRE_NORM
             s.weights_of = -1 if layer.get("weights_of") is None else layer["weights_of"]
             s.kv_heads, s.scale, s.window, s.chunk = mix["kv_heads"], mix["scale"], mix["window"], mix["chunk"]
@@ -398,7 +504,7 @@ def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: i
     if cfg["arch"] in LAYERED:
         s.vocab_size, s.hidden_size, s.num_hidden_layers = cfg["vocab_size"], cfg["hidden_size"], len(cfg["layers"])
         s.max_position_embeddings = cfg.get("max_positions", 0)
-        s.norm_eps, s.logit_softcap = cfg["norm_eps"], cfg.get("logit_softcap", 0.0)
+        s.norm_eps, s.logit_softcap, s.norm_groups = cfg["norm_eps"], cfg.get("logit_softcap", 0.0), cfg.get("norm_groups", 1)
         return s
     for k in ("vocab_size", "hidden_size", "intermediate_size", "num_hidden_layers", "num_attention_heads",
               "max_position_embeddings"):
@@ -409,7 +515,6 @@ def to_struct(cfg: dict, dtype: int, max_batch: int, max_seq: int, max_tokens: i
     s.tie_word_embeddings = int(tied(cfg))
     # only qwen2's mask has the sliding-window term (qwen2.rs:316-327); the other families' masks are plain causal
     s.sliding_window = int(cfg.get("sliding_window") or 0) if cfg["arch"] == "qwen2" else 0
-    s.reserved0 = 0
     s.rope_theta = float(cfg["rope_theta"])
     s.norm_eps = float(norm_eps(cfg))
     return s

@@ -308,7 +308,7 @@ extern "C" int32_t rb_kv_cache_create_shared(rb_ctx* ctx, int32_t layers, int32_
   RB_REQUIRE(ctx && out, "rb_kv_cache_create_shared: null argument");
   RB_REQUIRE(layers > 0 && kv_heads > 0 && head_dim > 0 && max_batch > 0 && max_seq > 0, "rb_kv_cache_create_shared: bad sizes");
   RB_REQUIRE(dtype == RB_BF16 || dtype == RB_F32, "rb_kv_cache_create_shared: dtype %d unsupported", dtype);
-  RB_REQUIRE(head_dim % 8 == 0 && head_dim <= 256, "rb_kv_cache_create_shared: head_dim %d unsupported", head_dim);
+  RB_REQUIRE(head_dim % 8 == 0 && head_dim <= 1024, "rb_kv_cache_create_shared: head_dim %d unsupported", head_dim);
   return kv_cache_create(ctx, nullptr, layers, kv_heads, head_dim, max_batch, max_seq, dtype, out, true);
 }
 
@@ -530,7 +530,7 @@ extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache*
   x.value_dim = o->value_dim ? o->value_dim : c->head_dim;
   x.out_ld = o->out_ld ? o->out_ld : (int64_t)q_heads * x.value_dim;
   x.temp_every = o->temp_every; x.temp_coef = o->temp_coef; x.softcap = o->softcap; x.sink = o->sink;
-  x.chunk = o->chunk; x.head_gate = o->gate && o->head_gate; x.out_scale = o->out_scale != 0.f ? o->out_scale : 1.f;
+  x.talk = o->talk; x.chunk = o->chunk; x.head_gate = o->gate && o->head_gate; x.out_scale = o->out_scale != 0.f ? o->out_scale : 1.f;
   RB_REQUIRE(x.value_dim > 0 && x.value_dim <= c->head_dim, "rb_attention_general: value size %d of a %d-wide cache", x.value_dim,
              c->head_dim);
   RB_REQUIRE(x.window >= 0 && x.window <= (1 << 30), "rb_attention_general: bad window %d", x.window);
@@ -561,6 +561,11 @@ extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache*
   ProfScope prof(ctx, RB_PROF_ATTENTION,
                  es * ((c->shared() ? 1.0 : 2.0) * kv_tokens * c->kv_heads * d + (x.gate ? 3.0 : 2.0) * batch * s_new * q_heads * d),
                  4.0 * pairs * q_heads * d);
+  if (x.talk) {
+    RB_REQUIRE(!x.alibi && !x.gate && !x.temp_every && x.softcap == 0.f && x.out_scale == 1.f,
+               "rb_attention_general: mixed heads go with window, chunk, sink and value_dim only");
+    return attention_talk_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, x);
+  }
   if (!ctx->debug_simple_attn && attention_mma_takes(c, q_heads))
     return attention_mma_bf16(ctx, q, c, layer, batch, s_new, q_heads, scale, out, &x);
   return attention_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, &x);

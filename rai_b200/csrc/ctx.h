@@ -217,6 +217,27 @@ struct JoinSpec {
 };
 int add_then_norm(rb_ctx* ctx, const JoinSpec& s, int dtype);
 
+// sandwich.cu: rb_sandwich_join
+struct SandwichSpec {
+  const void* y = nullptr;
+  const float* acc = nullptr;
+  int n_acc = 0;
+  const void* post_gain = nullptr;
+  int groups = 1;
+  float eps = 0.f;
+  int64_t rows = 0;
+  int width = 0, ld = 0;
+  const float* h_in = nullptr;
+  float* h_out = nullptr;
+  const void* depth = nullptr;
+  int n_depth = 0;
+  float* history = nullptr;
+  int64_t history_stride = 0;
+  const void* gain = nullptr;
+  void* out = nullptr;
+};
+int sandwich_join(rb_ctx* ctx, const SandwichSpec& s, int dtype);
+
 // What an attention layer may have beyond the plain causal form.
 struct AttnExtra {
   int window = 0;              // rolling window: how many keys, its own included, a row sees; 0 = all
@@ -232,6 +253,7 @@ struct AttnExtra {
   float temp_coef = 0.f;
   float softcap = 0.f;         // > 0: score <- softcap tanh(score / softcap)
   const void* sink = nullptr;  // [q_heads], cache dtype: exp(sink) joins the softmax denominator
+  const void* talk = nullptr;  // [q_heads][q_heads], cache dtype: score[h] <- sum_g talk[h][g] score[g] before the mask
 };
 // the earliest position that the row at position `pos` sees (window 2^30: no window; chunk 0: no chunks)
 __host__ __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
@@ -282,6 +304,9 @@ int attention_reserve_scratch(rb_ctx* ctx, size_t bytes);
 bool attention_prefill_tc_supported(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const void* out);
 int attention_prefill_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
                          void* out, const AttnExtra* ext = nullptr);
+// plain_kernels.cu: attention whose heads' scores are mixed (x.talk), any sizes
+int attention_talk_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                          int dtype, const AttnExtra& x);
 int attention_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
                      float scale, void* out, int dtype, const AttnExtra* ext = nullptr);
 }  // namespace rb

@@ -376,6 +376,21 @@ int head_append_run(rb_ctx* ctx, const HeadArgs<T>& a) {
 
 using namespace rb;
 
+// amplitude * cos and sin of position * f[i], made in double precision
+static int rotary_upload(rb_ctx* ctx, const std::vector<double>& f, int max_pos, double amplitude, float* cos_dev, float* sin_dev) {
+  const size_t half = f.size();
+  std::vector<float> c((size_t)max_pos * half), s((size_t)max_pos * half);
+  for (int p = 0; p < max_pos; ++p)
+    for (size_t i = 0; i < half; ++i) {
+      c[(size_t)p * half + i] = (float)(amplitude * cos(p * f[i]));
+      s[(size_t)p * half + i] = (float)(amplitude * sin(p * f[i]));
+    }
+  RB_CUDA(cudaMemcpyAsync(cos_dev, c.data(), c.size() * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
+  RB_CUDA(cudaMemcpyAsync(sin_dev, s.data(), s.size() * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
+  RB_CUDA(cudaStreamSynchronize(ctx->stream));  // the staging vectors die with this frame
+  return RB_OK;
+}
+
 extern "C" int32_t rb_rotary_tables(rb_ctx* ctx, int32_t dims, int32_t max_pos, double base, double factor, double low, double high,
                                     double original, float* cos_dev, float* sin_dev) {
   RB_REQUIRE(ctx && cos_dev && sin_dev, "rb_rotary_tables: null argument");
@@ -390,16 +405,23 @@ extern "C" int32_t rb_rotary_tables(rb_ctx* ctx, int32_t dims, int32_t max_pos, 
     const double s = turns < low ? 0.0 : (turns - low) / (high - low);
     f[i] = (1.0 - s) * f[i] / factor + s * f[i];
   }
-  std::vector<float> c((size_t)max_pos * half), s((size_t)max_pos * half);
-  for (int p = 0; p < max_pos; ++p)
-    for (int i = 0; i < half; ++i) {
-      c[(size_t)p * half + i] = (float)cos(p * f[i]);
-      s[(size_t)p * half + i] = (float)sin(p * f[i]);
-    }
-  RB_CUDA(cudaMemcpyAsync(cos_dev, c.data(), c.size() * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
-  RB_CUDA(cudaMemcpyAsync(sin_dev, s.data(), s.size() * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
-  RB_CUDA(cudaStreamSynchronize(ctx->stream));  // the staging vectors die with this frame
-  return RB_OK;
+  return rotary_upload(ctx, f, max_pos, 1.0, cos_dev, sin_dev);
+}
+
+extern "C" int32_t rb_rotary_tables_yarn(rb_ctx* ctx, int32_t dims, int32_t max_pos, double base, double factor, double fast, double slow,
+                                         double original, float* cos_dev, float* sin_dev) {
+  RB_REQUIRE(ctx && cos_dev && sin_dev, "rb_rotary_tables_yarn: null argument");
+  RB_REQUIRE(dims > 0 && (dims % 2) == 0 && max_pos > 0 && base > 0.0 && base != 1.0 && factor > 0.0 && fast > 0.0 && slow > 0.0 && original > 0.0,
+             "rb_rotary_tables_yarn: bad sizes");
+  const double two_pi = 2.0 * 3.14159265358979323846;
+  auto index = [&](double turns) { return dims * log(original / (two_pi * turns)) / (2.0 * log(base)); };
+  const double lo = std::max(floor(index(fast)), 0.0), hi = std::min(ceil(index(slow)), dims - 1.0);
+  std::vector<double> f(dims / 2);
+  for (int i = 0; i < dims / 2; ++i) {
+    const double plain = pow(base, -2.0 * i / dims), stretch = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+    f[i] = plain / factor * stretch + plain * (1.0 - stretch);
+  }
+  return rotary_upload(ctx, f, max_pos, 0.1 * log(factor) + 1.0, cos_dev, sin_dev);
 }
 
 extern "C" int32_t rb_head_norm_rope_append(rb_ctx* ctx, const void* src, const float* acc, int32_t n_acc, const void* bias, int64_t src_ld,

@@ -20,12 +20,23 @@
 //     -> experts' gated GEMM -> experts' down GEMM;  attention;  output GEMM over [heads | shared expert]
 //     -> x += m (.), h = norm(x)
 //
+// or, with a norm on both sides of each sublayer (sandwich block), attention whose heads' scores are mixed or latent attention,
+// then a dense feed-forward, and an average over the depth so far:
+//
+//   h -> [q|k|v] GEMM -> q/k norm + rotary positions + cache append -> attention with mixed heads
+//   h -> [query latent|latent, key part|gate] GEMM -> norms + rotation + latent append -> query GEMM
+//        steps:   -> into the latent's space, per head -> attention over the latents -> out of it, per head (+ gate)
+//        prompts: latents GEMM to keys and values -> head split -> attention (+ gate)
+//     -> output GEMM -> x += norm(.), h = norm(x)
+//   h -> up GEMM (+ squared ReLU) -> down GEMM -> x += norm(.), x = depth average, h = norm(x)
+//
 // Single-token GEMMs leave float32 split-K slabs that the next kernel sums, as in the other families.  The driver around
 // this walk (lengths, the captured decode step, sampling, loading) is model.cu's.
 #include <string.h>
 
 #include <algorithm>
 #include <map>
+#include <tuple>
 
 #include "model.h"
 
@@ -95,18 +106,18 @@ int mixer(rb_model* m, const MixLayer& w, int batch, int seq, const int32_t* new
                              m->attn, w.mix_k, dt);
 }
 
-// m->act = xIELU(x . Wup^T): in the GEMM's epilogue, or, when that would leave most SMs idle, from split-K slabs
-int mlp_up(rb_model* m, const MixLayer& w, int64_t rows) {
+// m->act = act(x . Wup^T): in the GEMM's epilogue, or, when that would leave most SMs idle, from split-K slabs
+int mlp_up(rb_model* m, const MixLayer& w, int64_t rows, int act) {
   rb_ctx* ctx = m->ctx;
   const int64_t tiles = (w.mlp_k + 127) / 128;
   if (!ctx->debug_simple && tiles * 4 < (int64_t)ctx->sm_count * 3) {
     const int s = slab_count(m, rows, w.mlp_k, m->ld);
     if (s > 1) {
       RB_TRY(rb_linear_partials(ctx, m->h, w.up, m->scratch, rows, w.mlp_k, m->ld, s));
-      return act_from_partials(ctx, m->scratch, s, rows, w.mlp_k, w.mlp_k, false, nullptr, RB_ACT_XIELU, m->act, w.act);
+      return act_from_partials(ctx, m->scratch, s, rows, w.mlp_k, w.mlp_k, false, nullptr, act, m->act, w.act);
     }
   }
-  return rb_linear_act(ctx, m->h, w.up, nullptr, m->act, rows, w.mlp_k, m->ld, RB_ACT_XIELU, w.act, m->cfg.dtype);
+  return rb_linear_act(ctx, m->h, w.up, nullptr, m->act, rows, w.mlp_k, m->ld, act, w.act, m->cfg.dtype);
 }
 
 // A parallel block on m->h (the stream, normalised): the stream moves on, and m->h is what the next block (gain, or NULL after
@@ -276,14 +287,128 @@ int parallel_embed(rb_model* m, const uint32_t* tokens, int batch, int seq, cons
   return add_then_norm(m->ctx, j, c.dtype);
 }
 
+// A product of m->h (or another operand): slabs for the consumer to sum at single-token steps, a tensor otherwise
+struct Projected {
+  const void* src = nullptr;
+  const float* acc = nullptr;
+  int n_acc = 0;
+};
+int project(rb_model* m, const void* x, const void* w, const void* bias, void* dst, int64_t rows, int n, int k, int seq, Projected* out) {
+  const int s = seq == 1 ? slab_count(m, rows, n, k) : 0;
+  if (s > 0) {
+    RB_TRY(rb_linear_partials(m->ctx, x, w, m->scratch, rows, n, k, s));
+    *out = Projected{nullptr, m->scratch, s};
+    return RB_OK;
+  }
+  RB_TRY(rb_linear(m->ctx, x, w, bias, nullptr, dst, rows, n, k, RB_ACT_NONE, m->cfg.dtype));
+  *out = Projected{dst, nullptr, 0};
+  return RB_OK;
+}
+
+// Attention whose heads' scores are mixed, from m->h to m->attn
+int talking_mixer(rb_model* m, const MixLayer& w, int batch, int seq) {
+  const rb_layer_config& c = w.c;
+  const int dt = m->cfg.dtype;
+  Projected u;
+  RB_TRY(project(m, m->h, w.in_w, w.in_b, m->mix_in, (int64_t)batch * seq, w.n_in, m->ld, seq, &u));
+  RB_TRY(rb_head_norm_rope_append(m->ctx, u.src, u.acc, u.n_acc, w.in_b, w.n_in, w.q_norm, w.k_norm, (float)m->cfg.norm_eps, w.rope_cos,
+                                  w.rope_sin, w.rot_dims, batch, seq, c.heads, c.kv_heads, c.key_dim, c.value_dim, w.kv, w.kv_layer, m->q,
+                                  nullptr, 0, dt));
+  rb_attention_options o{};
+  o.value_dim = c.value_dim; o.out_ld = w.mix_k; o.talk = w.talk; o.sink = w.sink;
+  return rb_attention_general(m->ctx, m->q, w.kv, w.kv_layer, batch, seq, c.heads, (float)c.scale, &o, m->attn, dt);
+}
+
+// Latent attention, from m->h to m->attn
+int latent_mixer(rb_model* m, const MixLayer& w, int batch, int seq) {
+  rb_ctx* ctx = m->ctx;
+  const rb_layer_config& c = w.c;
+  const int dt = m->cfg.dtype, kv_rank = c.kv_rank;
+  const int64_t rows = (int64_t)batch * seq;
+  const bool own = c.kv_from < 0;
+  // sequences that all start here multiply their latents out; everything else stays in the latent's space
+  bool fresh = seq > 1 && w.prompt_kv >= 0;
+  for (int b = 0; b < batch && fresh; ++b) fresh = m->cache->host_lens[b] == seq;
+  Projected u;
+  RB_TRY(project(m, m->h, w.in_w, nullptr, m->mix_in, rows, w.n_in, m->ld, seq, &u));
+  const int gates = c.head_gate ? c.heads : c.heads * c.value_dim;
+  const bool gate_copy = u.acc != nullptr;
+  RB_TRY(rb_latent_append(ctx, u.src, u.acc, u.n_acc, w.n_in, c.q_rank, own ? kv_rank : 0, c.rot_dim, w.dq_norm, w.dkv_norm,
+                          (float)m->cfg.norm_eps, w.rope_cos, w.rope_sin, w.rot_dims, c.rot_interleaved, batch, seq, w.kv, w.kv_layer,
+                          m->q_latent, own && fresh ? m->latent : nullptr, gate_copy ? m->gate : nullptr, gate_copy ? gates : 0, dt));
+  const void* gate = gate_copy ? m->gate : (const char*)m->mix_in + (size_t)w.gate_col * m->es;
+  const int64_t gate_ld = gate_copy ? pad8(gates) : w.n_in;
+  rb_attention_options o{};
+  o.sink = w.sink;
+  if (fresh) {
+    rb_kv_cache* prompt = m->prompt_kv[w.prompt_kv];
+    prompt->pages_per_seq = (seq + kPageTokens - 1) / kPageTokens;
+    prompt->max_seq = prompt->pages_per_seq * kPageTokens;
+    if (!own) RB_TRY(rb_latent_gather(ctx, w.kv, w.kv_layer, kv_rank, batch, seq, m->latent, dt));
+    RB_TRY(rb_linear(ctx, m->q_latent, w.uq, nullptr, nullptr, m->q_raw, rows, w.n_q, w.qr_p, RB_ACT_NONE, dt));
+    RB_TRY(rb_linear(ctx, m->latent, w.uk, nullptr, nullptr, m->kv_raw, rows, w.n_kv, w.kr_p, RB_ACT_NONE, dt));
+    RB_TRY(rb_latent_heads(ctx, m->q_raw, w.n_q, m->kv_raw, w.n_kv, w.v_col, c.heads, c.key_dim, c.rot_dim, c.value_dim, kv_rank, w.rope_cos,
+                           w.rope_sin, w.rot_dims, c.rot_interleaved, batch, seq, w.kv, w.kv_layer, prompt, m->q, dt));
+    o.value_dim = c.value_dim; o.out_ld = w.mix_k; o.gate = gate; o.gate_ld = gate_ld; o.head_gate = c.head_gate;
+    return rb_attention_general(ctx, m->q, prompt, 0, batch, seq, c.heads, (float)c.scale, &o, m->attn, dt);
+  }
+  RB_TRY(project(m, m->q_latent, w.uq, nullptr, m->q_raw, rows, w.n_q, w.qr_p, seq, &u));
+  RB_TRY(rb_latent_query(ctx, u.src, u.acc, u.n_acc, w.n_q, w.uk, c.heads, c.key_dim, c.rot_dim, kv_rank, w.rope_cos, w.rope_sin, w.rot_dims,
+                         c.rot_interleaved, batch, seq, w.kv, m->q, dt));
+  o.value_dim = w.kr_p;
+  RB_TRY(rb_attention_general(ctx, m->q, w.kv, w.kv_layer, batch, seq, c.heads, (float)c.scale, &o, m->lat_out, dt));
+  return rb_latent_output(ctx, m->lat_out, w.uv, c.heads, kv_rank, c.value_dim, gate, gate_ld, c.head_gate, rows, m->attn, w.mix_k, dt);
+}
+
+// A sandwich block on m->h (the stream, normalised for the mixer), the l-th; m->h is then what the next block (gain, or NULL after
+// the last) reads.  The stream that enters block 0 is the history's first entry.
+int sandwich_block(rb_model* m, const MixLayer& w, int l, int batch, int seq, const void* next_gain) {
+  const rb_model_config& cfg = m->cfg;
+  const int64_t rows = (int64_t)batch * seq;
+  RB_TRY(w.c.mixer == RB_MIXER_LATENT ? latent_mixer(m, w, batch, seq) : talking_mixer(m, w, batch, seq));
+  const bool mlp = w.c.mlp_size > 0;
+  SandwichSpec j;
+  j.groups = cfg.norm_groups; j.eps = (float)cfg.norm_eps; j.rows = rows; j.width = cfg.hidden_size; j.ld = m->ld;
+  j.h_in = l == 0 ? m->history : m->stream; j.h_out = m->stream;
+  auto join = [&](const void* x, const void* weight, int k, const void* post, bool last, const void* gain) -> int {
+    const int s = slab_count(m, rows, m->ld, k);
+    if (s > 0) {
+      RB_TRY(rb_linear_partials(m->ctx, x, weight, m->scratch, rows, m->ld, k, s));
+      j.acc = m->scratch; j.n_acc = s; j.y = nullptr;
+    } else {
+      RB_TRY(rb_linear(m->ctx, x, weight, nullptr, nullptr, m->sub_out, rows, m->ld, k, RB_ACT_NONE, cfg.dtype));
+      j.y = m->sub_out; j.acc = nullptr; j.n_acc = 0;
+    }
+    j.post_gain = post;
+    if (last) { j.depth = w.depth; j.n_depth = l + 2; j.history = m->history; j.history_stride = (int64_t)cfg.max_tokens * m->ld; }
+    j.gain = gain; j.out = gain ? m->h : nullptr;
+    return sandwich_join(m->ctx, j, cfg.dtype);
+  };
+  RB_TRY(join(m->attn, w.o_w, w.mix_k, w.norm1b, !mlp, mlp ? w.norm2 : next_gain));
+  if (!mlp) return RB_OK;
+  RB_TRY(mlp_up(m, w, rows, RB_ACT_RELU2));
+  j.h_in = m->stream;
+  return join(m->act, w.down, w.mlp_k, w.norm2b, true, next_gain);
+}
+
+int sandwich_embed(rb_model* m, const uint32_t* tokens, int64_t rows) {
+  const rb_model_config& c = m->cfg;
+  RB_TRY(rb_embed_stream(m->ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->history, nullptr));
+  SandwichSpec j;
+  j.groups = c.norm_groups; j.eps = (float)c.norm_eps; j.rows = rows; j.width = c.hidden_size; j.ld = m->ld; j.h_in = m->history;
+  j.gain = m->mix[0].norm1; j.out = m->h;
+  return sandwich_join(m->ctx, j, c.dtype);
+}
+
 }  // namespace
 
 int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq, const int32_t* new_lens) {
   const rb_model_config& c = m->cfg;
   rb_ctx* ctx = m->ctx;
   const int64_t rows = (int64_t)batch * seq;
-  const bool parallel = c.arch == RB_ARCH_VOTAPEL, prenorm = c.arch == RB_ARCH_KUFULIX;
-  if (parallel) RB_TRY(parallel_embed(m, tokens, batch, seq, new_lens));
+  const bool parallel = c.arch == RB_ARCH_VOTAPEL, prenorm = c.arch == RB_ARCH_KUFULIX, sandwich = c.arch == RB_ARCH_FIZADRA;
+  if (sandwich) RB_TRY(sandwich_embed(m, tokens, rows));
+  else if (parallel) RB_TRY(parallel_embed(m, tokens, batch, seq, new_lens));
   else if (prenorm) RB_TRY(prenorm_embed(m, tokens, rows));
   else
     RB_TRY(rb_embed_stream(ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->stream,
@@ -291,7 +416,9 @@ int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq,
   for (size_t l = 0; l < m->mix.size(); ++l) {
     const MixLayer& w = m->mix[l];
     const void* next_gain = l + 1 < m->mix.size() ? m->mix[l + 1].norm1 : nullptr;
-    if (parallel) {
+    if (sandwich) {
+      RB_TRY(sandwich_block(m, w, (int)l, batch, seq, next_gain));
+    } else if (parallel) {
       RB_TRY(parallel_block(m, w, batch, seq, next_gain));
     } else if (prenorm) {
       RB_TRY(prenorm_block(m, w, batch, seq, new_lens, next_gain));
@@ -299,7 +426,7 @@ int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq,
       RB_TRY(mixer(m, w, batch, seq, new_lens));
       RB_TRY(sublayer_out(m, m->attn, w.o_w, w.mix_k, w.norm1, rows));
       if (w.c.mlp_size > 0) {
-        RB_TRY(mlp_up(m, w, rows));
+        RB_TRY(mlp_up(m, w, rows, RB_ACT_XIELU));
         RB_TRY(sublayer_out(m, m->act, w.down, w.mlp_k, w.norm2, rows));
       }
     }
@@ -313,7 +440,9 @@ int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq,
 int rb::layered_logits(rb_model* m, const int32_t* rows, int seq, int n, float* out) {
   const rb_model_config& c = m->cfg;
   const auto norm = c.arch == RB_ARCH_MALASUN ? rb_scalar_norm_rows : rb_one_plus_norm_rows;
-  RB_TRY(norm(m->ctx, m->stream, rows, seq, m->norm_w, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
+  if (c.arch == RB_ARCH_FIZADRA)
+    RB_TRY(rb_group_norm_rows(m->ctx, m->stream, rows, seq, m->norm_w, c.norm_groups, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
+  else RB_TRY(norm(m->ctx, m->stream, rows, seq, m->norm_w, (float)c.norm_eps, n, c.hidden_size, m->ld, m->xn, c.dtype));
   if (c.dtype == RB_F32) {
     RB_TRY(rb_linear(m->ctx, m->xn, m->lm_head, nullptr, nullptr, out, n, c.vocab_size, m->ld, RB_ACT_NONE, RB_F32));
   } else {
@@ -377,11 +506,39 @@ static int check_prenorm(const rb_layer_config* layers, int n, int l) {
   return RB_OK;
 }
 
+// What a sandwich layer may be
+static int check_sandwich(const rb_layer_config* layers, int l) {
+  const rb_layer_config& y = layers[l];
+  RB_REQUIRE(y.block == RB_BLOCK_SANDWICH && (y.mixer == RB_MIXER_ATTENTION || y.mixer == RB_MIXER_LATENT) &&
+                 (y.mlp_size == 0 || y.mlp_kind == RB_MLP_DENSE_RELU2) && y.mlp_size >= 0,
+             "layer %d: block, mixer or feed-forward kind does not belong to this architecture", l);
+  RB_REQUIRE(y.heads > 0 && y.key_dim > 0 && y.value_dim > 0 && y.scale > 0.0, "layer %d: bad heads", l);
+  RB_REQUIRE(y.rot_dims >= 0 && (y.rot_dims % 2) == 0 && y.rot_dims <= (y.mixer == RB_MIXER_LATENT ? y.rot_dim : y.key_dim),
+             "layer %d: %d dimensions cannot turn", l, y.rot_dims);
+  if (y.mixer == RB_MIXER_ATTENTION) {
+    RB_REQUIRE(y.kv_heads > 0 && y.heads % y.kv_heads == 0 && y.kv_from < 0 && y.talk && y.softmax_one && y.qk_norm && !y.rot_interleaved,
+               "layer %d: bad attention", l);
+    if (y.key_dim > 256 || y.value_dim > 256) return fail(RB_ERR_UNIMPLEMENTED, "layer %d: head sizes above 256", l);
+    return RB_OK;
+  }
+  RB_REQUIRE(y.q_rank > 0 && y.kv_rank > 0 && y.rot_dim >= 0, "layer %d: bad latent sizes", l);
+  if (pad8(y.kv_rank) + y.rot_dim > 960) return fail(RB_ERR_UNIMPLEMENTED, "layer %d: a latent of more than 960 numbers", l);
+  if (y.kv_from < 0) return RB_OK;
+  RB_REQUIRE(y.kv_from < l && layers[y.kv_from].mixer == RB_MIXER_LATENT && layers[y.kv_from].kv_from < 0,
+             "layer %d: kv_from %d is not an earlier layer with a latent of its own", l, y.kv_from);
+  const rb_layer_config& o = layers[y.kv_from];
+  RB_REQUIRE(o.kv_rank == y.kv_rank && o.rot_dim == y.rot_dim && o.rot_dims == y.rot_dims && o.rot_base == y.rot_base &&
+                 o.rot_interleaved == y.rot_interleaved && o.rot_yarn == y.rot_yarn && o.rot_original == y.rot_original &&
+                 o.rot_factor == y.rot_factor && o.rot_low == y.rot_low && o.rot_high == y.rot_high,
+             "layer %d: its latent or rotation differs from that of layer %d", l, y.kv_from);
+  return RB_OK;
+}
+
 extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cfg, const rb_layer_config* layers, rb_model** out) {
   RB_REQUIRE(ctx && cfg && layers && out, "rb_model_create_layers: null argument");
   const rb_model_config& c = *cfg;
-  const bool parallel = c.arch == RB_ARCH_VOTAPEL, prenorm = c.arch == RB_ARCH_KUFULIX;
-  RB_REQUIRE(c.arch == RB_ARCH_MALASUN || parallel || prenorm, "rb_model_create_layers: architecture %d is not described layer by layer", c.arch);
+  const bool parallel = c.arch == RB_ARCH_VOTAPEL, prenorm = c.arch == RB_ARCH_KUFULIX, sandwich = c.arch == RB_ARCH_FIZADRA;
+  RB_REQUIRE(c.arch == RB_ARCH_MALASUN || parallel || prenorm || sandwich, "rb_model_create_layers: architecture %d is not described layer by layer", c.arch);
   RB_REQUIRE(c.dtype == RB_BF16 || c.dtype == RB_F32, "rb_model_create_layers: dtype %d unsupported", c.dtype);
   RB_REQUIRE(c.hidden_size > 0 && c.vocab_size > 0 && c.num_hidden_layers > 0, "rb_model_create_layers: bad sizes");
   RB_REQUIRE(c.max_batch > 0 && c.max_seq > 0 && c.max_tokens >= c.max_batch, "rb_model_create_layers: bad capacities");
@@ -389,11 +546,13 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   if (c.tp_size > 1) return fail(RB_ERR_UNIMPLEMENTED, "rb_model_create_layers: tensor parallelism is not available for this design");
   RB_REQUIRE(!parallel || c.max_position_embeddings > 0, "rb_model_create_layers: learned positions need their number");
   RB_REQUIRE(c.logit_softcap >= 0.0, "rb_model_create_layers: bad logit cap");
+  RB_REQUIRE(!sandwich || (c.norm_groups > 0 && c.hidden_size % c.norm_groups == 0), "rb_model_create_layers: %d parts of a row of %d", c.norm_groups,
+             c.hidden_size);
   const int L = c.num_hidden_layers;
   for (int l = 0; l < L; ++l) {
     const rb_layer_config& y = layers[l];
-    if (prenorm) {
-      RB_TRY(check_prenorm(layers, L, l));
+    if (prenorm || sandwich) {
+      RB_TRY(prenorm ? check_prenorm(layers, L, l) : check_sandwich(layers, l));
       continue;
     }
     RB_REQUIRE(y.block == (parallel ? RB_BLOCK_PARALLEL : RB_BLOCK_POST_NORM) &&
@@ -461,15 +620,128 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
     vec("embed.norm", W, m->embed_norm);
   }
   m->mix.resize(L);
-  std::map<std::pair<int, int>, std::vector<int>> geometry;  // (key/value heads, cache head size) -> layers with K and V of their own
+  // (key/value heads, cache head size, the values are the keys) -> layers with K and V of their own
+  std::map<std::tuple<int, int, bool>, std::vector<int>> geometry;
+  auto cached = [&](MixLayer& w, int l, int kv_heads, int head_dim) {
+    auto& group = geometry[{kv_heads, head_dim, parallel || w.c.mixer == RB_MIXER_LATENT}];
+    w.kv_layer = (int)group.size();
+    group.push_back(l);
+  };
   int max_in = 8, max_q = 8, max_gate = 8, max_mix = 8, max_mlp = 8, max_experts = 0, max_top = 0, max_ff = 8;
   int max_chan = 0, max_inner = 0, max_gates = 0;
   std::map<std::vector<double>, std::pair<float*, float*>> rotations;  // tables, one set per kind of rotation
+  auto turn = [&](MixLayer& w) {
+    const rb_layer_config& y = w.c;
+    w.rot_dims = y.rot_dims;
+    if (y.rot_dims == 0 || st != RB_OK) return;
+    const double original = y.rot_original;
+    const int positions = (c.max_seq + kPageTokens - 1) / kPageTokens * kPageTokens;   // those of whole pages: padding may sit there
+    auto& t = rotations[{(double)y.rot_dims, y.rot_base, original, y.rot_factor, y.rot_low, y.rot_high, (double)y.rot_yarn}];
+    if (!t.first) {
+      const size_t bytes = (size_t)positions * (y.rot_dims / 2) * sizeof(float);
+      st = dev_alloc(m, bytes, (void**)&t.first, false);
+      if (st == RB_OK) st = dev_alloc(m, bytes, (void**)&t.second, false);
+      if (st == RB_OK)
+        st = y.rot_yarn ? rb_rotary_tables_yarn(ctx, y.rot_dims, positions, y.rot_base, y.rot_factor, y.rot_high, y.rot_low, original, t.first, t.second)
+                        : rb_rotary_tables(ctx, y.rot_dims, positions, y.rot_base, y.rot_factor, y.rot_low, y.rot_high, original, t.first, t.second);
+    }
+    w.rope_cos = t.first;
+    w.rope_sin = t.second;
+  };
+  int max_qr = 0, max_kr = 0, max_nq = 0, max_nkv = 0, max_lat = 0, zero_heads = 0;
+  std::map<std::pair<int, int>, int> prompt_shapes;   // (heads, head size) -> index into m->prompt_kv
   for (int l = 0; l < L && st == RB_OK; ++l) {
     MixLayer& w = m->mix[l];
     w.c = layers[l];
     const rb_layer_config& y = w.c;
     const std::string pre = "l" + std::to_string(l) + ".", mix = pre + "mix.";
+    if (sandwich) {
+      const bool latent = y.mixer == RB_MIXER_LATENT, mlp = y.mlp_size > 0;
+      auto part = [&](const std::string& name, int64_t n, int64_t row, void* dst) { mat(mix + name, n, W, at(dst, row * ld), ld); };
+      turn(w);
+      w.mix_k = pad8((int64_t)y.heads * y.value_dim);
+      w.mlp_k = pad8(y.mlp_size);
+      for (void** p : {&w.norm1, &w.norm1b}) A(ld, p);
+      if (mlp) for (void** p : {&w.norm2, &w.norm2b}) A(ld, p);
+      A(pad8(l + 2), &w.depth);
+      A((int64_t)ld * w.mix_k, &w.o_w);
+      if (mlp) { A((int64_t)w.mlp_k * ld, &w.up); A((int64_t)ld * w.mlp_k, &w.down); }
+      if (latent) {
+        const bool own = y.kv_from < 0;
+        const int gates = y.head_gate ? y.heads : y.heads * y.value_dim, nk = y.heads * y.key_dim, nv = y.heads * y.value_dim;
+        w.qr_p = pad8(y.q_rank); w.kr_p = pad8(y.kv_rank); w.kv_p = own ? pad8(y.kv_rank + y.rot_dim) : 0;
+        w.gate_col = w.qr_p + w.kv_p;
+        w.n_in = w.gate_col + pad8(gates);
+        w.n_q = pad8((int64_t)y.heads * (y.key_dim + y.rot_dim)); w.v_col = pad8(nk); w.n_kv = w.v_col + pad8(nv);
+        A((int64_t)w.n_in * ld, &w.in_w);
+        A(w.qr_p, &w.dq_norm);
+        if (own) A(w.kr_p, &w.dkv_norm);
+        A((int64_t)w.n_q * w.qr_p, &w.uq);
+        A((int64_t)w.n_kv * w.kr_p, &w.uk);
+        if (y.sink) A(pad8(y.heads), &w.sink);
+        if (st != RB_OK) break;
+        w.uv = at(w.uk, (int64_t)w.v_col * w.kr_p);
+        part("dq", y.q_rank, 0, w.in_w);
+        vec(mix + "dq.norm", y.q_rank, w.dq_norm);
+        mat(mix + "uq", (int64_t)y.heads * (y.key_dim + y.rot_dim), y.q_rank, w.uq, w.qr_p);
+        const int head_dim = c.dtype == RB_BF16 ? (w.kr_p + y.rot_dim + 63) / 64 * 64 : pad8(w.kr_p + y.rot_dim);
+        if (own) {
+          part("dkv", y.kv_rank + y.rot_dim, w.qr_p, w.in_w);
+          vec(mix + "dkv.norm", y.kv_rank, w.dkv_norm);
+          cached(w, l, 1, head_dim);
+        }
+        mat(mix + "uk", nk, y.kv_rank, w.uk, w.kr_p);
+        mat(mix + "uv", nv, y.kv_rank, w.uv, w.kr_p);
+        if (y.sink) vec(mix + "sink", y.heads, w.sink);
+        part("g", gates, w.gate_col, w.in_w);
+        const int wide = std::max(y.key_dim + y.rot_dim, y.value_dim), prompt_dim = cache_dim(c.dtype, y.key_dim + y.rot_dim, y.value_dim);
+        if (wide <= 256) {
+          auto it = prompt_shapes.insert({{y.heads, prompt_dim}, (int)prompt_shapes.size()});
+          w.prompt_kv = it.first->second;
+          max_q = std::max(max_q, y.heads * prompt_dim);
+        }
+        max_q = std::max(max_q, y.heads * head_dim);
+        max_gate = std::max(max_gate, pad8(gates));
+        max_qr = std::max(max_qr, w.qr_p); max_kr = std::max(max_kr, w.kr_p); max_nq = std::max(max_nq, w.n_q);
+        max_nkv = std::max(max_nkv, w.n_kv); max_lat = std::max(max_lat, y.heads * w.kr_p);
+      } else {
+        const int nq = y.heads * y.key_dim, nk = y.kv_heads * y.key_dim, nv = y.kv_heads * y.value_dim, qp = pad8(nq), kp = pad8(nk);
+        const int widest = std::max(y.key_dim, y.value_dim), head_dim = c.dtype == RB_BF16 ? (widest + 63) / 64 * 64 : pad8(widest);
+        w.n_in = qp + kp + pad8(nv);
+        A((int64_t)w.n_in * ld, &w.in_w);
+        A(w.n_in, &w.in_b);
+        for (void** p : {&w.q_norm, &w.k_norm}) A(pad8(y.key_dim), p);
+        A(pad8((int64_t)y.heads * y.heads), &w.talk);
+        if (st != RB_OK) break;
+        const int n[3] = {nq, nk, nv}, row[3] = {0, qp, qp + kp};
+        for (int i = 0; i < 3; ++i) {
+          const std::string name(1, "qkv"[i]);
+          part(name, n[i], row[i], w.in_w);
+          vec(mix + name + ".b", n[i], at(w.in_b, row[i]));
+        }
+        vec(mix + "q.norm", y.key_dim, w.q_norm);
+        vec(mix + "k.norm", y.key_dim, w.k_norm);
+        mat(mix + "talk", y.heads, y.heads, w.talk, y.heads);
+        cached(w, l, y.kv_heads, head_dim);
+        max_q = std::max(max_q, y.heads * head_dim);
+        zero_heads = std::max(zero_heads, y.heads);
+      }
+      if (st != RB_OK) break;
+      vec(pre + "norm1", W, w.norm1);
+      vec(pre + "norm1b", W, w.norm1b);
+      mat(mix + "o", W, (int64_t)y.heads * y.value_dim, w.o_w, w.mix_k);
+      if (mlp) {
+        vec(pre + "norm2", W, w.norm2);
+        vec(pre + "norm2b", W, w.norm2b);
+        mat(pre + "mlp.up", y.mlp_size, W, w.up, ld);
+        mat(pre + "mlp.down", W, y.mlp_size, w.down, w.mlp_k);
+      }
+      vec(pre + "dwa", l + 2, w.depth);
+      max_in = std::max(max_in, w.n_in);
+      max_mix = std::max(max_mix, w.mix_k);
+      max_mlp = std::max(max_mlp, w.mlp_k);
+      continue;
+    }
     if (prenorm) {
       const bool ssd = y.mixer == RB_MIXER_ATTENTION_SSD, own = y.weights_of < 0;
       const int nq = y.heads * y.key_dim, nk = y.kv_heads * y.key_dim, nv = y.kv_heads * y.value_dim, qp = pad8(nq), kp = pad8(nk), vp = pad8(nv);
@@ -483,9 +755,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
       w.mix_k = w.attn_cols + ip;
       w.ff_p = pad8(y.mlp_size);
       w.n_router = y.mlp_size > 0 ? pad8(y.experts + y.identity) : 0;
-      auto& group = geometry[{y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim)}];
-      w.kv_layer = (int)group.size();
-      group.push_back(l);
+      cached(w, l, y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim));
       if (ssd && st == RB_OK) st = dev_alloc(m, (size_t)c.max_batch * y.ssd_heads * y.ssd_state * y.ssd_value_dim * sizeof(float), (void**)&w.state, true);
       if (ssd && st == RB_OK) st = dev_alloc(m, (size_t)c.max_batch * std::max(1, taps - 1) * C * sizeof(float), (void**)&w.ring, true);
       max_q = std::max(max_q, y.heads * cache_dim(c.dtype, y.key_dim, y.value_dim));
@@ -500,20 +770,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
         max_top = std::max(max_top, y.top);
         max_ff = std::max(max_ff, w.ff_p);
       }
-      w.rot_dims = y.rot_dims;
-      if (y.rot_dims > 0 && st == RB_OK) {
-        const double original = y.rot_original;
-        auto& t = rotations[{(double)y.rot_dims, y.rot_base, original, y.rot_factor, y.rot_low, y.rot_high}];
-        if (!t.first) {
-          const size_t bytes = (size_t)c.max_seq * (y.rot_dims / 2) * sizeof(float);
-          st = dev_alloc(m, bytes, (void**)&t.first, false);
-          if (st == RB_OK) st = dev_alloc(m, bytes, (void**)&t.second, false);
-          if (st == RB_OK)
-            st = rb_rotary_tables(ctx, y.rot_dims, c.max_seq, y.rot_base, y.rot_factor, y.rot_low, y.rot_high, original, t.first, t.second);
-        }
-        w.rope_cos = t.first;
-        w.rope_sin = t.second;
-      }
+      turn(w);
       if (!own) continue;   // parameters: below
       A(ld, &w.norm1);
       A((int64_t)w.n_in * ld, &w.in_w);
@@ -626,9 +883,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
         mat(mlp + "shared.up", y.shared_size, W, at(w.in_w, (int64_t)(qp + kp + w.glu_p) * ld), ld);
         mat(mlp + "shared.down", W, y.shared_size, at(w.o_w, w.attn_cols), w.mix_k);
       }
-      auto& group = geometry[{y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim)}];
-      w.kv_layer = (int)group.size();
-      group.push_back(l);
+      cached(w, l, y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim));
       max_q = std::max(max_q, y.heads * cache_dim(c.dtype, y.key_dim, y.value_dim));
       max_in = std::max(max_in, w.n_in);
       max_mix = std::max(max_mix, w.mix_k);
@@ -683,9 +938,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
       if (own) {
         part("k", nk, qp, w.k_norm);
         part("v", nv, qp + kp, nullptr);
-        auto& group = geometry[{y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim)}];
-        w.kv_layer = (int)group.size();
-        group.push_back(l);
+        cached(w, l, y.kv_heads, cache_dim(c.dtype, y.key_dim, y.value_dim));
       }
       mat(mix + "g", (int64_t)y.heads * y.value_dim, W, at(w.in_w, (int64_t)C * ld), ld);
       if (taps > 1) st = dev_alloc(m, (size_t)c.max_batch * (taps - 1) * C * sizeof(float), (void**)&w.state, true);
@@ -718,10 +971,10 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
       w = m->mix[o];
       w.c = own.c; w.kv_layer = own.kv_layer; w.state = own.state; w.ring = own.ring;
     }
-  A(parallel || prenorm ? ld : 8, &m->norm_w);
+  A(parallel || prenorm || sandwich ? ld : 8, &m->norm_w);
   A((int64_t)V * ld, &m->lm_head);
   if (st == RB_OK) {
-    if (parallel || prenorm) vec("final.norm", W, m->norm_w);
+    if (parallel || prenorm || sandwich) vec("final.norm", W, m->norm_w);
     else num("final.norm", m->norm_w);
     mat("head", V, W, m->lm_head, ld);
     m->vocab_l = V;
@@ -731,14 +984,15 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   if (st == RB_OK) st = kv_cache_create(ctx, nullptr, 0, 1, 8, c.max_batch, c.max_seq, c.dtype, &m->cache);
   for (auto& g : geometry) {
     rb_kv_cache* view = nullptr;
-    if (st == RB_OK) st = kv_cache_create(ctx, m->cache, (int)g.second.size(), g.first.first, g.first.second, 0, 0, c.dtype, &view, parallel);
+    if (st == RB_OK)
+      st = kv_cache_create(ctx, m->cache, (int)g.second.size(), std::get<0>(g.first), std::get<1>(g.first), 0, 0, c.dtype, &view, std::get<2>(g.first));
     if (st != RB_OK) break;
     m->views.push_back(view);
     for (int l : g.second) m->mix[l].kv = view;
   }
   if (st == RB_OK)
     for (MixLayer& w : m->mix)
-      if (w.c.mixer == RB_MIXER_ATTENTION && w.c.kv_from >= 0) {
+      if ((w.c.mixer == RB_MIXER_ATTENTION || w.c.mixer == RB_MIXER_LATENT) && w.c.kv_from >= 0) {
         w.kv = m->mix[w.c.kv_from].kv;
         w.kv_layer = m->mix[w.c.kv_from].kv_layer;
       }
@@ -755,7 +1009,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   const size_t MT = c.max_tokens, few = std::min<size_t>(MT, 256);
   B(MT * sizeof(uint32_t), (void**)&m->ids);
   B(MT * ld * sizeof(float), (void**)&m->stream);
-  if (c.dtype == RB_F32 && !parallel && !prenorm) m->h = m->stream;
+  if (c.dtype == RB_F32 && !parallel && !prenorm && !sandwich) m->h = m->stream;
   else B(MT * ld * m->es, &m->h);
   B(MT * max_in * m->es, &m->mix_in);
   B(MT * max_q * m->es, &m->q);
@@ -768,6 +1022,39 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   B((size_t)c.max_batch * sizeof(uint32_t), (void**)&m->next_ids);
   B(MT * sizeof(int32_t), (void**)&m->last_rows);
   if (parallel || prenorm) B(kMaxExperts * sizeof(int32_t), (void**)&m->route_count);
+  if (sandwich) {
+    B((size_t)(L + 1) * MT * ld * sizeof(float), (void**)&m->history);
+    void* zeros = nullptr;   // sinks of score 0: one more in the softmax denominator
+    B((size_t)pad8(zero_heads) * m->es, &zeros);
+    for (MixLayer& w : m->mix)
+      if (w.c.softmax_one) w.sink = zeros;
+  }
+  if (max_qr > 0) {
+    B(MT * max_qr * m->es, &m->q_latent);
+    B(MT * max_kr * m->es, &m->latent);
+    B(MT * max_nq * m->es, &m->q_raw);
+    // keys and values multiplied out, or each head's weighted latent: never both
+    B(MT * std::max(max_nkv, max_lat) * m->es, &m->kv_raw);
+    m->lat_out = m->kv_raw;
+    const int pages = (int)(MT / kPageTokens) + c.max_batch;   // every sequence of a call may end in a page of its own
+    size_t elems = 0;
+    for (auto& g : prompt_shapes) elems = std::max(elems, (size_t)pages * kPageTokens * g.first.first * g.first.second);
+    void *k = nullptr, *v = nullptr, *table = nullptr;
+    if (!prompt_shapes.empty()) { B(elems * m->es, &k); B(elems * m->es, &v); }
+    B((size_t)pages * sizeof(int32_t), &table);
+    std::vector<int32_t> in_order(pages);
+    for (int i = 0; i < pages; ++i) in_order[i] = i;
+    if (st == RB_OK) st = rb_upload(ctx, table, in_order.data(), in_order.size() * sizeof(int32_t));
+    if (st == RB_OK) RB_CUDA(cudaStreamSynchronize(ctx->stream));   // (the vector dies with this frame)
+    m->prompt_kv.resize(prompt_shapes.size(), nullptr);
+    for (auto& g : prompt_shapes) {
+      if (st != RB_OK) break;
+      rb_kv_cache* p = new rb_kv_cache(m->cache);
+      p->ctx = ctx; p->layers = 1; p->kv_heads = g.first.first; p->head_dim = g.first.second; p->dtype = c.dtype; p->max_batch = c.max_batch;
+      p->num_pages = pages; p->k = k; p->v = v; p->block_table = (int32_t*)table; p->seq_lens = m->cache->seq_lens; p->slots = m->cache->slots;
+      m->prompt_kv[g.second] = p;
+    }
+  }
   if (max_inner > 0) {
     B(MT * max_chan * m->es + (size_t)c.max_batch * max_gates * 2 * sizeof(float), &m->chan);
     B(MT * max_inner * m->es, &m->rec_out);
@@ -782,7 +1069,7 @@ extern "C" int32_t rb_model_create_layers(rb_ctx* ctx, const rb_model_config* cf
   }
   B((size_t)c.max_batch * sizeof(int32_t), (void**)&m->new_lens);
   if (c.dtype == RB_BF16) {
-    m->scratch_floats = (size_t)16 * few * std::max(std::max(std::max(max_in, max_mlp), ld), max_experts);
+    m->scratch_floats = (size_t)16 * few * std::max({max_in, max_mlp, ld, max_experts, max_nq});
     B(m->scratch_floats * sizeof(float), (void**)&m->scratch);
   }
   if (st != RB_OK) { rb_model_destroy(m); return st; }

@@ -752,6 +752,7 @@ extern "C" int32_t rb_model_destroy(rb_model* m) {
     if (m->peer_base[r] && m->peer_base[r] != m->xchg_base) cudaIpcCloseMemHandle(m->peer_base[r]);
   if (m->comm && nccl().CommDestroy) nccl().CommDestroy(m->comm);
   for (rb_kv_cache* v : m->views) rb_kv_cache_destroy(v);
+  for (rb_kv_cache* v : m->prompt_kv) delete v;   // (their memory is the model's)
   if (m->cache) rb_kv_cache_destroy(m->cache);
   for (void* p : m->owned) rb_free(m->ctx, p);
   delete m;

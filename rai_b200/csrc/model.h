@@ -59,6 +59,12 @@ struct MixLayer {
   const float *rope_cos = nullptr, *rope_sin = nullptr;
   void *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *skip = nullptr, *router = nullptr, *correction = nullptr;
   float* ring = nullptr;       // Mamba-2: earlier channel values [slot][taps - 1][channels]
+  // sandwich block: norms behind the sublayers, weights of the depth average; head-mixing attention (zero: sinks of score 0);
+  // latent attention (fused input projection [query latent | latent, key part | gate])
+  void *norm1b = nullptr, *norm2b = nullptr, *depth = nullptr, *talk = nullptr;
+  void *dq_norm = nullptr, *dkv_norm = nullptr, *uq = nullptr, *uk = nullptr, *uv = nullptr;   // uk, uv: one matrix [keys | values]
+  int qr_p = 0, kv_p = 0, kr_p = 0, n_q = 0, n_kv = 0, v_col = 0;   // padded sizes: latents, their columns, heads multiplied out
+  int prompt_kv = -1;          // index into rb_model::prompt_kv; -1: prompts, too, attend in the latent's space
   rb_kv_cache* kv = nullptr;   // the cache (of this layer's geometry) its keys and values are in, and the layer there
   int kv_layer = 0;
   float* state = nullptr;      // attention: ring of projected values [slot][taps - 1][channels]; recurrences: [slot][head][key][value]
@@ -134,6 +140,11 @@ struct rb_model {
   void *expert_act = nullptr, *expert_out = nullptr;
   float* route_own = nullptr;             // weight of a row's identity experts
   void *chan = nullptr, *rec_out = nullptr;  // a recurrence's channels after their convolution, and its output
+  // sandwich blocks: the embedding and every layer's result [layers + 1][max_tokens][ld]; latent attention's intermediate rows,
+  // and where a prompt's keys and values go when its latents are multiplied out (pages in order, one buffer for all layers)
+  float* history = nullptr;
+  void *q_latent = nullptr, *latent = nullptr, *q_raw = nullptr, *kv_raw = nullptr, *lat_out = nullptr;
+  std::vector<rb_kv_cache*> prompt_kv;
   float* layer_trace = nullptr;
   int logits_dtype = RB_BF16;
   int32_t* new_lens = nullptr;            // device [max_batch]: tokens each sequence feeds in this call

@@ -128,23 +128,23 @@ __global__ void __launch_bounds__(256) gemv_f32_kernel(const float* __restrict__
 
 // One block per (token, query head): its 8 warps take every 8th key of the paged cache, each with an online
 // softmax of its own (lanes split head_dim), and their (max, sum, O) states are merged through shared memory.
-// float32 throughout.  Correct for any head_dim <= 256.
+// float32 throughout.  Correct for any head_dim <= 32 * NJ.
 constexpr int kPlainAttnWarps = 8;
-template <typename T>
+template <typename T, int NJ>
 __global__ void __launch_bounds__(kPlainAttnWarps * 32)
 attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                        const int32_t* __restrict__ block_table, const int32_t* __restrict__ seq_lens, int pages_per_seq,
                        int s_new, int q_heads, int kv_heads, int d, float scale, int window, T* __restrict__ out, int ext,
                        const AttnExtra x) {
-  __shared__ float sm_m[kPlainAttnWarps], sm_l[kPlainAttnWarps], sm_o[kPlainAttnWarps][256];
+  __shared__ float sm_m[kPlainAttnWarps], sm_l[kPlainAttnWarps], sm_o[kPlainAttnWarps][32 * NJ];
   const int m = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = m / s_new, s = m % s_new;
   const int limit = seq_lens[b] - s_new + s;  // last visible key
   const int kvh = h / (q_heads / kv_heads);
-  float qv[8], o[8];
+  float qv[NJ], o[NJ];
 #pragma unroll
-  for (int j = 0; j < 8; ++j) {
+  for (int j = 0; j < NJ; ++j) {
     const int i = lane + 32 * j;
     qv[j] = i < d ? Cvt<T>::to_f(q[((size_t)m * q_heads + h) * d + i]) : 0.f;
     o[j] = 0.f;
@@ -161,7 +161,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
     const size_t off = (((size_t)page * kv_heads + kvh) * kPageTokens + (t % kPageTokens)) * d;
     float dot = 0.f;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
+    for (int j = 0; j < NJ; ++j) {
       const int i = lane + 32 * j;
       if (i < d) dot += qv[j] * Cvt<T>::to_f(k_cache[off + i]);
     }
@@ -172,7 +172,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
     const float corr = expf(mx - mn), p = expf(dot - mn);
     l = l * corr + p;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
+    for (int j = 0; j < NJ; ++j) {
       const int i = lane + 32 * j;
       if (i < d) o[j] = o[j] * corr + p * Cvt<T>::to_f(v_cache[off + i]);
     }
@@ -180,7 +180,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
   }
   if (lane == 0) { sm_m[warp] = mx; sm_l[warp] = l; }
 #pragma unroll
-  for (int j = 0; j < 8; ++j) {
+  for (int j = 0; j < NJ; ++j) {
     const int i = lane + 32 * j;
     if (i < d) sm_o[warp][i] = o[j];
   }
@@ -205,6 +205,69 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
     } else {
       out[((size_t)m * q_heads + h) * d + i] = Cvt<T>::from_f(O / L);
     }
+  }
+}
+
+// The same where the heads' scores are mixed before the softmax: one block per token with all its heads, 32 keys at a time.
+// Shared memory: q [heads][d], scores and weights [heads][33] each, max, sum and rescaling factor per head, O [heads][d].
+constexpr int kTalkKeys = 32;
+template <typename T>
+__global__ void __launch_bounds__(256)
+attention_talk_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+                            const int32_t* __restrict__ block_table, const int32_t* __restrict__ seq_lens, int pages_per_seq, int s_new,
+                            int q_heads, int kv_heads, int d, float scale, T* __restrict__ out, const AttnExtra x) {
+  extern __shared__ float smem_talk[];
+  float* q_s = smem_talk;
+  float* s_s = q_s + q_heads * d;
+  float* p_s = s_s + q_heads * (kTalkKeys + 1);
+  float* m_s = p_s + q_heads * (kTalkKeys + 1);
+  float* l_s = m_s + q_heads;
+  float* c_s = l_s + q_heads;
+  float* o_s = c_s + q_heads;
+  const int m = blockIdx.x, b = m / s_new, limit = seq_lens[b] - s_new + m % s_new, group = q_heads / kv_heads;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const T* talk = (const T*)x.talk;
+  for (int i = threadIdx.x; i < q_heads * d; i += blockDim.x) { q_s[i] = Cvt<T>::to_f(q[(size_t)m * q_heads * d + i]); o_s[i] = 0.f; }
+  for (int h = threadIdx.x; h < q_heads; h += blockDim.x) { m_s[h] = -INFINITY; l_s[h] = 0.f; }
+  const int first = first_visible(limit, x.window > 0 ? x.window : 1 << 30, x.chunk);
+  for (int t0 = first / kTalkKeys * kTalkKeys; t0 <= limit; t0 += kTalkKeys) {
+    const int page = block_table[(size_t)b * pages_per_seq + t0 / kPageTokens];
+    auto row = [&](const T* cache, int kvh, int key) {
+      return cache + (((size_t)page * kv_heads + kvh) * kPageTokens + (t0 + key) % kPageTokens) * d;
+    };
+    __syncthreads();
+    for (int it = warp; it < q_heads * kTalkKeys; it += warps) {
+      const int h = it / kTalkKeys, key = it % kTalkKeys;
+      const T* kr = row(k_cache, h / group, key);
+      float dot = 0.f;
+      for (int i = lane; i < d; i += 32) dot = fmaf(q_s[h * d + i], Cvt<T>::to_f(kr[i]), dot);
+      dot = warp_sum(dot);
+      if (lane == 0) s_s[h * (kTalkKeys + 1) + key] = dot * scale;
+    }
+    __syncthreads();
+    for (int h = warp; h < q_heads; h += warps) {   // a lane has a key
+      float s = 0.f;
+      for (int g = 0; g < q_heads; ++g) s = fmaf(Cvt<T>::to_f(talk[h * q_heads + g]), s_s[g * (kTalkKeys + 1) + lane], s);
+      if (t0 + lane < first || t0 + lane > limit) s = -INFINITY;
+      const float top = fmaxf(m_s[h], warp_max(s)), use = top == -INFINITY ? 0.f : top;
+      const float p = expf(s - use), sum = warp_sum(p);
+      p_s[h * (kTalkKeys + 1) + lane] = p;
+      __syncwarp();
+      if (lane == 0) { c_s[h] = expf(m_s[h] - use); l_s[h] = l_s[h] * c_s[h] + sum; m_s[h] = top; }
+    }
+    __syncthreads();
+    for (int it = threadIdx.x; it < q_heads * x.value_dim; it += blockDim.x) {
+      const int h = it / x.value_dim, i = it % x.value_dim;
+      float o = o_s[h * d + i] * c_s[h];
+      for (int key = 0; key < kTalkKeys; ++key) o = fmaf(p_s[h * (kTalkKeys + 1) + key], Cvt<T>::to_f(row(v_cache, h / group, key)[i]), o);
+      o_s[h * d + i] = o;
+    }
+  }
+  __syncthreads();
+  for (int it = threadIdx.x; it < q_heads * x.value_dim; it += blockDim.x) {
+    const int h = it / x.value_dim, i = it % x.value_dim;
+    const float l = l_s[h] + (x.sink ? expf(Cvt<T>::to_f(((const T*)x.sink)[h]) - m_s[h]) : 0.f);
+    out[(size_t)m * x.out_ld + it] = Cvt<T>::from_f(o_s[h * d + i] / l);
   }
 }
 
@@ -253,25 +316,48 @@ int gemm_simple(rb_ctx* ctx, const GemmArgs& a, int dtype) {
   return fail(RB_ERR_DTYPE, "gemm: dtype %d unsupported", dtype);
 }
 
-int attention_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
-                     float scale, void* out, int dtype, const AttnExtra* ext) {
-  const AttnExtra x = ext ? *ext : AttnExtra();
+template <typename T, int NJ>
+static int attention_plain_launch(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
+                                  void* out, const AttnExtra* ext) {
   const size_t loff = (size_t)layer * c->layer_stride_elems();
-  const int warps = kPlainAttnWarps;
   dim3 grid((unsigned)(batch * s_new), (unsigned)q_heads);
-  if (dtype == RB_F32)
-    attention_plain_kernel<float><<<grid, warps * 32, 0, ctx->stream>>>(
-        (const float*)q, (const float*)c->k + loff, (const float*)c->v + loff, c->block_table, c->seq_lens,
-        c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (float*)out, ext ? 1 : 0, x);
-  else if (dtype == RB_BF16)
-    attention_plain_kernel<__nv_bfloat16><<<grid, warps * 32, 0, ctx->stream>>>(
-        (const __nv_bfloat16*)q, (const __nv_bfloat16*)c->k + loff, (const __nv_bfloat16*)c->v + loff, c->block_table,
-        c->seq_lens, c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim, scale, c->window, (__nv_bfloat16*)out,
-        ext ? 1 : 0, x);
-  else
-    return fail(RB_ERR_DTYPE, "attention: dtype %d unsupported", dtype);
+  attention_plain_kernel<T, NJ><<<grid, kPlainAttnWarps * 32, 0, ctx->stream>>>(
+      (const T*)q, (const T*)c->k + loff, (const T*)c->v + loff, c->block_table, c->seq_lens, c->pages_per_seq, s_new, q_heads, c->kv_heads,
+      c->head_dim, scale, c->window, (T*)out, ext ? 1 : 0, ext ? *ext : AttnExtra());
   ctx->launches++;
   return launch_status("attention_plain");
+}
+
+int attention_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads,
+                     float scale, void* out, int dtype, const AttnExtra* ext) {
+  RB_REQUIRE(dtype == RB_F32 || dtype == RB_BF16, "attention: dtype %d unsupported", dtype);
+  RB_REQUIRE(c->head_dim <= 1024, "attention: head_dim %d exceeds 1024", c->head_dim);
+  const bool wide = c->head_dim > 256;
+  const auto run = dtype == RB_F32 ? (wide ? attention_plain_launch<float, 32> : attention_plain_launch<float, 8>)
+                                   : (wide ? attention_plain_launch<__nv_bfloat16, 32> : attention_plain_launch<__nv_bfloat16, 8>);
+  return run(ctx, q, c, layer, batch, s_new, q_heads, scale, out, ext);
+}
+
+template <typename T>
+static int talk_plain_launch(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                             const AttnExtra& x) {
+  const size_t loff = (size_t)layer * c->layer_stride_elems();
+  const size_t smem = (size_t)q_heads * (2 * c->head_dim + 2 * (kTalkKeys + 1) + 3) * sizeof(float);
+  if (smem > 200 * 1024) return fail(RB_ERR_UNIMPLEMENTED, "attention: %d mixed heads of %d exceed shared memory", q_heads, c->head_dim);
+  auto kern = attention_talk_plain_kernel<T>;
+  if (smem > 48 * 1024) RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<dim3((unsigned)(batch * s_new)), 256, smem, ctx->stream>>>((const T*)q, (const T*)c->k + loff, (const T*)c->v + loff, c->block_table,
+                                                                   c->seq_lens, c->pages_per_seq, s_new, q_heads, c->kv_heads, c->head_dim,
+                                                                   scale, (T*)out, x);
+  ctx->launches++;
+  return launch_status("attention_talk_plain");
+}
+
+int attention_talk_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                          int dtype, const AttnExtra& x) {
+  if (dtype == RB_F32) return talk_plain_launch<float>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, x);
+  if (dtype == RB_BF16) return talk_plain_launch<__nv_bfloat16>(ctx, q, c, layer, batch, s_new, q_heads, scale, out, x);
+  return fail(RB_ERR_DTYPE, "attention: dtype %d unsupported", dtype);
 }
 
 }  // namespace rb

@@ -27,6 +27,8 @@ def param_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
         return _votapel_shapes(cfg)
     if a == "kufulix":
         return _kufulix_shapes(cfg)
+    if a == "fizadra":
+        return _fizadra_shapes(cfg)
     H, I, V = cfg["hidden_size"], cfg["intermediate_size"], cfg["vocab_size"]
     nq = cfg["num_attention_heads"]
     nkv = cfg.get("num_key_value_heads") or nq
@@ -156,6 +158,34 @@ def _kufulix_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     return out + [("final.norm", (W,), "delta"), ("head", (V, W), "fan_in")]
 
 
+def _fizadra_shapes(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """Kinds as in _votapel_shapes; 'talk' is how heads mix their scores, 'depth' a layer's weights of everything before it."""
+    W, V = cfg["hidden_size"], cfg["vocab_size"]
+    out: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        mix, mlp, p = layer["mixer"], layer["mlp"], f"l{i}."
+        H, d, e, m = mix["heads"], mix["dim"], mix["vdim"], f"l{i}.mix."
+        out += [(p + n, (W,), "norm_w") for n in (("norm1", "norm2", "norm1b", "norm2b") if mlp else ("norm1", "norm1b"))]
+        if mix["type"] == "latent_attention":
+            out += [(m + "dq", (mix["q_rank"], W), "fan_in"), (m + "dq.norm", (mix["q_rank"],), "norm_w"),
+                    (m + "uq", (H * (d + mix["rot_dim"]), mix["q_rank"]), "fan_in")]
+            if mix["kv_from"] is None:
+                out += [(m + "dkv", (mix["kv_rank"] + mix["rot_dim"], W), "fan_in"), (m + "dkv.norm", (mix["kv_rank"],), "norm_w")]
+            out += [(m + "uk", (H * d, mix["kv_rank"]), "fan_in"), (m + "uv", (H * e, mix["kv_rank"]), "fan_in")]
+            if mix["sink"]:
+                out.append((m + "sink", (H,), "sink"))
+            out.append((m + "g", (H * e if mix["gate"] == "elements" else H, W), "fan_in"))
+        else:
+            for n, rows in (("q", H * d), ("k", mix["kv_heads"] * d), ("v", mix["kv_heads"] * e)):
+                out += [(m + n, (rows, W), "fan_in"), (m + n + ".b", (rows,), "bias")]
+            out += [(m + "q.norm", (d,), "norm_w"), (m + "k.norm", (d,), "norm_w"), (m + "talk", (H, H), "talk")]
+        out.append((m + "o", (W, H * e), "fan_in"))
+        if mlp:
+            out += [(p + "mlp.up", (mlp["ff"], W), "fan_in"), (p + "mlp.down", (W, mlp["ff"]), "fan_in")]
+        out.append((p + "dwa", (i + 2,), "depth"))
+    return out + [("final.norm", (W,), "norm_w"), ("head", (V, W), "fan_in")]
+
+
 def bf16_round(x: np.ndarray) -> np.ndarray:
     """float32 -> nearest-even bfloat16 -> float32 (so the CPU oracle and the GPU see the same values)."""
     u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
@@ -177,6 +207,8 @@ _DRAWS = {
     "decay": lambda r, s: r.uniform(-1.0, 2.5, s),
     "skip": lambda r, s: 1.0 + 0.3 * r.standard_normal(s),
     "correction": lambda r, s: 0.05 * r.standard_normal(s),
+    "talk": lambda r, s: np.eye(s[0]) + r.standard_normal(s) / np.sqrt(s[0]),
+    "depth": lambda r, s: np.append(0.3 * r.standard_normal(s[0] - 1), 1.0),
 }
 
 
