@@ -134,7 +134,7 @@ extern "C" int32_t rb_sync(rb_ctx* ctx) {
     if (code == RB_ERR_TIMEOUT) {
       // blocks that gave up returned before they were counted: re-arm the self-resetting arrival counters
       for (rb_kv_cache* kc : ctx->caches)
-        RB_CUDA(cudaMemset(kc->split_count, 0, (size_t)kc->max_batch * kc->kv_heads * sizeof(uint32_t)));
+        RB_CUDA(cudaMemset(kc->split_count, 0, kc->split_counters() * sizeof(uint32_t)));
       RB_CUDA(cudaMemset(ctx->argmax_best, 0, kArgmaxRows * sizeof(unsigned long long)));
       RB_CUDA(cudaMemset(ctx->argmax_count, 0, kArgmaxRows * sizeof(unsigned int)));
       RB_CUDA(cudaMemset(ctx->gemm_tile_count, 0, 2 * kGemmMaxReduceTiles * sizeof(uint32_t)));
@@ -265,7 +265,7 @@ int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_hea
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->num_pages * sizeof(int32_t), (void**)&c->block_table);
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->seq_lens);
   if (st == RB_OK && !shared) st = rb_malloc(ctx, (size_t)c->max_batch * sizeof(int32_t), (void**)&c->slots);
-  if (st == RB_OK) st = rb_malloc(ctx, (size_t)c->max_batch * kv_heads * sizeof(uint32_t), (void**)&c->split_count);
+  if (st == RB_OK) st = rb_malloc(ctx, c->split_counters() * sizeof(uint32_t), (void**)&c->split_count);
   if (st != RB_OK) { rb_kv_cache_destroy(c); return st; }
   // Zero the pages: the tail of a sequence's last page is read (and masked) by the attention
   // kernels, so it must hold finite values.
@@ -287,7 +287,7 @@ int rb::kv_cache_create(rb_ctx* ctx, rb_kv_cache* shared, int layers, int kv_hea
     RB_CUDA(cudaMemsetAsync(c->seq_lens, 0, (size_t)c->max_batch * sizeof(int32_t), ctx->stream));
     c->own_lens.assign(c->max_batch, 0);
   }
-  RB_CUDA(cudaMemsetAsync(c->split_count, 0, (size_t)c->max_batch * kv_heads * sizeof(uint32_t), ctx->stream));
+  RB_CUDA(cudaMemsetAsync(c->split_count, 0, c->split_counters() * sizeof(uint32_t), ctx->stream));
   RB_CUDA(cudaStreamSynchronize(ctx->stream));
   ctx->caches.push_back(c);
   *out = c;
@@ -564,8 +564,9 @@ extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache*
   if (x.talk) {
     RB_REQUIRE(!x.alibi && !x.gate && !x.temp_every && x.softcap == 0.f && x.out_scale == 1.f,
                "rb_attention_general: mixed heads go with window, chunk, sink and value_dim only");
-    return attention_talk_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, x);
   }
+  if (!ctx->debug_simple_attn && attention_joint_takes(c, x)) return attention_joint(ctx, q, c, layer, batch, s_new, q_heads, scale, out, x);
+  if (x.talk) return attention_talk_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, x);
   if (!ctx->debug_simple_attn && attention_mma_takes(c, q_heads))
     return attention_mma_bf16(ctx, q, c, layer, batch, s_new, q_heads, scale, out, &x);
   return attention_simple(ctx, q, c, layer, batch, s_new, q_heads, scale, out, dtype, &x);

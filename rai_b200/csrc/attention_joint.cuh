@@ -1,0 +1,592 @@
+// Attention in which one block has every head of its tokens, over the paged bf16 cache: heads whose scores are mixed before the
+// softmax (score[h] <- sum_g talk[h][g] score[g]), and latent attention, where all heads read one wide vector per token that
+// serves as key and, up to the latent's size, as value.  Prompts, portions of them and single tokens run the same kernel.
+//
+// Eight consumer warps and one that issues tiled copies.  Per tile of KT keys:
+//   1  scores, transposed: S^T[keys x rows] = K . Q^T on mma.sync, a row being a (token, query head) that reads the tile's
+//      key/value head; keys fill the 16-row side, so a single token's few heads waste nothing.  Raw scores go to shared memory.
+//   2  a warp takes eight heads of a token (or eight rows): lanes are keys.  It mixes the raw scores of all heads (float32),
+//      masks, and turns them into weights against a reference point that follows the running maximum lazily; weights go to
+//      shared memory in bf16, the sum of a row stays in float32.
+//   3  O^T[dims x rows] += V^T . P^T, accumulators in registers for the whole walk.
+// The eight warps form teams of WG; a team has every TEAMS-th key/value head and reads only that head's tiles.  Inside a team the
+// warps share out the dimensions of V, and for K two key halves times parts of the dot product (partial scores add in step 2).
+// Copies run ahead through a ring of tiles: K of every head, then V of every head, and so on.
+//
+// Every wait is bounded; after a give-up the block runs on without waiting, writes nothing, reports, lets its copies land and
+// returns.
+#pragma once
+#include <algorithm>
+#include <vector>
+
+#include "ctx.h"
+#include "mma.cuh"
+#include "ptx.cuh"
+
+namespace rb {
+
+using bf16 = __nv_bfloat16;
+
+namespace joint {
+
+constexpr float kLog2e = 1.4426950408889634f;
+// Two warpgroups of consumers and one for the copies, which hands its registers over: 384 x 168 = 256 x 232 + 128 x 40.
+constexpr int kConsumers = 256, kThreads = 384;
+constexpr int kMaxStages = 24;
+constexpr int kMaxSplits = 32;
+
+struct Params {
+  const bf16* q;               // [tokens][q_heads][D]
+  const int32_t *block_table, *seq_lens;
+  int pages_per_seq, s_new, D, q_heads, kv_heads, group;
+  int row_tiles, tile_rows;    // rows (token, head of a key/value head) of a block: tile_rows <= 8 NT
+  int nbk, nbv;                // 64-column blocks of a key and of a value that matter
+  int stages, stage_bytes;
+  int n_splits;
+  int window, chunk, value_dim;
+  float scale_log2;
+  const bf16 *talk, *sink;
+  bf16* out;
+  int64_t out_ld;
+  float *part_o, *part_ml;
+  uint32_t *split_count, *status;
+  long long wait_cycles;
+};
+
+// LATENT: one key/value head whose keys are the values, nothing mixed
+template <int KT_, int WG_, int GP_, int DW_, int NT_, bool LATENT_>
+struct Shape {
+  static constexpr int KT = KT_, WG = WG_, GP = GP_, DW = DW_, NT = NT_;
+  static constexpr bool LATENT = LATENT_;
+  static constexpr int TEAMS = 8 / WG;
+  static constexpr int SM = WG < 2 ? 1 : 2, SK = WG / SM;     // key halves, parts of the dot product
+  static constexpr int MK = KT / 16 / SM;                     // 16-key tiles of a warp
+  static constexpr int R = 8 * NT;                            // rows per key/value head
+  static constexpr int SP = KT + 4, PP = KT + 8;              // pitches of scores (floats) and weights (bf16)
+  static constexpr int KL = KT / 32;                          // keys per lane
+};
+
+struct Layout {   // byte offsets behind the ring
+  size_t q, s, p, talk, m, total;
+};
+template <typename S>
+__host__ __device__ inline Layout layout_of(int G, int H, int nbk) {
+  Layout l;
+  size_t at = 0;
+  const size_t rows = (size_t)G * S::R;
+  l.q = at; at += rows * (nbk * 64 + 8) * 2;
+  l.s = at; at += (size_t)S::SK * rows * S::SP * 4;
+  l.p = at; at += rows * S::PP * 2;
+  l.talk = at; at += S::LATENT ? 0 : (size_t)H * ((H + 7) / 8 * 8) * 4;
+  l.m = at; at += rows * 3 * 4;
+  l.total = at;
+  return l;
+}
+
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)),
+        "l"(reinterpret_cast<unsigned long long&>(c)));
+  return r;
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t& r0, uint32_t& r1, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+__device__ __forceinline__ void take_registers() { asm volatile("setmaxnreg.inc.sync.aligned.u32 232;"); }
+__device__ __forceinline__ void give_registers() { asm volatile("setmaxnreg.dec.sync.aligned.u32 40;"); }
+__device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+
+// byte offset of the 16-byte chunk with (key, dims dc..dc+8) in a tile of column blocks [KT keys][128 bytes], 128-byte swizzle
+template <int KT>
+__device__ __forceinline__ int tile_off(int key, int dc) {
+  return (dc >> 6) * (KT * 128) + key * 128 + ((((dc & 63) >> 3) ^ (key & 7)) << 4);
+}
+
+// Merges the splits of a single token's rows (the consumer warps; w_s: [row][split] weights over the row's sum)
+template <typename S>
+__device__ __forceinline__ void merge_splits(const Params& p, float* w_s, int b, int r0, int n_rows) {
+  const int H = p.q_heads, vd = p.value_dim, ns = p.n_splits;
+  const int live = S::LATENT ? n_rows : H;   // heads of the tile, or of the token
+  auto head_of = [&](int i) { return S::LATENT ? (r0 + i) % p.group : i; };
+  for (int i = threadIdx.x; i < live; i += kConsumers) {
+    const int head = head_of(i);
+    const float* ml = p.part_ml + ((size_t)b * H + head) * ns * 2;
+    float M = -INFINITY, L = 0.f;
+    for (int s = 0; s < ns; ++s) M = fmaxf(M, __ldcg(ml + 2 * s));
+    for (int s = 0; s < ns; ++s) {
+      const float w = ex2_fast(__ldcg(ml + 2 * s) - M);
+      L = fmaf(w, __ldcg(ml + 2 * s + 1), L);
+      w_s[i * kMaxSplits + s] = w;
+    }
+    if (p.sink) L += ex2_fast(fmaf(__bfloat162float(p.sink[head]), kLog2e, -M));
+    const float inv = 1.0f / L;
+    for (int s = 0; s < ns; ++s) w_s[i * kMaxSplits + s] *= inv;
+  }
+  consumers_sync();
+  for (int i = threadIdx.x; i < live * vd; i += kConsumers) {
+    const int row = i / vd, dim = i % vd, head = head_of(row);
+    const float* src = p.part_o + ((size_t)b * H + head) * ns * vd + dim;
+    float v = 0.f;
+    for (int s0 = 0; s0 < ns; s0 += 8) {
+      float t[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) t[k] = s0 + k < ns ? __ldcg(src + (size_t)(s0 + k) * vd) : 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+        if (s0 + k < ns) v = fmaf(t[k], w_s[row * kMaxSplits + s0 + k], v);
+    }
+    p.out[(size_t)b * p.out_ld + (size_t)head * vd + dim] = __float2bfloat16_rn(v);
+  }
+}
+
+template <typename S>
+__global__ void __launch_bounds__(kThreads, 1) kernel(const Params p, const __grid_constant__ CUtensorMap tm_k,
+                                                      const __grid_constant__ CUtensorMap tm_v) {
+  constexpr int KT = S::KT, NT = S::NT, R = S::R, GP = S::GP, DW = S::DW, SP = S::SP, PP = S::PP, KL = S::KL;
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t full_bar[kMaxStages];
+  __shared__ __align__(8) uint64_t empty_bar[kMaxStages];
+  __shared__ volatile uint32_t abort_flag;
+  __shared__ volatile int rescale_flag[2];
+  __shared__ uint32_t issued_count, is_last;
+  uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int G = p.kv_heads, H = p.q_heads, group = p.group;
+  const Layout lay = layout_of<S>(G, H, p.nbk);
+  uint8_t* rest = ring + (size_t)p.stages * p.stage_bytes;
+  bf16* q_s = reinterpret_cast<bf16*>(rest + lay.q);
+  float* s_s = reinterpret_cast<float*>(rest + lay.s);
+  bf16* p_s = reinterpret_cast<bf16*>(rest + lay.p);
+  float* t_s = reinterpret_cast<float*>(rest + lay.talk);     // [g][h]: scale * log2(e) * talk[h][g]
+  float* m_s = reinterpret_cast<float*>(rest + lay.m);        // reference point, sum, rescaling factor per row
+  const int rows = G * R, qp = p.nbk * 64 + 8, hp = (H + 7) / 8 * 8;
+  float* l_s = m_s + rows;
+  float* c_s = l_s + rows;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(&full_bar[s], 1); ptx::mbar_init(&empty_bar[s], S::WG); }
+    abort_flag = 0;
+    rescale_flag[0] = rescale_flag[1] = 0;
+    issued_count = 0;
+    ptx::fence_barrier_init();
+    ptx::fence_proxy_async();
+    ptx::tma_prefetch_desc(&tm_k);
+    if (!S::LATENT) ptx::tma_prefetch_desc(&tm_v);
+  }
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();   // q, lengths and the newest keys come from kernels before this one
+
+  const int split = blockIdx.x, b = blockIdx.z;
+  const int tile_row = p.s_new > 1 ? (int)gridDim.y - 1 - (int)blockIdx.y : (int)blockIdx.y;   // longest walks first
+  const int r0 = tile_row * p.tile_rows, total_rows = p.s_new * group;
+  const int n_rows = min(p.tile_rows, total_rows - r0);
+  const int len = p.seq_lens[b], base = len - p.s_new;
+  const int first_token = r0 / group, last_token = (r0 + n_rows - 1) / group;
+  int tile_lo = first_visible(base + first_token, p.window, p.chunk) / KT;
+  int tile_hi = (min(base + last_token + 1, len) + KT - 1) / KT;
+  if (p.n_splits > 1) {
+    const int per = (tile_hi - tile_lo + p.n_splits - 1) / p.n_splits;
+    tile_lo += split * per;
+    tile_hi = min(tile_hi, tile_lo + per);
+  }
+  const int units = S::LATENT ? 1 : 2 * G;   // copies per key tile
+
+  if (warp >= 8) {
+    // ------------------------------------------------------------------ copies
+    give_registers();
+    if (warp == 8 && lane == 0) {
+      uint32_t u = 0;
+      bool ok = true;
+      for (int tile = tile_lo; tile < tile_hi && ok; ++tile) {
+        const int page = p.block_table[(size_t)b * p.pages_per_seq + tile * KT / kPageTokens];
+        for (int i = 0; i < units && ok; ++i, ++u) {
+          const int st = u % p.stages;
+          if (!ptx::mbar_wait(&empty_bar[st], ((u / p.stages) & 1u) ^ 1u, &abort_flag, p.wait_cycles)) { ok = false; break; }
+          const bool v = i >= G;
+          const int nb = v ? p.nbv : p.nbk, y = (page * G + (v ? i - G : i)) * kPageTokens + tile * KT % kPageTokens;
+          ptx::mbar_expect_tx(&full_bar[st], (uint32_t)nb * KT * 128);
+          for (int cb = 0; cb < nb; ++cb)
+            ptx::tma_load_2d(ring + (size_t)st * p.stage_bytes + cb * (KT * 128), v ? &tm_v : &tm_k, &full_bar[st], cb * 64, y);
+          issued_count = u + 1;
+        }
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ what the walk starts from
+    take_registers();
+    float o[GP][DW][NT][4];
+    for (int i = threadIdx.x; i < rows * (p.nbk * 8); i += kConsumers) {
+      const int row = i / (p.nbk * 8), c = i % (p.nbk * 8) * 8, g = row / R, n = row % R;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (n < n_rows) {
+        const int token = (r0 + n) / group, head = g * group + (r0 + n) % group;
+        v = *reinterpret_cast<const uint4*>(p.q + (((size_t)b * p.s_new + token) * H + head) * p.D + c);
+      }
+      *reinterpret_cast<uint4*>(q_s + (size_t)row * qp + c) = v;
+    }
+    for (int i = threadIdx.x; i < rows * (PP / 8); i += kConsumers) reinterpret_cast<uint4*>(p_s)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < rows; i += kConsumers) { m_s[i] = -INFINITY; l_s[i] = 0.f; c_s[i] = 1.f; }
+    if (!S::LATENT)
+      for (int i = threadIdx.x; i < H * hp; i += kConsumers) {
+        const int g = i / hp, h = i % hp;
+        t_s[i] = h < H ? __bfloat162float(p.talk[h * H + g]) * p.scale_log2 : 0.f;
+      }
+    consumers_sync();
+#pragma unroll
+    for (int a = 0; a < GP; ++a)
+#pragma unroll
+      for (int d = 0; d < DW; ++d)
+#pragma unroll
+        for (int n = 0; n < NT; ++n) { o[a][d][n][0] = o[a][d][n][1] = o[a][d][n][2] = o[a][d][n][3] = 0.f; }
+
+    const int team = warp / S::WG, wi = warp % S::WG, g8 = lane >> 2, t4 = lane & 3;
+    const int km = wi % S::SM, ks = wi / S::SM;
+    const int steps = p.nbk * 4, per_part = (steps + S::SK - 1) / S::SK, k_lo = ks * per_part, k_hi = min(steps, k_lo + per_part);
+    const int live_heads = p.value_dim;
+    for (int tile = tile_lo; tile < tile_hi; ++tile) {
+      const int it = tile - tile_lo, key0 = tile * KT;
+      // ---------------------------------------------------------------- 1: raw scores
+#pragma unroll
+      for (int a = 0; a < GP; ++a) {
+        const int g = a * S::TEAMS + team;
+        if (g >= G) continue;
+        const uint32_t u = (uint32_t)it * units + g, st = u % p.stages;
+        ptx::mbar_wait(&full_bar[st], (u / p.stages) & 1u, &abort_flag, p.wait_cycles);
+        __syncwarp();
+        const uint32_t kt = s_u32(ring + (size_t)st * p.stage_bytes);
+        constexpr int NC = NT < 4 ? NT : 4;
+#pragma unroll
+        for (int nc = 0; nc < NT / NC; ++nc) {
+          float s[S::MK][NC][4];
+#pragma unroll
+          for (int m = 0; m < S::MK; ++m)
+#pragma unroll
+            for (int n = 0; n < NC; ++n) { s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f; }
+          const uint32_t qa = s_u32(q_s + (size_t)(g * R + nc * NC * 8) * qp);
+#pragma unroll 4
+          for (int kk = k_lo; kk < k_hi; ++kk) {
+            uint32_t af[S::MK][4];
+#pragma unroll
+            for (int m = 0; m < S::MK; ++m)
+              ldsm_x4(af[m], kt + tile_off<KT>(km * (KT / S::SM) + m * 16 + (lane & 15), kk * 16 + (lane >> 4) * 8));
+            if constexpr (NC == 1) {
+              uint32_t b0, b1;
+              ldsm_x2(b0, b1, qa + (uint32_t)(((lane & 7) * qp + kk * 16 + ((lane >> 3) & 1) * 8) * 2));
+#pragma unroll
+              for (int m = 0; m < S::MK; ++m) mma16816(s[m][0], af[m], b0, b1);
+            } else {
+#pragma unroll
+              for (int j = 0; j < NC / 2; ++j) {
+                uint32_t bf[4];
+                ldsm_x4(bf, qa + (uint32_t)(((j * 16 + (lane & 7) + ((lane >> 4) << 3)) * qp + kk * 16 + ((lane >> 3) & 1) * 8) * 2));
+#pragma unroll
+                for (int m = 0; m < S::MK; ++m) { mma16816(s[m][2 * j], af[m], bf[0], bf[1]); mma16816(s[m][2 * j + 1], af[m], bf[2], bf[3]); }
+              }
+            }
+          }
+          float* dst = s_s + ((size_t)ks * rows + g * R + nc * NC * 8) * SP + km * (KT / S::SM);
+#pragma unroll
+          for (int m = 0; m < S::MK; ++m)
+#pragma unroll
+            for (int n = 0; n < NC; ++n)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) dst[(n * 8 + 2 * t4 + (e & 1)) * SP + m * 16 + g8 + (e >> 1) * 8] = s[m][n][e];
+        }
+        if (!S::LATENT) {
+          __syncwarp();
+          if (lane == 0) ptx::mbar_arrive(&empty_bar[st]);
+        }
+      }
+      consumers_sync();
+      // ---------------------------------------------------------------- 2: mixing, mask, weights
+      if (threadIdx.x == 0) rescale_flag[(it + 1) & 1] = 0;
+      const int chunks = S::LATENT ? (n_rows + 7) / 8 : hp / 8, n_units = S::LATENT ? chunks : chunks * (n_rows / group);
+      for (int unit = warp; unit < n_units; unit += 8) {
+        const int tok = S::LATENT ? 0 : unit / chunks, h0 = (S::LATENT ? unit : unit % chunks) * 8;   // eight heads, or eight rows
+        float2 acc[4][KL];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(0.f, 0.f);
+        auto raw = [&](int row, float* v) {
+#pragma unroll
+          for (int e = 0; e < KL; ++e) v[e] = 0.f;
+#pragma unroll
+          for (int k = 0; k < S::SK; ++k) {
+            const float* src = s_s + ((size_t)k * rows + row) * SP + lane * KL;
+            if constexpr (KL == 1) v[0] += src[0];
+            else { const float2 t = *reinterpret_cast<const float2*>(src); v[0] += t.x; v[KL - 1] += t.y; }
+          }
+        };
+        if (S::LATENT) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            float x[KL], y[KL];
+            raw(h0 + 2 * i, x);
+            raw(h0 + 2 * i + 1, y);
+#pragma unroll
+            for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(x[e] * p.scale_log2, y[e] * p.scale_log2);
+          }
+        } else {
+          int row = tok * group, j = 0;
+#pragma unroll 4
+          for (int g = 0; g < H; ++g) {
+            float x[KL];
+            raw(row, x);
+            const float4 t0 = *reinterpret_cast<const float4*>(t_s + g * hp + h0), t1 = *reinterpret_cast<const float4*>(t_s + g * hp + h0 + 4);
+#pragma unroll
+            for (int e = 0; e < KL; ++e) {
+              const float2 xx = make_float2(x[e], x[e]);
+              acc[0][e] = fma2(make_float2(t0.x, t0.y), xx, acc[0][e]);
+              acc[1][e] = fma2(make_float2(t0.z, t0.w), xx, acc[1][e]);
+              acc[2][e] = fma2(make_float2(t1.x, t1.y), xx, acc[2][e]);
+              acc[3][e] = fma2(make_float2(t1.z, t1.w), xx, acc[3][e]);
+            }
+            ++row;
+            if (++j == group) { j = 0; row += R - group; }
+          }
+        }
+        float sum[8];
+        int seen_lo = 0, seen_hi = 0;
+        if (!S::LATENT) {
+          seen_hi = base + r0 / group + tok;
+          seen_lo = first_visible(seen_hi, p.window, p.chunk);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          sum[i] = 0.f;
+          int row;
+          if (S::LATENT) {
+            row = h0 + i;
+            if (row >= n_rows) continue;
+            seen_hi = base + (r0 + row) / group;
+            seen_lo = first_visible(seen_hi, p.window, p.chunk);
+          } else {
+            const int h = h0 + i;
+            if (h >= H) continue;
+            row = h / group * R + tok * group + h % group;
+          }
+          float v[KL], top = -INFINITY;
+#pragma unroll
+          for (int e = 0; e < KL; ++e) {
+            const int key = key0 + lane * KL + e;
+            const float x = (i & 1) ? acc[i >> 1][e].y : acc[i >> 1][e].x;
+            v[e] = key <= seen_hi && key >= seen_lo ? x : -INFINITY;
+            top = fmaxf(top, v[e]);
+          }
+          // the reference point moves only when the maximum has outgrown it by 2^8
+          const float m_old = m_s[row];
+          float m_new = m_old;
+          if (__any_sync(0xffffffffu, top > m_old + 8.0f)) m_new = fmaxf(m_old, warp_max(top));
+          const float use = m_new == -INFINITY ? 0.f : m_new;
+#pragma unroll
+          for (int e = 0; e < KL; ++e) { v[e] = ex2_fast(v[e] - use); sum[i] += v[e]; }
+          bf16* dst = p_s + (size_t)row * PP + lane * KL;
+          if constexpr (KL == 1) dst[0] = __float2bfloat16_rn(v[0]);
+          else *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v[0], v[KL - 1]);
+          if (m_new != m_old) {   // warp-uniform, rare
+            __syncwarp();         // every lane has read the old one
+            if (lane == 0) {
+              const float c = ex2_fast(m_old - use);
+              m_s[row] = m_new;
+              c_s[row] = c;
+              l_s[row] *= c;
+              if (m_old != -INFINITY) rescale_flag[it & 1] = 1;
+            }
+          } else if (lane == 0) {
+            c_s[row] = 1.f;
+          }
+        }
+        // eight sums over the lanes at once; lane 4 i ends up with the i-th
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const bool up = lane & 16;
+          const float keep = up ? sum[i + 4] : sum[i], send = up ? sum[i] : sum[i + 4];
+          sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, 16);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const bool up = lane & 8;
+          const float keep = up ? sum[i + 2] : sum[i], send = up ? sum[i] : sum[i + 2];
+          sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
+        }
+        {
+          const bool up = lane & 4;
+          const float keep = up ? sum[1] : sum[0], send = up ? sum[0] : sum[1];
+          sum[0] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+        }
+        sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 2);
+        sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 1);
+        __syncwarp();   // (lane 0 may have rescaled a row's sum)
+        if ((lane & 3) == 0) {
+          const int h = h0 + (lane >> 2);
+          if (S::LATENT ? h < n_rows : h < H) l_s[S::LATENT ? h : h / group * R + tok * group + h % group] += sum[0];
+        }
+        __syncwarp();
+      }
+      consumers_sync();
+      // ---------------------------------------------------------------- 3: values
+      const bool rescale = rescale_flag[it & 1] != 0;
+#pragma unroll
+      for (int a = 0; a < GP; ++a) {
+        const int g = a * S::TEAMS + team;
+        if (g >= G) continue;
+        const uint32_t u = (uint32_t)it * units + (S::LATENT ? 0 : G + g), st = u % p.stages;
+        if (!S::LATENT) {
+          ptx::mbar_wait(&full_bar[st], (u / p.stages) & 1u, &abort_flag, p.wait_cycles);
+          __syncwarp();
+        }
+        const uint32_t vt = s_u32(ring + (size_t)st * p.stage_bytes);
+        if (rescale) {
+#pragma unroll
+          for (int n = 0; n < NT; ++n) {
+            const float c0 = c_s[g * R + n * 8 + 2 * t4], c1 = c_s[g * R + n * 8 + 2 * t4 + 1];
+#pragma unroll
+            for (int d = 0; d < DW; ++d) { o[a][d][n][0] *= c0; o[a][d][n][1] *= c1; o[a][d][n][2] *= c0; o[a][d][n][3] *= c1; }
+          }
+        }
+#pragma unroll
+        for (int k2 = 0; k2 < KL; ++k2) {
+          uint32_t pf[NT][4];   // weights of 32 keys
+#pragma unroll
+          for (int n = 0; n < NT; ++n)
+            ldsm_x4(pf[n], s_u32(p_s + (size_t)(g * R + n * 8 + (lane & 7)) * PP + k2 * 32 + (lane >> 3) * 8));
+#pragma unroll
+          for (int d = 0; d < DW; ++d) {
+            const int dim0 = (wi * DW + d) * 16;
+            if (dim0 >= live_heads) continue;
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+              uint32_t af[4];
+              ldsm_x4_t(af, vt + tile_off<KT>(k2 * 32 + hf * 16 + (lane & 7) + ((lane >> 4) << 3), dim0 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+              for (int n = 0; n < NT; ++n) mma16816(o[a][d][n], af, pf[n][2 * hf], pf[n][2 * hf + 1]);
+            }
+          }
+        }
+        __syncwarp();
+        if (lane == 0) ptx::mbar_arrive(&empty_bar[st]);
+      }
+    }
+    consumers_sync();
+    if (!abort_flag) {
+      // ---------------------------------------------------------------- output
+      const int vd = p.value_dim, ns = p.n_splits;
+#pragma unroll
+      for (int a = 0; a < GP; ++a) {
+        const int g = a * S::TEAMS + team;
+        if (g >= G) continue;
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int e2 = 0; e2 < 2; ++e2) {
+            const int row = n * 8 + 2 * t4 + e2;
+            if (row >= n_rows) continue;
+            const int token = (r0 + row) / group, head = g * group + (r0 + row) % group;
+            const float m = m_s[g * R + row];
+            float l = l_s[g * R + row];
+            if (ns == 1) {
+              if (p.sink) l += ex2_fast(fmaf(__bfloat162float(p.sink[head]), kLog2e, -m));
+              const float inv = 1.0f / l;
+              bf16* dst = p.out + ((size_t)b * p.s_new + token) * p.out_ld + (size_t)head * vd;
+#pragma unroll
+              for (int d = 0; d < DW; ++d) {
+                const int dim = (wi * DW + d) * 16 + g8;
+                if (dim < vd) dst[dim] = __float2bfloat16_rn(o[a][d][n][e2] * inv);
+                if (dim + 8 < vd) dst[dim + 8] = __float2bfloat16_rn(o[a][d][n][2 + e2] * inv);
+              }
+            } else {
+              const size_t at = ((size_t)b * H + head) * ns + split;   // (single tokens)
+#pragma unroll
+              for (int d = 0; d < DW; ++d) {
+                const int dim = (wi * DW + d) * 16 + g8;
+                if (dim < vd) p.part_o[at * vd + dim] = o[a][d][n][e2];
+                if (dim + 8 < vd) p.part_o[at * vd + dim + 8] = o[a][d][n][2 + e2];
+              }
+              if (wi == 0 && g8 == 0) { p.part_ml[at * 2] = m; p.part_ml[at * 2 + 1] = l; }
+            }
+          }
+      }
+      if (ns > 1) {
+        // The block that arrives last for these rows merges all splits, in split order.
+        __threadfence();
+        consumers_sync();
+        if (threadIdx.x == 0) {
+          uint32_t* cnt = p.split_count + (size_t)b * p.row_tiles + tile_row;
+          is_last = atomicAdd(cnt, 1u) == (uint32_t)ns - 1u ? 1u : 0u;
+          if (is_last) *cnt = 0u;   // re-armed for the next launch
+          __threadfence();
+        }
+        consumers_sync();
+        if (is_last) merge_splits<S>(p, reinterpret_cast<float*>(ring), b, r0, n_rows);
+      }
+    }
+  }
+  __syncthreads();
+  if (abort_flag && threadIdx.x == 0) {
+    p.status[0] = (uint32_t)(-RB_ERR_TIMEOUT); p.status[1] = 0xA701u; p.status[2] = blockIdx.y; p.status[3] = blockIdx.z;
+    volatile uint32_t never = 0;   // copies already on their way get a bounded chance to land
+    for (uint32_t u = issued_count > (uint32_t)p.stages ? issued_count - p.stages : 0; u < issued_count; ++u)
+      ptx::mbar_wait(&full_bar[u % p.stages], (u / p.stages) & 1u, &never, p.wait_cycles);
+  }
+}
+
+constexpr size_t kSmemLimit = 227 * 1024 - 4096;   // (the static part and alignment)
+
+// Ring depth that fits; 0: not even two tiles do
+template <typename S>
+int ring_of(const Params& p, size_t* bytes) {
+  const Layout l = layout_of<S>(p.kv_heads, p.q_heads, p.nbk);
+  if (l.total + 2 * (size_t)p.stage_bytes > kSmemLimit) return 0;
+  const int stages = (int)std::min<size_t>({(size_t)kMaxStages, (kSmemLimit - l.total) / p.stage_bytes, (size_t)std::max(3, 2 * 96 * 1024 / p.stage_bytes)});
+  *bytes = l.total + (size_t)stages * p.stage_bytes + 1024;
+  return stages;
+}
+
+// RB_ERR_UNIMPLEMENTED (without an error text): this shape does not fit
+template <typename S>
+int launch(rb_ctx* ctx, rb_kv_cache* c, Params p, int layer, int batch, int max_len) {
+  p.stage_bytes = S::KT * 128 * std::max(p.nbk, S::LATENT ? 0 : p.nbv);
+  size_t smem = 0;
+  p.stages = ring_of<S>(p, &smem);
+  const int whole = p.s_new * p.group;
+  p.tile_rows = std::min(whole, S::LATENT ? S::R : S::R / p.group * p.group);
+  if (p.stages == 0 || p.tile_rows == 0) return RB_ERR_UNIMPLEMENTED;
+  p.row_tiles = (whole + p.tile_rows - 1) / p.tile_rows;
+  p.n_splits = 1;
+  if (p.s_new == 1 && p.row_tiles <= (S::LATENT ? ::kLatentRowTiles : 1)) {
+    p.n_splits = attention_decode_splits(ctx, batch, p.row_tiles, max_len, 256);
+    if (p.n_splits > kMaxSplits) p.n_splits = kMaxSplits;
+    if (p.n_splits > 1) {
+      const size_t parts = (size_t)batch * p.q_heads * p.n_splits;
+      RB_TRY(attention_reserve_scratch(ctx, parts * (p.value_dim + 2) * sizeof(float)));
+      p.part_o = ctx->attn_scratch;
+      p.part_ml = ctx->attn_scratch + parts * p.value_dim;
+    }
+  }
+  auto kern = kernel<S>;
+  static size_t set[64] = {};
+  const int dv = ctx->device & 63;
+  if (smem > set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set[dv] = smem; }
+  CUtensorMap tk{}, tv{};
+  const size_t off = (size_t)layer * c->layer_stride_elems();
+  const int64_t rows = (int64_t)c->num_pages * c->kv_heads * kPageTokens;
+  RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->k + off, rows, p.D, p.D, S::KT, &tk));
+  if (!S::LATENT) RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->v + off, rows, p.D, p.D, S::KT, &tv));
+  const dim3 grid((unsigned)p.n_splits, (unsigned)p.row_tiles, (unsigned)batch);
+  if (grid.y > 65535) return RB_ERR_UNIMPLEMENTED;
+  RB_CUDA(launch_kernel(kern, grid, dim3(kThreads), smem, ctx->stream, ctx->pdl, p, tk, tv));
+  ctx->launches++;
+  return RB_OK;
+}
+
+}  // namespace joint
+
+}  // namespace rb

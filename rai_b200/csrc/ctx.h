@@ -58,6 +58,8 @@ struct rb_ctx {
 // A design whose layers differ in head counts or sizes has one cache per geometry over ONE set of sequences: the
 // first owns the tables (block table, lengths, state slots), the others are views that share them (`tables`).  A
 // cache with layers == 0 is only the tables.
+constexpr int kLatentRowTiles = 16;   // arrival counters per sequence of a cache with one head that is key and value
+
 struct rb_kv_cache {
   explicit rb_kv_cache(rb_kv_cache* shared = nullptr)
       : tables(shared), host_lens(shared ? shared->host_lens : own_lens) {}
@@ -74,8 +76,9 @@ struct rb_kv_cache {
   int32_t* seq_lens = nullptr;     // device [max_batch]
   int32_t* slots = nullptr;        // device [max_batch]: where sequence b keeps its recurrent and convolution state
   std::vector<int32_t> host_table, host_slots;  // host copies of block_table and slots
-  uint32_t* split_count = nullptr;  // device [max_batch][kv_heads]: arrivals of a split decode attention; self-resetting
+  uint32_t* split_count = nullptr;  // device [max_batch][kv_heads] (one shared head: [max_batch][kLatentRowTiles]): arrivals of a split decode attention; self-resetting
   std::vector<int32_t>& host_lens;
+  size_t split_counters() const { return (size_t)max_batch * (shared() && kv_heads == 1 ? kLatentRowTiles : kv_heads); }
   size_t layer_stride_elems() const { return (size_t)num_pages * kv_heads * 64 * head_dim; }
 };
 
@@ -304,6 +307,11 @@ int attention_reserve_scratch(rb_ctx* ctx, size_t bytes);
 bool attention_prefill_tc_supported(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const void* out);
 int attention_prefill_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale,
                          void* out, const AttnExtra* ext = nullptr);
+// attention_latent.cu, attention_talk.cu: attention with mixed heads or over latents, one block for all heads of its tokens
+bool attention_joint_takes(const rb_kv_cache* c, const AttnExtra& x);
+int attention_joint_row_tiles(const rb_kv_cache* c, int q_heads);   // blocks a single token's heads take
+int attention_joint(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                    const AttnExtra& x);
 // plain_kernels.cu: attention whose heads' scores are mixed (x.talk), any sizes
 int attention_talk_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
                           int dtype, const AttnExtra& x);

@@ -459,7 +459,9 @@ int rb::layered_decode_plan(rb_model* m, int batch) {
   for (int b = 0; b < batch; ++b) max_len = std::max(max_len, m->cache->host_lens[b]);
   uint32_t plan = 17;
   for (const MixLayer& w : m->mix)
-    if (w.kv)
+    if (w.kv && w.c.block == RB_BLOCK_SANDWICH)
+      plan = plan * 31 + (uint32_t)attention_decode_splits(m->ctx, batch, attention_joint_row_tiles(w.kv, w.c.heads), max_len, 256);
+    else if (w.kv)
       plan = plan * 31 + (uint32_t)attention_decode_splits(m->ctx, batch, w.c.kv_heads, attention_walk_len(max_len, w.c.window, w.c.chunk),
                                                            w.kv->head_dim);
   return (int)(plan & 0x7fffffffu);
