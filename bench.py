@@ -55,7 +55,7 @@ def parse_args():
     ap.add_argument("--skip-parity", action="store_true", help="skip the oracle comparison that follows the timed region")
     ap.add_argument("--skip-other-configs", action="store_true",
                     help="skip the short decode runs of the other benchmark configurations (single-GPU default run only)")
-    ap.add_argument("--design", default="", choices=["", "malasun", "votapel", "kufulix"],
+    ap.add_argument("--design", default="", choices=["", "malasun", "votapel", "kufulix", "fizadra"],
                     help="instead of the headline: prefill and decode of this design at a few sizes, each beside a qwen2 "
                          "model of equal width, heads, depth and parameter count; with routed experts also beside one with as "
                          "many parameters as a token uses (one JSON line)")
@@ -640,7 +640,9 @@ def random_param(kind, shape, gen):
     w = {"norm_w": lambda: torch.ones(shape, device="cuda"), "gain": lambda: torch.ones(shape, device="cuda"), "embed": n,
          "fan_in": lambda: n() / shape[1] ** 0.5, "conv": lambda: n() / shape[1] ** 0.5, "lower": lambda: u(0.0, 0.9),
          "forget_b": lambda: u(0.0, 6.0), "delta": lambda: n() * 0.2, "sink": n, "act": lambda: u(-1.0, 1.0),
-         "step_b": lambda: u(-5.0, 0.0), "decay": lambda: u(-1.0, 2.5), "skip": lambda: 1.0 + n() * 0.3, "correction": lambda: n() * 0.05}.get(kind, lambda: n() * 0.02)()
+         "step_b": lambda: u(-5.0, 0.0), "decay": lambda: u(-1.0, 2.5), "skip": lambda: 1.0 + n() * 0.3, "correction": lambda: n() * 0.05,
+         "talk": lambda: torch.eye(shape[0], device="cuda") + n() / shape[0] ** 0.5,
+         "depth": lambda: torch.cat([n()[1:] * 0.1, torch.ones(1, device="cuda")])}.get(kind, lambda: n() * 0.02)()
     return w.to(torch.bfloat16)
 
 
@@ -674,8 +676,11 @@ def equal_size_qwen2(cfg, active=False):
 
 def relatives(name, cfg):
     """Kufulix beside the designs that have what qwen2 lacks: routed experts (Votapel of equal width, heads, depth, experts and
-    parameter count) and a recurrence (the Malasun configuration of the same width and heads)."""
+    parameter count) and a recurrence (the Malasun configuration of the same width and heads).  Fizadra beside Malasun, whose
+    joints norm a sublayer's output on a float32 stream."""
     from rai_b200 import configs
+    if cfg["arch"] == "fizadra":
+        return {"malasun": configs.get(name.replace("fizadra", "malasun"))}
     if cfg["arch"] != "kufulix":
         return {}
     votapel, malasun = configs.get(name.replace("kufulix", "votapel")), configs.get(name.replace("kufulix", "malasun"))

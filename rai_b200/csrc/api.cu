@@ -559,8 +559,9 @@ extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache*
   }
   const double es = (double)dtype_size(dtype), d = c->head_dim;
   ProfScope prof(ctx, RB_PROF_ATTENTION,
-                 es * ((c->shared() ? 1.0 : 2.0) * kv_tokens * c->kv_heads * d + (x.gate ? 3.0 : 2.0) * batch * s_new * q_heads * d),
-                 4.0 * pairs * q_heads * d);
+                 es * ((c->shared() ? 1.0 : 2.0) * kv_tokens * c->kv_heads * d +
+                       (double)batch * s_new * q_heads * (d + (x.gate && !x.head_gate ? 2.0 : 1.0) * x.value_dim)),
+                 2.0 * pairs * q_heads * (d + x.value_dim));
   if (x.talk) {
     RB_REQUIRE(!x.alibi && !x.gate && !x.temp_every && x.softcap == 0.f && x.out_scale == 1.f,
                "rb_attention_general: mixed heads go with window, chunk, sink and value_dim only");
