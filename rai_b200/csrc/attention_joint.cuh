@@ -146,8 +146,8 @@ __device__ __forceinline__ void merge_splits(const Params& p, float* w_s, int b,
 }
 
 template <typename S>
-__global__ void __launch_bounds__(kThreads, 1) kernel(const Params p, const __grid_constant__ CUtensorMap tm_k,
-                                                      const __grid_constant__ CUtensorMap tm_v) {
+__global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Params p, const __grid_constant__ CUtensorMap tm_k,
+                                                                      const __grid_constant__ CUtensorMap tm_v) {
   constexpr int KT = S::KT, NT = S::NT, R = S::R, GP = S::GP, DW = S::DW, SP = S::SP, PP = S::PP, KL = S::KL;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t full_bar[kMaxStages];
@@ -571,7 +571,7 @@ int launch(rb_ctx* ctx, rb_kv_cache* c, Params p, int layer, int batch, int max_
       p.part_ml = ctx->attn_scratch + parts * p.value_dim;
     }
   }
-  auto kern = kernel<S>;
+  auto kern = joint_attention_kernel<S>;
   static size_t set[64] = {};
   const int dv = ctx->device & 63;
   if (smem > set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set[dv] = smem; }

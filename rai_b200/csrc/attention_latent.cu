@@ -41,6 +41,8 @@ bool attention_joint_takes(const rb_kv_cache* c, const AttnExtra& x) {
 
 int attention_joint(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
                     const AttnExtra& x) {
+  if (x.talk && ctx->attn_tc && attention_mix_tc_takes(c, s_new, q_heads, q, x))
+    return attention_mix_tc(ctx, q, c, layer, batch, s_new, q_heads, scale, out, x);
   joint::Params p{};
   p.q = (const bf16*)q; p.block_table = c->block_table; p.seq_lens = c->seq_lens; p.pages_per_seq = c->pages_per_seq; p.s_new = s_new;
   p.D = c->head_dim; p.q_heads = q_heads; p.kv_heads = c->kv_heads; p.group = q_heads / c->kv_heads;

@@ -1,0 +1,534 @@
+// Causal attention of prompts whose heads' scores are mixed before the softmax (score[h] <- sum_g talk[h][g] score[g]), on the
+// 5th-generation tensor cores, for head sizes up to 128 and up to 32 heads over the paged bf16 cache.
+//
+// One CTA has MT = 256 / HP tokens with all their heads (HP: the number of heads rounded up to 8, 16 or 32), so that no raw score
+// is computed twice.  Both products are transposed: keys, then dimensions, fill the 128 lanes of tensor memory, and a column is
+// a (head, token):
+//   S^T [128 keys x 256]  = K . Q^T      per key/value head: its heads' columns, K and Q K-major
+//   O^T [128 dims x 256] += V^T . P^T    V and P MN-major, straight from their [keys][...] tiles
+// which fills the 512 columns of tensor memory.  Twelve warps:
+//   warps 0-7   a thread has one key (its lane) and 64 columns at a time, all heads of a few tokens: it reads the raw scores,
+//               mixes them in float32 (packed FMAs), masks, and stores the weights in bf16.  The reference point of the
+//               exponentials is one number per column for all 128 keys; it moves only when some score has outgrown it by
+//               2^8, which all warps learn at a barrier before they exponentiate (always at the first tile).  The sums of
+//               the weights over the keys come from a product with ones on mma.sync, in float32.
+//   warp 8      tiled copies: Q once, then K of every head, V of every head, ... through a ring of 128-key tiles (two pages);
+//   warp 9      owns the tensor memory; one lane issues the products: the scores of the next tile as soon as the raw scores of
+//               this one have been read, so that they are there when its weights are done.
+// Every wait is bounded; after a give-up the block runs on without waiting, writes nothing, reports, lets its copies land, frees its
+// tensor memory and returns.
+#include <algorithm>
+
+#include "ctx.h"
+#include "mma.cuh"
+#include "ptx.cuh"
+
+namespace rb {
+
+using bf16 = __nv_bfloat16;
+
+namespace {
+
+constexpr int kKeys = 128;                   // keys per tile = lanes
+constexpr int kThreads = 384;                // 384 x 168 = 256 x 232 + 128 x 40 registers
+constexpr int kWarps = 8, kSoftmax = 256;
+constexpr int kCols = 256;                   // columns of S and of O
+constexpr int kBlock = kKeys * 128;          // 64 columns of 128 keys (or of P's rows), 128-byte swizzle; a stage of the ring
+constexpr int kPageBlock = kPageTokens * 128;
+constexpr int kMaxStages = 8;
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct MixParams {
+  const int32_t *block_table, *seq_lens;
+  int pages_per_seq, s_new, q_heads, kv_heads, group, D, nb, nbv;
+  int head_cols;              // columns of a key/value head: group * MT, rounded up so that no block of 64 is crossed
+  int stages, value_dim;
+  float scale_log2;
+  const bf16 *talk, *sink;
+  bf16* out;
+  int64_t out_ld;
+  uint32_t* status;
+  long long wait_cycles;
+};
+
+struct MixCtrl {
+  uint64_t q_full, full[kMaxStages], empty[kMaxStages], s_full, s_empty, p_full, o_done;
+  uint32_t tmem_base, abort_flag, issued, grow[2];
+};
+
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)),
+        "l"(reinterpret_cast<unsigned long long&>(c)));
+  return r;
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) {
+  float2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+  return r;
+}
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+
+template <int HP>
+struct MixShape {
+  static constexpr int MT = kCols / HP;      // tokens of a CTA
+  static constexpr int TC = 64 / HP;         // tokens of a thread at a time
+  // behind Q, P and the ring: talk (every coefficient twice), minus the reference points and their shifts, per column
+  static constexpr int kTalkBytes = HP * HP * 8;
+  static constexpr size_t fixed_bytes(int nb) { return (size_t)nb * kCols * 128 + 4 * kBlock + kTalkBytes + 2 * kCols * 4 + sizeof(MixCtrl); }
+};
+
+template <int HP>
+__global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __grid_constant__ CUtensorMap tm_q,
+                                                                      const __grid_constant__ CUtensorMap tm_k,
+                                                                      const __grid_constant__ CUtensorMap tm_v, const MixParams p) {
+  using C = MixShape<HP>;
+  constexpr int MT = C::MT, TC = C::TC;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  uint8_t* q_s = smem;                                                  // [nb][256 columns][128 bytes]
+  uint8_t* p_s = q_s + (size_t)p.nb * kCols * 128;                      // [4][128 keys][128 bytes]
+  uint8_t* ring = p_s + 4 * kBlock;
+  float2* t_s = reinterpret_cast<float2*>(ring + (size_t)p.stages * kBlock);   // [h][g]
+  float* m_s = reinterpret_cast<float*>(t_s + HP * HP);                 // minus the reference point, per column
+  float* shift_s = m_s + kCols;                                         // by how much it has just moved; at the end 1 / sum
+  MixCtrl* ctl = reinterpret_cast<MixCtrl*>(shift_s + kCols);
+  volatile uint32_t* abort_flag = &ctl->abort_flag;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int G = p.kv_heads, H = p.q_heads, group = p.group;
+
+  if (threadIdx.x == 0) {
+    ptx::mbar_init(&ctl->q_full, 1);
+    for (int i = 0; i < p.stages; ++i) { ptx::mbar_init(&ctl->full[i], 1); ptx::mbar_init(&ctl->empty[i], 1); }
+    ptx::mbar_init(&ctl->s_full, 1);
+    ptx::mbar_init(&ctl->s_empty, kWarps);
+    ptx::mbar_init(&ctl->p_full, kWarps);
+    ptx::mbar_init(&ctl->o_done, 1);
+    ctl->abort_flag = ctl->issued = ctl->grow[0] = ctl->grow[1] = 0;
+    ptx::fence_barrier_init();
+    ptx::fence_proxy_async();
+    ptx::tma_prefetch_desc(&tm_q);
+    ptx::tma_prefetch_desc(&tm_k);
+    ptx::tma_prefetch_desc(&tm_v);
+  }
+  if (warp == 9) {
+    ptx::tmem_alloc(&ctl->tmem_base, 512);
+    ptx::tmem_relinquish();
+  }
+  ptx::tc_fence_before();
+  __syncthreads();
+  ptx::tc_fence_after();
+  const uint32_t tmem_s = ctl->tmem_base, tmem_o = tmem_s + kCols;
+  pdl_launch_dependents();
+  pdl_wait();   // q, lengths and the newest keys come from kernels before this one
+
+  const int t0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * MT, b = blockIdx.y;   // longest walks first
+  const int len = p.seq_lens[b], base = len - p.s_new;
+  const int n = (min(base + t0 + MT, len) + kKeys - 1) / kKeys;                  // tiles
+  // the swizzle atoms must sit on 1024-byte boundaries
+  const bool layout_ok = (ptx::smem_u32(smem) & 1023u) == 0u && n >= 1;
+  if (!layout_ok && threadIdx.x == 0) { p.status[0] = (uint32_t)(-RB_ERR_CUDA); p.status[1] = 0xA710u; p.status[2] = blockIdx.x; }
+
+  if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 40;");
+    if (layout_ok && warp == 8 && lane == 0) {
+      // ------------------------------------------------------------------ copies
+      ptx::mbar_expect_tx(&ctl->q_full, (uint32_t)(H * p.nb * MT * 128));
+      for (int h = 0; h < H; ++h)
+        for (int cb = 0; cb < p.nb; ++cb)
+          ptx::tma_load_2d(q_s + (size_t)cb * kCols * 128 + (size_t)(h / group * p.head_cols + h % group * MT) * 128, &tm_q, &ctl->q_full,
+                           h * p.D + cb * 64, b * p.s_new + t0);
+      uint32_t u = 0;
+      bool ok = true;
+      // a stage is 64 columns of a tile's keys, or one page of its values
+      auto next_stage = [&](uint32_t bytes) -> uint8_t* {
+        const int st = u % p.stages;
+        if (!ptx::mbar_wait(&ctl->empty[st], ((u / p.stages) & 1u) ^ 1u, abort_flag, p.wait_cycles)) { ok = false; return nullptr; }
+        ptx::mbar_expect_tx(&ctl->full[st], bytes);
+        return ring + (size_t)st * kBlock;
+      };
+      auto page_of = [&](int i) { return p.block_table[(size_t)b * p.pages_per_seq + min(i, p.pages_per_seq - 1)]; };
+      auto load_keys = [&](int tile) {
+        const int page0 = page_of(tile * 2), page1 = page_of(tile * 2 + 1);
+        for (int i = 0; i < G * p.nb && ok; ++i, ++u) {
+          const int g = i / p.nb, cb = i % p.nb, st = u % p.stages;
+          uint8_t* dst = next_stage(kBlock);
+          if (!dst) return;
+          ptx::tma_load_2d(dst, &tm_k, &ctl->full[st], cb * 64, (page0 * G + g) * kPageTokens);
+          ptx::tma_load_2d(dst + kPageBlock, &tm_k, &ctl->full[st], cb * 64, (page1 * G + g) * kPageTokens);
+          ctl->issued = u + 1;
+        }
+      };
+      auto load_values = [&](int tile) {
+        const int page[2] = {page_of(tile * 2), page_of(tile * 2 + 1)};
+        for (int i = 0; i < G * 2 && ok; ++i, ++u) {
+          const int st = u % p.stages, y = (page[i & 1] * G + (i >> 1)) * kPageTokens;
+          uint8_t* dst = next_stage((uint32_t)p.nbv * kPageBlock);
+          if (!dst) return;
+          for (int cb = 0; cb < p.nbv; ++cb) ptx::tma_load_2d(dst + cb * kPageBlock, &tm_v, &ctl->full[st], cb * 64, y);
+          ctl->issued = u + 1;
+        }
+      };
+      load_keys(0);
+      for (int j = 0; j < n && ok; ++j) {
+        if (j + 1 < n) load_keys(j + 1);
+        if (ok) load_values(j);
+      }
+    } else if (layout_ok && warp == 9 && lane == 0) {
+      // ------------------------------------------------------------------ products
+      const uint32_t idesc_s = ptx::umma_idesc_bf16(kKeys, p.head_cols), idesc_o = ptx::umma_idesc_bf16(128, p.head_cols, true, true);
+      const uint32_t qa = ptx::smem_u32(q_s), pa = ptx::smem_u32(p_s), ra = ptx::smem_u32(ring);
+      uint32_t u = 0;
+      auto full = [&]() -> bool {
+        if (!ptx::mbar_wait(&ctl->full[u % p.stages], (u / p.stages) & 1u, abort_flag, p.wait_cycles)) return false;
+        ptx::tc_fence_after();
+        return true;
+      };
+      auto scores = [&](int j) -> bool {
+        if (!ptx::mbar_wait(&ctl->s_empty, ((uint32_t)j & 1u) ^ 1u, abort_flag, p.wait_cycles)) return false;
+        for (int g = 0; g < G; ++g)
+          for (int cb = 0; cb < p.nb; ++cb, ++u) {
+            if (!full()) return false;
+            const uint32_t ka = ra + (u % p.stages) * kBlock, qb = qa + cb * (kCols * 128) + g * p.head_cols * 128;
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk)
+              ptx::umma_bf16(tmem_s + (uint32_t)(g * p.head_cols), ptx::umma_desc_k_sw128(ka + kk * 32), ptx::umma_desc_k_sw128(qb + kk * 32), idesc_s,
+                             (cb > 0 || kk > 0) ? 1u : 0u);
+            ptx::umma_commit(&ctl->empty[u % p.stages]);
+          }
+        ptx::umma_commit(&ctl->s_full);
+        return true;
+      };
+      bool ok = ptx::mbar_wait(&ctl->q_full, 0u, abort_flag, p.wait_cycles);
+      if (ok) ok = scores(0);
+      for (int j = 0; j < n && ok; ++j) {
+        if (j + 1 < n && !scores(j + 1)) break;
+        if (!ptx::mbar_wait(&ctl->p_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles)) break;
+        for (int i = 0; i < G * 2 && ok; ++i, ++u) {
+          if (!full()) { ok = false; break; }
+          const int col = (i >> 1) * p.head_cols, page = i & 1;
+          const uint32_t va = ra + (u % p.stages) * kBlock, pb = pa + (col >> 6) * kBlock + (col & 63) * 2 + page * kPageBlock;
+#pragma unroll
+          for (int ks = 0; ks < kPageTokens / 16; ++ks)   // 16 keys are 16 rows of 128 bytes further in both tiles
+            ptx::umma_bf16(tmem_o + (uint32_t)col, ptx::umma_desc_mn_sw128(va + ks * (16 * 128), kPageBlock, 1024),
+                           ptx::umma_desc_mn_sw128(pb + ks * (16 * 128), kBlock, 1024), idesc_o, (j > 0 || page > 0 || ks > 0) ? 1u : 0u);
+          ptx::umma_commit(&ctl->empty[u % p.stages]);
+        }
+        if (ok) ptx::umma_commit(&ctl->o_done);
+      }
+    }
+  } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 232;");
+    // ------------------------------------------------------------------ mixing, softmax, output
+    const int quarter = warp & 3, half = warp >> 2, key = quarter * 32 + lane;
+    const uint32_t t_lane = (uint32_t)(quarter * 32) << 16;
+    const int g8 = lane >> 2, t4 = lane & 3;
+    for (int i = threadIdx.x; i < HP * HP; i += kSoftmax) {
+      const int h = i / HP, g = i % HP;
+      const float t = h < H && g < H ? __bfloat162float(p.talk[h * H + g]) * p.scale_log2 : 0.f;
+      t_s[i] = make_float2(t, t);
+    }
+    m_s[threadIdx.x] = 0.f;
+    softmax_sync();
+    auto column = [&](int h) { return h / group * p.head_cols + h % group * MT; };
+    float sums[4][4];   // columns 32 warp .. + 32, the same in every row of the fragment
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { sums[i][0] = sums[i][1] = sums[i][2] = sums[i][3] = 0.f; }
+    for (int j = 0; j < (layout_ok ? n : 0); ++j) {
+      const int key_pos = j * kKeys + key;
+      const bool edge = j * kKeys + kKeys - 1 > base + t0;
+      ptx::mbar_wait(&ctl->s_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles);
+      __syncwarp();
+      ptx::tc_fence_after();
+#pragma unroll 1
+      for (int c = 0; c < 2; ++c) {
+        const int i0 = half * (MT / 2) + c * TC;   // first token
+        float2 x[HP][TC / 2];                      // raw scores of the token pairs
+        {
+          int col = i0, in_group = 0;
+#pragma unroll
+          for (int h = 0; h < HP; ++h) {
+            uint32_t r[TC];
+            if (h < H) {   // uniform
+              ptx::tmem_ld_32xn<TC>(tmem_s + t_lane + (uint32_t)col, r);
+            } else {
+#pragma unroll
+              for (int i = 0; i < TC; ++i) r[i] = 0u;
+            }
+#pragma unroll
+            for (int i = 0; i < TC / 2; ++i) x[h][i] = make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
+            col += MT;
+            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+          }
+        }
+        ptx::tmem_wait_ld();
+        if (c == 1) {
+          ptx::tc_fence_before();
+          __syncwarp();
+          if (lane == 0) ptx::mbar_arrive(&ctl->s_empty);   // the next tile's scores may come
+        }
+        // mixed scores less their reference points
+        float2 d[HP][TC / 2];
+        float top = -INFINITY;
+        {
+          int col = i0, in_group = 0;
+#pragma unroll
+          for (int h = 0; h < HP; ++h) {
+#pragma unroll
+            for (int i = 0; i < TC / 2; ++i) d[h][i] = *reinterpret_cast<const float2*>(m_s + (h < H ? col : 0) + 2 * i);
+#pragma unroll
+            for (int g = 0; g < HP; g += 2) {
+              const float4 t = *reinterpret_cast<const float4*>(t_s + h * HP + g);
+#pragma unroll
+              for (int i = 0; i < TC / 2; ++i) {
+                d[h][i] = fma2(make_float2(t.x, t.y), x[g][i], d[h][i]);
+                d[h][i] = fma2(make_float2(t.z, t.w), x[g + 1][i], d[h][i]);
+              }
+            }
+            if (edge) {
+#pragma unroll
+              for (int i = 0; i < TC / 2; ++i) {
+                const int pos = base + t0 + i0 + 2 * i;
+                if (key_pos > pos) d[h][i].x = -INFINITY;
+                if (key_pos > pos + 1) d[h][i].y = -INFINITY;
+              }
+            }
+#pragma unroll
+            for (int i = 0; i < TC / 2; ++i)
+              if (h < H) top = fmaxf(top, fmaxf(d[h][i].x, d[h][i].y));
+            col += MT;
+            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+          }
+        }
+        volatile uint32_t* grow = ctl->grow + c;   // (a flag of its own for each half of a tile: a fast warp may already be in the next)
+        if (__any_sync(0xffffffffu, top > 8.0f) && lane == 0) *grow = 1u;
+        softmax_sync();
+        if (j == 0 || *grow != 0u) {   // uniform over the eight warps
+          constexpr int kLowest = (int)0x807fffff;   // -inf in an order of integers that is the order of floats
+          int* best = reinterpret_cast<int*>(shift_s);
+          best[threadIdx.x] = kLowest;
+          softmax_sync();
+          {
+            int col = i0, in_group = 0;
+#pragma unroll
+            for (int h = 0; h < HP; ++h) {
+#pragma unroll
+              for (int i = 0; i < TC; ++i) {
+                const float m = warp_max((i & 1) ? d[h][i / 2].y : d[h][i / 2].x);
+                const int o = __float_as_int(m);
+                if (lane == 0 && h < H) atomicMax(best + col + i, o >= 0 ? o : o ^ 0x7fffffff);
+              }
+              col += MT;
+              if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+            }
+          }
+          softmax_sync();
+          if (threadIdx.x == 0) *grow = 0u;
+          {
+            const int o = best[threadIdx.x];
+            const float up = __int_as_float(o >= 0 ? o : o ^ 0x7fffffff);
+            const float shift = o > kLowest && (j == 0 || up > 8.0f) ? up : 0.f;
+            m_s[threadIdx.x] -= shift;
+            shift_s[threadIdx.x] = shift;
+          }
+          softmax_sync();
+          {
+            int col = i0, in_group = 0;
+#pragma unroll
+            for (int h = 0; h < HP; ++h) {
+#pragma unroll
+              for (int i = 0; i < TC / 2; ++i) {
+                const float2 s = *reinterpret_cast<const float2*>(shift_s + (h < H ? col : 0) + 2 * i);
+                d[h][i] = add2(d[h][i], make_float2(-s.x, -s.y));
+              }
+              col += MT;
+              if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+            }
+          }
+          if (j > 0) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float c0 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4]), c1 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4 + 1]);
+              sums[i][0] *= c0; sums[i][1] *= c1; sums[i][2] *= c0; sums[i][3] *= c1;
+            }
+            ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
+            __syncwarp();
+            ptx::tc_fence_after();
+            for (int h = 0; h < H; ++h) {
+              const int col = column(h) + i0;
+              uint32_t r[TC];
+              ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
+              ptx::tmem_wait_ld();
+#pragma unroll
+              for (int i = 0; i < TC; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * ex2_fast(-shift_s[col + i]));
+              ptx::tmem_st_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
+            }
+            ptx::tmem_wait_st();
+          }
+        }
+        if (c == 0 && j > 0) {   // P of the tile before has been read
+          ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
+          __syncwarp();
+        }
+        {
+          int col = i0, in_group = 0;
+#pragma unroll
+          for (int h = 0; h < HP; ++h) {
+            if (h < H) {
+              uint32_t w[TC / 2];
+#pragma unroll
+              for (int i = 0; i < TC / 2; ++i) {
+                const __nv_bfloat162 v = __floats2bfloat162_rn(ex2_fast(d[h][i].x), ex2_fast(d[h][i].y));
+                w[i] = *reinterpret_cast<const uint32_t*>(&v);
+              }
+              uint8_t* dst = p_s + (col >> 6) * kBlock + key * 128 + ((((col & 63) >> 3) ^ (key & 7)) << 4) + (col & 7) * 2;
+              if constexpr (TC == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(w[0], w[1], w[2], w[3]);
+              else if constexpr (TC == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(w[0], w[1]);
+              else *reinterpret_cast<uint32_t*>(dst) = w[0];
+            }
+            col += MT;
+            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+          }
+        }
+      }
+      ptx::fence_proxy_async();   // the weights become visible to the tensor core's reads
+      ptx::tc_fence_before();
+      __syncwarp();
+      if (lane == 0) ptx::mbar_arrive(&ctl->p_full);
+      ptx::mbar_wait(&ctl->p_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles);
+      __syncwarp();
+      // sums over the keys: ones . P
+      const uint32_t ones[4] = {0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int col = warp * 32 + i * 8;
+        const uint32_t src = s_u32(p_s + (col >> 6) * kBlock);
+#pragma unroll
+        for (int k = 0; k < kKeys / 32; ++k) {
+          uint32_t bb[4];
+          const int row = k * 32 + lane;
+          ldsm_x4_t(bb, src + (uint32_t)(row * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4)));
+          mma16816(sums[i], ones, bb[0], bb[1]);
+          mma16816(sums[i], ones, bb[2], bb[3]);
+        }
+      }
+    }
+    // ------------------------------------------------------------------ output
+    if (layout_ok) {
+      ptx::mbar_wait(&ctl->o_done, (uint32_t)(n - 1) & 1u, abort_flag, p.wait_cycles);
+      __syncwarp();
+      ptx::tc_fence_after();
+      softmax_sync();
+      if (g8 == 0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { shift_s[warp * 32 + i * 8 + 2 * t4] = sums[i][0]; shift_s[warp * 32 + i * 8 + 2 * t4 + 1] = sums[i][1]; }
+      }
+      softmax_sync();
+      for (int v = threadIdx.x; v < H * MT; v += kSoftmax) {
+        const int h = v / MT, col = column(h) + v % MT;
+        const float l = shift_s[col] + (p.sink ? ex2_fast(fmaf(__bfloat162float(p.sink[h]), kLog2e, m_s[col])) : 0.f);
+        shift_s[col] = 1.0f / l;
+      }
+      softmax_sync();
+      const int dim = quarter * 32 + lane;
+      if (!*abort_flag && quarter * 32 < p.value_dim) {
+        for (int h = 0; h < H; ++h) {
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const int i0 = half * (MT / 2) + c * TC, col = column(h) + i0;
+            uint32_t r[TC];
+            ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
+            ptx::tmem_wait_ld();
+#pragma unroll
+            for (int i = 0; i < TC; ++i) {
+              const int token = t0 + i0 + i;
+              if (token < p.s_new && dim < p.value_dim)
+                p.out[((size_t)b * p.s_new + token) * p.out_ld + (size_t)h * p.value_dim + dim] = __float2bfloat16_rn(__uint_as_float(r[i]) * shift_s[col + i]);
+            }
+          }
+        }
+      }
+    }
+  }
+
+  // ------------------------------------------------------------------ teardown
+  ptx::tc_fence_before();
+  __syncthreads();
+  if (*abort_flag && threadIdx.x == 0) {
+    p.status[0] = (uint32_t)(-RB_ERR_TIMEOUT); p.status[1] = 0xA711u; p.status[2] = blockIdx.x; p.status[3] = blockIdx.y;
+    volatile uint32_t never = 0;   // copies already on their way get a bounded chance to land
+    ptx::mbar_wait(&ctl->q_full, 0u, &never, p.wait_cycles);
+    const uint32_t issued = ctl->issued;
+    for (uint32_t u = issued > (uint32_t)p.stages ? issued - p.stages : 0; u < issued; ++u)
+      ptx::mbar_wait(&ctl->full[u % p.stages], (u / p.stages) & 1u, &never, p.wait_cycles);
+  }
+  __syncthreads();
+  if (warp == 9) {
+    __syncwarp();
+    ptx::tc_fence_after();
+    ptx::tmem_dealloc(tmem_s, 512);
+  }
+}
+
+// columns a key/value head takes: whole 16s that do not cross a block of 64
+int head_columns(int n) {
+  if (n > 64) return (n + 63) / 64 * 64;
+  return n <= 16 ? 16 : n <= 32 ? 32 : 64;
+}
+int padded_heads(int H) { return H <= 8 ? 8 : H <= 16 ? 16 : 32; }
+
+template <int HP>
+int launch_mix(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, MixParams p) {
+  using C = MixShape<HP>;
+  constexpr size_t kLimit = 227 * 1024;
+  const size_t fixed = C::fixed_bytes(p.nb);
+  p.stages = (int)std::min<size_t>(kMaxStages, (kLimit - fixed) / kBlock);
+  const size_t smem = fixed + (size_t)p.stages * kBlock;
+  auto kern = attention_mix_tc_kernel<HP>;
+  static size_t set[64] = {};
+  const int dv = ctx->device & 63;
+  if (smem > set[dv]) { RB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); set[dv] = smem; }
+  CUtensorMap tq, tk, tv;
+  const size_t off = (size_t)layer * c->layer_stride_elems();
+  const int64_t rows = (int64_t)c->num_pages * c->kv_heads * kPageTokens;
+  // q rows are (sequence, position), columns (head, lane): a box is one head's tokens x 64
+  RB_TRY(tmap_2d_bf16(ctx, q, (int64_t)batch * p.s_new, (int64_t)p.q_heads * p.D, (int64_t)p.q_heads * p.D, C::MT, &tq));
+  RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->k + off, rows, p.D, p.D, kPageTokens, &tk));
+  RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->v + off, rows, p.D, p.D, kPageTokens, &tv));
+  RB_CUDA(launch_kernel(kern, dim3((unsigned)((p.s_new + C::MT - 1) / C::MT), (unsigned)batch), dim3(kThreads), smem, ctx->stream, ctx->pdl, tq, tk,
+                        tv, p));
+  ctx->launches++;
+  return RB_OK;
+}
+
+}  // namespace
+
+bool attention_mix_tc_takes(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const AttnExtra& x) {
+  if (c->dtype != RB_BF16 || c->shared() || (c->head_dim != 64 && c->head_dim != 128) || q_heads > 32 || q_heads % c->kv_heads != 0) return false;
+  if (x.window > 0 || x.chunk > 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0) return false;
+  const int mt = kCols / padded_heads(q_heads);
+  return s_new >= 16 && c->kv_heads * head_columns(q_heads / c->kv_heads * mt) <= kCols;
+}
+
+int attention_mix_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                     const AttnExtra& x) {
+  MixParams p{};
+  const int hp = padded_heads(q_heads);
+  p.block_table = c->block_table; p.seq_lens = c->seq_lens; p.pages_per_seq = c->pages_per_seq; p.s_new = s_new; p.q_heads = q_heads;
+  p.kv_heads = c->kv_heads; p.group = q_heads / c->kv_heads; p.D = c->head_dim; p.nb = c->head_dim / 64; p.nbv = (x.value_dim + 63) / 64;
+  p.head_cols = head_columns(p.group * (kCols / hp)); p.value_dim = x.value_dim; p.scale_log2 = scale * kLog2e;
+  p.talk = (const bf16*)x.talk; p.sink = (const bf16*)x.sink; p.out = (bf16*)out; p.out_ld = x.out_ld; p.status = ctx->status_dev;
+  p.wait_cycles = ctx->local_wait_cycles();
+  RB_REQUIRE(batch <= 65535, "attention: batch %d too large", batch);
+  if (hp == 8) return launch_mix<8>(ctx, q, c, layer, batch, p);
+  if (hp == 16) return launch_mix<16>(ctx, q, c, layer, batch, p);
+  return launch_mix<32>(ctx, q, c, layer, batch, p);
+}
+
+}  // namespace rb

@@ -312,6 +312,10 @@ bool attention_joint_takes(const rb_kv_cache* c, const AttnExtra& x);
 int attention_joint_row_tiles(const rb_kv_cache* c, int q_heads);   // blocks a single token's heads take
 int attention_joint(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
                     const AttnExtra& x);
+// attention_mix_tc.cu: attention of prompts with mixed heads on tcgen05 (head sizes up to 128, up to 32 heads)
+bool attention_mix_tc_takes(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const AttnExtra& x);
+int attention_mix_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
+                     const AttnExtra& x);
 // plain_kernels.cu: attention whose heads' scores are mixed (x.talk), any sizes
 int attention_talk_simple(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, int s_new, int q_heads, float scale, void* out,
                           int dtype, const AttnExtra& x);
