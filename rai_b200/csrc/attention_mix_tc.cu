@@ -9,9 +9,11 @@
 // which fills the 512 columns of tensor memory.  Twelve warps:
 //   warps 0-7   a thread has one key (its lane) and 64 columns at a time, all heads of a few tokens: it reads the raw scores,
 //               mixes them in float32 (packed FMAs), masks, and stores the weights in bf16.  The reference point of the
-//               exponentials is one number per column for all 128 keys; it moves only when some score has outgrown it by
-//               2^8, which all warps learn at a barrier before they exponentiate (always at the first tile).  The sums of
-//               the weights over the keys come from a product with ones on mma.sync, in float32.
+//               exponentials is one number per column for all 128 keys, 2^6 above the maximum when it was set.  A tile is
+//               computed on the reference points as they are; only if a weight comes out at 2 or more (always at the first tile)
+//               do the warps set new ones and compute the tile again, from raw scores that the warp in question has not
+//               given back.  One barrier per tile, which the sums over the keys need anyway: they come from a product with
+//               ones on mma.sync, in float32.
 //   warp 8      tiled copies: Q once, then K of every head, V of every head, ... through a ring of 128-key tiles (two pages);
 //   warp 9      owns the tensor memory; one lane issues the products: the scores of the next tile as soon as the raw scores of
 //               this one have been read, so that they are there when its weights are done.
@@ -63,18 +65,15 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
         "l"(reinterpret_cast<unsigned long long&>(c)));
   return r;
 }
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-  float2 r;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r))
-      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
-  return r;
-}
 __device__ __forceinline__ float ex2_fast(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+__device__ __forceinline__ void softmax_sync() {
+  __syncwarp();
+  asm volatile("bar.sync 1, 256;" ::: "memory");
+}
 
 template <int HP>
 struct MixShape {
@@ -240,169 +239,172 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
     float sums[4][4];   // columns 32 warp .. + 32, the same in every row of the fragment
 #pragma unroll
     for (int i = 0; i < 4; ++i) { sums[i][0] = sums[i][1] = sums[i][2] = sums[i][3] = 0.f; }
+    // Chunk c of tile j: raw scores of TC tokens and all heads -> mixed scores less their reference points
+    auto mix = [&](int j, int c, float2 (&d)[HP][TC / 2]) {
+      const int i0 = half * (MT / 2) + c * TC;   // first token
+      float2 x[HP][TC / 2];                      // raw scores of the token pairs
+      int col = i0, in_group = 0;
+      auto next_head = [&]() {
+        col += MT;
+        if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+      };
+#pragma unroll
+      for (int h = 0; h < HP; ++h) {
+        uint32_t r[TC];
+        if (h < H) {   // uniform
+          ptx::tmem_ld_32xn<TC>(tmem_s + t_lane + (uint32_t)col, r);
+        } else {
+#pragma unroll
+          for (int i = 0; i < TC; ++i) r[i] = 0u;
+        }
+#pragma unroll
+        for (int i = 0; i < TC / 2; ++i) x[h][i] = make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
+        next_head();
+      }
+      ptx::tmem_wait_ld();
+      col = i0;
+      in_group = 0;
+#pragma unroll
+      for (int h = 0; h < HP; ++h) {
+#pragma unroll
+        for (int i = 0; i < TC / 2; ++i) d[h][i] = *reinterpret_cast<const float2*>(m_s + (h < H ? col : 0) + 2 * i);
+#pragma unroll
+        for (int g = 0; g < HP; g += 2) {
+          const float4 t = *reinterpret_cast<const float4*>(t_s + h * HP + g);
+#pragma unroll
+          for (int i = 0; i < TC / 2; ++i) {
+            d[h][i] = fma2(make_float2(t.x, t.y), x[g][i], d[h][i]);
+            d[h][i] = fma2(make_float2(t.z, t.w), x[g + 1][i], d[h][i]);
+          }
+        }
+        next_head();
+      }
+      if (j * kKeys + kKeys - 1 > base + t0) {   // a tile that the diagonal cuts
+        const int first = j * kKeys + key - (base + t0 + i0);   // token i sees this key from i = first on
+#pragma unroll
+        for (int h = 0; h < HP; ++h)
+#pragma unroll
+          for (int i = 0; i < TC / 2; ++i) {
+            if (first > 2 * i) d[h][i].x = -INFINITY;
+            if (first > 2 * i + 1) d[h][i].y = -INFINITY;
+          }
+      }
+    };
+    // The chunk's weights into P; all their bits together (a weight of 2 or more has bit 14 of its half set, no smaller one has)
+    auto weights = [&](int c, const float2 (&d)[HP][TC / 2]) -> uint32_t {
+      int col = half * (MT / 2) + c * TC, in_group = 0;
+      uint32_t bits = 0u;
+#pragma unroll
+      for (int h = 0; h < HP; ++h) {
+        if (h < H) {
+          uint32_t w[TC / 2];
+#pragma unroll
+          for (int i = 0; i < TC / 2; ++i) {
+            const __nv_bfloat162 v = __floats2bfloat162_rn(ex2_fast(d[h][i].x), ex2_fast(d[h][i].y));
+            w[i] = *reinterpret_cast<const uint32_t*>(&v);
+            bits |= w[i];
+          }
+          uint8_t* dst = p_s + (col >> 6) * kBlock + key * 128 + ((((col & 63) >> 3) ^ (key & 7)) << 4) + (col & 7) * 2;
+          if constexpr (TC == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(w[0], w[1], w[2], w[3]);
+          else if constexpr (TC == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(w[0], w[1]);
+          else *reinterpret_cast<uint32_t*>(dst) = w[0];
+        }
+        col += MT;
+        if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
+      }
+      return bits;
+    };
     for (int j = 0; j < (layout_ok ? n : 0); ++j) {
-      const int key_pos = j * kKeys + key;
-      const bool edge = j * kKeys + kKeys - 1 > base + t0;
       ptx::mbar_wait(&ctl->s_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles);
       __syncwarp();
       ptx::tc_fence_after();
-#pragma unroll 1
-      for (int c = 0; c < 2; ++c) {
-        const int i0 = half * (MT / 2) + c * TC;   // first token
-        float2 x[HP][TC / 2];                      // raw scores of the token pairs
-        {
-          int col = i0, in_group = 0;
+      volatile uint32_t* grow = ctl->grow + (j & 1);   // (a fast warp may already be in the next tile)
+      bool kept = j == 0;   // this warp has not given the raw scores back
+      float2 d[HP][TC / 2];
+      if (j > 0) {
+        uint32_t bits = 0u;
 #pragma unroll
-          for (int h = 0; h < HP; ++h) {
-            uint32_t r[TC];
-            if (h < H) {   // uniform
-              ptx::tmem_ld_32xn<TC>(tmem_s + t_lane + (uint32_t)col, r);
-            } else {
-#pragma unroll
-              for (int i = 0; i < TC; ++i) r[i] = 0u;
-            }
-#pragma unroll
-            for (int i = 0; i < TC / 2; ++i) x[h][i] = make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
-            col += MT;
-            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
-          }
-        }
-        ptx::tmem_wait_ld();
-        if (c == 1) {
-          ptx::tc_fence_before();
-          __syncwarp();
-          if (lane == 0) ptx::mbar_arrive(&ctl->s_empty);   // the next tile's scores may come
-        }
-        // mixed scores less their reference points
-        float2 d[HP][TC / 2];
-        float top = -INFINITY;
-        {
-          int col = i0, in_group = 0;
-#pragma unroll
-          for (int h = 0; h < HP; ++h) {
-#pragma unroll
-            for (int i = 0; i < TC / 2; ++i) d[h][i] = *reinterpret_cast<const float2*>(m_s + (h < H ? col : 0) + 2 * i);
-#pragma unroll
-            for (int g = 0; g < HP; g += 2) {
-              const float4 t = *reinterpret_cast<const float4*>(t_s + h * HP + g);
-#pragma unroll
-              for (int i = 0; i < TC / 2; ++i) {
-                d[h][i] = fma2(make_float2(t.x, t.y), x[g][i], d[h][i]);
-                d[h][i] = fma2(make_float2(t.z, t.w), x[g + 1][i], d[h][i]);
-              }
-            }
-            if (edge) {
-#pragma unroll
-              for (int i = 0; i < TC / 2; ++i) {
-                const int pos = base + t0 + i0 + 2 * i;
-                if (key_pos > pos) d[h][i].x = -INFINITY;
-                if (key_pos > pos + 1) d[h][i].y = -INFINITY;
-              }
-            }
-#pragma unroll
-            for (int i = 0; i < TC / 2; ++i)
-              if (h < H) top = fmaxf(top, fmaxf(d[h][i].x, d[h][i].y));
-            col += MT;
-            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
-          }
-        }
-        volatile uint32_t* grow = ctl->grow + c;   // (a flag of its own for each half of a tile: a fast warp may already be in the next)
-        if (__any_sync(0xffffffffu, top > 8.0f) && lane == 0) *grow = 1u;
-        softmax_sync();
-        if (j == 0 || *grow != 0u) {   // uniform over the eight warps
-          constexpr int kLowest = (int)0x807fffff;   // -inf in an order of integers that is the order of floats
-          int* best = reinterpret_cast<int*>(shift_s);
-          best[threadIdx.x] = kLowest;
-          softmax_sync();
-          {
-            int col = i0, in_group = 0;
-#pragma unroll
-            for (int h = 0; h < HP; ++h) {
-#pragma unroll
-              for (int i = 0; i < TC; ++i) {
-                const float m = warp_max((i & 1) ? d[h][i / 2].y : d[h][i / 2].x);
-                const int o = __float_as_int(m);
-                if (lane == 0 && h < H) atomicMax(best + col + i, o >= 0 ? o : o ^ 0x7fffffff);
-              }
-              col += MT;
-              if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
-            }
-          }
-          softmax_sync();
-          if (threadIdx.x == 0) *grow = 0u;
-          {
-            const int o = best[threadIdx.x];
-            const float up = __int_as_float(o >= 0 ? o : o ^ 0x7fffffff);
-            const float shift = o > kLowest && (j == 0 || up > 8.0f) ? up : 0.f;
-            m_s[threadIdx.x] -= shift;
-            shift_s[threadIdx.x] = shift;
-          }
-          softmax_sync();
-          {
-            int col = i0, in_group = 0;
-#pragma unroll
-            for (int h = 0; h < HP; ++h) {
-#pragma unroll
-              for (int i = 0; i < TC / 2; ++i) {
-                const float2 s = *reinterpret_cast<const float2*>(shift_s + (h < H ? col : 0) + 2 * i);
-                d[h][i] = add2(d[h][i], make_float2(-s.x, -s.y));
-              }
-              col += MT;
-              if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
-            }
-          }
-          if (j > 0) {
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const float c0 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4]), c1 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4 + 1]);
-              sums[i][0] *= c0; sums[i][1] *= c1; sums[i][2] *= c0; sums[i][3] *= c1;
-            }
+        for (int c = 0; c < 2; ++c) {
+          mix(j, c, d);
+          if (c == 0) {   // P of the tile before has been read
             ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
             __syncwarp();
-            ptx::tc_fence_after();
-            for (int h = 0; h < H; ++h) {
-              const int col = column(h) + i0;
-              uint32_t r[TC];
-              ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
-              ptx::tmem_wait_ld();
-#pragma unroll
-              for (int i = 0; i < TC; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * ex2_fast(-shift_s[col + i]));
-              ptx::tmem_st_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
-            }
-            ptx::tmem_wait_st();
           }
+          bits |= weights(c, d);
         }
-        if (c == 0 && j > 0) {   // P of the tile before has been read
-          ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
+        kept = __any_sync(0xffffffffu, (bits & 0x40004000u) != 0u);
+        if (kept) {
+          if (lane == 0) *grow = 1u;
+        } else {   // the next tile's scores may come, once every warp has said so
+          ptx::tc_fence_before();
           __syncwarp();
+          if (lane == 0) ptx::mbar_arrive(&ctl->s_empty);
         }
-        {
-          int col = i0, in_group = 0;
+        ptx::fence_proxy_async();   // the weights become visible to the tensor core's reads
+      }
+      softmax_sync();
+      const bool again = j == 0 || *grow != 0u;
+      if (again) {
+        // Uniform over the eight warps, and rare but for the first tile: the raw scores are still there, since at least one
+        // warp has kept them.  New reference points, 2^6 above the maximum, for columns that have outgrown theirs; sums and O
+        // follow; the tile's weights once more.
+        constexpr int kLowest = (int)0x807fffff;   // -inf in an order of integers that is the order of floats
+        int* best = reinterpret_cast<int*>(shift_s);
+        ptx::tc_fence_after();
+        best[threadIdx.x] = kLowest;
+        softmax_sync();
+        if (threadIdx.x == 0) *grow = 0u;
+#pragma unroll 1
+        for (int c = 0; c < 2; ++c) {
+          mix(j, c, d);
+          int col = half * (MT / 2) + c * TC, in_group = 0;
 #pragma unroll
           for (int h = 0; h < HP; ++h) {
-            if (h < H) {
-              uint32_t w[TC / 2];
 #pragma unroll
-              for (int i = 0; i < TC / 2; ++i) {
-                const __nv_bfloat162 v = __floats2bfloat162_rn(ex2_fast(d[h][i].x), ex2_fast(d[h][i].y));
-                w[i] = *reinterpret_cast<const uint32_t*>(&v);
-              }
-              uint8_t* dst = p_s + (col >> 6) * kBlock + key * 128 + ((((col & 63) >> 3) ^ (key & 7)) << 4) + (col & 7) * 2;
-              if constexpr (TC == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(w[0], w[1], w[2], w[3]);
-              else if constexpr (TC == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(w[0], w[1]);
-              else *reinterpret_cast<uint32_t*>(dst) = w[0];
+            for (int i = 0; i < TC; ++i) {
+              const int o = __float_as_int(warp_max((i & 1) ? d[h][i / 2].y : d[h][i / 2].x));
+              if (lane == 0 && h < H) atomicMax(best + col + i, o >= 0 ? o : o ^ 0x7fffffff);
             }
             col += MT;
             if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
           }
         }
+        softmax_sync();
+        {
+          const int o = best[threadIdx.x];
+          const float up = __int_as_float(o >= 0 ? o : o ^ 0x7fffffff);
+          const float shift = o > kLowest && (j == 0 || up > 0.9f) ? up + 6.0f : 0.f;
+          m_s[threadIdx.x] -= shift;
+          shift_s[threadIdx.x] = shift;
+        }
+        softmax_sync();
+        if (j > 0) {   // (the product of the tile before has been waited for above)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float c0 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4]), c1 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4 + 1]);
+            sums[i][0] *= c0; sums[i][1] *= c1; sums[i][2] *= c0; sums[i][3] *= c1;
+          }
+          for (int v = 0; v < 2 * H; ++v) {
+            const int col = column(v >> 1) + half * (MT / 2) + (v & 1) * TC;
+            uint32_t r[TC];
+            ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
+            ptx::tmem_wait_ld();
+#pragma unroll
+            for (int i = 0; i < TC; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * ex2_fast(-shift_s[col + i]));
+            ptx::tmem_st_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
+          }
+          ptx::tmem_wait_st();
+        }
+#pragma unroll 1
+        for (int c = 0; c < 2; ++c) {
+          mix(j, c, d);
+          weights(c, d);
+        }
+        ptx::tc_fence_before();
+        ptx::fence_proxy_async();
+        softmax_sync();   // every warp has read the raw scores for the last time
+        if (kept && lane == 0) ptx::mbar_arrive(&ctl->s_empty);
       }
-      ptx::fence_proxy_async();   // the weights become visible to the tensor core's reads
-      ptx::tc_fence_before();
-      __syncwarp();
-      if (lane == 0) ptx::mbar_arrive(&ctl->p_full);
-      ptx::mbar_wait(&ctl->p_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles);
-      __syncwarp();
       // sums over the keys: ones . P
       const uint32_t ones[4] = {0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u};
 #pragma unroll
@@ -418,6 +420,8 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
           mma16816(sums[i], ones, bb[2], bb[3]);
         }
       }
+      __syncwarp();
+      if (lane == 0) ptx::mbar_arrive(&ctl->p_full);   // (now: once the product with V is through, P is free for the next tile)
     }
     // ------------------------------------------------------------------ output
     if (layout_ok) {
