@@ -10,10 +10,10 @@
 //   warps 0-7   a thread has one key (its lane) and 64 columns at a time, all heads of a few tokens: it reads the raw scores,
 //               mixes them in float32 (packed FMAs), masks, and stores the weights in bf16.  The reference point of the
 //               exponentials is one number per column for all 128 keys, 2^6 above the maximum when it was set.  A tile is
-//               computed on the reference points as they are; only if a weight comes out at 2 or more (always at the first tile)
-//               do the warps set new ones and compute the tile again, from raw scores that the warp in question has not
-//               given back.  One barrier per tile, which the sums over the keys need anyway: they come from a product with
-//               ones on mma.sync, in float32.
+//               computed on the reference points as they are; only if a score has outgrown its own by 2 (always at the first
+//               tile) do the warps set new ones and compute the tile again, from raw scores that the warp in question has
+//               not given back.  The sums of the weights over the keys come from a product with ones on mma.sync, in
+//               float32.
 //   warp 8      tiled copies: Q once, then K of every head, V of every head, ... through a ring of 128-key tiles (two pages);
 //   warp 9      owns the tensor memory; one lane issues the products: the scores of the next tile as soon as the raw scores of
 //               this one have been read, so that they are there when its weights are done.
@@ -45,6 +45,7 @@ struct MixParams {
   int pages_per_seq, s_new, q_heads, kv_heads, group, D, nb, nbv;
   int head_cols;              // columns of a key/value head: group * MT, rounded up so that no block of 64 is crossed
   int stages, value_dim;
+  int column[32];             // of a head's first token
   float scale_log2;
   const bf16 *talk, *sink;
   bf16* out;
@@ -55,7 +56,7 @@ struct MixParams {
 
 struct MixCtrl {
   uint64_t q_full, full[kMaxStages], empty[kMaxStages], s_full, s_empty, p_full, o_done;
-  uint32_t tmem_base, abort_flag, issued, grow[2];
+  uint32_t tmem_base, abort_flag, issued, grow[2][2];   // grow: [half][tile & 1]
 };
 
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
@@ -70,15 +71,38 @@ __device__ __forceinline__ float ex2_fast(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// among the eight softmax warps, and among the four of a half
 __device__ __forceinline__ void softmax_sync() {
   __syncwarp();
   asm volatile("bar.sync 1, 256;" ::: "memory");
+}
+template <bool kHalves>
+__device__ __forceinline__ void half_sync(int half) {
+  if (!kHalves) return softmax_sync();
+  __syncwarp();
+  asm volatile("bar.sync %0, 128;" ::"r"(2 + half) : "memory");
+}
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float r;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+  return r;
 }
 
 template <int HP>
 struct MixShape {
   static constexpr int MT = kCols / HP;      // tokens of a CTA
   static constexpr int TC = 64 / HP;         // tokens of a thread at a time
+  // Warps 0-3 have the first half of the tokens, warps 4-7 the second.  Where eight neighbouring columns belong to one half, each
+  // half goes its own way within a tile; otherwise all eight warps move together.
+  static constexpr bool kHalves = MT >= 16;
+  static __device__ __forceinline__ int eighth(int warp, int k) {   // the k-th of the four groups of 8 columns a warp adds up
+    const int i = (warp & 3) * 4 + k;
+    return !kHalves ? warp * 4 + k : i / (MT / 16) * (MT / 8) + (warp >> 2) * (MT / 16) + i % (MT / 16);
+  }
+  static __device__ __forceinline__ int own_column(int thread) {     // one column per thread, of its half
+    const int i = thread & 127;
+    return !kHalves ? thread : i / (MT / 2) * MT + (thread >> 7) * (MT / 2) + i % (MT / 2);
+  }
   // behind Q, P and the ring: talk (every coefficient twice), minus the reference points and their shifts, per column
   static constexpr int kTalkBytes = HP * HP * 8;
   static constexpr size_t fixed_bytes(int nb) { return (size_t)nb * kCols * 128 + 4 * kBlock + kTalkBytes + 2 * kCols * 4 + sizeof(MixCtrl); }
@@ -99,8 +123,8 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
   float* shift_s = m_s + kCols;                                         // by how much it has just moved; at the end 1 / sum
   MixCtrl* ctl = reinterpret_cast<MixCtrl*>(shift_s + kCols);
   volatile uint32_t* abort_flag = &ctl->abort_flag;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int G = p.kv_heads, H = p.q_heads, group = p.group;
+  const int warp = __shfl_sync(0xffffffffu, (int)threadIdx.x >> 5, 0), lane = threadIdx.x & 31;   // (uniform, and seen to be)
+  const int G = p.kv_heads, H = p.q_heads;
 
   if (threadIdx.x == 0) {
     ptx::mbar_init(&ctl->q_full, 1);
@@ -109,7 +133,8 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
     ptx::mbar_init(&ctl->s_empty, kWarps);
     ptx::mbar_init(&ctl->p_full, kWarps);
     ptx::mbar_init(&ctl->o_done, 1);
-    ctl->abort_flag = ctl->issued = ctl->grow[0] = ctl->grow[1] = 0;
+    ctl->abort_flag = ctl->issued = 0;
+    ctl->grow[0][0] = ctl->grow[0][1] = ctl->grow[1][0] = ctl->grow[1][1] = 0;
     ptx::fence_barrier_init();
     ptx::fence_proxy_async();
     ptx::tma_prefetch_desc(&tm_q);
@@ -141,37 +166,41 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
       ptx::mbar_expect_tx(&ctl->q_full, (uint32_t)(H * p.nb * MT * 128));
       for (int h = 0; h < H; ++h)
         for (int cb = 0; cb < p.nb; ++cb)
-          ptx::tma_load_2d(q_s + (size_t)cb * kCols * 128 + (size_t)(h / group * p.head_cols + h % group * MT) * 128, &tm_q, &ctl->q_full,
+          ptx::tma_load_2d(q_s + (size_t)cb * kCols * 128 + (size_t)p.column[h] * 128, &tm_q, &ctl->q_full,
                            h * p.D + cb * 64, b * p.s_new + t0);
-      uint32_t u = 0;
+      uint32_t phase = 1u;
+      int st = 0;
       bool ok = true;
       // a stage is 64 columns of a tile's keys, or one page of its values
       auto next_stage = [&](uint32_t bytes) -> uint8_t* {
-        const int st = u % p.stages;
-        if (!ptx::mbar_wait(&ctl->empty[st], ((u / p.stages) & 1u) ^ 1u, abort_flag, p.wait_cycles)) { ok = false; return nullptr; }
+        if (!ptx::mbar_wait(&ctl->empty[st], phase, abort_flag, p.wait_cycles)) { ok = false; return nullptr; }
         ptx::mbar_expect_tx(&ctl->full[st], bytes);
         return ring + (size_t)st * kBlock;
+      };
+      auto advance = [&]() {
+        ++ctl->issued;
+        if (++st == p.stages) { st = 0; phase ^= 1u; }
       };
       auto page_of = [&](int i) { return p.block_table[(size_t)b * p.pages_per_seq + min(i, p.pages_per_seq - 1)]; };
       auto load_keys = [&](int tile) {
         const int page0 = page_of(tile * 2), page1 = page_of(tile * 2 + 1);
-        for (int i = 0; i < G * p.nb && ok; ++i, ++u) {
-          const int g = i / p.nb, cb = i % p.nb, st = u % p.stages;
-          uint8_t* dst = next_stage(kBlock);
-          if (!dst) return;
-          ptx::tma_load_2d(dst, &tm_k, &ctl->full[st], cb * 64, (page0 * G + g) * kPageTokens);
-          ptx::tma_load_2d(dst + kPageBlock, &tm_k, &ctl->full[st], cb * 64, (page1 * G + g) * kPageTokens);
-          ctl->issued = u + 1;
-        }
+        for (int g = 0; g < G; ++g)
+          for (int cb = 0; cb < p.nb; ++cb) {
+            uint8_t* dst = next_stage(kBlock);
+            if (!dst) return;
+            ptx::tma_load_2d(dst, &tm_k, &ctl->full[st], cb * 64, (page0 * G + g) * kPageTokens);
+            ptx::tma_load_2d(dst + kPageBlock, &tm_k, &ctl->full[st], cb * 64, (page1 * G + g) * kPageTokens);
+            advance();
+          }
       };
       auto load_values = [&](int tile) {
         const int page[2] = {page_of(tile * 2), page_of(tile * 2 + 1)};
-        for (int i = 0; i < G * 2 && ok; ++i, ++u) {
-          const int st = u % p.stages, y = (page[i & 1] * G + (i >> 1)) * kPageTokens;
+        for (int i = 0; i < G * 2; ++i) {
+          const int y = (page[i & 1] * G + (i >> 1)) * kPageTokens;
           uint8_t* dst = next_stage((uint32_t)p.nbv * kPageBlock);
           if (!dst) return;
           for (int cb = 0; cb < p.nbv; ++cb) ptx::tma_load_2d(dst + cb * kPageBlock, &tm_v, &ctl->full[st], cb * 64, y);
-          ctl->issued = u + 1;
+          advance();
         }
       };
       load_keys(0);
@@ -183,23 +212,30 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
       // ------------------------------------------------------------------ products
       const uint32_t idesc_s = ptx::umma_idesc_bf16(kKeys, p.head_cols), idesc_o = ptx::umma_idesc_bf16(128, p.head_cols, true, true);
       const uint32_t qa = ptx::smem_u32(q_s), pa = ptx::smem_u32(p_s), ra = ptx::smem_u32(ring);
-      uint32_t u = 0;
+      // descriptors of the ring's first stage, of Q and of P; addresses in them count 16 bytes
+      const uint64_t dk = ptx::umma_desc_k_sw128(ra), dq = ptx::umma_desc_k_sw128(qa);
+      const uint64_t dv = ptx::umma_desc_mn_sw128(ra, kPageBlock, 1024), dp = ptx::umma_desc_mn_sw128(pa, kBlock, 1024);
+      uint32_t phase = 0u;
+      int st = 0;
       auto full = [&]() -> bool {
-        if (!ptx::mbar_wait(&ctl->full[u % p.stages], (u / p.stages) & 1u, abort_flag, p.wait_cycles)) return false;
+        if (!ptx::mbar_wait(&ctl->full[st], phase, abort_flag, p.wait_cycles)) return false;
         ptx::tc_fence_after();
         return true;
+      };
+      auto release = [&]() {
+        ptx::umma_commit(&ctl->empty[st]);
+        if (++st == p.stages) { st = 0; phase ^= 1u; }
       };
       auto scores = [&](int j) -> bool {
         if (!ptx::mbar_wait(&ctl->s_empty, ((uint32_t)j & 1u) ^ 1u, abort_flag, p.wait_cycles)) return false;
         for (int g = 0; g < G; ++g)
-          for (int cb = 0; cb < p.nb; ++cb, ++u) {
+          for (int cb = 0; cb < p.nb; ++cb) {
             if (!full()) return false;
-            const uint32_t ka = ra + (u % p.stages) * kBlock, qb = qa + cb * (kCols * 128) + g * p.head_cols * 128;
+            const uint64_t a = dk + (uint32_t)(st * (kBlock / 16)), bq = dq + (uint32_t)(cb * (kCols * 128 / 16) + g * p.head_cols * (128 / 16));
 #pragma unroll
             for (int kk = 0; kk < 4; ++kk)
-              ptx::umma_bf16(tmem_s + (uint32_t)(g * p.head_cols), ptx::umma_desc_k_sw128(ka + kk * 32), ptx::umma_desc_k_sw128(qb + kk * 32), idesc_s,
-                             (cb > 0 || kk > 0) ? 1u : 0u);
-            ptx::umma_commit(&ctl->empty[u % p.stages]);
+              ptx::umma_bf16(tmem_s + (uint32_t)(g * p.head_cols), a + kk * 2, bq + kk * 2, idesc_s, (cb > 0 || kk > 0) ? 1u : 0u);
+            release();
           }
         ptx::umma_commit(&ctl->s_full);
         return true;
@@ -209,15 +245,15 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
       for (int j = 0; j < n && ok; ++j) {
         if (j + 1 < n && !scores(j + 1)) break;
         if (!ptx::mbar_wait(&ctl->p_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles)) break;
-        for (int i = 0; i < G * 2 && ok; ++i, ++u) {
+        for (int i = 0; i < G * 2 && ok; ++i) {
           if (!full()) { ok = false; break; }
           const int col = (i >> 1) * p.head_cols, page = i & 1;
-          const uint32_t va = ra + (u % p.stages) * kBlock, pb = pa + (col >> 6) * kBlock + (col & 63) * 2 + page * kPageBlock;
+          const uint64_t a = dv + (uint32_t)(st * (kBlock / 16)),
+                         bp = dp + (uint32_t)(((col >> 6) * kBlock + (col & 63) * 2 + page * kPageBlock) / 16);
 #pragma unroll
           for (int ks = 0; ks < kPageTokens / 16; ++ks)   // 16 keys are 16 rows of 128 bytes further in both tiles
-            ptx::umma_bf16(tmem_o + (uint32_t)col, ptx::umma_desc_mn_sw128(va + ks * (16 * 128), kPageBlock, 1024),
-                           ptx::umma_desc_mn_sw128(pb + ks * (16 * 128), kBlock, 1024), idesc_o, (j > 0 || page > 0 || ks > 0) ? 1u : 0u);
-          ptx::umma_commit(&ctl->empty[u % p.stages]);
+            ptx::umma_bf16(tmem_o + (uint32_t)col, a + ks * 128, bp + ks * 128, idesc_o, (j > 0 || page > 0 || ks > 0) ? 1u : 0u);
+          release();
         }
         if (ok) ptx::umma_commit(&ctl->o_done);
       }
@@ -235,39 +271,39 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
     }
     m_s[threadIdx.x] = 0.f;
     softmax_sync();
-    auto column = [&](int h) { return h / group * p.head_cols + h % group * MT; };
-    float sums[4][4];   // columns 32 warp .. + 32, the same in every row of the fragment
+    float sums[4][4];   // of four groups of 8 columns, the same in every row of the fragment
 #pragma unroll
     for (int i = 0; i < 4; ++i) { sums[i][0] = sums[i][1] = sums[i][2] = sums[i][3] = 0.f; }
     // Chunk c of tile j: raw scores of TC tokens and all heads -> mixed scores less their reference points
     auto mix = [&](int j, int c, float2 (&d)[HP][TC / 2]) {
       const int i0 = half * (MT / 2) + c * TC;   // first token
       float2 x[HP][TC / 2];                      // raw scores of the token pairs
-      int col = i0, in_group = 0;
-      auto next_head = [&]() {
-        col += MT;
-        if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
-      };
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
         uint32_t r[TC];
         if (h < H) {   // uniform
-          ptx::tmem_ld_32xn<TC>(tmem_s + t_lane + (uint32_t)col, r);
+          ptx::tmem_ld_32xn<TC>(tmem_s + t_lane + (uint32_t)(p.column[h] + i0), r);
         } else {
 #pragma unroll
           for (int i = 0; i < TC; ++i) r[i] = 0u;
         }
 #pragma unroll
         for (int i = 0; i < TC / 2; ++i) x[h][i] = make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
-        next_head();
       }
       ptx::tmem_wait_ld();
-      col = i0;
-      in_group = 0;
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
+        const float* m = m_s + p.column[h] + i0;   // (column 0 for heads that are not there)
+        if constexpr (TC >= 4) {
 #pragma unroll
-        for (int i = 0; i < TC / 2; ++i) d[h][i] = *reinterpret_cast<const float2*>(m_s + (h < H ? col : 0) + 2 * i);
+          for (int i = 0; i < TC / 4; ++i) {
+            const float4 v = *reinterpret_cast<const float4*>(m + 4 * i);
+            d[h][2 * i] = make_float2(v.x, v.y);
+            d[h][2 * i + 1] = make_float2(v.z, v.w);
+          }
+        } else {
+          d[h][0] = *reinterpret_cast<const float2*>(m);
+        }
 #pragma unroll
         for (int g = 0; g < HP; g += 2) {
           const float4 t = *reinterpret_cast<const float4*>(t_s + h * HP + g);
@@ -277,7 +313,6 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
             d[h][i] = fma2(make_float2(t.z, t.w), x[g + 1][i], d[h][i]);
           }
         }
-        next_head();
       }
       if (j * kKeys + kKeys - 1 > base + t0) {   // a tile that the diagonal cuts
         const int first = j * kKeys + key - (base + t0 + i0);   // token i sees this key from i = first on
@@ -290,102 +325,103 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
           }
       }
     };
-    // The chunk's weights into P; all their bits together (a weight of 2 or more has bit 14 of its half set, no smaller one has)
-    auto weights = [&](int c, const float2 (&d)[HP][TC / 2]) -> uint32_t {
-      int col = half * (MT / 2) + c * TC, in_group = 0;
-      uint32_t bits = 0u;
+    // The chunk's weights into P
+    auto weights = [&](int c, const float2 (&d)[HP][TC / 2]) {
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
         if (h < H) {
+          const int col = p.column[h] + half * (MT / 2) + c * TC;
           uint32_t w[TC / 2];
 #pragma unroll
           for (int i = 0; i < TC / 2; ++i) {
             const __nv_bfloat162 v = __floats2bfloat162_rn(ex2_fast(d[h][i].x), ex2_fast(d[h][i].y));
             w[i] = *reinterpret_cast<const uint32_t*>(&v);
-            bits |= w[i];
           }
           uint8_t* dst = p_s + (col >> 6) * kBlock + key * 128 + ((((col & 63) >> 3) ^ (key & 7)) << 4) + (col & 7) * 2;
           if constexpr (TC == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(w[0], w[1], w[2], w[3]);
           else if constexpr (TC == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(w[0], w[1]);
           else *reinterpret_cast<uint32_t*>(dst) = w[0];
         }
-        col += MT;
-        if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
       }
-      return bits;
     };
     for (int j = 0; j < (layout_ok ? n : 0); ++j) {
       ptx::mbar_wait(&ctl->s_full, (uint32_t)j & 1u, abort_flag, p.wait_cycles);
       __syncwarp();
       ptx::tc_fence_after();
-      volatile uint32_t* grow = ctl->grow + (j & 1);   // (a fast warp may already be in the next tile)
+      volatile uint32_t* grow = &ctl->grow[C::kHalves ? half : 0][j & 1];   // (a fast warp may already be in the next tile)
       bool kept = j == 0;   // this warp has not given the raw scores back
       float2 d[HP][TC / 2];
       if (j > 0) {
-        uint32_t bits = 0u;
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          mix(j, c, d);
-          if (c == 0) {   // P of the tile before has been read
-            ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
-            __syncwarp();
-          }
-          bits |= weights(c, d);
-        }
-        kept = __any_sync(0xffffffffu, (bits & 0x40004000u) != 0u);
-        if (kept) {
-          if (lane == 0) *grow = 1u;
-        } else {   // the next tile's scores may come, once every warp has said so
-          ptx::tc_fence_before();
-          __syncwarp();
-          if (lane == 0) ptx::mbar_arrive(&ctl->s_empty);
-        }
-        ptx::fence_proxy_async();   // the weights become visible to the tensor core's reads
-      }
-      softmax_sync();
-      const bool again = j == 0 || *grow != 0u;
-      if (again) {
-        // Uniform over the eight warps, and rare but for the first tile: the raw scores are still there, since at least one
-        // warp has kept them.  New reference points, 2^6 above the maximum, for columns that have outgrown theirs; sums and O
-        // follow; the tile's weights once more.
-        constexpr int kLowest = (int)0x807fffff;   // -inf in an order of integers that is the order of floats
-        int* best = reinterpret_cast<int*>(shift_s);
-        ptx::tc_fence_after();
-        best[threadIdx.x] = kLowest;
-        softmax_sync();
-        if (threadIdx.x == 0) *grow = 0u;
 #pragma unroll 1
         for (int c = 0; c < 2; ++c) {
           mix(j, c, d);
-          int col = half * (MT / 2) + c * TC, in_group = 0;
+          float top = -INFINITY;
+#pragma unroll
+          for (int h = 0; h < HP; ++h)
+            if (h < H) {
+#pragma unroll
+              for (int i = 0; i < TC / 2; ++i) top = max3(top, d[h][i].x, d[h][i].y);
+            }
+          kept |= __any_sync(0xffffffffu, top > 1.0f) != 0;
+          if (c == 0) {   // P of the tile before has been read, by the product and by this half's sums
+            half_sync<C::kHalves>(half);
+            ptx::mbar_wait(&ctl->o_done, (uint32_t)(j - 1) & 1u, abort_flag, p.wait_cycles);
+            __syncwarp();
+          } else if (kept) {
+            if (lane == 0) *grow = 1u;
+          } else {   // the next tile's scores may come, once every warp has said so
+            ptx::tc_fence_before();
+            __syncwarp();
+            if (lane == 0) ptx::mbar_arrive(&ctl->s_empty);
+          }
+          weights(c, d);
+        }
+        ptx::fence_proxy_async();   // the weights become visible to the tensor core's reads
+      }
+      half_sync<C::kHalves>(half);
+      const bool again = j == 0 || *grow != 0u;
+      if (again) {
+        // Uniform over the half's four warps, and rare but for the first tile: the raw scores are still there, since at least
+        // one warp has kept them.  New reference points, 2^6 above the maximum, for columns that have outgrown theirs; sums and O
+        // follow; the tile's weights once more.
+        constexpr int kLowest = (int)0x807fffff;   // -inf in an order of integers that is the order of floats
+        int* best = reinterpret_cast<int*>(shift_s);
+        const int mine = C::own_column(threadIdx.x);
+        ptx::tc_fence_after();
+        best[mine] = kLowest;
+        half_sync<C::kHalves>(half);
+        if ((threadIdx.x & (C::kHalves ? 127 : 255)) == 0) *grow = 0u;
+#pragma unroll 1
+        for (int c = 0; c < 2; ++c) {
+          mix(j, c, d);
 #pragma unroll
           for (int h = 0; h < HP; ++h) {
+            if (h >= H) continue;
 #pragma unroll
             for (int i = 0; i < TC; ++i) {
               const int o = __float_as_int(warp_max((i & 1) ? d[h][i / 2].y : d[h][i / 2].x));
-              if (lane == 0 && h < H) atomicMax(best + col + i, o >= 0 ? o : o ^ 0x7fffffff);
+              if (lane == 0) atomicMax(best + p.column[h] + half * (MT / 2) + c * TC + i, o >= 0 ? o : o ^ 0x7fffffff);
             }
-            col += MT;
-            if (++in_group == group) { in_group = 0; col += p.head_cols - group * MT; }
           }
         }
-        softmax_sync();
+        half_sync<C::kHalves>(half);
         {
-          const int o = best[threadIdx.x];
+          const int o = best[mine];
           const float up = __int_as_float(o >= 0 ? o : o ^ 0x7fffffff);
           const float shift = o > kLowest && (j == 0 || up > 0.9f) ? up + 6.0f : 0.f;
-          m_s[threadIdx.x] -= shift;
-          shift_s[threadIdx.x] = shift;
+          m_s[mine] -= shift;
+          shift_s[mine] = shift;
         }
-        softmax_sync();
+        half_sync<C::kHalves>(half);
         if (j > 0) {   // (the product of the tile before has been waited for above)
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            const float c0 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4]), c1 = ex2_fast(-shift_s[warp * 32 + i * 8 + 2 * t4 + 1]);
+            const float* by = shift_s + C::eighth(warp, i) * 8 + 2 * t4;
+            const float c0 = ex2_fast(-by[0]), c1 = ex2_fast(-by[1]);
             sums[i][0] *= c0; sums[i][1] *= c1; sums[i][2] *= c0; sums[i][3] *= c1;
           }
           for (int v = 0; v < 2 * H; ++v) {
-            const int col = column(v >> 1) + half * (MT / 2) + (v & 1) * TC;
+            const int col = p.column[v >> 1] + half * (MT / 2) + (v & 1) * TC;
             uint32_t r[TC];
             ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
             ptx::tmem_wait_ld();
@@ -402,14 +438,15 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
         }
         ptx::tc_fence_before();
         ptx::fence_proxy_async();
-        softmax_sync();   // every warp has read the raw scores for the last time
+        half_sync<C::kHalves>(half);   // every warp has read the raw scores for the last time
         if (kept && lane == 0) ptx::mbar_arrive(&ctl->s_empty);
       }
+      if (lane == 0) ptx::mbar_arrive(&ctl->p_full);
       // sums over the keys: ones . P
       const uint32_t ones[4] = {0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u};
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int col = warp * 32 + i * 8;
+        const int col = C::eighth(warp, i) * 8;
         const uint32_t src = s_u32(p_s + (col >> 6) * kBlock);
 #pragma unroll
         for (int k = 0; k < kKeys / 32; ++k) {
@@ -420,8 +457,6 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
           mma16816(sums[i], ones, bb[2], bb[3]);
         }
       }
-      __syncwarp();
-      if (lane == 0) ptx::mbar_arrive(&ctl->p_full);   // (now: once the product with V is through, P is free for the next tile)
     }
     // ------------------------------------------------------------------ output
     if (layout_ok) {
@@ -431,11 +466,15 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
       softmax_sync();
       if (g8 == 0) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) { shift_s[warp * 32 + i * 8 + 2 * t4] = sums[i][0]; shift_s[warp * 32 + i * 8 + 2 * t4 + 1] = sums[i][1]; }
+        for (int i = 0; i < 4; ++i) {
+          float* l = shift_s + C::eighth(warp, i) * 8 + 2 * t4;
+          l[0] = sums[i][0];
+          l[1] = sums[i][1];
+        }
       }
       softmax_sync();
       for (int v = threadIdx.x; v < H * MT; v += kSoftmax) {
-        const int h = v / MT, col = column(h) + v % MT;
+        const int h = v / MT, col = p.column[h] + v % MT;
         const float l = shift_s[col] + (p.sink ? ex2_fast(fmaf(__bfloat162float(p.sink[h]), kLog2e, m_s[col])) : 0.f);
         shift_s[col] = 1.0f / l;
       }
@@ -445,7 +484,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
         for (int h = 0; h < H; ++h) {
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
-            const int i0 = half * (MT / 2) + c * TC, col = column(h) + i0;
+            const int i0 = half * (MT / 2) + c * TC, col = p.column[h] + i0;
             uint32_t r[TC];
             ptx::tmem_ld_32xn<TC>(tmem_o + t_lane + (uint32_t)col, r);
             ptx::tmem_wait_ld();
@@ -526,7 +565,10 @@ int attention_mix_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int 
   const int hp = padded_heads(q_heads);
   p.block_table = c->block_table; p.seq_lens = c->seq_lens; p.pages_per_seq = c->pages_per_seq; p.s_new = s_new; p.q_heads = q_heads;
   p.kv_heads = c->kv_heads; p.group = q_heads / c->kv_heads; p.D = c->head_dim; p.nb = c->head_dim / 64; p.nbv = (x.value_dim + 63) / 64;
-  p.head_cols = head_columns(p.group * (kCols / hp)); p.value_dim = x.value_dim; p.scale_log2 = scale * kLog2e;
+  const int mt = kCols / hp;
+  p.head_cols = head_columns(p.group * mt);
+  for (int h = 0; h < q_heads; ++h) p.column[h] = h / p.group * p.head_cols + h % p.group * mt;
+  p.value_dim = x.value_dim; p.scale_log2 = scale * kLog2e;
   p.talk = (const bf16*)x.talk; p.sink = (const bf16*)x.sink; p.out = (bf16*)out; p.out_ld = x.out_ld; p.status = ctx->status_dev;
   p.wait_cycles = ctx->local_wait_cycles();
   RB_REQUIRE(batch <= 65535, "attention: batch %d too large", batch);
