@@ -317,6 +317,8 @@ typedef struct rb_attention_options {
   int32_t reserved0;
   const void* talk;                /* [q_heads][q_heads], model dtype: score[h] <- sum over g of talk[h][g] * score[g], after scale and
                                       before mask and softmax; goes with window, chunk, sink and value_dim only */
+  const float* talk_host;          /* the numbers of `talk` once more, in host memory (read during the call), or NULL: with them
+                                      prompts run on the tensor cores' own kernel */
 } rb_attention_options;
 int32_t rb_attention_general(rb_ctx* ctx, const void* q_dev, rb_kv_cache* cache, int32_t layer, int32_t batch, int32_t s_new,
                              int32_t q_heads, float scale, const rb_attention_options* options, void* out_dev, int32_t dtype);

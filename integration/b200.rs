@@ -139,6 +139,7 @@ pub struct rb_attention_options {
     pub out_scale: f32,
     pub reserved0: i32,
     pub talk: *const c_void,
+    pub talk_host: *const f32,
 }
 
 /// `struct rb_route_options` of include/rai_b200.h, field for field.

@@ -69,7 +69,7 @@ class AttentionOptions(ctypes.Structure):
                 ("temp_coef", ctypes.c_float), ("softcap", ctypes.c_float), ("value_dim", ctypes.c_int32),
                 ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64), ("sink", ctypes.c_void_p), ("out_ld", ctypes.c_int64),
                 ("chunk", ctypes.c_int32), ("head_gate", ctypes.c_int32), ("out_scale", ctypes.c_float), ("reserved0", ctypes.c_int32),
-                ("talk", ctypes.c_void_p)]
+                ("talk", ctypes.c_void_p), ("talk_host", ctypes.c_void_p)]
 
 
 class RouteOptions(ctypes.Structure):

@@ -530,7 +530,7 @@ extern "C" int32_t rb_attention_general(rb_ctx* ctx, const void* q, rb_kv_cache*
   x.value_dim = o->value_dim ? o->value_dim : c->head_dim;
   x.out_ld = o->out_ld ? o->out_ld : (int64_t)q_heads * x.value_dim;
   x.temp_every = o->temp_every; x.temp_coef = o->temp_coef; x.softcap = o->softcap; x.sink = o->sink;
-  x.talk = o->talk; x.chunk = o->chunk; x.head_gate = o->gate && o->head_gate; x.out_scale = o->out_scale != 0.f ? o->out_scale : 1.f;
+  x.talk = o->talk; x.talk_host = o->talk ? o->talk_host : nullptr; x.chunk = o->chunk; x.head_gate = o->gate && o->head_gate; x.out_scale = o->out_scale != 0.f ? o->out_scale : 1.f;
   RB_REQUIRE(x.value_dim > 0 && x.value_dim <= c->head_dim, "rb_attention_general: value size %d of a %d-wide cache", x.value_dim,
              c->head_dim);
   RB_REQUIRE(x.window >= 0 && x.window <= (1 << 30), "rb_attention_general: bad window %d", x.window);

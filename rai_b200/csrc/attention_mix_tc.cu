@@ -46,8 +46,7 @@ struct MixParams {
   int head_cols;              // columns of a key/value head: group * MT, rounded up so that no block of 64 is crossed
   int stages, value_dim;
   int column[32];             // of a head's first token
-  float scale_log2;
-  const bf16 *talk, *sink;
+  const bf16* sink;
   bf16* out;
   int64_t out_ld;
   uint32_t* status;
@@ -103,23 +102,29 @@ struct MixShape {
     const int i = thread & 127;
     return !kHalves ? thread : i / (MT / 2) * MT + (thread >> 7) * (MT / 2) + i % (MT / 2);
   }
-  // behind Q, P and the ring: talk (every coefficient twice), minus the reference points and their shifts, per column
-  static constexpr int kTalkBytes = HP * HP * 8;
-  static constexpr size_t fixed_bytes(int nb) { return (size_t)nb * kCols * 128 + 4 * kBlock + kTalkBytes + 2 * kCols * 4 + sizeof(MixCtrl); }
+  // behind Q, P and the ring: minus the reference points and their shifts, per column
+  static constexpr size_t fixed_bytes(int nb) { return (size_t)nb * kCols * 128 + 4 * kBlock + 2 * kCols * 4 + sizeof(MixCtrl); }
+};
+
+// scale * log2(e) * talk[h][g], every number twice, as operands of the launch: constants to the mixing, which would otherwise spend
+// more on fetching them from shared memory than on its multiply-adds
+template <int HP>
+struct MixTalk {
+  float2 t[HP * HP];
 };
 
 template <int HP>
 __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __grid_constant__ CUtensorMap tm_q,
                                                                       const __grid_constant__ CUtensorMap tm_k,
-                                                                      const __grid_constant__ CUtensorMap tm_v, const MixParams p) {
+                                                                      const __grid_constant__ CUtensorMap tm_v, const MixParams p,
+                                                                      const __grid_constant__ MixTalk<HP> talk) {
   using C = MixShape<HP>;
   constexpr int MT = C::MT, TC = C::TC;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* q_s = smem;                                                  // [nb][256 columns][128 bytes]
   uint8_t* p_s = q_s + (size_t)p.nb * kCols * 128;                      // [4][128 keys][128 bytes]
   uint8_t* ring = p_s + 4 * kBlock;
-  float2* t_s = reinterpret_cast<float2*>(ring + (size_t)p.stages * kBlock);   // [h][g]
-  float* m_s = reinterpret_cast<float*>(t_s + HP * HP);                 // minus the reference point, per column
+  float* m_s = reinterpret_cast<float*>(ring + (size_t)p.stages * kBlock);   // minus the reference point, per column
   float* shift_s = m_s + kCols;                                         // by how much it has just moved; at the end 1 / sum
   MixCtrl* ctl = reinterpret_cast<MixCtrl*>(shift_s + kCols);
   volatile uint32_t* abort_flag = &ctl->abort_flag;
@@ -264,11 +269,6 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
     const int quarter = warp & 3, half = warp >> 2, key = quarter * 32 + lane;
     const uint32_t t_lane = (uint32_t)(quarter * 32) << 16;
     const int g8 = lane >> 2, t4 = lane & 3;
-    for (int i = threadIdx.x; i < HP * HP; i += kSoftmax) {
-      const int h = i / HP, g = i % HP;
-      const float t = h < H && g < H ? __bfloat162float(p.talk[h * H + g]) * p.scale_log2 : 0.f;
-      t_s[i] = make_float2(t, t);
-    }
     m_s[threadIdx.x] = 0.f;
     softmax_sync();
     float sums[4][4];   // of four groups of 8 columns, the same in every row of the fragment
@@ -305,14 +305,9 @@ __global__ void __launch_bounds__(kThreads, 1) attention_mix_tc_kernel(const __g
           d[h][0] = *reinterpret_cast<const float2*>(m);
         }
 #pragma unroll
-        for (int g = 0; g < HP; g += 2) {
-          const float4 t = *reinterpret_cast<const float4*>(t_s + h * HP + g);
+        for (int g = 0; g < HP; ++g)
 #pragma unroll
-          for (int i = 0; i < TC / 2; ++i) {
-            d[h][i] = fma2(make_float2(t.x, t.y), x[g][i], d[h][i]);
-            d[h][i] = fma2(make_float2(t.z, t.w), x[g + 1][i], d[h][i]);
-          }
-        }
+          for (int i = 0; i < TC / 2; ++i) d[h][i] = fma2(talk.t[h * HP + g], x[g][i], d[h][i]);
       }
       if (j * kKeys + kKeys - 1 > base + t0) {   // a tile that the diagonal cuts
         const int first = j * kKeys + key - (base + t0 + i0);   // token i sees this key from i = first on
@@ -527,12 +522,17 @@ int head_columns(int n) {
 int padded_heads(int H) { return H <= 8 ? 8 : H <= 16 ? 16 : 32; }
 
 template <int HP>
-int launch_mix(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, MixParams p) {
+int launch_mix(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch, MixParams p, const float* talk, float scale) {
   using C = MixShape<HP>;
   constexpr size_t kLimit = 227 * 1024;
   const size_t fixed = C::fixed_bytes(p.nb);
   p.stages = (int)std::min<size_t>(kMaxStages, (kLimit - fixed) / kBlock);
   const size_t smem = fixed + (size_t)p.stages * kBlock;
+  MixTalk<HP> coef;
+  for (int i = 0; i < HP * HP; ++i) {
+    const int h = i / HP, g = i % HP;
+    coef.t[i].x = coef.t[i].y = h < p.q_heads && g < p.q_heads ? talk[h * p.q_heads + g] * scale * kLog2e : 0.f;
+  }
   auto kern = attention_mix_tc_kernel<HP>;
   static size_t set[64] = {};
   const int dv = ctx->device & 63;
@@ -545,7 +545,7 @@ int launch_mix(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch,
   RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->k + off, rows, p.D, p.D, kPageTokens, &tk));
   RB_TRY(tmap_2d_bf16(ctx, (const bf16*)c->v + off, rows, p.D, p.D, kPageTokens, &tv));
   RB_CUDA(launch_kernel(kern, dim3((unsigned)((p.s_new + C::MT - 1) / C::MT), (unsigned)batch), dim3(kThreads), smem, ctx->stream, ctx->pdl, tq, tk,
-                        tv, p));
+                        tv, p, coef));
   ctx->launches++;
   return RB_OK;
 }
@@ -554,7 +554,7 @@ int launch_mix(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int batch,
 
 bool attention_mix_tc_takes(const rb_kv_cache* c, int s_new, int q_heads, const void* q, const AttnExtra& x) {
   if (c->dtype != RB_BF16 || c->shared() || (c->head_dim != 64 && c->head_dim != 128) || q_heads > 32 || q_heads % c->kv_heads != 0) return false;
-  if (x.window > 0 || x.chunk > 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0) return false;
+  if (!x.talk_host || x.window > 0 || x.chunk > 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0) return false;
   const int mt = kCols / padded_heads(q_heads);
   return s_new >= 16 && c->kv_heads * head_columns(q_heads / c->kv_heads * mt) <= kCols;
 }
@@ -568,13 +568,13 @@ int attention_mix_tc(rb_ctx* ctx, const void* q, rb_kv_cache* c, int layer, int 
   const int mt = kCols / hp;
   p.head_cols = head_columns(p.group * mt);
   for (int h = 0; h < q_heads; ++h) p.column[h] = h / p.group * p.head_cols + h % p.group * mt;
-  p.value_dim = x.value_dim; p.scale_log2 = scale * kLog2e;
-  p.talk = (const bf16*)x.talk; p.sink = (const bf16*)x.sink; p.out = (bf16*)out; p.out_ld = x.out_ld; p.status = ctx->status_dev;
+  p.value_dim = x.value_dim;
+  p.sink = (const bf16*)x.sink; p.out = (bf16*)out; p.out_ld = x.out_ld; p.status = ctx->status_dev;
   p.wait_cycles = ctx->local_wait_cycles();
   RB_REQUIRE(batch <= 65535, "attention: batch %d too large", batch);
-  if (hp == 8) return launch_mix<8>(ctx, q, c, layer, batch, p);
-  if (hp == 16) return launch_mix<16>(ctx, q, c, layer, batch, p);
-  return launch_mix<32>(ctx, q, c, layer, batch, p);
+  if (hp == 8) return launch_mix<8>(ctx, q, c, layer, batch, p, x.talk_host, scale);
+  if (hp == 16) return launch_mix<16>(ctx, q, c, layer, batch, p, x.talk_host, scale);
+  return launch_mix<32>(ctx, q, c, layer, batch, p, x.talk_host, scale);
 }
 
 }  // namespace rb

@@ -257,6 +257,7 @@ struct AttnExtra {
   float softcap = 0.f;         // > 0: score <- softcap tanh(score / softcap)
   const void* sink = nullptr;  // [q_heads], cache dtype: exp(sink) joins the softmax denominator
   const void* talk = nullptr;  // [q_heads][q_heads], cache dtype: score[h] <- sum_g talk[h][g] score[g] before the mask
+  const float* talk_host = nullptr;   // the same numbers on the host, or NULL
 };
 // the earliest position that the row at position `pos` sees (window 2^30: no window; chunk 0: no chunks)
 __host__ __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {

@@ -306,8 +306,17 @@ int project(rb_model* m, const void* x, const void* w, const void* bias, void* d
 }
 
 // Attention whose heads' scores are mixed, from m->h to m->attn
-int talking_mixer(rb_model* m, const MixLayer& w, int batch, int seq) {
+int talking_mixer(rb_model* m, MixLayer& w, int batch, int seq) {
   const rb_layer_config& c = w.c;
+  if (seq > 1 && w.talk_version != m->params_loaded) {   // the first prompt with these parameters (never a captured step)
+    const int n = c.heads * c.heads;
+    std::vector<__nv_bfloat16> half(n);
+    w.talk_host.resize(n);
+    RB_TRY(rb_download(m->ctx, m->cfg.dtype == RB_F32 ? (void*)w.talk_host.data() : (void*)half.data(), w.talk, n * m->es));
+    if (m->cfg.dtype == RB_BF16)
+      for (int i = 0; i < n; ++i) w.talk_host[i] = __bfloat162float(half[i]);
+    w.talk_version = m->params_loaded;
+  }
   const int dt = m->cfg.dtype;
   Projected u;
   RB_TRY(project(m, m->h, w.in_w, w.in_b, m->mix_in, (int64_t)batch * seq, w.n_in, m->ld, seq, &u));
@@ -316,6 +325,7 @@ int talking_mixer(rb_model* m, const MixLayer& w, int batch, int seq) {
                                   nullptr, 0, dt));
   rb_attention_options o{};
   o.value_dim = c.value_dim; o.out_ld = w.mix_k; o.talk = w.talk; o.sink = w.sink;
+  o.talk_host = w.talk_version == m->params_loaded ? w.talk_host.data() : nullptr;
   return rb_attention_general(m->ctx, m->q, w.kv, w.kv_layer, batch, seq, c.heads, (float)c.scale, &o, m->attn, dt);
 }
 
@@ -362,7 +372,7 @@ int latent_mixer(rb_model* m, const MixLayer& w, int batch, int seq) {
 
 // A sandwich block on m->h (the stream, normalised for the mixer), the l-th; m->h is then what the next block (gain, or NULL after
 // the last) reads.  The stream that enters block 0 is the history's first entry.
-int sandwich_block(rb_model* m, const MixLayer& w, int l, int batch, int seq, const void* next_gain) {
+int sandwich_block(rb_model* m, MixLayer& w, int l, int batch, int seq, const void* next_gain) {
   const rb_model_config& cfg = m->cfg;
   const int64_t rows = (int64_t)batch * seq;
   RB_TRY(w.c.mixer == RB_MIXER_LATENT ? latent_mixer(m, w, batch, seq) : talking_mixer(m, w, batch, seq));
@@ -414,7 +424,7 @@ int rb::layered_forward(rb_model* m, const uint32_t* tokens, int batch, int seq,
     RB_TRY(rb_embed_stream(ctx, m->embed, c.dtype, c.vocab_size, c.hidden_size, m->ld, tokens, rows, m->stream,
                            c.dtype == RB_F32 ? nullptr : m->h));
   for (size_t l = 0; l < m->mix.size(); ++l) {
-    const MixLayer& w = m->mix[l];
+    MixLayer& w = m->mix[l];
     const void* next_gain = l + 1 < m->mix.size() ? m->mix[l + 1].norm1 : nullptr;
     if (sandwich) {
       RB_TRY(sandwich_block(m, w, (int)l, batch, seq, next_gain));

@@ -768,6 +768,7 @@ extern "C" rb_kv_cache* rb_model_kv_cache(rb_model* m) { return m ? m->cache : n
 
 template <typename S>
 static int copy_pieces(rb_model* m, const ParamSpec& sp, const S* src_dev) {
+  ++m->params_loaded;
   for (const Piece& pc : sp.pieces) {
     const int64_t n = pc.rows * pc.cols;
     if (n == 0) continue;

@@ -63,6 +63,8 @@ struct MixLayer {
   // latent attention (fused input projection [query latent | latent, key part | gate])
   void *norm1b = nullptr, *norm2b = nullptr, *depth = nullptr, *talk = nullptr;
   void *dq_norm = nullptr, *dkv_norm = nullptr, *uq = nullptr, *uk = nullptr, *uv = nullptr;   // uk, uv: one matrix [keys | values]
+  std::vector<float> talk_host;   // as of talk_version of rb_model::params_loaded
+  int64_t talk_version = -1;
   int qr_p = 0, kv_p = 0, kr_p = 0, n_q = 0, n_kv = 0, v_col = 0;   // padded sizes: latents, their columns, heads multiplied out
   int prompt_kv = -1;          // index into rb_model::prompt_kv; -1: prompts, too, attend in the latent's space
   rb_kv_cache* kv = nullptr;   // the cache (of this layer's geometry) its keys and values are in, and the layer there
@@ -87,6 +89,7 @@ struct rb_model {
   std::vector<std::string> names;
   std::map<std::string, rb::ParamSpec> params;
   int64_t param_bytes = 0;
+  int64_t params_loaded = 0;   // grows with every parameter that is loaded
   // workspace
   uint32_t* ids = nullptr;
   void *h = nullptr, *xn = nullptr, *tmp = nullptr, *qkv = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;

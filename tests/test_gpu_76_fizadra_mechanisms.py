@@ -262,7 +262,8 @@ def test_into_the_latents_space_and_out(cuda, dtype, H, d, rd, turning, interlea
 
 # ---- attention
 
-def talking_case(cuda, dtype, H, G, d, e, base, s_new, scale=0.2, B=2, sink=None, plant=None, seed=0, window=0, chunk=0):
+def talking_case(cuda, dtype, H, G, d, e, base, s_new, scale=0.2, B=2, sink=None, plant=None, seed=0, window=0, chunk=0,
+                 on_host=True):
     """(got, want) [B, s_new, H, e]: `base` tokens are cached, `s_new` are fed.  plant = (row, key): that query's and that key's
     scores stand out after mixing, and the key's value is 5."""
     rng, T = np.random.default_rng(seed), base + s_new
@@ -279,6 +280,7 @@ def talking_case(cuda, dtype, H, G, d, e, base, s_new, scale=0.2, B=2, sink=None
     fused = np.zeros((B, T, offs[-1]))
     for a, o in zip((q, k, v), offs):
         fused[:, :, o:o + a[0, 0].size] = a.reshape(B, T, -1)
+    host = np.ascontiguousarray(talk, dtype=np.float32)
     td, sd, out_ld = dev(talk, dtype), None if sink is None else dev(sink, dtype), pad8(H * e) + 8
     for lo, hi in ((0, base), (base, T)):
         if hi == lo:
@@ -289,7 +291,8 @@ def talking_case(cuda, dtype, H, G, d, e, base, s_new, scale=0.2, B=2, sink=None
         _lib.call("rb_head_norm_rope_append", cuda.ctx, ptr(src), None, 0, None, fused.shape[2], None, None, 1e-5, None, None, 0, B, hi - lo, H, G, d, e,
                   cache.h, 0, ptr(qd), None, 0, dtype)
         if lo == base:
-            o = _lib.AttentionOptions(value_dim=e, out_ld=out_ld, talk=ptr(td), sink=ptr(sd), window=window, chunk=chunk)
+            o = _lib.AttentionOptions(value_dim=e, out_ld=out_ld, talk=ptr(td), sink=ptr(sd), window=window, chunk=chunk,
+                                      talk_host=host.ctypes.data if on_host else None)
             _lib.call("rb_attention_general", cuda.ctx, ptr(qd), cache.h, 0, B, hi - lo, H, scale, ctypes.byref(o), ptr(out), dtype)
         cuda.synchronize()
     cache.close()
