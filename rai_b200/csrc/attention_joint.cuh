@@ -5,7 +5,7 @@
 // Eight consumer warps and one that issues tiled copies.  Per tile of KT keys:
 //   1  scores, transposed: S^T[keys x rows] = K . Q^T on mma.sync, a row being a (token, query head) that reads the tile's
 //      key/value head; keys fill the 16-row side, so a single token's few heads waste nothing.  Raw scores go to shared memory.
-//   2  a warp takes eight heads of a token (or eight rows): lanes are keys.  It mixes the raw scores of all heads (float32),
+//   2  a warp takes a few heads of a token (or a few rows): lanes are keys.  It mixes the raw scores of all heads (float32),
 //      masks, and turns them into weights against a reference point that follows the running maximum lazily; weights go to
 //      shared memory in bf16, the sum of a row stays in float32.
 //   3  O^T[dims x rows] += V^T . P^T, accumulators in registers for the whole walk.
@@ -42,6 +42,7 @@ struct Params {
   int row_tiles, tile_rows;    // rows (token, head of a key/value head) of a block: tile_rows <= 8 NT
   int nbk, nbv;                // 64-column blocks of a key and of a value that matter
   int stages, stage_bytes;
+  uint32_t stages_inv;         // ceil(2^32 / stages)
   int n_splits;
   int window, chunk, value_dim;
   float scale_log2;
@@ -64,10 +65,11 @@ struct Shape {
   static constexpr int R = 8 * NT;                            // rows per key/value head
   static constexpr int SP = KT + 4, PP = KT + 8;              // pitches of scores (floats) and weights (bf16)
   static constexpr int KL = KT / 32;                          // keys per lane
+  static constexpr int CH = NT == 1 ? 2 : 8;                  // heads that a warp mixes at a time
 };
 
 struct Layout {   // byte offsets behind the ring
-  size_t q, s, p, talk, m, total;
+  size_t q, s, p, talk, row, m, total;
 };
 template <typename S>
 __host__ __device__ inline Layout layout_of(int G, int H, int nbk) {
@@ -78,6 +80,7 @@ __host__ __device__ inline Layout layout_of(int G, int H, int nbk) {
   l.s = at; at += (size_t)S::SK * rows * S::SP * 4;
   l.p = at; at += rows * S::PP * 2;
   l.talk = at; at += S::LATENT ? 0 : (size_t)H * ((H + 7) / 8 * 8) * 4;
+  l.row = at; at += S::LATENT ? 0 : (size_t)H * 4;
   l.m = at; at += rows * 3 * 4;
   l.total = at;
   return l;
@@ -163,6 +166,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
   float* s_s = reinterpret_cast<float*>(rest + lay.s);
   bf16* p_s = reinterpret_cast<bf16*>(rest + lay.p);
   float* t_s = reinterpret_cast<float*>(rest + lay.talk);     // [g][h]: scale * log2(e) * talk[h][g]
+  int* row_s = reinterpret_cast<int*>(rest + lay.row);        // first row of a head
   float* m_s = reinterpret_cast<float*>(rest + lay.m);        // reference point, sum, rescaling factor per row
   const int rows = G * R, qp = p.nbk * 64 + 8, hp = (H + 7) / 8 * 8;
   float* l_s = m_s + rows;
@@ -197,6 +201,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     tile_hi = min(tile_hi, tile_lo + per);
   }
   const int units = S::LATENT ? 1 : 2 * G;   // copies per key tile
+  auto turn_of = [&](uint32_t u) { return __umulhi(u, p.stages_inv); };   // u / stages (u < 2^20)
 
   if (warp >= 8) {
     // ------------------------------------------------------------------ copies
@@ -207,8 +212,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       for (int tile = tile_lo; tile < tile_hi && ok; ++tile) {
         const int page = p.block_table[(size_t)b * p.pages_per_seq + tile * KT / kPageTokens];
         for (int i = 0; i < units && ok; ++i, ++u) {
-          const int st = u % p.stages;
-          if (!ptx::mbar_wait(&empty_bar[st], ((u / p.stages) & 1u) ^ 1u, &abort_flag, p.wait_cycles)) { ok = false; break; }
+          const uint32_t turn = turn_of(u), st = u - turn * p.stages;
+          if (!ptx::mbar_wait(&empty_bar[st], (turn & 1u) ^ 1u, &abort_flag, p.wait_cycles)) { ok = false; break; }
           const bool v = i >= G;
           const int nb = v ? p.nbv : p.nbk, y = (page * G + (v ? i - G : i)) * kPageTokens + tile * KT % kPageTokens;
           ptx::mbar_expect_tx(&full_bar[st], (uint32_t)nb * KT * 128);
@@ -234,6 +239,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     for (int i = threadIdx.x; i < rows * (PP / 8); i += kConsumers) reinterpret_cast<uint4*>(p_s)[i] = make_uint4(0, 0, 0, 0);
     for (int i = threadIdx.x; i < rows; i += kConsumers) { m_s[i] = -INFINITY; l_s[i] = 0.f; c_s[i] = 1.f; }
     if (!S::LATENT)
+      for (int h = threadIdx.x; h < H; h += kConsumers) row_s[h] = h / group * R + h % group;
+    if (!S::LATENT)
       for (int i = threadIdx.x; i < H * hp; i += kConsumers) {
         const int g = i / hp, h = i % hp;
         t_s[i] = h < H ? __bfloat162float(p.talk[h * H + g]) * p.scale_log2 : 0.f;
@@ -249,7 +256,19 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     const int team = warp / S::WG, wi = warp % S::WG, g8 = lane >> 2, t4 = lane & 3;
     const int km = wi % S::SM, ks = wi / S::SM;
     const int steps = p.nbk * 4, per_part = (steps + S::SK - 1) / S::SK, k_lo = ks * per_part, k_hi = min(steps, k_lo + per_part);
-    const int live_heads = p.value_dim;
+    const int live_dims = p.value_dim, n_tokens = S::LATENT ? 1 : n_rows / group;
+    float m_row[NT], l_row[NT];   // LATENT: of this warp's rows
+    int seen_from[NT], seen_to[NT];
+    if constexpr (S::LATENT) {
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int row = warp * NT + i;
+        m_row[i] = -INFINITY;
+        l_row[i] = 0.f;
+        seen_to[i] = row < n_rows ? base + (r0 + row) / group : -1;
+        seen_from[i] = row < n_rows ? first_visible(seen_to[i], p.window, p.chunk) : 0;
+      }
+    }
     for (int tile = tile_lo; tile < tile_hi; ++tile) {
       const int it = tile - tile_lo, key0 = tile * KT;
       // ---------------------------------------------------------------- 1: raw scores
@@ -257,8 +276,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       for (int a = 0; a < GP; ++a) {
         const int g = a * S::TEAMS + team;
         if (g >= G) continue;
-        const uint32_t u = (uint32_t)it * units + g, st = u % p.stages;
-        ptx::mbar_wait(&full_bar[st], (u / p.stages) & 1u, &abort_flag, p.wait_cycles);
+        const uint32_t u = (uint32_t)it * units + g, turn = turn_of(u), st = u - turn * p.stages;
+        ptx::mbar_wait(&full_bar[st], turn & 1u, &abort_flag, p.wait_cycles);
         __syncwarp();
         const uint32_t kt = s_u32(ring + (size_t)st * p.stage_bytes);
         constexpr int NC = NT < 4 ? NT : 4;
@@ -307,129 +326,135 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       consumers_sync();
       // ---------------------------------------------------------------- 2: mixing, mask, weights
       if (threadIdx.x == 0) rescale_flag[(it + 1) & 1] = 0;
-      const int chunks = S::LATENT ? (n_rows + 7) / 8 : hp / 8, n_units = S::LATENT ? chunks : chunks * (n_rows / group);
-      for (int unit = warp; unit < n_units; unit += 8) {
-        const int tok = S::LATENT ? 0 : unit / chunks, h0 = (S::LATENT ? unit : unit % chunks) * 8;   // eight heads, or eight rows
-        float2 acc[4][KL];
+      auto raw = [&](int row, float (&v)[KL]) {   // the parts of the dot product added up
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+        for (int e = 0; e < KL; ++e) v[e] = 0.f;
 #pragma unroll
-          for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(0.f, 0.f);
-        auto raw = [&](int row, float* v) {
+        for (int k = 0; k < S::SK; ++k) {
+          const float* src = s_s + ((size_t)k * rows + row) * SP + lane * KL;
+          if constexpr (KL == 1) v[0] += src[0];
+          else { const float2 t = *reinterpret_cast<const float2*>(src); v[0] += t.x; v[KL - 1] += t.y; }
+        }
+      };
+      auto store_weights = [&](int row, const float (&v)[KL]) {
+        bf16* dst = p_s + (size_t)row * PP + lane * KL;
+        if constexpr (KL == 1) dst[0] = __float2bfloat16_rn(v[0]);
+        else *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v[0], v[KL - 1]);
+      };
+      if constexpr (S::LATENT) {   // a warp has NT rows for the whole walk: reference points and sums stay in registers
+        float v[NT][KL];
 #pragma unroll
-          for (int e = 0; e < KL; ++e) v[e] = 0.f;
+        for (int i = 0; i < NT; ++i) raw(warp * NT + i, v[i]);
 #pragma unroll
-          for (int k = 0; k < S::SK; ++k) {
-            const float* src = s_s + ((size_t)k * rows + row) * SP + lane * KL;
-            if constexpr (KL == 1) v[0] += src[0];
-            else { const float2 t = *reinterpret_cast<const float2*>(src); v[0] += t.x; v[KL - 1] += t.y; }
+        for (int i = 0; i < NT; ++i) {
+          float top = -INFINITY;
+#pragma unroll
+          for (int e = 0; e < KL; ++e) {
+            const int k = key0 + lane * KL + e;
+            v[i][e] = k <= seen_to[i] && k >= seen_from[i] ? v[i][e] * p.scale_log2 : -INFINITY;
+            top = fmaxf(top, v[i][e]);
           }
-        };
-        if (S::LATENT) {
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            float x[KL], y[KL];
-            raw(h0 + 2 * i, x);
-            raw(h0 + 2 * i + 1, y);
-#pragma unroll
-            for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(x[e] * p.scale_log2, y[e] * p.scale_log2);
+          // the reference point moves only when the maximum has outgrown it by 2^8
+          if (__any_sync(0xffffffffu, top > m_row[i] + 8.0f)) {
+            const float m_new = fmaxf(m_row[i], warp_max(top)), c = ex2_fast(m_row[i] - m_new);
+            l_row[i] *= c;
+            if (lane == 0) {
+              c_s[warp * NT + i] = c;
+              if (m_row[i] != -INFINITY) rescale_flag[it & 1] = 1;
+            }
+            m_row[i] = m_new;
+          } else if (lane == 0) {
+            c_s[warp * NT + i] = 1.f;
           }
-        } else {
+          const float use = m_row[i] == -INFINITY ? 0.f : m_row[i];
+#pragma unroll
+          for (int e = 0; e < KL; ++e) { v[i][e] = ex2_fast(v[i][e] - use); l_row[i] += v[i][e]; }
+          store_weights(warp * NT + i, v[i]);
+        }
+      } else {
+        constexpr int CH = S::CH;
+        const int chunks = (H + CH - 1) / CH, n_units = chunks * n_tokens;
+        for (int unit = warp; unit < n_units; unit += 8) {
+          const int tok = n_tokens == 1 ? 0 : unit / chunks, h0 = (unit - tok * chunks) * CH;
+          float2 acc[CH / 2][KL];
+#pragma unroll
+          for (int i = 0; i < CH / 2; ++i)
+#pragma unroll
+            for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(0.f, 0.f);
           int row = tok * group, j = 0;
-#pragma unroll 4
+#pragma unroll 8
           for (int g = 0; g < H; ++g) {
             float x[KL];
             raw(row, x);
-            const float4 t0 = *reinterpret_cast<const float4*>(t_s + g * hp + h0), t1 = *reinterpret_cast<const float4*>(t_s + g * hp + h0 + 4);
+            const float* t = t_s + g * hp + h0;
 #pragma unroll
-            for (int e = 0; e < KL; ++e) {
-              const float2 xx = make_float2(x[e], x[e]);
-              acc[0][e] = fma2(make_float2(t0.x, t0.y), xx, acc[0][e]);
-              acc[1][e] = fma2(make_float2(t0.z, t0.w), xx, acc[1][e]);
-              acc[2][e] = fma2(make_float2(t1.x, t1.y), xx, acc[2][e]);
-              acc[3][e] = fma2(make_float2(t1.z, t1.w), xx, acc[3][e]);
+            for (int i = 0; i < CH / 2; ++i) {
+              const float2 t2 = *reinterpret_cast<const float2*>(t + 2 * i);
+#pragma unroll
+              for (int e = 0; e < KL; ++e) acc[i][e] = fma2(t2, make_float2(x[e], x[e]), acc[i][e]);
             }
             ++row;
             if (++j == group) { j = 0; row += R - group; }
           }
-        }
-        float sum[8];
-        int seen_lo = 0, seen_hi = 0;
-        if (!S::LATENT) {
-          seen_hi = base + r0 / group + tok;
-          seen_lo = first_visible(seen_hi, p.window, p.chunk);
-        }
+          const int seen_hi = base + r0 / group + tok, seen_lo = first_visible(seen_hi, p.window, p.chunk);
+          float sum[CH], m_old[CH];
+          int at[CH];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          sum[i] = 0.f;
-          int row;
-          if (S::LATENT) {
-            row = h0 + i;
-            if (row >= n_rows) continue;
-            seen_hi = base + (r0 + row) / group;
-            seen_lo = first_visible(seen_hi, p.window, p.chunk);
-          } else {
-            const int h = h0 + i;
-            if (h >= H) continue;
-            row = h / group * R + tok * group + h % group;
+          for (int i = 0; i < CH; ++i) {
+            at[i] = row_s[min(h0 + i, H - 1)] + tok * group;
+            m_old[i] = m_s[at[i]];
           }
-          float v[KL], top = -INFINITY;
 #pragma unroll
-          for (int e = 0; e < KL; ++e) {
-            const int key = key0 + lane * KL + e;
-            const float x = (i & 1) ? acc[i >> 1][e].y : acc[i >> 1][e].x;
-            v[e] = key <= seen_hi && key >= seen_lo ? x : -INFINITY;
-            top = fmaxf(top, v[e]);
-          }
-          // the reference point moves only when the maximum has outgrown it by 2^8
-          const float m_old = m_s[row];
-          float m_new = m_old;
-          if (__any_sync(0xffffffffu, top > m_old + 8.0f)) m_new = fmaxf(m_old, warp_max(top));
-          const float use = m_new == -INFINITY ? 0.f : m_new;
+          for (int i = 0; i < CH; ++i) {
+            sum[i] = 0.f;
+            if (h0 + i >= H) continue;
+            float v[KL], top = -INFINITY;
 #pragma unroll
-          for (int e = 0; e < KL; ++e) { v[e] = ex2_fast(v[e] - use); sum[i] += v[e]; }
-          bf16* dst = p_s + (size_t)row * PP + lane * KL;
-          if constexpr (KL == 1) dst[0] = __float2bfloat16_rn(v[0]);
-          else *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v[0], v[KL - 1]);
-          if (m_new != m_old) {   // warp-uniform, rare
-            __syncwarp();         // every lane has read the old one
-            if (lane == 0) {
-              const float c = ex2_fast(m_old - use);
-              m_s[row] = m_new;
-              c_s[row] = c;
-              l_s[row] *= c;
-              if (m_old != -INFINITY) rescale_flag[it & 1] = 1;
+            for (int e = 0; e < KL; ++e) {
+              const int key = key0 + lane * KL + e;
+              const float x = (i & 1) ? acc[i >> 1][e].y : acc[i >> 1][e].x;
+              v[e] = key <= seen_hi && key >= seen_lo ? x : -INFINITY;
+              top = fmaxf(top, v[e]);
             }
-          } else if (lane == 0) {
-            c_s[row] = 1.f;
+            float m_new = m_old[i];
+            const bool moves = __any_sync(0xffffffffu, top > m_old[i] + 8.0f);
+            if (moves) m_new = fmaxf(m_old[i], warp_max(top));
+            const float use = m_new == -INFINITY ? 0.f : m_new;
+#pragma unroll
+            for (int e = 0; e < KL; ++e) { v[e] = ex2_fast(v[e] - use); sum[i] += v[e]; }
+            store_weights(at[i], v);
+            if (lane == 0) {
+              const float c = moves ? ex2_fast(m_old[i] - use) : 1.f;
+              c_s[at[i]] = c;
+              if (moves) {
+                m_s[at[i]] = m_new;
+                l_s[at[i]] *= c;
+                if (m_old[i] != -INFINITY) rescale_flag[it & 1] = 1;
+              }
+            }
+          }
+          if constexpr (CH == 8) {   // eight sums over the lanes at once; lane 4 i ends up with the i-th
+#pragma unroll
+            for (int half = 4; half >= 1; half >>= 1)
+#pragma unroll
+              for (int i = 0; i < half; ++i) {
+                const bool up = lane & (half * 4);
+                const float keep = up ? sum[i + half] : sum[i], send = up ? sum[i] : sum[i + half];
+                sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, half * 4);
+              }
+            sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 2);
+            sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 1);
+            __syncwarp();   // (lane 0 may have rescaled a row's sum)
+            if ((lane & 3) == 0 && h0 + (lane >> 2) < H) l_s[row_s[h0 + (lane >> 2)] + tok * group] += sum[0];
+            __syncwarp();
+          } else {
+#pragma unroll
+            for (int i = 0; i < CH; ++i) sum[i] = warp_sum(sum[i]);
+            if (lane == 0)
+              for (int i = 0; i < CH; ++i)
+                if (h0 + i < H) l_s[at[i]] += sum[i];
           }
         }
-        // eight sums over the lanes at once; lane 4 i ends up with the i-th
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const bool up = lane & 16;
-          const float keep = up ? sum[i + 4] : sum[i], send = up ? sum[i] : sum[i + 4];
-          sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, 16);
-        }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const bool up = lane & 8;
-          const float keep = up ? sum[i + 2] : sum[i], send = up ? sum[i] : sum[i + 2];
-          sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
-        }
-        {
-          const bool up = lane & 4;
-          const float keep = up ? sum[1] : sum[0], send = up ? sum[0] : sum[1];
-          sum[0] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
-        }
-        sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 2);
-        sum[0] += __shfl_xor_sync(0xffffffffu, sum[0], 1);
-        __syncwarp();   // (lane 0 may have rescaled a row's sum)
-        if ((lane & 3) == 0) {
-          const int h = h0 + (lane >> 2);
-          if (S::LATENT ? h < n_rows : h < H) l_s[S::LATENT ? h : h / group * R + tok * group + h % group] += sum[0];
-        }
-        __syncwarp();
       }
       consumers_sync();
       // ---------------------------------------------------------------- 3: values
@@ -438,9 +463,9 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       for (int a = 0; a < GP; ++a) {
         const int g = a * S::TEAMS + team;
         if (g >= G) continue;
-        const uint32_t u = (uint32_t)it * units + (S::LATENT ? 0 : G + g), st = u % p.stages;
+        const uint32_t u = (uint32_t)it * units + (S::LATENT ? 0 : G + g), turn = turn_of(u), st = u - turn * p.stages;
         if (!S::LATENT) {
-          ptx::mbar_wait(&full_bar[st], (u / p.stages) & 1u, &abort_flag, p.wait_cycles);
+          ptx::mbar_wait(&full_bar[st], turn & 1u, &abort_flag, p.wait_cycles);
           __syncwarp();
         }
         const uint32_t vt = s_u32(ring + (size_t)st * p.stage_bytes);
@@ -461,7 +486,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
 #pragma unroll
           for (int d = 0; d < DW; ++d) {
             const int dim0 = (wi * DW + d) * 16;
-            if (dim0 >= live_heads) continue;
+            if (dim0 >= live_dims) continue;
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
               uint32_t af[4];
@@ -473,6 +498,13 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
         }
         __syncwarp();
         if (lane == 0) ptx::mbar_arrive(&empty_bar[st]);
+      }
+    }
+    if constexpr (S::LATENT) {
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const float l = warp_sum(l_row[i]);
+        if (lane == 0) { m_s[warp * NT + i] = m_row[i]; l_s[warp * NT + i] = l; }
       }
     }
     consumers_sync();
@@ -557,6 +589,7 @@ int launch(rb_ctx* ctx, rb_kv_cache* c, Params p, int layer, int batch, int max_
   size_t smem = 0;
   p.stages = ring_of<S>(p, &smem);
   const int whole = p.s_new * p.group;
+  if (p.stages > 0) p.stages_inv = (uint32_t)(((1ull << 32) + p.stages - 1) / p.stages);
   p.tile_rows = std::min(whole, S::LATENT ? S::R : S::R / p.group * p.group);
   if (p.stages == 0 || p.tile_rows == 0) return RB_ERR_UNIMPLEMENTED;
   p.row_tiles = (whole + p.tile_rows - 1) / p.tile_rows;
