@@ -42,7 +42,8 @@ struct Params {
   int row_tiles, tile_rows;    // rows (token, head of a key/value head) of a block: tile_rows <= 8 NT
   int nbk, nbv;                // 64-column blocks of a key and of a value that matter
   int stages, stage_bytes;
-  uint32_t stages_inv;         // ceil(2^32 / stages)
+  int ring, own_rings;         // stages of a ring; whether each team has a ring of its own
+  uint32_t ring_inv;           // ceil(2^32 / ring)
   int n_splits;
   int window, chunk, value_dim;
   float scale_log2;
@@ -157,7 +158,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
   __shared__ __align__(8) uint64_t empty_bar[kMaxStages];
   __shared__ volatile uint32_t abort_flag;
   __shared__ volatile int rescale_flag[2];
-  __shared__ uint32_t issued_count, is_last;
+  __shared__ uint32_t full_turn[kMaxStages], is_last;   // copies issued into each stage
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int G = p.kv_heads, H = p.q_heads, group = p.group;
   const Layout lay = layout_of<S>(G, H, p.nbk);
@@ -177,7 +178,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(&full_bar[s], 1); ptx::mbar_init(&empty_bar[s], S::WG); }
     abort_flag = 0;
     rescale_flag[0] = rescale_flag[1] = 0;
-    issued_count = 0;
+    for (int s = 0; s < p.stages; ++s) full_turn[s] = 0;
     ptx::fence_barrier_init();
     ptx::fence_proxy_async();
     ptx::tma_prefetch_desc(&tm_k);
@@ -201,25 +202,40 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     tile_hi = min(tile_hi, tile_lo + per);
   }
   const int units = S::LATENT ? 1 : 2 * G;   // copies per key tile
-  auto turn_of = [&](uint32_t u) { return __umulhi(u, p.stages_inv); };   // u / stages (u < 2^20)
+  // Stage of the copy of head g's keys or values of the it-th tile, and how often the stage has been used before.  One ring serves
+  // all heads if it holds a tile of each: a team then never waits for a copy into a stage whose earlier copy, another
+  // team's, may still be on its way (it would take that one for its own).  Otherwise each team has a ring of its own.
+  auto place = [&](int it, int g, bool values, uint32_t& st) -> uint32_t {
+    uint32_t u, first = 0;
+    if (!p.own_rings) {
+      u = (uint32_t)it * units + (values ? G + g : g);
+    } else {
+      const int t = g % S::TEAMS, heads = (G - t + S::TEAMS - 1) / S::TEAMS, a = g / S::TEAMS;
+      u = (uint32_t)it * (2 * heads) + (values ? heads + a : a);
+      first = t * p.ring;
+    }
+    const uint32_t turn = p.ring == 1 ? u : __umulhi(u, p.ring_inv);   // u / ring (u < 2^20)
+    st = first + u - turn * p.ring;
+    return turn;
+  };
 
   if (warp >= 8) {
     // ------------------------------------------------------------------ copies
     give_registers();
     if (warp == 8 && lane == 0) {
-      uint32_t u = 0;
       bool ok = true;
       for (int tile = tile_lo; tile < tile_hi && ok; ++tile) {
         const int page = p.block_table[(size_t)b * p.pages_per_seq + tile * KT / kPageTokens];
-        for (int i = 0; i < units && ok; ++i, ++u) {
-          const uint32_t turn = turn_of(u), st = u - turn * p.stages;
+        for (int i = 0; i < units && ok; ++i) {
+          uint32_t st;
+          const uint32_t turn = place(tile - tile_lo, i < G ? i : i - G, i >= G, st);
           if (!ptx::mbar_wait(&empty_bar[st], (turn & 1u) ^ 1u, &abort_flag, p.wait_cycles)) { ok = false; break; }
           const bool v = i >= G;
           const int nb = v ? p.nbv : p.nbk, y = (page * G + (v ? i - G : i)) * kPageTokens + tile * KT % kPageTokens;
           ptx::mbar_expect_tx(&full_bar[st], (uint32_t)nb * KT * 128);
           for (int cb = 0; cb < nb; ++cb)
             ptx::tma_load_2d(ring + (size_t)st * p.stage_bytes + cb * (KT * 128), v ? &tm_v : &tm_k, &full_bar[st], cb * 64, y);
-          issued_count = u + 1;
+          full_turn[st] = turn + 1;
         }
       }
     }
@@ -276,7 +292,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       for (int a = 0; a < GP; ++a) {
         const int g = a * S::TEAMS + team;
         if (g >= G) continue;
-        const uint32_t u = (uint32_t)it * units + g, turn = turn_of(u), st = u - turn * p.stages;
+        uint32_t st;
+        const uint32_t turn = place(it, g, false, st);
         ptx::mbar_wait(&full_bar[st], turn & 1u, &abort_flag, p.wait_cycles);
         __syncwarp();
         const uint32_t kt = s_u32(ring + (size_t)st * p.stage_bytes);
@@ -463,7 +480,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       for (int a = 0; a < GP; ++a) {
         const int g = a * S::TEAMS + team;
         if (g >= G) continue;
-        const uint32_t u = (uint32_t)it * units + (S::LATENT ? 0 : G + g), turn = turn_of(u), st = u - turn * p.stages;
+        uint32_t st;
+        const uint32_t turn = place(it, g, !S::LATENT, st);
         if (!S::LATENT) {
           ptx::mbar_wait(&full_bar[st], turn & 1u, &abort_flag, p.wait_cycles);
           __syncwarp();
@@ -565,8 +583,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
   if (abort_flag && threadIdx.x == 0) {
     p.status[0] = (uint32_t)(-RB_ERR_TIMEOUT); p.status[1] = 0xA701u; p.status[2] = blockIdx.y; p.status[3] = blockIdx.z;
     volatile uint32_t never = 0;   // copies already on their way get a bounded chance to land
-    for (uint32_t u = issued_count > (uint32_t)p.stages ? issued_count - p.stages : 0; u < issued_count; ++u)
-      ptx::mbar_wait(&full_bar[u % p.stages], (u / p.stages) & 1u, &never, p.wait_cycles);
+    for (int st = 0; st < p.stages; ++st)
+      if (full_turn[st] > 0) ptx::mbar_wait(&full_bar[st], (full_turn[st] - 1u) & 1u, &never, p.wait_cycles);
   }
 }
 
@@ -589,9 +607,12 @@ int launch(rb_ctx* ctx, rb_kv_cache* c, Params p, int layer, int batch, int max_
   size_t smem = 0;
   p.stages = ring_of<S>(p, &smem);
   const int whole = p.s_new * p.group;
-  if (p.stages > 0) p.stages_inv = (uint32_t)(((1ull << 32) + p.stages - 1) / p.stages);
+  p.own_rings = !S::LATENT && p.stages < p.kv_heads;
+  p.ring = p.own_rings ? p.stages / S::TEAMS : p.stages;
+  if (p.ring == 0) return RB_ERR_UNIMPLEMENTED;
+  p.ring_inv = (uint32_t)std::min<uint64_t>(0xffffffffull, ((1ull << 32) + p.ring - 1) / p.ring);
   p.tile_rows = std::min(whole, S::LATENT ? S::R : S::R / p.group * p.group);
-  if (p.stages == 0 || p.tile_rows == 0) return RB_ERR_UNIMPLEMENTED;
+  if (p.tile_rows == 0) return RB_ERR_UNIMPLEMENTED;
   p.row_tiles = (whole + p.tile_rows - 1) / p.tile_rows;
   p.n_splits = 1;
   if (p.s_new == 1 && p.row_tiles <= (S::LATENT ? ::kLatentRowTiles : 1)) {

@@ -16,10 +16,12 @@ int attention_talk_tc(rb_ctx* ctx, const joint::Params& p, rb_kv_cache* c, int l
   if (G == 2) { if (wide) RB_TALK(4, 1, 4, 8); RB_TALK(4, 1, 2, 8); }
   if (G <= 4) { if (wide) RB_TALK(2, 1, 8, 4); RB_TALK(2, 1, 4, 8); }
   if (G <= 8) { if (wide) RB_TALK(1, 1, 16, 2); RB_TALK(1, 1, 8, 4); }
-  if (G <= 16 && !wide) RB_TALK(1, 2, 8, 2);
+  if (G <= 16 && !wide)
+    return rows <= 8 ? joint::launch<Shape<32, 1, 2, 8, 1, false>>(ctx, c, p, layer, batch, max_len)
+                     : joint::launch<Shape<32, 1, 2, 8, 2, false>>(ctx, c, p, layer, batch, max_len);
 #undef RB_TALK
-  if (G <= 16) return joint::launch<Shape<64, 1, 2, 16, 1, false>>(ctx, c, p, layer, batch, max_len);
-  if (G <= 32 && !wide) return joint::launch<Shape<64, 1, 4, 8, 1, false>>(ctx, c, p, layer, batch, max_len);
+  if (G <= 16) return joint::launch<Shape<32, 1, 2, 16, 1, false>>(ctx, c, p, layer, batch, max_len);
+  if (G <= 32 && !wide) return joint::launch<Shape<32, 1, 4, 8, 1, false>>(ctx, c, p, layer, batch, max_len);
   return RB_ERR_UNIMPLEMENTED;
 }
 

@@ -305,12 +305,13 @@ def rounded_sink(rng, H, dtype):
 
 
 TALKS = [(4, 2, 40, 24), (3, 3, 72, 80), (6, 1, 96, 56), (8, 8, 96, 128), (9, 3, 20, 13), (16, 4, 128, 64), (12, 12, 64, 64), (4, 2, 200, 160), (6, 6, 64, 200),
-         (2, 1, 256, 40), (24, 24, 32, 32), (1, 1, 64, 64), (40, 2, 32, 32), (32, 8, 128, 128), (10, 10, 136, 136), (20, 20, 64, 144), (36, 36, 24, 16)]
+         (2, 1, 256, 40), (24, 24, 32, 32), (1, 1, 64, 64), (40, 2, 32, 32), (32, 8, 128, 128), (10, 10, 136, 136), (20, 20, 64, 144), (36, 36, 24, 16),
+         (32, 32, 128, 128), (16, 16, 128, 64), (12, 12, 128, 128), (8, 8, 128, 128), (7, 7, 200, 256), (12, 3, 96, 96), (5, 5, 64, 64), (24, 8, 64, 32)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,d,e", TALKS)
-@pytest.mark.parametrize("base,s_new", [(0, 1), (0, 2), (0, 70), (33, 2), (70, 45), (130, 1)])
+@pytest.mark.parametrize("base,s_new", [(0, 1), (0, 2), (0, 70), (33, 2), (70, 45), (130, 1), (230, 9), (300, 1)])
 def test_attention_with_mixed_heads(cuda, dtype, H, G, d, e, base, s_new):
     sink = rounded_sink(np.random.default_rng(H), H, dtype)
     got, (q, k, v, talk) = talking_case(cuda, dtype, H, G, d, e, base, s_new, sink=sink)
