@@ -122,7 +122,9 @@ __device__ __forceinline__ void merge_splits(const Params& p, float* w_s, int b,
     const int head = head_of(i);
     const float* ml = p.part_ml + ((size_t)b * H + head) * ns * 2;
     float M = -INFINITY, L = 0.f;
+#pragma unroll 4
     for (int s = 0; s < ns; ++s) M = fmaxf(M, __ldcg(ml + 2 * s));
+#pragma unroll 4
     for (int s = 0; s < ns; ++s) {
       const float w = ex2_fast(__ldcg(ml + 2 * s) - M);
       L = fmaf(w, __ldcg(ml + 2 * s + 1), L);
@@ -133,18 +135,36 @@ __device__ __forceinline__ void merge_splits(const Params& p, float* w_s, int b,
     for (int s = 0; s < ns; ++s) w_s[i * kMaxSplits + s] *= inv;
   }
   consumers_sync();
+  if ((vd & 3) == 0) {
+    const int quads = vd >> 2;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < live * quads; i += kConsumers) {
+      const int row = i / quads, dim = (i - row * quads) * 4, head = head_of(row);
+      const float4* src = reinterpret_cast<const float4*>(p.part_o + ((size_t)b * H + head) * ns * vd + dim);
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int s0 = 0; s0 < ns; s0 += 4) {
+        float4 t[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (s0 + k < ns) t[k] = __ldcg(src + (size_t)(s0 + k) * quads);
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (s0 + k < ns) {
+            const float w = w_s[row * kMaxSplits + s0 + k];
+            v.x = fmaf(t[k].x, w, v.x); v.y = fmaf(t[k].y, w, v.y); v.z = fmaf(t[k].z, w, v.z); v.w = fmaf(t[k].w, w, v.w);
+          }
+      }
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      *reinterpret_cast<uint2*>(p.out + (size_t)b * p.out_ld + (size_t)head * vd + dim) =
+          make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < live * vd; i += kConsumers) {
     const int row = i / vd, dim = i % vd, head = head_of(row);
     const float* src = p.part_o + ((size_t)b * H + head) * ns * vd + dim;
     float v = 0.f;
-    for (int s0 = 0; s0 < ns; s0 += 8) {
-      float t[8];
-#pragma unroll
-      for (int k = 0; k < 8; ++k) t[k] = s0 + k < ns ? __ldcg(src + (size_t)(s0 + k) * vd) : 0.f;
-#pragma unroll
-      for (int k = 0; k < 8; ++k)
-        if (s0 + k < ns) v = fmaf(t[k], w_s[row * kMaxSplits + s0 + k], v);
-    }
+    for (int sp = 0; sp < ns; ++sp) v = fmaf(__ldcg(src + (size_t)sp * vd), w_s[row * kMaxSplits + sp], v);
     p.out[(size_t)b * p.out_ld + (size_t)head * vd + dim] = __float2bfloat16_rn(v);
   }
 }
@@ -245,22 +265,27 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     float o[GP][DW][NT][4];
     for (int i = threadIdx.x; i < rows * (p.nbk * 8); i += kConsumers) {
       const int row = i / (p.nbk * 8), c = i % (p.nbk * 8) * 8, g = row / R, n = row % R;
-      uint4 v = make_uint4(0, 0, 0, 0);
+      bf16* dst = q_s + (size_t)row * qp + c;
       if (n < n_rows) {
-        const int token = (r0 + n) / group, head = g * group + (r0 + n) % group;
-        v = *reinterpret_cast<const uint4*>(p.q + (((size_t)b * p.s_new + token) * H + head) * p.D + c);
+        const int token = p.s_new == 1 ? 0 : (r0 + n) / group, head = g * group + r0 + n - token * group;
+        cp_async16(dst, p.q + (((size_t)b * p.s_new + token) * H + head) * p.D + c);
+      } else {
+        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
       }
-      *reinterpret_cast<uint4*>(q_s + (size_t)row * qp + c) = v;
     }
+    cp_async_commit();
     for (int i = threadIdx.x; i < rows * (PP / 8); i += kConsumers) reinterpret_cast<uint4*>(p_s)[i] = make_uint4(0, 0, 0, 0);
     for (int i = threadIdx.x; i < rows; i += kConsumers) { m_s[i] = -INFINITY; l_s[i] = 0.f; c_s[i] = 1.f; }
     if (!S::LATENT)
       for (int h = threadIdx.x; h < H; h += kConsumers) row_s[h] = h / group * R + h % group;
-    if (!S::LATENT)
+    if (!S::LATENT) {
+#pragma unroll 4
       for (int i = threadIdx.x; i < H * hp; i += kConsumers) {
-        const int g = i / hp, h = i % hp;
-        t_s[i] = h < H ? __bfloat162float(p.talk[h * H + g]) * p.scale_log2 : 0.f;
+        const int h = i / H, g = i - h * H;   // (neighbouring threads read neighbours)
+        t_s[g * hp + h] = h < H ? __bfloat162float(__ldg(p.talk + min(i, H * H - 1))) * p.scale_log2 : 0.f;
       }
+    }
+    cp_async_wait<0>();
     consumers_sync();
 #pragma unroll
     for (int a = 0; a < GP; ++a)
@@ -273,6 +298,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
     const int km = wi % S::SM, ks = wi / S::SM;
     const int steps = p.nbk * 4, per_part = (steps + S::SK - 1) / S::SK, k_lo = ks * per_part, k_hi = min(steps, k_lo + per_part);
     const int live_dims = p.value_dim, n_tokens = S::LATENT ? 1 : n_rows / group;
+    const bool windowed = p.window < (1 << 30) || p.chunk > 0;
+    bool rescaled = false;        // this warp's rows had other factors than 1 in the tile before
     float m_row[NT], l_row[NT];   // LATENT: of this warp's rows
     int seen_from[NT], seen_to[NT];
     if constexpr (S::LATENT) {
@@ -359,30 +386,46 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
         else *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v[0], v[KL - 1]);
       };
       if constexpr (S::LATENT) {   // a warp has NT rows for the whole walk: reference points and sums stay in registers
-        float v[NT][KL];
+        float v[NT][KL], top[NT];
 #pragma unroll
         for (int i = 0; i < NT; ++i) raw(warp * NT + i, v[i]);
+        const bool edge = key0 + KT - 1 > base + first_token || windowed;   // a key that some row does not see
+        bool outgrown = false;
 #pragma unroll
         for (int i = 0; i < NT; ++i) {
-          float top = -INFINITY;
+          top[i] = -INFINITY;
 #pragma unroll
           for (int e = 0; e < KL; ++e) {
+            v[i][e] *= p.scale_log2;
             const int k = key0 + lane * KL + e;
-            v[i][e] = k <= seen_to[i] && k >= seen_from[i] ? v[i][e] * p.scale_log2 : -INFINITY;
-            top = fmaxf(top, v[i][e]);
+            if (edge && (k > seen_to[i] || k < seen_from[i])) v[i][e] = -INFINITY;
+            top[i] = fmaxf(top[i], v[i][e]);
           }
-          // the reference point moves only when the maximum has outgrown it by 2^8
-          if (__any_sync(0xffffffffu, top > m_row[i] + 8.0f)) {
-            const float m_new = fmaxf(m_row[i], warp_max(top)), c = ex2_fast(m_row[i] - m_new);
-            l_row[i] *= c;
-            if (lane == 0) {
-              c_s[warp * NT + i] = c;
-              if (m_row[i] != -INFINITY) rescale_flag[it & 1] = 1;
+          outgrown |= top[i] > m_row[i] + 8.0f;   // the reference point moves only when the maximum has outgrown it by 2^8
+        }
+        if (rescaled) {   // (the factors of the tile before have been read)
+          if (lane == 0)
+            for (int i = 0; i < NT; ++i) c_s[warp * NT + i] = 1.f;
+          rescaled = false;
+        }
+        if (__any_sync(0xffffffffu, outgrown)) {
+#pragma unroll
+          for (int i = 0; i < NT; ++i) {
+            const float best = warp_max(top[i]);
+            if (best > m_row[i] + 8.0f) {
+              const float c = ex2_fast(m_row[i] - best);
+              l_row[i] *= c;
+              if (lane == 0) {
+                c_s[warp * NT + i] = c;
+                if (m_row[i] != -INFINITY) rescale_flag[it & 1] = 1;
+              }
+              m_row[i] = best;
             }
-            m_row[i] = m_new;
-          } else if (lane == 0) {
-            c_s[warp * NT + i] = 1.f;
           }
+          rescaled = true;
+        }
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
           const float use = m_row[i] == -INFINITY ? 0.f : m_row[i];
 #pragma unroll
           for (int e = 0; e < KL; ++e) { v[i][e] = ex2_fast(v[i][e] - use); l_row[i] += v[i][e]; }
@@ -391,6 +434,8 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
       } else {
         constexpr int CH = S::CH;
         const int chunks = (H + CH - 1) / CH, n_units = chunks * n_tokens;
+        const bool any_factors = rescaled;
+        bool any_moved = false;
         for (int unit = warp; unit < n_units; unit += 8) {
           const int tok = n_tokens == 1 ? 0 : unit / chunks, h0 = (unit - tok * chunks) * CH;
           float2 acc[CH / 2][KL];
@@ -398,57 +443,73 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
           for (int i = 0; i < CH / 2; ++i)
 #pragma unroll
             for (int e = 0; e < KL; ++e) acc[i][e] = make_float2(0.f, 0.f);
-          int row = tok * group, j = 0;
-#pragma unroll 8
-          for (int g = 0; g < H; ++g) {
-            float x[KL];
-            raw(row, x);
-            const float* t = t_s + g * hp + h0;
+          constexpr int B = CH == 8 ? 4 : 8;   // raw heads in flight
+          for (int g0 = 0; g0 < H; g0 += B) {
+            float x[B][KL];
+            float2 t2[B][CH / 2];
 #pragma unroll
-            for (int i = 0; i < CH / 2; ++i) {
-              const float2 t2 = *reinterpret_cast<const float2*>(t + 2 * i);
+            for (int g = 0; g < B; ++g) {
+              const int gg = min(g0 + g, H - 1);
+              raw(row_s[gg] + tok * group, x[g]);
 #pragma unroll
-              for (int e = 0; e < KL; ++e) acc[i][e] = fma2(t2, make_float2(x[e], x[e]), acc[i][e]);
+              for (int i = 0; i < CH / 2; ++i) t2[g][i] = *reinterpret_cast<const float2*>(t_s + gg * hp + h0 + 2 * i);
             }
-            ++row;
-            if (++j == group) { j = 0; row += R - group; }
+#pragma unroll
+            for (int g = 0; g < B; ++g)
+              if (g0 + g < H) {
+#pragma unroll
+                for (int i = 0; i < CH / 2; ++i)
+#pragma unroll
+                  for (int e = 0; e < KL; ++e) acc[i][e] = fma2(t2[g][i], make_float2(x[g][e], x[g][e]), acc[i][e]);
+              }
           }
           const int seen_hi = base + r0 / group + tok, seen_lo = first_visible(seen_hi, p.window, p.chunk);
-          float sum[CH], m_old[CH];
+          float sum[CH], m[CH], v[CH][KL], top[CH];
           int at[CH];
+          bool outgrown = false;
 #pragma unroll
           for (int i = 0; i < CH; ++i) {
             at[i] = row_s[min(h0 + i, H - 1)] + tok * group;
-            m_old[i] = m_s[at[i]];
+            m[i] = m_s[at[i]];
+          }
+#pragma unroll
+          for (int i = 0; i < CH; ++i) {
+            top[i] = -INFINITY;
+#pragma unroll
+            for (int e = 0; e < KL; ++e) {
+              const int key = key0 + lane * KL + e;
+              const float x = (i & 1) ? acc[i >> 1][e].y : acc[i >> 1][e].x;
+              v[i][e] = key <= seen_hi && key >= seen_lo ? x : -INFINITY;
+              top[i] = fmaxf(top[i], v[i][e]);
+            }
+            outgrown |= h0 + i < H && top[i] > m[i] + 8.0f;   // the reference point moves only when the maximum has outgrown it by 2^8
+          }
+          const bool moves = __any_sync(0xffffffffu, outgrown);
+          if (moves || any_factors) {   // (factors other than 1 of the tile before have been read)
+#pragma unroll
+            for (int i = 0; i < CH; ++i) {
+              const float best = moves ? warp_max(top[i]) : -INFINITY, old = m[i];
+              const bool move = best > old + 8.0f;
+              if (move) m[i] = best;
+              __syncwarp();
+              if (lane == 0 && h0 + i < H) {
+                const float c = move ? ex2_fast(old - best) : 1.f;
+                c_s[at[i]] = c;
+                m_s[at[i]] = m[i];
+                l_s[at[i]] *= c;
+                if (move && old != -INFINITY) rescale_flag[it & 1] = 1;
+              }
+            }
+            any_moved |= moves;
           }
 #pragma unroll
           for (int i = 0; i < CH; ++i) {
             sum[i] = 0.f;
             if (h0 + i >= H) continue;
-            float v[KL], top = -INFINITY;
+            const float use = m[i] == -INFINITY ? 0.f : m[i];
 #pragma unroll
-            for (int e = 0; e < KL; ++e) {
-              const int key = key0 + lane * KL + e;
-              const float x = (i & 1) ? acc[i >> 1][e].y : acc[i >> 1][e].x;
-              v[e] = key <= seen_hi && key >= seen_lo ? x : -INFINITY;
-              top = fmaxf(top, v[e]);
-            }
-            float m_new = m_old[i];
-            const bool moves = __any_sync(0xffffffffu, top > m_old[i] + 8.0f);
-            if (moves) m_new = fmaxf(m_old[i], warp_max(top));
-            const float use = m_new == -INFINITY ? 0.f : m_new;
-#pragma unroll
-            for (int e = 0; e < KL; ++e) { v[e] = ex2_fast(v[e] - use); sum[i] += v[e]; }
-            store_weights(at[i], v);
-            if (lane == 0) {
-              const float c = moves ? ex2_fast(m_old[i] - use) : 1.f;
-              c_s[at[i]] = c;
-              if (moves) {
-                m_s[at[i]] = m_new;
-                l_s[at[i]] *= c;
-                if (m_old[i] != -INFINITY) rescale_flag[it & 1] = 1;
-              }
-            }
+            for (int e = 0; e < KL; ++e) { v[i][e] = ex2_fast(v[i][e] - use); sum[i] += v[i][e]; }
+            store_weights(at[i], v[i]);
           }
           if constexpr (CH == 8) {   // eight sums over the lanes at once; lane 4 i ends up with the i-th
 #pragma unroll
@@ -472,6 +533,7 @@ __global__ void __launch_bounds__(kThreads, 1) joint_attention_kernel(const Para
                 if (h0 + i < H) l_s[at[i]] += sum[i];
           }
         }
+        rescaled = any_moved;
       }
       consumers_sync();
       // ---------------------------------------------------------------- 3: values

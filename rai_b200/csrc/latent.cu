@@ -202,22 +202,32 @@ struct HeadProduct {
 };
 
 // what lies behind the product in a query's row, for rows m0 .. m0 + n_rows of head h
+// `part` of `parts`: rows are shared out over the blocks that hold the same rows' columns.
 template <typename T>
-__device__ __forceinline__ void query_tail(const HeadProduct<T>& p, int64_t m0, int n_rows, int h) {
+__device__ __forceinline__ void query_tail(const HeadProduct<T>& p, int64_t m0, int n_rows, int h, int part, int parts) {
   const int tail = p.out_head - p.n;
-  for (int it = threadIdx.x; it < n_rows * tail; it += blockDim.x) {
-    const int64_t m = m0 + it / tail;
-    const int i = it % tail;
-    if (m >= p.rows) break;
+  const int mine = (n_rows - part + parts - 1) / parts;
+#pragma unroll 4
+  for (int it = threadIdx.x; it < mine * tail; it += blockDim.x) {
+    const int r = it / tail, i = it - r * tail;
+    const int64_t m = m0 + part + (int64_t)r * parts;
+    if (m >= p.rows) continue;
     float y = 0.f;
     if (i < p.rot_dim) {
-      const int pos = p.pages.seq_lens[m / p.s_new] - p.s_new + (int)(m % p.s_new);
+      const int seq = p.s_new == 1 ? (int)m : (int)(m / p.s_new);
+      const int pos = p.pages.seq_lens[seq] - p.s_new + (int)(m - (int64_t)seq * p.s_new);
       if (pos < 0 || pos >= p.pages.max_seq) continue;   // (the append has recorded it)
       const size_t base = (size_t)m * p.a_ld + (size_t)h * p.a_head + p.k;
       y = turned(p.rot, pos, i, [&](int j) {
         if (p.a) return Cvt<T>::to_f(p.a[base + j]);
         float s = 0.f;
-        for (int t = 0; t < p.n_acc; ++t) s += p.acc[(size_t)t * p.acc_stride + base + j];
+        for (int t0 = 0; t0 < p.n_acc; t0 += 4) {
+          float v[4];
+#pragma unroll
+          for (int t = 0; t < 4; ++t) v[t] = t0 + t < p.n_acc ? p.acc[(size_t)(t0 + t) * p.acc_stride + base + j] : 0.f;
+#pragma unroll
+          for (int t = 0; t < 4; ++t) s += v[t];
+        }
         return s;
       });
     }
@@ -247,7 +257,7 @@ __global__ void __launch_bounds__(128) head_product_plain_kernel(const HeadProdu
     if (!QUERY) s *= gate_of(p, m, h, c);
     p.out[(size_t)m * p.out_ld + (size_t)h * p.out_head + c] = Cvt<T>::from_f(s);
   }
-  if (QUERY) query_tail(p, m, 1, h);
+  if (QUERY) query_tail(p, m, 1, h, 0, 1);
 }
 
 constexpr int kHpRows = 64, kHpCols = 32, kHpMaxK = 512;
@@ -307,6 +317,7 @@ __global__ void __launch_bounds__(128) head_product_mma_kernel(const HeadProduct
       }
     }
     cp_async_commit();
+    if (QUERY && k0 == 0) query_tail(p, m0, kHpRows, h, (int)blockIdx.x, (int)gridDim.x);   // (while the copies land)
     cp_async_wait<0>();
     __syncthreads();
     for (int kk = 0; kk < kc; kk += 16) {
@@ -340,7 +351,6 @@ __global__ void __launch_bounds__(128) head_product_mma_kernel(const HeadProduct
       for (int e = 0; e < 2; ++e)
         if (c + e < p.n) dst[e] = __float2bfloat16_rn(QUERY ? o[i][hf * 2 + e] : o[i][hf * 2 + e] * gate_of(p, m, h, c + e));
     }
-  if (QUERY && blockIdx.x == 0) query_tail(p, m0, kHpRows, h);
 }
 
 template <typename T, bool QUERY>
