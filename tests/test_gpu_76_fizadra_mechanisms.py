@@ -319,6 +319,14 @@ def test_attention_with_mixed_heads(cuda, dtype, H, G, d, e, base, s_new):
     assert rms_err(got, want) < TOL[dtype]
 
 
+@pytest.mark.parametrize("H,G,d,e", [(8, 4, 64, 64), (16, 16, 128, 128), (5, 1, 128, 64)])
+@pytest.mark.parametrize("base,s_new", [(0, 70), (70, 45)])
+def test_mixing_known_on_the_device_only(cuda, H, G, d, e, base, s_new):
+    got, (q, k, v, talk) = talking_case(cuda, _lib.BF16, H, G, d, e, base, s_new, on_host=False)
+    want = np.stack([ref.attention(q[b, base:], k[b], v[b], 0.2, None, talk, base) for b in range(2)])
+    assert rms_err(got, want) < TOL[_lib.BF16]
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,d,e", [(8, 8, 96, 128), (16, 4, 128, 64), (6, 1, 96, 56)])
 @pytest.mark.parametrize("base,s_new", [(0, 300), (999, 1), (700, 1), (301, 64)])
